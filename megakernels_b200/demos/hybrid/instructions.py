@@ -1,0 +1,178 @@
+"""Decode instruction set of layer-list models and the globals its kernels run on.
+
+Same encoding as the latency set (``Instruction.serialize``): opcode, then the fields.  One
+instruction covers a run of whole output rows (projections), a block of value columns of one
+recurrence head, or one split of the visible keys of a KV head; the phases of a layer are ordered
+by one arrival counter per layer and opcode.
+"""
+
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+
+import torch
+from torch import Tensor
+
+from megakernels_b200.instructions import Instruction
+from megakernels_b200.utils import get_sm_count
+
+COUNTERS_PER_LAYER = 8  # MKBH_BARRIERS_PER_LAYER
+PARTIAL_SUMS = 4096  # per-row, per-column-group sums an instruction may hold
+
+
+@dataclass
+class HybridGlobals:
+    """Everything a launch reads or writes; prefill and decode share the activation buffers."""
+
+    model: object
+    device: torch.device
+    portion: int
+
+    tokens: Tensor  # int32 [portion]
+    want_rows: Tensor  # int32 [portion]
+    x: Tensor  # fp32 [portion, width]: the residual stream
+    proj: Tensor  # fp32 [portion, stacked projection rows or ff]
+    mixed: Tensor  # fp32 [portion, mixer output]
+    decay: Tensor  # fp32 [portion, recurrence channels]
+    act: Tensor  # model dtype [portion, widest matrix input]
+    logits: Tensor  # fp32 [vocab]
+    argmax_out: Tensor  # int32 [1]
+    counters: Tensor  # int32, zeroed by every decode launch
+    arrivals: Tensor  # int32 [layers + 1, COUNTERS_PER_LAYER]
+    attn_part: Tensor  # fp32 [max heads, 2, max_splits, max vdim + 2]
+    status: Tensor  # int32 [16]
+    max_splits: int
+    max_kv_heads: int
+    part_vdim: int
+
+    slot: int = 0
+    pos_id: int = 0
+    pos_id_device: Tensor | None = None  # int32 [1]; overrides pos_id in decode launches
+    instructions: Tensor | None = None
+    timings: Tensor | None = None
+    batch_size: int = 1
+    hooks: dict = field(default_factory=dict)
+
+    def sm_count(self) -> int:
+        return get_sm_count(self.device)
+
+    @property
+    def dtype_bytes(self) -> int:
+        return 4 if self.model.dtype == torch.float32 else 2
+
+
+def matrix_shape(globs: HybridGlobals, opcode: int, layer: int) -> tuple[int, int]:
+    """(rows, input columns) of the matrix an instruction streams."""
+    cfg = globs.model.config
+    if opcode == Head.opcode():
+        return cfg.vocab_size, cfg.width
+    spec = cfg.layers[layer]
+    return {
+        NormProj.opcode(): (spec.mixer.in_rows, cfg.width),
+        OutProj.opcode(): (cfg.width, spec.mixer.out_features),
+        NormUp.opcode(): (spec.mlp.ff if spec.mlp else 0, cfg.width),
+        Down.opcode(): (cfg.width, spec.mlp.ff if spec.mlp else 0),
+    }[opcode]
+
+
+@dataclass
+class RowRange(Instruction):
+    layer_idx: int
+    row_start: int
+    row_end: int
+
+    @classmethod
+    def tags(cls):
+        return {"pool": "memory"}
+
+    def cost(self, globs) -> float:
+        return (self.row_end - self.row_start) * matrix_shape(globs, self.opcode(), self.layer_idx)[1]
+
+
+@dataclass
+class NormProj(RowRange):
+    """Layer norm of the residual stream, stacked input projection of the mixer."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 1
+
+
+@dataclass
+class DeltaStep(Instruction):
+    """One step of a head's recurrence for value columns ``[col_start, col_end)``."""
+
+    layer_idx: int
+    head_idx: int
+    col_start: int
+    col_end: int
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 2
+
+    @classmethod
+    def tags(cls):
+        return {"pool": "compute"}
+
+    def cost(self, globs) -> float:
+        m = globs.model.config.layers[self.layer_idx].mixer
+        return (self.col_end - self.col_start) * m.dim * 4
+
+
+@dataclass
+class WindowAttention(Instruction):
+    """One split of the keys a KV head's queries see; the last split to arrive merges them."""
+
+    layer_idx: int
+    kv_head_idx: int
+    split_idx: int
+    num_splits: int
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 3
+
+    @classmethod
+    def tags(cls):
+        return {"pool": "compute"}
+
+    def cost(self, globs) -> float:
+        m = globs.model.config.layers[self.layer_idx].mixer
+        return (m.window + m.keep_first) * (2 * m.dim + m.vdim) / self.num_splits
+
+
+@dataclass
+class OutProj(RowRange):
+    """Output projection of the mixer, layer scale, residual add."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 4
+
+
+@dataclass
+class NormUp(RowRange):
+    """Layer norm, up projection of the feed-forward."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 5
+
+
+@dataclass
+class Down(RowRange):
+    """PolyNorm, down projection, layer scale, residual add."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 6
+
+
+@dataclass
+class Head(RowRange):
+    """Final layer norm, logits and their running argmax."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 7

@@ -217,13 +217,130 @@ class MK_Generator(Generator):
             out = self.run(ids[:, pos : pos + 1], pos_id=pos)
         return out.reshape(-1)
 
+    def step(self, tokens: list[int], position: int, want: list[int], slot: int = 0) -> Tensor:
+        """Feed a sequence's next ``tokens`` (the first one at ``position``) and return fp32 logits
+        ``[len(want), vocab]`` at the listed places among them."""
+        globs = self.schedule.globs
+        rows = []
+        for i, token in enumerate(tokens):
+            self.run(torch.tensor([[token]], device=globs.hidden_states.device), pos_id=position + i)
+            if i in want:
+                rows.append(globs.logits.float().reshape(-1).clone())
+        self.check()
+        order = sorted(set(want))
+        out = torch.stack(rows) if rows else torch.zeros(0, globs.vocab_size, device=globs.hidden_states.device)
+        return out[[order.index(i) for i in want]]
+
     def check(self):
         """Synchronise and raise if any device-side wait gave up."""
         if self.last_call is None:
             return None
-        import mk_llama  # the module get_mk_func imported
+        return self.interpreter.module.sync_status(self.last_call)
 
-        return mk_llama.sync_status(self.last_call)
+
+class Hybrid_Generator(MK_Generator):
+    """Layer-list models: prompts in portions through the prefill kernels, then one megakernel
+    launch per token.  ``slot`` selects the sequence whose state a call reads and advances."""
+
+    def __init__(self, model, interpreter, schedule, **kw):
+        # the kernel always computes the argmax; there is no barrier fill (the launch clears its counters)
+        self.slot = 0
+        self.model, self.interpreter, self.schedule = model, interpreter, schedule
+        self.skip_mk, self.skip_rest = kw.get("skip_mk", False), kw.get("skip_rest", False)
+        self.last_call = None
+
+    def fill(self):
+        """Nothing to reset: counters are cleared by the launch, recurrent state at position 0."""
+
+    def _place(self, tokens, position: int) -> int:
+        globs = self.schedule.globs
+        ids = torch.as_tensor(tokens).reshape(-1)
+        if ids.device.type == "cpu":
+            if ids.numel() and not (0 <= int(ids.min()) and int(ids.max()) < self.model.config.vocab_size):
+                raise ValueError("token id outside the vocabulary")
+        globs.tokens[: ids.numel()].copy_(ids, non_blocking=True)
+        globs.slot, globs.pos_id = self.slot, position
+        return ids.numel()
+
+    def run(self, input_ids: Tensor, pos_id: int):
+        if getattr(self, "_graph", None) is not None:
+            return self._replay(input_ids, pos_id)
+        globs = self.schedule.globs
+        if not self.skip_rest:
+            self._place(input_ids, int(pos_id))
+        else:
+            globs.slot, globs.pos_id = self.slot, int(pos_id)
+        if not self.skip_mk:
+            self.last_call = self.interpreter.interpret(globs)
+        return input_ids if self.skip_rest else globs.argmax_out.to(torch.long)
+
+    def enable_cuda_graph(self, warmup_pos: int = 0):
+        """Capture one decode step of the current slot; token and position come from device words."""
+        globs = self.schedule.globs
+        self.last_call = self.interpreter.bind(globs)
+        self.last_call._schedule()  # validates the schedule, which copies from the device
+        globs.slot = self.slot
+        globs.pos_id_device = torch.full((1,), warmup_pos, dtype=torch.int32, device=globs.device)
+        self._graph_out = torch.zeros(1, dtype=torch.long, device=globs.device)
+        self.interpreter.module.sync_status(self.last_call)
+        self._graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(self._graph):
+            self.interpreter.interpret(globs)
+            self._graph_out.copy_(globs.argmax_out)
+        return self
+
+    def disable_cuda_graph(self):
+        self._graph = None
+        self.schedule.globs.pos_id_device = None
+
+    def _replay(self, input_ids: Tensor, pos_id: int):
+        globs = self.schedule.globs
+        globs.tokens[:1].copy_(input_ids.reshape(-1), non_blocking=True)
+        globs.pos_id_device.fill_(int(pos_id))
+        self._graph.replay()
+        return self._graph_out
+
+    def feed(self, tokens, position: int, want: list[int], layers_out: list | None = None) -> Tensor:
+        """``step`` without the final synchronisation; any number of tokens, any cut."""
+        globs, model = self.schedule.globs, self.model
+        ids = torch.as_tensor(tokens).reshape(-1)
+        if position + ids.numel() > model.max_len():
+            raise ValueError(f"position {position + ids.numel() - 1} of {model.max_len()}")
+        V = model.config.vocab_size
+        out = torch.empty(len(want), V, device=globs.device, dtype=torch.float32)
+        n = globs.portion
+        for a in range(0, ids.numel(), n):
+            part = ids[a : a + n]
+            here = [(k, w - a) for k, w in enumerate(want) if a <= w < a + n]
+            count = self._place(part, position + a)
+            if count == 1 and layers_out is None and not getattr(self, "_graph", None):
+                self.last_call = self.interpreter.interpret(globs)
+                for k, _ in here:
+                    out[k] = globs.logits
+                continue
+            logits = None
+            if here:
+                globs.want_rows[: len(here)].copy_(torch.tensor([w for _, w in here], dtype=torch.int32))
+                logits = torch.empty(len(here), V, device=globs.device, dtype=torch.float32)
+            trace = None
+            if layers_out is not None:
+                trace = torch.empty(len(model.layers), count, model.config.width, device=globs.device)
+                layers_out.append(trace)
+            self.last_call = self.interpreter.prefill(globs, count, len(here), logits, trace)
+            if here:
+                out[[k for k, _ in here]] = logits
+        return out
+
+    def step(self, tokens: list[int], position: int, want: list[int], slot: int = 0) -> Tensor:
+        self.slot = slot
+        out = self.feed(tokens, position, want)
+        self.check()
+        return out
+
+    def prefill(self, prompt_ids: Tensor) -> Tensor:
+        """Run a prompt from position 0; returns the first generated token ``[1]``."""
+        n = prompt_ids.numel()
+        return self.feed(prompt_ids, 0, [n - 1]).argmax(dim=-1)
 
 
 class TP_MK_Generator(MK_Generator):

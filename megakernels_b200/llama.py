@@ -26,6 +26,7 @@ import torch
 from torch import Tensor
 
 from megakernels_b200.model_types import BatchState, DeviceType, ExtraModelConfig
+from megakernels_b200.state import SlotPool
 
 
 # --------------------------------------------------------------------------- #
@@ -235,6 +236,8 @@ def compute_shard_bounds(dim_size: int, num_shards: int, shard_index: int) -> sl
 class LlamaForCausalLM:
     """Weights, KV cache and RoPE tables in the layout the megakernel reads."""
 
+    setting = "latency"  # schedule builder, interpreter and generator (dispatch.py)
+
     def __init__(
         self,
         config: LlamaConfig,
@@ -289,6 +292,10 @@ class LlamaForCausalLM:
         )
         k_cache = torch.zeros(shape, device=self.device, dtype=self.dtype)
         self.stacked_kv_cache = (k_cache, torch.zeros_like(k_cache))
+        self.slots = SlotPool(1)  # a single-sequence launch always decodes slot 0 of the cache
+
+    def max_len(self) -> int:
+        return self.kv_len()
 
     # -- construction ----------------------------------------------------- #
     @classmethod

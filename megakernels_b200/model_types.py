@@ -47,3 +47,4 @@ class ExtraModelConfig:
     interleave_rope: bool = False
     max_len_override: int | None = None
     max_batch_size: int = 1
+    prefill_portion: int = 2048  # most tokens of one prefill call (layer-list models)

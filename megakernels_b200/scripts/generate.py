@@ -4,8 +4,8 @@ Same ``key=value`` command line and timing method as the reference script
 (megakernels/scripts/generate.py:28-207): CUDA events around a whole
 generation of ``ntok - 1`` tokens, ``num_warmup`` + ``num_iters`` repeats.
 Differences: ``model=`` names an architecture preset (``llama-1b``,
-``llama-8b``, ``llama-70b``) initialised from ``seed=`` or a local checkpoint
-directory, and the prompt is a list of token ids (``prompt_ids=1,2,3`` or
+``llama-8b``, ``llama-70b``, ``torirax-1b``, ``torirax-8b``) initialised from
+``seed=`` or a local checkpoint directory of either family (``registry.py``), and the prompt is a list of token ids (``prompt_ids=1,2,3`` or
 ``prompt_len=32`` random ids) because no tokenizer ships with this package.
 Only ``mode=mk`` exists here.
 """
@@ -19,24 +19,13 @@ from pathlib import Path
 
 import torch
 
-from megakernels_b200.dispatch import make_mk_interpreter, make_schedule_builder
 from megakernels_b200.demos.latency.scheduler import (
     LatencyScheduleOptions,
     pick_num_attention_partitions,
 )
-from megakernels_b200.generators import MK_Generator
-from megakernels_b200.llama import LlamaConfig, LlamaForCausalLM
+from megakernels_b200.dispatch import BUILDER_MAP, make_generator
 from megakernels_b200.model_types import ExtraModelConfig
-from megakernels_b200.scheduler import assign_to_sms, tensorize_instructions
-
-PRESETS = {
-    "llama-1b": LlamaConfig.llama_3_2_1b,
-    "llama-8b": LlamaConfig.llama_3_1_8b,
-    "llama-70b": LlamaConfig.llama_3_1_70b,
-    "meta-llama/Llama-3.2-1B-Instruct": LlamaConfig.llama_3_2_1b,
-    "meta-llama/Llama-3.1-8B-Instruct": LlamaConfig.llama_3_1_8b,
-}
-
+from megakernels_b200.registry import family_of_preset, load_model
 
 @dataclass
 class ScriptConfig:
@@ -60,7 +49,8 @@ class ScriptConfig:
     skip_mk: bool = False
     skip_rest: bool = False
     sched: str = "rr"
-    setting: str = "latency"
+    setting: str = "latency"  # layer-list models bring their own ("hybrid")
+    dtype: str = "bfloat16"
     memory_fraction: float = 0.0
     attn_partitions: int = 0
     coalesce_o_proj: bool = False
@@ -73,6 +63,8 @@ class ScriptConfig:
                 "paths of the reference are CPU checkers under oracle/)"
             )
         assert self.interleave_rope, "interleave_rope must be True for mk mode"
+        if self.setting not in BUILDER_MAP:
+            raise SystemExit(f"unknown setting {self.setting!r}; available: {sorted(BUILDER_MAP)}")
         assert self.batch_size == 1, "the latency megakernel decodes one sequence"
 
     def once(self):
@@ -119,17 +111,22 @@ def main(config: ScriptConfig):
         max_len_override=config.max_len_override,
         max_batch_size=config.batch_size,
     )
-    if config.model in PRESETS:
+    dtype = getattr(torch, config.dtype)
+    family = family_of_preset(config.model)
+    if family is not None:
         overrides = {"num_hidden_layers": config.layers} if config.layers else {}
-        model = LlamaForCausalLM.from_random(
-            PRESETS[config.model](**overrides),
+        if overrides and family.name != "llama":
+            raise SystemExit("layers= applies to the llama presets")
+        model = family.model_class.from_random(
+            family.presets[config.model](**overrides),
             extra,
             device=config.device,
+            dtype=dtype,
             seed=config.seed,
             draw_on="device",
         )
     else:
-        model = LlamaForCausalLM.from_pretrained(Path(config.model), extra, device=config.device)
+        model = load_model(Path(config.model), extra, device=config.device, dtype=dtype)
 
     if config.prompt_ids:
         prompt = torch.tensor([int(t) for t in config.prompt_ids.split(",")], dtype=torch.long)
@@ -140,24 +137,21 @@ def main(config: ScriptConfig):
     prompt_len = prompt.numel()
     print(f"Input ids shape: {tuple(prompt.shape)}")
 
-    n_part = config.attn_partitions or pick_num_attention_partitions(
-        prompt_len, config.ntok, model.device, model.num_kv_heads()
-    )
-    options = LatencyScheduleOptions(
-        num_attention_partitions=n_part, coalesce_o_proj=config.coalesce_o_proj,
-        merge_in_last_partial=config.merge_in_last_partial,
-    )
-    schedule = make_schedule_builder(config.setting, options).build(model)
-    queues = assign_to_sms(
-        config.sched, schedule=schedule, memory_fraction=config.memory_fraction or None
-    )
-    tensorize_instructions(schedule.globs, queues)
-
-    interpreter = make_mk_interpreter(config.setting, Path(config.mk_dir) if config.mk_dir else None)
-    gen = MK_Generator(
+    options = None  # the setting's defaults
+    if model.setting == "latency":
+        n_part = config.attn_partitions or pick_num_attention_partitions(
+            prompt_len, config.ntok, model.device, model.num_kv_heads()
+        )
+        options = LatencyScheduleOptions(
+            num_attention_partitions=n_part, coalesce_o_proj=config.coalesce_o_proj,
+            merge_in_last_partial=config.merge_in_last_partial,
+        )
+    gen = make_generator(
         model,
-        interpreter,
-        schedule,
+        options,
+        sched=config.sched,
+        mk_dir=Path(config.mk_dir) if config.mk_dir else None,
+        memory_fraction=config.memory_fraction or None,
         barrier_fill_val=config.barrier_fill_val,
         skip_mk=config.skip_mk,
         skip_rest=config.skip_rest,
