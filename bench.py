@@ -85,6 +85,9 @@ def parse_args():
     ap.add_argument("--batch", type=int, default=1,
                     help="independent sequences decoded per launch (2..8: the batched kernel; 9..64: its tcgen05 "
                          "build; each sequence gets a seeded random KV length in [256, 4096] unless --prefill is given)")
+    ap.add_argument("--layer-list", default="", choices=["", "torirax-1b", "torirax-8b"],
+                    help="instead of the llama workload: prefill and decode of a layer-list model, beside the llama "
+                         "preset of its width (one GPU)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true")
     ap.add_argument("--no-e2e", action="store_true")
@@ -754,7 +757,15 @@ def log(msg: str):
 
 def main():
     args = parse_args()
-    if args.impl == "reference":
+    if args.layer_list:
+        from megakernels_b200.scripts import bench_layers
+
+        peaks = {"hbm_gbs": FALLBACK_HBM_GBS, "bf16_tflops_sustained": 1400.0}
+        path = ROOT / "MEASURED_PEAKS.json"
+        if path.exists():
+            peaks.update({k: v for k, v in json.loads(path.read_text()).items() if k in peaks})
+        bench_layers.run(args, ClockSampler, peaks)
+    elif args.impl == "reference":
         run_reference_arm(args)
     else:
         run_ours(args)

@@ -56,7 +56,7 @@ enum MkbhOpcode {
 #define MKBH_FLAG_RECORD_TIMINGS 1u
 
 /* Matrices are row-major [out, in] in the model dtype with `in` padded with zeros to a multiple
- * of 8 elements; vectors, biases and the low-rank decay factor are float. */
+ * of 8 elements; vectors and biases are float. */
 typedef struct MkbhLayer {
     int32_t mixer;             /* MkbhMixer */
     int32_t heads, kv_heads;   /* delta rule: heads only */
@@ -74,12 +74,12 @@ typedef struct MkbhLayer {
     const void *in_w, *out_w, *up_w, *down_w;
     const float *in_bias;      /* [in_rows] or NULL */
     const float *norm1, *norm2, *ls1, *ls2;
-    const float *decay_w2;     /* [heads*dim, rank] */
+    const void *decay_w2;      /* [heads*dim, rank], model dtype, not padded */
     const float *decay_w0;     /* [heads*dim] */
     const float *out_norm;     /* [heads*dim] */
     void *k_cache;             /* [slots, cache_keep + cache_ring, kv_heads, 2, dim] */
     void *v_cache;             /* [slots, cache_keep + cache_ring, kv_heads, vdim] */
-    float *state;              /* [slots, heads, dim (key channel), dim (value channel)] */
+    float *state;              /* [slots, heads, dim (value channel), dim (key channel)] */
 } MkbhLayer;
 
 typedef struct MkbhGlobals {
@@ -118,10 +118,10 @@ typedef struct MkbhGlobals {
     int32_t max_splits, part_vdim; /* largest split count and vdim of any attention layer */
 
     /* activations: x [rows, width]; proj [rows, max in_rows, ff]; act [rows, ld] in the model dtype;
-     * mixed [rows, max heads*dim] float; decay the same */
+     * mixed [rows, widest mixer output]; decay [rows, max of heads*dim + 2*heads of a recurrence] */
     float *x, *proj, *mixed, *decay;
     void *act;
-    int64_t x_elems, proj_elems, mixed_elems, act_elems; /* capacities, checked before launching */
+    int64_t x_elems, proj_elems, mixed_elems, act_elems, decay_elems; /* capacities, checked before launching */
     int32_t portion_capacity;
 
     uint32_t flags;

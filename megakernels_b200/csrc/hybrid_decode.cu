@@ -11,8 +11,11 @@
 //     activations stay in registers for the whole instruction;
 //   * every output row has exactly one owner, which also adds it to the 32-bit residual stream: no
 //     atomics on data, bit-identical results from run to run;
-//   * whatever does not depend on the token (recurrent state, older keys and values, low-rank decay
-//     factors) is fetched before an instruction waits for its producers;
+//   * an operand warp runs one instruction ahead: it fetches the next instruction's words, its layer
+//     descriptor and its vectors (norm weights, layer scales, biases, decay factors) into shared
+//     memory, so that no pointer or vector is chased through HBM on the critical path;
+//   * what else does not depend on the token (recurrent state, older keys and values) is fetched
+//     before an instruction waits for its producers;
 //   * every wait is bounded and reports into the status record.
 #include "hybrid_kernels.h"
 
@@ -34,62 +37,72 @@ using mkb::smem_u32;
 
 constexpr int kConsumerWarps = 16;
 constexpr int kConsumers = kConsumerWarps * 32;
-constexpr int kBlock = kConsumers + 32;
+constexpr int kOperandWarp = kConsumerWarps + 1;  // (warp 16 is the loader)
+constexpr int kBlock = kConsumers + 64;
 constexpr int kStage = 32768;
 constexpr int kMaxStages = 6;
 constexpr int kPartFloats = 4096;      // per-row, per-column-group partial sums of an instruction
+constexpr int kMaxRows = 512;          // output rows of an instruction
+static_assert(kPartFloats * 4 <= 40 * 1024, "");
 constexpr int kScratchMin = 40 * 1024; // activation / mixer scratch, at least
+constexpr int kRowVecBytes = kMaxRows * 4 + 32;
 constexpr int kSmemLimit = 226 * 1024;
-constexpr int kMaxStateRows = 16;      // key channels of one column a thread carries (DELTA_STEP)
-constexpr int kMaxAcc = 16;            // outputs a thread carries (ATTENTION)
+constexpr int kMaxChannels = 8;        // key channels of one column a lane carries (dim <= 256)
 
 struct Params {
     MkbhGlobals g;
-    int stages, act_bytes;
+    int stages, act_bytes, vec_bytes;
     int attn_chunk;        // keys staged at a time
-    int l2_window;         // stages the loader may prefetch into L2 beyond the ring
+    int l2_window;         // stages the loader may prefetch into L2, ring included
     unsigned long long timeout_ns;
 };
 
+// What the operand warp prepares for one instruction.
+struct Desc {
+    int op, layer, a0, a1, a2;
+    int wait_idx, wait_thr;   // phase counter to wait for (index -1: none)
+    int arrive_idx, arrive_thr;
+    int row_bytes, per_stage, groups;
+    int has_vec, vec_off, row_off;  // vector operands: present, byte offsets inside their buffers
+    int pad;
+    MkbhLayer L;
+};
+static_assert(sizeof(MkbhLayer) % 8 == 0, "");
+constexpr int kDescBytes = (sizeof(Desc) + 127) & ~127;
+
+enum Bar { kDescFull = 0, kDescEmpty = 2, kVecFull = 4, kVecEmpty = 5, kRing = 6 };
+
 struct Smem {  // byte offsets from the 128-byte aligned base
-    int act, part, red, bars, ctl, total;
-    __host__ __device__ Smem(int stages, int act_bytes) {
-        act = stages * kStage;
-        part = act + act_bytes;
-        red = part + kPartFloats * 4;
-        bars = red + 128 * 4;
-        ctl = bars + 2 * kMaxStages * 8;
+    int act, vec, rows, desc, red, bars, ctl, total;
+    __host__ __device__ Smem(int stages, int act_bytes, int vec_bytes) {
+        act = stages * kStage;          // activations; partial sums once they are in registers
+        vec = act + act_bytes;          // norm weights / decay factor
+        rows = vec + vec_bytes;         // two slots: per-row vectors (bias, layer scale, decay bias)
+        desc = rows + 2 * kRowVecBytes;
+        red = (desc + 2 * kDescBytes + 127) & ~127;
+        bars = red + 2 * 3 * kConsumerWarps * 4;
+        ctl = bars + (kRing + 2 * kMaxStages) * 8;
         total = ctl + 16 * 4;
     }
 };
 
-struct Ctx {
-    const Params* p;
-    const MkbhGlobals* g;
-    uint32_t base;       // shared-window address
-    float *act, *part, *red;
-    uint32_t bars;
-    volatile int* ctl;   // [0] CTA abort, [1] last-arriver verdict, [2] agreed abort
-    int instr, opcode, pos;
-    uint32_t slot, phase;  // consumer view of the ring
-    __device__ uint32_t full(int s) const { return bars + s * 8; }
-    __device__ uint32_t empty(int s) const { return bars + (kMaxStages + s) * 8; }
+struct Cta {  // small and passed by reference to inlined code only: stays in registers
+    uint32_t base, bars;
+    uint8_t* gb;
+    volatile int* ctl;  // [0] CTA abort, [1] last-arriver verdict, [2], [3] agreed abort
+    int instr, opcode, pos, turn;
+    __device__ __forceinline__ uint32_t bar(int i) const { return bars + i * 8; }
+    __device__ __forceinline__ uint32_t full(int s) const { return bars + (kRing + s) * 8; }
+    __device__ __forceinline__ uint32_t empty(int s) const { return bars + (kRing + kMaxStages + s) * 8; }
 };
 
 __device__ __forceinline__ void csync() { asm volatile("bar.sync 1, %0;" ::"n"(kConsumers) : "memory"); }
 
-__device__ __forceinline__ void rec(const Ctx& c, int slot) {
-    if (c.g->timings != nullptr && threadIdx.x == 0)
-        c.g->timings[((size_t)blockIdx.x * c.g->queue_len + c.instr) * MKBH_TIMING_SLOTS + slot] =
-            (int)(uint32_t)globaltimer_ns();
-}
-
-__device__ __noinline__ void report(const Ctx& c, int code, int role, int d0, int d1, int d2) {
-    int* st = c.g->status;
+__device__ __noinline__ void report(int* st, volatile int* ctl, int code, int role, int instr, int op, int d0, int d1, int d2) {
     if (atomicCAS(&st[0], 0, code) == 0) {
         st[1] = blockIdx.x;
-        st[2] = c.instr;
-        st[3] = c.opcode;
+        st[2] = instr;
+        st[3] = op;
         st[4] = role;
         st[5] = d0;
         st[6] = d1;
@@ -97,75 +110,64 @@ __device__ __noinline__ void report(const Ctx& c, int code, int role, int d0, in
         __threadfence();
     }
     atomicExch(&st[15], 1);
-    c.ctl[0] = 1;
-}
-__device__ __forceinline__ bool global_abort(const Ctx& c) {
-    return *reinterpret_cast<volatile int*>(&c.g->status[15]) != 0;
+    ctl[0] = 1;
 }
 
-__device__ __noinline__ bool bar_wait_slow(const Ctx& c, uint32_t bar, uint32_t parity, int role, bool honour_abort) {
+__device__ __noinline__ bool bar_wait_slow(uint32_t bar, uint32_t parity, volatile int* ctl, int* status,
+                                           unsigned long long timeout_ns, int role, int instr, int op, bool honour_abort) {
     const unsigned long long t0 = globaltimer_ns();
     for (uint32_t spins = 1;; ++spins) {
         if (mbar_try_wait(bar, parity)) return true;
         if ((spins & 63u) == 0) {
-            if (honour_abort && c.ctl[0]) return false;
-            if (globaltimer_ns() - t0 > c.p->timeout_ns) {
-                report(c, MKBH_ERR_DEVICE_TIMEOUT, role, -1, 0, 0);
+            if (honour_abort && ctl[0]) return false;
+            if (globaltimer_ns() - t0 > timeout_ns) {
+                report(status, ctl, MKBH_ERR_DEVICE_TIMEOUT, role, instr, op, -1, 0, 0);
                 return false;
             }
         }
     }
 }
-
-__device__ __forceinline__ int* counter(const Ctx& c, int layer, int op) {
-    return c.g->counters + 2 + layer * MKBH_BARRIERS_PER_LAYER + op;
-}
-__device__ __forceinline__ int threshold(const Ctx& c, int layer, int op) {
-    return __ldg(c.g->arrivals + layer * MKBH_BARRIERS_PER_LAYER + op);
+__device__ __forceinline__ bool bar_wait(const Params& p, const Cta& c, uint32_t bar, uint32_t parity, int role,
+                                         bool honour_abort = true) {
+    return mbar_try_wait(bar, parity) ||
+           bar_wait_slow(bar, parity, c.ctl, p.g.status, p.timeout_ns, role, c.instr, c.opcode, honour_abort);
 }
 
-// One consumer thread's view of the abort word for all of them (the loader may set it at any time):
-// true if they go on together.
-__device__ __forceinline__ bool agree(const Ctx& c) {
-    if (threadIdx.x == 0) c.ctl[2] = c.ctl[0];
+// One consumer thread's view of the abort word for all of them (the loaders may set it at any
+// time): true if they go on together.
+__device__ __forceinline__ bool agree(Cta& c) {
+    // two words in turn: a slow thread may still read the previous verdict while the next is written
+    const int w = 2 + (c.turn++ & 1);
+    if (threadIdx.x == 0) c.ctl[w] = c.ctl[0];
     csync();
-    return c.ctl[2] == 0;
+    return c.ctl[w] == 0;
 }
 
-// All consumers: wait until phase `op` of `layer` is complete.  false (uniformly): aborting.
-__device__ bool wait_phase(const Ctx& c, int layer, int op) {
-    if (threadIdx.x == 0) {
-        const int* addr = counter(c, layer, op);
-        const int thr = threshold(c, layer, op);
-        unsigned long long t0 = 0;
-        uint32_t spins = 0;
-        while (ld_acquire_gpu(addr) < thr) {
-            if ((++spins & 63u) == 0) {
-                if (c.ctl[0]) break;
-                if (global_abort(c)) {
-                    c.ctl[0] = 1;
-                    break;
-                }
-                const unsigned long long now = globaltimer_ns();
-                if (t0 == 0) t0 = now;
-                else if (now - t0 > c.p->timeout_ns) {
-                    report(c, MKBH_ERR_DEVICE_TIMEOUT, 1, layer, op, ld_acquire_gpu(addr));
-                    break;
-                }
+__device__ __noinline__ void poll_counter(const int* addr, int thr, volatile int* ctl, int* status,
+                                          unsigned long long timeout_ns, int instr, int op) {
+    unsigned long long t0 = 0;
+    uint32_t spins = 0;
+    while (ld_acquire_gpu(addr) < thr) {
+        if ((++spins & 63u) == 0) {
+            if (ctl[0]) return;
+            if (*reinterpret_cast<volatile int*>(&status[15])) {
+                ctl[0] = 1;
+                return;
+            }
+            const unsigned long long now = globaltimer_ns();
+            if (t0 == 0) t0 = now;
+            else if (now - t0 > timeout_ns) {
+                report(status, ctl, MKBH_ERR_DEVICE_TIMEOUT, 1, instr, op, thr, ld_acquire_gpu(addr), 0);
+                return;
             }
         }
+        __nanosleep(20);
     }
-    return agree(c);
 }
-// All consumers, after their global writes: announce one arrival.
-__device__ __forceinline__ void signal_phase(const Ctx& c, int layer, int op) {
-    csync();
-    if (threadIdx.x == 0) red_release_gpu_add(counter(c, layer, op), 1);
-}
-// Phase that completes the residual stream a layer reads.
-__device__ __forceinline__ int last_phase(const MkbhLayer& L) { return L.ff ? MKBH_OP_DOWN : MKBH_OP_OUT_PROJ; }
 
-// ---- the weight stream ------------------------------------------------------------------- //
+__device__ __forceinline__ int phase_index(int layer, int op) { return layer * MKBH_BARRIERS_PER_LAYER + op; }
+
+// ---- loader: the weight stream ----------------------------------------------------------- //
 struct Block {  // rows [r0, r1) of a matrix of `row_bytes` rows
     const uint8_t* w;
     int r0, r1, row_bytes;
@@ -194,7 +196,7 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, const int* w,
 
 template <typename T>
 struct Cursor {  // the queue's weight blocks as a flat sequence of stages
-    int i = 0, row = 0;
+    int i = 0, row = 0, per = 1;
     bool open = false;
     Block b;
     __device__ bool next(const MkbhGlobals& g, const int* queue, const uint8_t*& src, uint32_t& bytes) {
@@ -203,11 +205,12 @@ struct Cursor {  // the queue's weight blocks as a flat sequence of stages
             if (weight_block<T>(g, queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION, b) && b.r1 > b.r0) {
                 open = true;
                 row = b.r0;
+                per = kStage / b.row_bytes;
             } else {
                 ++i;
             }
         }
-        const int n = min(kStage / b.row_bytes, b.r1 - row);
+        const int n = min(per, b.r1 - row);
         src = b.w + (size_t)row * b.row_bytes;
         bytes = (uint32_t)(n * b.row_bytes);
         row += n;
@@ -220,8 +223,8 @@ struct Cursor {  // the queue's weight blocks as a flat sequence of stages
 };
 
 template <typename T>
-__device__ void loader_main(Ctx& c) {
-    const MkbhGlobals& g = *c.g;
+__device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
+    const MkbhGlobals& g = p.g;
     const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
     const uint64_t policy = mkb::l2_policy_evict_first();
     Cursor<T> cur, pre;
@@ -229,7 +232,7 @@ __device__ void loader_main(Ctx& c) {
     const uint8_t* src;
     uint32_t bytes;
     bool more = true;
-    const int S = c.p->stages;
+    const int S = p.stages;
     while (cur.next(g, queue, src, bytes)) {
         const int slot = issued % S;
         const uint32_t parity = ((issued / S) & 1u) ^ 1u;
@@ -239,29 +242,150 @@ __device__ void loader_main(Ctx& c) {
             more = pre.next(g, queue, s2, b2);
             ++ahead;
         }
+        bool ok = true;
         while (!mbar_try_wait(c.empty(slot), parity)) {
-            if (more && ahead < issued + (uint32_t)c.p->l2_window) {
+            if (more && ahead < issued + (uint32_t)p.l2_window) {
                 const uint8_t* s2;
                 uint32_t b2;
                 more = pre.next(g, queue, s2, b2);
-                if (more)
-                    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(s2), "r"(b2) : "memory");
+                if (more) asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(s2), "r"(b2) : "memory");
                 ++ahead;
                 continue;
             }
-            if (!bar_wait_slow(c, c.empty(slot), parity, 0, true)) goto drain;
+            ok = bar_wait(p, c, c.empty(slot), parity, 0);
             break;
         }
+        if (!ok) break;
         mbar_expect_tx(c.full(slot), bytes);
         mkb::tma_bulk_g2s(c.base + slot * kStage, src, bytes, c.full(slot), policy);
         ++issued;
     }
-drain:  // no copy may be in flight when the CTA's shared memory goes away
+    // no copy may be in flight when the CTA's shared memory goes away
     for (uint32_t s = issued > (uint32_t)S ? issued - S : 0u; s < issued; ++s)
-        if (!mbar_try_wait(c.full(s % S), (s / S) & 1u)) bar_wait_slow(c, c.full(s % S), (s / S) & 1u, 0, false);
+        bar_wait(p, c, c.full(s % S), (s / S) & 1u, 0, false);
 }
 
-// ---- matrix-vector products ---------------------------------------------------------------- //
+// ---- operand warp ------------------------------------------------------------------------- //
+// Column groups of an input of `chunks` 16-byte chunks: warps that share a row.
+__host__ __device__ inline int column_groups(int chunks) {
+    int n = 1;
+    while (n < kConsumerWarps && n * 32 < chunks) n *= 2;
+    return n;
+}
+// Phase that completes the residual stream a layer leaves.
+__device__ __forceinline__ int last_phase(int ff) { return ff ? MKBH_OP_DOWN : MKBH_OP_OUT_PROJ; }
+
+__device__ __forceinline__ void copy_vec(uint32_t dst, const void* src, int bytes, uint32_t bar, uint64_t policy) {
+    const uint64_t a = reinterpret_cast<uint64_t>(src) & ~15ull, e = (reinterpret_cast<uint64_t>(src) + bytes + 15) & ~15ull;
+    mkb::tma_bulk_g2s(dst, reinterpret_cast<const void*>(a), (uint32_t)(e - a), bar, policy);
+}
+__device__ __forceinline__ uint32_t vec_span(const void* src, int bytes) {
+    const uint64_t a = reinterpret_cast<uint64_t>(src);
+    return (uint32_t)(((a + bytes + 15) & ~15ull) - (a & ~15ull));
+}
+
+template <typename T>
+__device__ __forceinline__ void operand_main(const Params& p, Cta& c, const Smem& sm) {
+    const MkbhGlobals& g = p.g;
+    const int lane = threadIdx.x & 31;
+    const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
+    const uint64_t policy = mkb::l2_policy_evict_first();
+    uint32_t vecs = 0;  // vector operands issued
+    int done = 0;       // descriptors published
+    bool ok = true;
+    for (int i = 0; i < g.queue_len && ok; ++i) {
+        const int slot = i & 1;
+        Desc* d = reinterpret_cast<Desc*>(c.gb + sm.desc + slot * kDescBytes);
+        const int w = lane < 5 ? __ldg(queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION + lane) : 0;
+        const int op = __shfl_sync(0xffffffffu, w, 0), layer = __shfl_sync(0xffffffffu, w, 1);
+        c.instr = i;
+        c.opcode = op;
+        int flag = 1;
+        if (lane == 0) flag = bar_wait(p, c, c.bar(kDescEmpty + slot), ((i >> 1) & 1u) ^ 1u, 2);
+        ok = __shfl_sync(0xffffffffu, flag, 0) != 0;
+        if (!ok) break;
+        if (lane < 5) (&d->op)[lane] = w;
+        const uint2* src = reinterpret_cast<const uint2*>(g.layers_device + layer);
+        for (int k = lane; k < (int)sizeof(MkbhLayer) / 8; k += 32) reinterpret_cast<uint2*>(&d->L)[k] = __ldg(src + k);
+        __syncwarp();
+        const void *vec = nullptr, *rows = nullptr;
+        int vec_n = 0, row_n = 0, K = 0;
+        if (lane == 0) {
+            const MkbhLayer& L = d->L;
+            const bool delta = L.mixer == MKBH_DELTA_RULE;
+            int wl = layer, wop = 0;
+            switch (op) {
+                case MKBH_OP_NORM_PROJ:
+                    K = g.width; vec = L.norm1; vec_n = K * 4; rows = L.in_bias;
+                    wl = layer - 1;
+                    wop = layer > 0 ? last_phase(__ldg(&g.layers_device[layer - 1].ff)) : -1;
+                    break;
+                case MKBH_OP_DELTA_STEP:
+                    vec = (const uint8_t*)L.decay_w2 + (size_t)d->a0 * L.dim * L.rank * sizeof(T);
+                    vec_n = L.dim * L.rank * (int)sizeof(T);
+                    rows = L.decay_w0 + d->a0 * L.dim;
+                    row_n = L.dim * 4;
+                    wop = MKBH_OP_NORM_PROJ;
+                    break;
+                case MKBH_OP_ATTENTION: wop = MKBH_OP_NORM_PROJ; break;
+                case MKBH_OP_OUT_PROJ:
+                    K = L.heads * (delta ? L.dim : L.vdim);
+                    rows = L.ls1;
+                    if (delta) vec = L.out_norm, vec_n = K * 4;
+                    wop = delta ? MKBH_OP_DELTA_STEP : MKBH_OP_ATTENTION;
+                    break;
+                case MKBH_OP_NORM_UP: K = g.width; vec = L.norm2; vec_n = K * 4; wop = MKBH_OP_OUT_PROJ; break;
+                case MKBH_OP_DOWN: K = L.ff; rows = L.ls2; wop = MKBH_OP_NORM_UP; break;
+                case MKBH_OP_HEAD:
+                    K = g.width; vec = g.final_norm; vec_n = K * 4;
+                    wl = g.num_layers - 1;
+                    wop = last_phase(__ldg(&g.layers_device[wl].ff));
+                    break;
+                default: wop = -1; break;
+            }
+            if (K > 0 && rows != nullptr) {
+                rows = (const float*)rows + d->a0;
+                row_n = (d->a1 - d->a0) * 4;
+            }
+            d->wait_idx = wop < 0 ? -1 : phase_index(wl, wop);
+            d->wait_thr = wop < 0 ? 0 : __ldg(g.arrivals + phase_index(wl, wop));
+            d->arrive_idx = phase_index(op == MKBH_OP_HEAD ? g.num_layers : layer, op);
+            d->arrive_thr = op == MKBH_OP_HEAD ? __ldg(g.arrivals + d->arrive_idx) : 0;
+            d->row_bytes = pad8(K) * (int)sizeof(T);
+            d->per_stage = K > 0 ? kStage / d->row_bytes : 0;
+            d->groups = column_groups(d->row_bytes / 16);
+            d->has_vec = vec != nullptr;
+            d->vec_off = (int)(reinterpret_cast<uint64_t>(vec) & 15);
+            d->row_off = rows != nullptr && row_n > 0 ? (int)(reinterpret_cast<uint64_t>(rows) & 15) : -1;
+        }
+        __syncwarp();
+        if (lane == 0) {
+            const uint32_t full = c.bar(kDescFull + slot);
+            if (d->row_off >= 0) {
+                mbar_expect_tx(full, vec_span(rows, row_n));
+                copy_vec(c.base + sm.rows + slot * kRowVecBytes, rows, row_n, full, policy);
+            } else {
+                mbar_arrive(full);
+            }
+            if (vec != nullptr) {
+                flag = bar_wait(p, c, c.bar(kVecEmpty), (vecs & 1u) ^ 1u, 2);
+                if (flag) {
+                    mbar_expect_tx(c.bar(kVecFull), vec_span(vec, vec_n));
+                    copy_vec(c.base + sm.vec, vec, vec_n, c.bar(kVecFull), policy);
+                    ++vecs;
+                }
+            }
+        }
+        done = i + 1;
+        ok = __shfl_sync(0xffffffffu, flag, 0) != 0;
+    }
+    if (lane == 0) {  // nothing of it may be in flight at exit
+        for (int i = done > 2 ? done - 2 : 0; i < done; ++i) bar_wait(p, c, c.bar(kDescFull + (i & 1)), (i >> 1) & 1u, 2, false);
+        if (vecs > 0) bar_wait(p, c, c.bar(kVecFull), (vecs - 1) & 1u, 2, false);
+    }
+}
+
+// ---- consumers ------------------------------------------------------------------------------ //
 template <typename T> struct Chunk;  // 16 bytes of weights times the matching activations
 template <> struct Chunk<float> {
     static constexpr int kElems = 4;
@@ -276,30 +400,26 @@ template <> struct Chunk<bf16> {
     static constexpr int kElems = 8;
     __device__ static __forceinline__ float dot(const uint4& w, const float* a, float acc) {
         const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+        float acc2 = 0.f;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             acc = fmaf(mkb::bf16_lo(u[i]), a[2 * i], acc);
-            acc = fmaf(mkb::bf16_hi(u[i]), a[2 * i + 1], acc);
+            acc2 = fmaf(mkb::bf16_hi(u[i]), a[2 * i + 1], acc2);
         }
-        return acc;
+        return acc + acc2;
     }
 };
 
-// Column groups of an input of `chunks` 16-byte chunks: warps that share a row.
-__host__ __device__ inline int column_groups(int chunks) {
-    int n = 1;
-    while (n < kConsumerWarps && n * 32 < chunks) n *= 2;
-    return n;
-}
-
-// Multiply the instruction's rows with the activations in c.act; partial sums [row][group] to
-// c.part.  Ends with a consumer barrier.  false (uniformly): aborting.
+// Multiply the instruction's rows with the activations in `act` (fp32, zero beyond the matrix's
+// columns); partial sums [row][group] replace them.  Ends with a consumer barrier.
 template <typename T, int kPer>
-__device__ __noinline__ bool matvec_rows(Ctx& c, const Block& b, int groups) {
+__device__ __forceinline__ bool matvec_rows(const Params& p, Cta& c, const Desc& d, float* act, uint32_t& ring_slot,
+                                            uint32_t& ring_phase) {
     constexpr int E = Chunk<T>::kElems;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int cg = warp & (groups - 1), rg = warp / groups, nrg = kConsumerWarps / groups;
-    const int chunks = b.row_bytes / 16;
+    const int groups = d.groups, row_bytes = d.row_bytes, per_stage = d.per_stage, rows = d.a1 - d.a0;
+    const int cg = warp & (groups - 1), nrg = kConsumerWarps / groups, rg = warp / groups;
+    const int chunks = row_bytes / 16, S = p.stages;
     float a[kPer * E];
     uint32_t off[kPer];
 #pragma unroll
@@ -307,14 +427,20 @@ __device__ __noinline__ bool matvec_rows(Ctx& c, const Block& b, int groups) {
         const int ch = (k * groups + cg) * 32 + lane;
         off[k] = ch < chunks ? (uint32_t)ch * 16u : 0u;
 #pragma unroll
-        for (int e = 0; e < E; ++e) a[k * E + e] = ch < chunks ? c.act[ch * E + e] : 0.f;
+        for (int e = 0; e < E; e += 4) {
+            const float4 f = ch < chunks ? *reinterpret_cast<const float4*>(act + ch * E + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+            a[k * E + e] = f.x;
+            a[k * E + e + 1] = f.y;
+            a[k * E + e + 2] = f.z;
+            a[k * E + e + 3] = f.w;
+        }
     }
-    const int per_stage = kStage / b.row_bytes;
-    uint32_t slot = c.slot, phase = c.phase;
+    csync();  // everybody holds its activations: the buffer takes the partial sums
+    uint32_t slot = ring_slot, phase = ring_phase;
     bool ok = true;
-    for (int r0 = b.r0; r0 < b.r1; r0 += per_stage) {
-        const int n = min(per_stage, b.r1 - r0);
-        bool mine = mbar_try_wait(c.full(slot), phase) || bar_wait_slow(c, c.full(slot), phase, 1, true);
+    for (int r0 = 0; r0 < rows; r0 += per_stage) {
+        const int n = min(per_stage, rows - r0);
+        const bool mine = bar_wait(p, c, c.full(slot), phase, 1);
         if (!__all_sync(0xffffffffu, mine)) {
             ok = false;
             break;
@@ -324,13 +450,11 @@ __device__ __noinline__ bool matvec_rows(Ctx& c, const Block& b, int groups) {
             float v[4];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const int row = r + j * nrg;
+                const int row = min(r + j * nrg, n - 1);  // (a repeated row's sum is dropped below)
+                const uint32_t addr = stage + (uint32_t)row * (uint32_t)row_bytes;
                 v[j] = 0.f;
-                if (row < n) {  // uniform over the warp
-                    const uint32_t addr = stage + (uint32_t)row * (uint32_t)b.row_bytes;
 #pragma unroll
-                    for (int k = 0; k < kPer; ++k) v[j] = Chunk<T>::dot(lds_v4(addr + off[k]), a + k * E, v[j]);
-                }
+                for (int k = 0; k < kPer; ++k) v[j] = Chunk<T>::dot(lds_v4(addr + off[k]), a + k * E, v[j]);
             }
             // four sums over 32 lanes in six shuffles: lane quarter q ends up with row q
             const bool up = lane & 16, up2 = lane & 8;
@@ -343,239 +467,281 @@ __device__ __noinline__ bool matvec_rows(Ctx& c, const Block& b, int groups) {
             y += __shfl_xor_sync(0xffffffffu, y, 2);
             y += __shfl_xor_sync(0xffffffffu, y, 1);
             const int row = r + (lane >> 3) * nrg;
-            if ((lane & 7) == 0 && row < n) c.part[(r0 - b.r0 + row) * groups + cg] = y;
+            if ((lane & 7) == 0 && row < n) act[(r0 + row) * groups + cg] = y;
         }
         __syncwarp();
         if (lane == 0) mbar_arrive(c.empty(slot));
-        if (++slot == (uint32_t)c.p->stages) {
+        if (++slot == (uint32_t)S) {
             slot = 0;
             phase ^= 1u;
         }
     }
-    c.slot = slot;
-    c.phase = phase;
+    ring_slot = slot;
+    ring_phase = phase;
     if (!ok) c.ctl[0] = 1;
     csync();
     return agree(c);
 }
 
-template <typename T>
-__device__ __forceinline__ bool matvec(Ctx& c, const Block& b, int& groups) {
-    const int chunks = b.row_bytes / 16;
-    groups = column_groups(chunks);
-    if (chunks <= groups * 32) return matvec_rows<T, 1>(c, b, groups);
-    if (chunks <= groups * 64) return matvec_rows<T, 2>(c, b, groups);
-    return matvec_rows<T, 4>(c, b, groups);
-}
-__device__ __forceinline__ float row_sum(const Ctx& c, int i, int groups) {
-    float s = 0.f;
-    for (int k = 0; k < groups; ++k) s += c.part[i * groups + k];
-    return s;
-}
-
+// Totals over the consumers; `red` alternates between two buffers, so that one barrier suffices.
 template <int N>
-__device__ __forceinline__ void csum(const Ctx& c, float (&v)[N]) {  // totals over the consumers
+__device__ __forceinline__ void csum(float* red, int& turn, float (&v)[N]) {
+    float* r = red + (turn & 1) * 3 * kConsumerWarps;
+    ++turn;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #pragma unroll
     for (int n = 0; n < N; ++n) {
         v[n] = warp_sum(v[n]);
-        if (lane == 0) c.red[n * kConsumerWarps + warp] = v[n];
+        if (lane == 0) r[n * kConsumerWarps + warp] = v[n];
     }
     csync();
 #pragma unroll
     for (int n = 0; n < N; ++n) {
         float s = 0.f;
 #pragma unroll
-        for (int w = 0; w < kConsumerWarps; ++w) s += c.red[n * kConsumerWarps + w];
+        for (int w = 0; w < kConsumerWarps; w += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(r + n * kConsumerWarps + w);
+            s += (f.x + f.y) + (f.z + f.w);
+        }
         v[n] = s;
     }
-    csync();
 }
 
-// ---- activations ------------------------------------------------------------------------- //
+// A vector of K floats spread over the consumers, kSlots per thread: four neighbours at a time
+// where K allows 16-byte accesses, else one by one.
+template <int kSlots>
+struct Spread {
+    float v[kSlots];
+    bool wide;
+    int K;
+    __device__ __forceinline__ int index(int s) const {
+        return wide ? 4 * ((int)threadIdx.x + kConsumers * (s >> 2)) + (s & 3) : (int)threadIdx.x + kConsumers * s;
+    }
+    __device__ __forceinline__ bool has(int s) const { return index(s) < K; }
+    __device__ __forceinline__ void load_cg(const float* src) {
+        if (wide) {
+#pragma unroll
+            for (int s = 0; s < kSlots; s += 4) {
+                uint4 u = make_uint4(0, 0, 0, 0);
+                if (has(s)) u = mkb::ld_cg_v4(src + index(s));
+                v[s] = __uint_as_float(u.x);
+                v[s + 1] = __uint_as_float(u.y);
+                v[s + 2] = __uint_as_float(u.z);
+                v[s + 3] = __uint_as_float(u.w);
+            }
+        } else {
+#pragma unroll
+            for (int s = 0; s < kSlots; ++s) v[s] = has(s) ? ld_cg_f32(src + index(s)) : 0.f;
+        }
+    }
+    __device__ __forceinline__ void store(float* dst) const {
+        if (wide) {
+#pragma unroll
+            for (int s = 0; s < kSlots; s += 4)
+                if (has(s)) *reinterpret_cast<float4*>(dst + index(s)) = make_float4(v[s], v[s + 1], v[s + 2], v[s + 3]);
+        } else {
+#pragma unroll
+            for (int s = 0; s < kSlots; ++s)
+                if (has(s)) dst[index(s)] = v[s];
+        }
+        const int z = K + (int)threadIdx.x;  // padding columns
+        if (z < pad8(K)) dst[z] = 0.f;
+    }
+};
+
 // Layer norm of the residual stream (or of the token's embedding, which `publish` also writes out).
-template <typename T>
-__device__ __noinline__ void norm_activation(const Ctx& c, const float* w, bool embedding, bool publish) {
-    const MkbhGlobals& g = *c.g;
-    const int K = g.width, tid = threadIdx.x;
-    float s[1] = {0.f};
+template <typename T, int kSlots>
+__device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, const float* w, float* act, float* red,
+                                                int& turn, bool embedding, bool publish) {
+    const MkbhGlobals& g = p.g;
+    Spread<kSlots> x;
+    x.K = g.width;
+    x.wide = g.width % 4 == 0;
     if (embedding) {
         int tok = __ldg(g.tokens);
         tok = tok < 0 ? 0 : tok >= g.vocab ? g.vocab - 1 : tok;
-        const T* e = static_cast<const T*>(g.embed) + (size_t)tok * K;
-        const T* q = static_cast<const T*>(g.pos) + (size_t)c.pos * K;
-        for (int i = tid; i < K; i += kConsumers) {
-            const float x = to_f(e[i]) * g.embed_scale + to_f(q[i]);
-            c.act[i] = x;
-            if (publish) g.x[i] = x;
-            s[0] += x;
+        const T* e = static_cast<const T*>(g.embed) + (size_t)tok * x.K;
+        const T* q = static_cast<const T*>(g.pos) + (size_t)c.pos * x.K;
+#pragma unroll
+        for (int s = 0; s < kSlots; ++s) {
+            const int i = x.index(s);
+            x.v[s] = i < x.K ? to_f(e[i]) * g.embed_scale + to_f(q[i]) : 0.f;
+            if (publish && i < x.K) g.x[i] = x.v[s];
         }
     } else {
-#pragma unroll 4
-        for (int i = tid; i < K; i += kConsumers) {
-            const float x = ld_cg_f32(g.x + i);
-            c.act[i] = x;
-            s[0] += x;
-        }
+        x.load_cg(g.x);
     }
-    csum<1>(c, s);
-    const float mean = s[0] / K;
-    s[0] = 0.f;
-    for (int i = tid; i < K; i += kConsumers) {
-        const float d = c.act[i] - mean;
-        s[0] += d * d;
+    float sum[1] = {0.f};
+#pragma unroll
+    for (int s = 0; s < kSlots; ++s) sum[0] += x.v[s];
+    csum<1>(red, turn, sum);
+    const float mean = sum[0] / x.K;
+    sum[0] = 0.f;
+#pragma unroll
+    for (int s = 0; s < kSlots; ++s) {
+        x.v[s] = x.has(s) ? x.v[s] - mean : 0.f;
+        sum[0] = fmaf(x.v[s], x.v[s], sum[0]);
     }
-    csum<1>(c, s);
-    const float inv = 1.f / sqrtf(s[0] / K + g.eps);
-    for (int i = tid; i < K; i += kConsumers) c.act[i] = (c.act[i] - mean) * inv * __ldg(w + i);
-    for (int i = K + tid; i < pad8(K); i += kConsumers) c.act[i] = 0.f;
-    csync();
+    csum<1>(red, turn, sum);
+    const float inv = 1.f / sqrtf(sum[0] / x.K + g.eps);
+#pragma unroll
+    for (int s = 0; s < kSlots; ++s)
+        if (x.has(s)) x.v[s] *= inv * w[x.index(s)];
+    x.store(act);
+}
+
+template <int kSlots>
+__device__ __forceinline__ void poly_activation(const Params& p, const MkbhLayer& L, float* act, float* red, int& turn) {
+    Spread<kSlots> z;
+    z.K = L.ff;
+    z.wide = L.ff % 4 == 0;
+    z.load_cg(p.g.proj);
+    float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < kSlots; ++k) {
+        const float a = z.v[k] * z.v[k];
+        s[0] += a;
+        s[1] = fmaf(a, a, s[1]);
+        s[2] = fmaf(a * a, a, s[2]);
+    }
+    csum<3>(red, turn, s);
+    const float f1 = L.act[0] / sqrtf(s[0] / z.K + p.g.eps), f2 = L.act[1] / sqrtf(s[1] / z.K + p.g.eps),
+                f3 = L.act[2] / sqrtf(s[2] / z.K + p.g.eps), e = L.act[3];
+#pragma unroll
+    for (int k = 0; k < kSlots; ++k) z.v[k] = z.v[k] * (f1 + z.v[k] * (f2 + z.v[k] * f3)) + e;
+    z.store(act);
 }
 
 // Mixer output as the output projection reads it.
-__device__ __noinline__ void mixed_activation(const Ctx& c, const MkbhLayer& L) {
-    const MkbhGlobals& g = *c.g;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    int K;
-    if (L.mixer == MKBH_DELTA_RULE) {
-        K = L.heads * L.dim;
-        for (int h = warp; h < L.heads; h += kConsumerWarps) {
-            float s = 0.f;
-            for (int i = lane; i < L.dim; i += 32) {
-                const float o = ld_cg_f32(g.mixed + h * L.dim + i);
-                c.act[h * L.dim + i] = o;
-                s += o * o;
-            }
-            const float inv = 1.f / sqrtf(warp_sum(s) / L.dim + g.eps);
-            for (int i = lane; i < L.dim; i += 32) {
-                const int j = h * L.dim + i;
-                c.act[j] *= inv * __ldg(L.out_norm + j) * sigmoid_f(ld_cg_f32(g.proj + 4 * K + j));
+template <int kSlots>
+__device__ __forceinline__ void plain_activation(const float* src, int K, float* act) {
+    Spread<kSlots> v;
+    v.K = K;
+    v.wide = K % 4 == 0;
+    v.load_cg(src);
+    v.store(act);
+}
+__device__ __forceinline__ void delta_activation(const Params& p, const MkbhLayer& L, const float* w, float* act) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = L.dim, HD = L.heads * D;
+    const float *o = p.g.mixed, *gate = p.g.proj + 4 * HD;
+    for (int h0 = warp; h0 < L.heads; h0 += 2 * kConsumerWarps) {  // two heads in flight
+        float v[2][kMaxChannels], g[2][kMaxChannels], s[2] = {0.f, 0.f};
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+            const int h = h0 + b * kConsumerWarps;
+#pragma unroll
+            for (int j = 0; j < kMaxChannels; ++j) {
+                const int i = lane + 32 * j;
+                const bool live = h < L.heads && i < D;
+                v[b][j] = live ? ld_cg_f32(o + h * D + i) : 0.f;
+                g[b][j] = live ? ld_cg_f32(gate + h * D + i) : 0.f;
             }
         }
-    } else {
-        K = L.heads * L.vdim;
-        for (int i = tid; i < K; i += kConsumers) c.act[i] = ld_cg_f32(g.mixed + i);
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+            const int h = h0 + b * kConsumerWarps;
+            if (h >= L.heads) break;  // uniform over the warp
+#pragma unroll
+            for (int j = 0; j < kMaxChannels; ++j) s[b] = fmaf(v[b][j], v[b][j], s[b]);
+            const float inv = 1.f / sqrtf(warp_sum(s[b]) / D + p.g.eps);
+#pragma unroll
+            for (int j = 0; j < kMaxChannels; ++j) {
+                const int i = lane + 32 * j;
+                if (i < D) act[h * D + i] = v[b][j] * inv * w[h * D + i] * sigmoid_f(g[b][j]);
+            }
+        }
     }
-    for (int i = K + tid; i < pad8(K); i += kConsumers) c.act[i] = 0.f;
-    csync();
-}
-
-__device__ __noinline__ void poly_activation(const Ctx& c, const MkbhLayer& L) {
-    const MkbhGlobals& g = *c.g;
-    const int tid = threadIdx.x, K = L.ff;
-    float s[3] = {0.f, 0.f, 0.f};
-#pragma unroll 4
-    for (int i = tid; i < K; i += kConsumers) {
-        const float z = ld_cg_f32(g.proj + i), a = z * z;
-        c.act[i] = z;
-        s[0] += a;
-        s[1] += a * a;
-        s[2] += a * a * a;
-    }
-    csum<3>(c, s);
-    const float f1 = L.act[0] / sqrtf(s[0] / K + g.eps), f2 = L.act[1] / sqrtf(s[1] / K + g.eps),
-                f3 = L.act[2] / sqrtf(s[2] / K + g.eps), e = L.act[3];
-    for (int i = tid; i < K; i += kConsumers) {
-        const float z = c.act[i];
-        c.act[i] = z * (f1 + z * (f2 + z * f3)) + e;
-    }
-    for (int i = K + tid; i < pad8(K); i += kConsumers) c.act[i] = 0.f;
-    csync();
+    const int z = HD + (int)threadIdx.x;
+    if (z < pad8(HD)) act[z] = 0.f;
 }
 
 // ---- generalized delta rule: one step for a block of value columns of one head --------------- //
-__device__ __noinline__ bool delta_step(Ctx& c, const int* w) {
-    const MkbhGlobals& g = *c.g;
-    const int layer = __ldg(w + 1), head = __ldg(w + 2), col0 = __ldg(w + 3), cols = __ldg(w + 4) - col0;
-    const MkbhLayer& L = g.layers_device[layer];
-    const int D = L.dim, HD = L.heads * D, R = L.rank, tid = threadIdx.x;
-    const int parts = min(kMaxStateRows, kConsumers / cols);
-    const int col = tid % cols, part = tid / cols;
-    const bool live = part < parts;
-    float* state = L.state + ((size_t)g.slot * L.heads + head) * D * D + col0 + col;
-    float S[kMaxStateRows];
+// The state is stored column by column ([head][value column][key channel]): a warp carries one
+// column, lane l the channels l, l + 32, ...; both sums over the old state (for the removal and for
+// the output) are taken in one pass.
+struct StateCol {
+    float S[kMaxChannels];
+    __device__ __forceinline__ void load(const float* col, int D, bool live) {
+        const int lane = threadIdx.x & 31;
 #pragma unroll
-    for (int j = 0; j < kMaxStateRows; ++j) {
-        const int i = part + j * parts;
-        S[j] = (live && i < D && c.pos > 0) ? state[(size_t)i * D] : 0.f;
+        for (int j = 0; j < kMaxChannels; ++j) S[j] = live && lane + 32 * j < D ? col[lane + 32 * j] : 0.f;
     }
-    // scratch: w2 [D][R + 1], inner [R], r k a w rw ck [D] each, partial sums [2][parts][cols]
-    float* w2 = c.act;
-    float* inner = w2 + D * (R + 1);
-    float *vr = inner + R, *vk = vr + D, *va = vk + D, *vw = va + D, *vrw = vw + D, *vck = vrw + D, *ps = vck + D;
-    for (int i = tid; i < D * R; i += kConsumers)
-        w2[(i / R) * (R + 1) + i % R] = __ldg(L.decay_w2 + (size_t)head * D * R + i);
+};
 
-    if (!wait_phase(c, layer, MKBH_OP_NORM_PROJ)) return false;
-    rec(c, 1);
+template <typename T>
+__device__ __forceinline__ void delta_step(const Params& p, const Cta& c, const Desc& d, float* act, const uint8_t* vec,
+                                           const float* w0, StateCol& first) {
+    const MkbhGlobals& g = p.g;
+    const MkbhLayer& L = d.L;
+    const int D = L.dim, HD = L.heads * D, R = L.rank, head = d.a0, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    float *inner = act, *decay = act + ((R + 3) & ~3);
+    const T* w2 = reinterpret_cast<const T*>(vec);
+    float k[kMaxChannels], r[kMaxChannels], a[kMaxChannels];
+    const float* src = g.proj + head * D;
+#pragma unroll
+    for (int j = 0; j < kMaxChannels; ++j) {
+        const int i = lane + 32 * j;
+        const bool live = i < D;
+        r[j] = live ? ld_cg_f32(src + i) : 0.f;
+        k[j] = live ? ld_cg_f32(src + HD + i) : 0.f;
+        a[j] = live ? ld_cg_f32(src + 3 * HD + i) : 0.f;
+    }
+    float v = d.a1 + warp < d.a2 ? ld_cg_f32(src + 2 * HD + d.a1 + warp) : 0.f;
     for (int i = tid; i < R; i += kConsumers) inner[i] = tanhf(ld_cg_f32(g.proj + 5 * HD + i));
-    for (int i = tid; i < 3 * D; i += kConsumers) {
-        const int which = i / D, j = i % D;
-        const float x = ld_cg_f32(g.proj + (which == 2 ? 3 : which) * HD + head * D + j);
-        if (which == 2) va[j] = sigmoid_f(x);
-        else (which ? vk : vr)[j] = x;
-    }
-    const float v = live ? ld_cg_f32(g.proj + 2 * HD + head * D + col0 + col) : 0.f;
-    csync();
-    // decays: four threads per channel
-    for (int i = tid >> 2; i < D; i += kConsumers / 4) {  // uniform over the four threads
-        float s = 0.f;
-        for (int r = tid & 3; r < R; r += 4) s = fmaf(w2[i * (R + 1) + r], inner[r], s);
-        const unsigned m = 0xfu << (tid & 28);
-        s += __shfl_xor_sync(m, s, 1);
-        s += __shfl_xor_sync(m, s, 2);
-        if ((tid & 3) == 0) {
-            const float d = expf(-L.decay_scale * sigmoid_f(s + __ldg(L.decay_w0 + head * D + i)));
-            vw[i] = d;
-            vrw[i] = vr[i] * d;
-        }
-    }
-    // every warp: |k|^2, r . (a k), r . k
+    // |k|^2, r . (a k), r . k
     float kk = 0.f, rak = 0.f, rk = 0.f;
-    for (int i = tid & 31; i < D; i += 32) {
-        const float k = vk[i], x = vr[i] * k;
-        kk = fmaf(k, k, kk);
+#pragma unroll
+    for (int j = 0; j < kMaxChannels; ++j) {
+        const float x = r[j] * k[j];
+        a[j] = sigmoid_f(a[j]);
+        kk = fmaf(k[j], k[j], kk);
         rk += x;
-        rak = fmaf(x, va[i], rak);
+        rak = fmaf(x, a[j], rak);
     }
     kk = warp_sum(kk);
     rk = warp_sum(rk);
     rak = warp_sum(rak);
     const float inv = 1.f / (kk + L.unit_eps);
-    for (int i = tid; i < D; i += kConsumers) vck[i] = va[i] * vk[i] * inv;
     csync();
-    float q = 0.f, o = 0.f;
-#pragma unroll
-    for (int j = 0; j < kMaxStateRows; ++j) {
-        const int i = part + j * parts;
-        if (live && i < D) {
-            q = fmaf(vk[i], S[j], q);
-            o = fmaf(vrw[i], S[j], o);
+    // decays: four threads per channel, their turns skewed over the banks
+    for (int i0 = 0; i0 < D; i0 += kConsumers / 4) {
+        const int i = i0 + (tid >> 2);
+        float s = 0.f;
+        if (i < D) {
+            int q = ((tid & 3) + 4 * i) % R;
+            for (int n = tid & 3; n < R; n += 4) {
+                s = fmaf(to_f(w2[i * R + q]), inner[q], s);
+                q += 4;
+                if (q >= R) q -= R;
+            }
         }
-    }
-    if (live) {
-        ps[part * cols + col] = q;
-        ps[(parts + part) * cols + col] = o;
+        s += __shfl_xor_sync(0xffffffffu, s, 1);
+        s += __shfl_xor_sync(0xffffffffu, s, 2);
+        if (i < D && (tid & 3) == 0) decay[i] = expf(-L.decay_scale * sigmoid_f(s + w0[i]));
     }
     csync();
-    if (live) {
-        q = o = 0.f;
-        for (int k = 0; k < parts; ++k) {
-            q += ps[k * cols + col];
-            o += ps[(parts + k) * cols + col];
-        }
-        if (part == 0) g.mixed[head * D + col0 + col] = o - rak * inv * q + rk * v;
+    float w[kMaxChannels];
 #pragma unroll
-        for (int j = 0; j < kMaxStateRows; ++j) {
-            const int i = part + j * parts;
-            if (i < D) state[(size_t)i * D] = fmaf(vk[i], v, fmaf(-vck[i], q, vw[i] * S[j]));
+    for (int j = 0; j < kMaxChannels; ++j) w[j] = lane + 32 * j < D ? decay[lane + 32 * j] : 0.f;
+    for (int col = d.a1 + warp; col < d.a2; col += kConsumerWarps) {  // uniform over the warp
+        float* S0 = L.state + (((size_t)g.slot * L.heads + head) * D + col) * D;
+        if (col != d.a1 + warp) {
+            first.load(S0, D, c.pos > 0);
+            v = ld_cg_f32(src + 2 * HD + col);
         }
+        float q = 0.f, o = 0.f;
+#pragma unroll
+        for (int j = 0; j < kMaxChannels; ++j) {
+            q = fmaf(k[j], first.S[j], q);
+            o = fmaf(r[j] * w[j], first.S[j], o);
+        }
+        q = warp_sum(q);
+        o = warp_sum(o);
+        if (lane == 0) g.mixed[head * D + col] = o - rak * inv * q + rk * v;
+#pragma unroll
+        for (int j = 0; j < kMaxChannels; ++j)
+            if (lane + 32 * j < D) S0[lane + 32 * j] = fmaf(k[j], v - a[j] * inv * q, w[j] * first.S[j]);
     }
-    signal_phase(c, layer, MKBH_OP_DELTA_STEP);
-    return true;
-}
-__host__ __device__ inline int delta_scratch_floats(int dim, int rank) {
-    return dim * (rank + 1) + rank + 6 * dim + 2 * kConsumers;
 }
 
 // ---- windowed differential attention: one split of the keys of one KV head -------------------- //
@@ -600,133 +766,161 @@ template <typename T>
 __host__ __device__ inline int attn_scratch_bytes(int nq, int dim, int vdim, int chunk) {
     return AttnScratch(nq, dim, chunk).tile * 4 + chunk * (key_stride<T>(dim) + vdim * (int)sizeof(T)) + 16;
 }
+__host__ __device__ inline int merge_scratch_floats(int nq, int splits, int per, int vdim) {
+    return nq * splits + per * (vdim + 1);
+}
 
 template <typename T>
-__device__ __noinline__ bool attention_split(Ctx& c, const int* w) {
-    const MkbhGlobals& g = *c.g;
-    const int layer = __ldg(w + 1), kvh = __ldg(w + 2), split = __ldg(w + 3), splits = __ldg(w + 4);
-    const MkbhLayer& L = g.layers_device[layer];
-    const int D = L.dim, E = L.vdim, G = L.kv_heads, per = L.heads / G, nq = 2 * per;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, KC = c.p->attn_chunk;
-    const AttnScratch a(nq, D, KC);
-    float *q = c.act + a.q, *p = c.act + a.p, *m = c.act + a.m, *l = c.act + a.l, *f = c.act + a.f;
-    T* kt = reinterpret_cast<T*>(c.act + a.tile);
-    const int ks = key_stride<T>(D) / (int)sizeof(T);
-    T* vt = kt + (size_t)KC * ks;
-
-    const KeyRange keys(c.pos, L.window, L.keep_first);
-    const int t_lo = (int)((long long)keys.count * split / splits), t_hi = (int)((long long)keys.count * (split + 1) / splits);
-    const size_t rows0 = (size_t)g.slot * (L.cache_keep + L.cache_ring);
-    T* kc = static_cast<T*>(L.k_cache) + rows0 * G * 2 * D + (size_t)kvh * 2 * D;
-    T* vc = static_cast<T*>(L.v_cache) + rows0 * G * E + (size_t)kvh * E;
-    // Rows of older positions: they do not depend on this step (other layers' caches included).
-    auto stage_rows = [&](int c0, int nk) {
-        const bool wide = (2 * D * sizeof(T)) % 16 == 0 && (E * sizeof(T)) % 16 == 0;
-        const int unit = wide ? 16 / (int)sizeof(T) : 1;
-        const int kn = 2 * D / unit, vn = E / unit;
-        for (int i = tid; i < nk * (kn + vn); i += kConsumers) {
-            const int t = i / (kn + vn), o = i % (kn + vn), j = keys.key(t_lo + c0 + t);
-            if (j == c.pos) continue;
-            const size_t row = cache_row(j, L.cache_keep, L.cache_ring);
-            const T* src = o < kn ? kc + row * G * 2 * D + o * unit : vc + row * G * E + (o - kn) * unit;
-            T* dst = o < kn ? kt + t * ks + o * unit : vt + t * E + (o - kn) * unit;
-            if (wide) *reinterpret_cast<uint4*>(dst) = mkb::ld_cg_v4(src);
-            else *dst = __ldcg(src);
-        }
-    };
-    const int n0 = min(KC, t_hi - t_lo);
-    stage_rows(0, n0);
-    for (int i = tid; i < nq; i += kConsumers) {
-        m[i] = -INFINITY;
-        l[i] = 0.f;
+struct AttnView {
+    int D, E, G, per, nq, ks, t_lo, count, keep, ring, pos;
+    KeyRange keys;
+    T *kc, *vc, *kt, *vt;
+    float *q, *p, *m, *l, *f;
+    __device__ __forceinline__ AttnView(const Params& pr, const Cta& c, const Desc& d, float* act)
+        : keys(c.pos, d.L.window, d.L.keep_first) {
+        const MkbhLayer& L = d.L;
+        D = L.dim; E = L.vdim; G = L.kv_heads; per = L.heads / G; nq = 2 * per;
+        keep = L.cache_keep; ring = L.cache_ring; pos = c.pos;
+        const AttnScratch a(nq, D, pr.attn_chunk);
+        q = act + a.q; p = act + a.p; m = act + a.m; l = act + a.l; f = act + a.f;
+        kt = reinterpret_cast<T*>(act + a.tile);
+        ks = key_stride<T>(D) / (int)sizeof(T);
+        vt = kt + (size_t)pr.attn_chunk * ks;
+        t_lo = (int)((long long)keys.count * d.a1 / d.a2);
+        count = (int)((long long)keys.count * (d.a1 + 1) / d.a2) - t_lo;
+        const size_t rows0 = (size_t)pr.g.slot * (keep + ring);
+        kc = static_cast<T*>(L.k_cache) + rows0 * G * 2 * D + (size_t)d.a0 * 2 * D;
+        vc = static_cast<T*>(L.v_cache) + rows0 * G * E + (size_t)d.a0 * E;
     }
-    if (!wait_phase(c, layer, MKBH_OP_NORM_PROJ)) return false;
-    rec(c, 1);
-    for (int i = tid; i < nq * D; i += kConsumers) q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
+    // Start copying rows [c0, c0 + nk) of the split, except this token's own: older rows do not
+    // depend on this step (other layers' caches included).  One warp per key.
+    __device__ __forceinline__ void stage(int c0, int nk) const {
+        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+        const bool wide = (D * sizeof(T)) % 16 == 0 && (E * sizeof(T)) % 16 == 0;
+        for (int t = warp; t < nk; t += kConsumerWarps) {
+            const int j = keys.key(t_lo + c0 + t);
+            if (j == pos) continue;
+            const size_t row = cache_row(j, keep, ring);
+            const T *ksrc = kc + row * G * 2 * D, *vsrc = vc + row * G * E;
+            T *kd = kt + t * ks, *vd = vt + t * E;
+            if (wide) {
+                const int U = 16 / (int)sizeof(T), kn = 2 * D / U, n = kn + E / U;
+                for (int u = lane; u < n; u += 32) {
+                    const void* s = u < kn ? (const void*)(ksrc + u * U) : (const void*)(vsrc + (u - kn) * U);
+                    const uint32_t dst = u < kn ? smem_u32(kd + u * U) : smem_u32(vd + (u - kn) * U);
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(s) : "memory");
+                }
+            } else {
+                for (int u = lane; u < 2 * D; u += 32) kd[u] = __ldcg(ksrc + u);
+                for (int u = lane; u < E; u += 32) vd[u] = __ldcg(vsrc + u);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+};
+
+template <typename T, int kAcc>
+__device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, const Desc& d) {
+    const MkbhGlobals& g = pr.g;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, KC = pr.attn_chunk;
+    const int D = A.D, E = A.E, nq = A.nq, kvh = d.a0;
+    const float scale = d.L.scale;
+    const bool owns = d.L.owns_kv != 0;
+    const int kv_off = d.L.heads * (2 * D + E);
     const int lanes_e = kConsumers / E;  // query vectors served side by side (E <= 512)
     const int e = tid % E, qv0 = tid / E;
     const bool has_e = qv0 < lanes_e;
-    float acc[kMaxAcc];
+    const bool dot16 = (D * sizeof(T)) % 16 == 0;
+    float acc[kAcc];
 #pragma unroll
-    for (int i = 0; i < kMaxAcc; ++i) acc[i] = 0.f;
+    for (int i = 0; i < kAcc; ++i) acc[i] = 0.f;
+    for (int i = tid; i < nq * D; i += kConsumers) A.q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
 
-    for (int c0 = 0; c0 < t_hi - t_lo; c0 += KC) {
-        const int nk = min(KC, t_hi - t_lo - c0);
-        if (c0 > 0) stage_rows(c0, nk);
-        if (keys.key(t_lo + c0 + nk - 1) == c.pos) {  // this token's own row (always the last key)
+    for (int c0 = 0; c0 < A.count; c0 += KC) {
+        const int nk = min(KC, A.count - c0);
+        if (c0 > 0) A.stage(c0, nk);
+        if (A.keys.key(A.t_lo + c0 + nk - 1) == A.pos) {  // this token's own row (always the last key)
             const int t = nk - 1;
-            const size_t row = cache_row(c.pos, L.cache_keep, L.cache_ring);
+            const size_t row = cache_row(A.pos, A.keep, A.ring);
             for (int i = tid; i < 2 * D + E; i += kConsumers) {
                 const bool is_k = i < 2 * D;
-                T* cell = is_k ? kc + row * G * 2 * D + i : vc + row * G * E + (i - 2 * D);
+                T* cell = is_k ? A.kc + row * A.G * 2 * D + i : A.vc + row * A.G * E + (i - 2 * D);
                 T x;
-                if (L.owns_kv) {
-                    const int off = L.heads * (2 * D + E) + (is_k ? kvh * 2 * D + i : G * 2 * D + kvh * E + (i - 2 * D));
-                    x = from_f<T>(ld_cg_f32(g.proj + off));
+                if (owns) {
+                    x = from_f<T>(ld_cg_f32(g.proj + kv_off + (is_k ? kvh * 2 * D + i : A.G * 2 * D + kvh * E + (i - 2 * D))));
                     *cell = x;
                 } else {
                     x = __ldcg(cell);
                 }
-                if (is_k) kt[t * ks + i] = x;
-                else vt[t * E + (i - 2 * D)] = x;
+                if (is_k) A.kt[t * A.ks + i] = x;
+                else A.vt[t * E + (i - 2 * D)] = x;
             }
         }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         csync();
         // scores: consecutive threads take consecutive keys of one query vector
         for (int i = tid; i < nq * KC; i += kConsumers) {
             const int t = i % KC, qv = i / KC;
             float s = -INFINITY;
             if (t < nk) {
-                const T* k = kt + t * ks + (qv & 1) * D;
-                const float* qq = q + qv * D;
+                const T* k = A.kt + t * A.ks + (qv & 1) * D;
+                const float* qq = A.q + qv * D;
                 s = 0.f;
-                int d = 0;
-                if ((D * sizeof(T)) % 16 == 0) {
+                if (dot16) {
                     constexpr int U = Chunk<T>::kElems;
-                    for (; d < D; d += U) s = Chunk<T>::dot(lds_v4(smem_u32(k + d)), qq + d, s);
+#pragma unroll 4
+                    for (int n = 0; n < D; n += U) {
+                        float f[U];
+#pragma unroll
+                        for (int x = 0; x < U; x += 4) {
+                            const float4 y = *reinterpret_cast<const float4*>(qq + n + x);
+                            f[x] = y.x; f[x + 1] = y.y; f[x + 2] = y.z; f[x + 3] = y.w;
+                        }
+                        s = Chunk<T>::dot(lds_v4(smem_u32(k + n)), f, s);
+                    }
                 } else {
-                    for (; d < D; ++d) s = fmaf(to_f(k[d]), qq[d], s);
+                    for (int n = 0; n < D; ++n) s = fmaf(to_f(k[n]), qq[n], s);
                 }
-                s *= L.scale;
+                s *= scale;
             }
-            p[qv * KC + t] = s;
+            A.p[qv * KC + t] = s;
         }
         csync();
         for (int qv = warp; qv < nq; qv += kConsumerWarps) {
+            const float old = c0 > 0 ? A.m[qv] : -INFINITY;
             float x = -INFINITY;
-            for (int t = lane; t < KC; t += 32) x = fmaxf(x, p[qv * KC + t]);
-            x = fmaxf(warp_max(x), m[qv]);
+            for (int t = lane; t < KC; t += 32) x = fmaxf(x, A.p[qv * KC + t]);
+            x = fmaxf(warp_max(x), old);
             float s = 0.f;
             for (int t = lane; t < KC; t += 32) {
-                const float y = expf(p[qv * KC + t] - x);
-                p[qv * KC + t] = y;
+                const float y = expf(A.p[qv * KC + t] - x);
+                A.p[qv * KC + t] = y;
                 s += y;
             }
             s = warp_sum(s);
             if (lane == 0) {
-                const float fac = expf(m[qv] - x);
-                f[qv] = fac;
-                l[qv] = l[qv] * fac + s;
-                m[qv] = x;
+                const float fac = expf(old - x);
+                A.l[qv] = (c0 > 0 ? A.l[qv] * fac : 0.f) + s;
+                A.f[qv] = fac;
+                A.m[qv] = x;
             }
-            __syncwarp();
         }
         csync();
         if (has_e) {
+            if (c0 > 0) {
 #pragma unroll
-            for (int i = 0; i < kMaxAcc; ++i) {
-                const int qv = qv0 + i * lanes_e;
-                if (qv < nq) acc[i] *= f[qv];
+                for (int i = 0; i < kAcc; ++i)
+                    if (qv0 + i * lanes_e < nq) acc[i] *= A.f[qv0 + i * lanes_e];
             }
             for (int t = 0; t < nk; t += 4) {  // weights beyond nk are zero
                 float v[4];
 #pragma unroll
-                for (int j = 0; j < 4; ++j) v[j] = t + j < nk ? to_f(vt[(t + j) * E + e]) : 0.f;
+                for (int j = 0; j < 4; ++j) v[j] = t + j < nk ? to_f(A.vt[(t + j) * E + e]) : 0.f;
 #pragma unroll
-                for (int i = 0; i < kMaxAcc; ++i) {
+                for (int i = 0; i < kAcc; ++i) {
                     const int qv = qv0 + i * lanes_e;
                     if (qv < nq) {
-                        const float4 w4 = *reinterpret_cast<const float4*>(p + qv * KC + t);
+                        const float4 w4 = *reinterpret_cast<const float4*>(A.p + qv * KC + t);
                         acc[i] = fmaf(w4.x, v[0], fmaf(w4.y, v[1], fmaf(w4.z, v[2], fmaf(w4.w, v[3], acc[i]))));
                     }
                 }
@@ -735,70 +929,74 @@ __device__ __noinline__ bool attention_split(Ctx& c, const int* w) {
         csync();
     }
     // partial rows [head][map][split][m, l, acc...]
-    const int PE = g.part_vdim + 2;
+    const int PE = g.part_vdim + 2, split = d.a1;
     float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
     if (has_e) {
 #pragma unroll
-        for (int i = 0; i < kMaxAcc; ++i) {
+        for (int i = 0; i < kAcc; ++i) {
             const int qv = qv0 + i * lanes_e;
             if (qv < nq) {
                 float* row = part + ((size_t)qv * g.max_splits + split) * PE;
                 row[2 + e] = acc[i];
                 if (e == 0) {
-                    row[0] = m[qv];
-                    row[1] = l[qv];
+                    row[0] = A.count > 0 ? A.m[qv] : -INFINITY;
+                    row[1] = A.count > 0 ? A.l[qv] : 0.f;
                 }
             }
         }
     }
-    csync();
-    if (tid == 0) {
-        int old;
-        int* cnt = g.counters + 2 + (g.num_layers + 1) * MKBH_BARRIERS_PER_LAYER + layer * g.max_kv_heads + kvh;
-        asm volatile("atom.acq_rel.gpu.global.add.s32 %0, [%1], 1;" : "=r"(old) : "l"(cnt) : "memory");
-        c.ctl[1] = old == splits - 1;
-    }
-    csync();
-    if (!c.ctl[1]) return true;
-    // the split of this KV head that arrives last merges the partial rows
-    for (int hh = warp; hh < per; hh += kConsumerWarps) {
-        float fac[2], inv[2];
-        const float* src[2];
-        for (int b = 0; b < 2; ++b) {
-            src[b] = part + (size_t)(2 * hh + b) * g.max_splits * PE;
-            float ms = lane < splits ? ld_cg_f32(src[b] + (size_t)lane * PE) : -INFINITY;
-            const float ls = lane < splits ? ld_cg_f32(src[b] + (size_t)lane * PE + 1) : 0.f;
-            const float M = warp_max(ms);
-            fac[b] = expf(ms - M);
-            inv[b] = 1.f / warp_sum(ls * fac[b]);
-        }
-        const int h = kvh * per + hh;
-        float* o = c.act + (size_t)warp * E;  // q, p and the tiles are no longer needed
-        float sq = 0.f;
-        for (int e2 = lane; e2 - lane < E; e2 += 32) {  // uniform trip count: the loop shuffles
-            float a1 = 0.f, a2 = 0.f;
-            for (int s = 0; s < splits; ++s) {
-                const float f1 = __shfl_sync(0xffffffffu, fac[0], s), f2 = __shfl_sync(0xffffffffu, fac[1], s);
-                if (e2 < E) {
-                    a1 = fmaf(f1, ld_cg_f32(src[0] + (size_t)s * PE + 2 + e2), a1);
-                    a2 = fmaf(f2, ld_cg_f32(src[1] + (size_t)s * PE + 2 + e2), a2);
-                }
-            }
-            if (e2 < E) {
-                const float x = a1 * inv[0] - L.lambda * (a2 * inv[1]);
-                o[e2] = x;
-                sq += x * x;
-            }
-        }
-        const float fin = (1.f - L.diff) / sqrtf(warp_sum(sq) / E + g.eps);
-        for (int e2 = lane; e2 < E; e2 += 32)
-            g.mixed[h * E + e2] = o[e2] * fin * sigmoid_f(ld_cg_f32(g.proj + L.heads * 2 * D + h * E + e2));
-    }
-    signal_phase(c, layer, MKBH_OP_ATTENTION);
-    return true;
 }
 
-// ---- output head: running argmax --------------------------------------------------------------- //
+// The split of a KV head that arrives last merges the partial rows, combines the maps, normalises
+// and gates.
+__device__ __forceinline__ void merge_splits(const Params& pr, const Desc& d, float* act) {
+    const MkbhGlobals& g = pr.g;
+    const MkbhLayer& L = d.L;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int E = L.vdim, per = L.heads / L.kv_heads, nq = 2 * per, kvh = d.a0, splits = d.a2, PE = g.part_vdim + 2;
+    const float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
+    float *fac = act, *o = act + nq * splits, *norm = o + per * E;
+    for (int qv = warp; qv < nq; qv += kConsumerWarps) {
+        const float* row = part + ((size_t)qv * g.max_splits + lane) * PE;
+        const float m = lane < splits ? ld_cg_f32(row) : -INFINITY, l = lane < splits ? ld_cg_f32(row + 1) : 0.f;
+        const float f = expf(m - warp_max(m)), total = warp_sum(l * f);
+        if (lane < splits) fac[qv * splits + lane] = f / total;
+    }
+    csync();
+    for (int i = tid; i < per * E; i += kConsumers) {
+        const int hh = i / E, e = i % E;
+        const float *s1 = part + (size_t)(2 * hh) * g.max_splits * PE + 2 + e, *s2 = s1 + (size_t)g.max_splits * PE;
+        const float *f1 = fac + 2 * hh * splits, *f2 = f1 + splits;
+        float a1 = 0.f, a2 = 0.f;
+        for (int s = 0; s < splits; s += 8) {
+            float x[8], y[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                x[j] = s + j < splits ? ld_cg_f32(s1 + (size_t)(s + j) * PE) : 0.f;
+                y[j] = s + j < splits ? ld_cg_f32(s2 + (size_t)(s + j) * PE) : 0.f;
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+                if (s + j < splits) {
+                    a1 = fmaf(f1[s + j], x[j], a1);
+                    a2 = fmaf(f2[s + j], y[j], a2);
+                }
+        }
+        o[i] = a1 - L.lambda * a2;
+    }
+    csync();
+    for (int hh = warp; hh < per; hh += kConsumerWarps) {
+        float s = 0.f;
+        for (int e = lane; e < E; e += 32) s = fmaf(o[hh * E + e], o[hh * E + e], s);
+        s = warp_sum(s);
+        if (lane == 0) norm[hh] = (1.f - L.diff) / sqrtf(s / E + g.eps);
+    }
+    csync();
+    const float* gate = g.proj + L.heads * 2 * L.dim + (size_t)kvh * per * E;
+    for (int i = tid; i < per * E; i += kConsumers)
+        g.mixed[(size_t)kvh * per * E + i] = o[i] * norm[i / E] * sigmoid_f(ld_cg_f32(gate + i));
+}
+
 __device__ __forceinline__ unsigned long long argmax_key(float v, int i) {
     uint32_t u = __float_as_uint(v);
     u = (u >> 31) ? ~u : (u | 0x80000000u);
@@ -806,69 +1004,122 @@ __device__ __forceinline__ unsigned long long argmax_key(float v, int i) {
 }
 
 template <typename T>
-__device__ bool run_instruction(Ctx& c, const int* w) {
-    const MkbhGlobals& g = *c.g;
-    const int op = __ldg(w), layer = __ldg(w + 1), tid = threadIdx.x;
-    if (op == MKBH_OP_DELTA_STEP) return delta_step(c, w);
-    if (op == MKBH_OP_ATTENTION) return attention_split<T>(c, w);
-    Block b;
-    if (!weight_block<T>(g, w, b)) {
-        if (tid == 0) report(c, MKBH_ERR_BAD_OPCODE, 1, op, 0, 0);
-        csync();
-        return false;
-    }
-    const MkbhLayer& L = g.layers_device[op == MKBH_OP_HEAD ? 0 : layer];
-    int groups = 1;
-    switch (op) {
-        case MKBH_OP_NORM_PROJ: {
-            if (layer > 0 && !wait_phase(c, layer - 1, last_phase(g.layers_device[layer - 1]))) return false;
-            rec(c, 1);
-            norm_activation<T>(c, L.norm1, layer == 0, layer == 0 && b.r0 == 0);
-            rec(c, 2);
-            if (!matvec<T>(c, b, groups)) return false;
-            for (int i = tid; i < b.r1 - b.r0; i += kConsumers)
-                g.proj[b.r0 + i] = row_sum(c, i, groups) + (L.in_bias ? __ldg(L.in_bias + b.r0 + i) : 0.f);
-        } break;
-        case MKBH_OP_OUT_PROJ:
-        case MKBH_OP_DOWN: {
-            const bool down = op == MKBH_OP_DOWN;
-            const float* ls = down ? L.ls2 : L.ls1;
-            const int prev = down ? MKBH_OP_NORM_UP : L.mixer == MKBH_DELTA_RULE ? MKBH_OP_DELTA_STEP : MKBH_OP_ATTENTION;
-            if (!wait_phase(c, layer, prev)) return false;
-            rec(c, 1);
-            if (down) poly_activation(c, L);
-            else mixed_activation(c, L);
-            rec(c, 2);
-            if (!matvec<T>(c, b, groups)) return false;
-            for (int i = tid; i < b.r1 - b.r0; i += kConsumers) {
-                float* x = g.x + b.r0 + i;  // this instruction is the only writer of its rows
-                *x = fmaf(__ldg(ls + b.r0 + i), row_sum(c, i, groups), ld_cg_f32(x));
+__device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Smem& sm) {
+    const MkbhGlobals& g = p.g;
+    const int tid = threadIdx.x, warp = tid >> 5;
+    float* act = reinterpret_cast<float*>(c.gb + sm.act);
+    float* red = reinterpret_cast<float*>(c.gb + sm.red);
+    int* counters = g.counters + 2;
+    uint32_t slot = 0, phase = 0, vecs = 0;
+    int turn = 0;
+    for (int i = 0; i < g.queue_len; ++i) {
+        c.instr = i;
+        c.opcode = -1;
+        bool ok = bar_wait(p, c, c.bar(kDescFull + (i & 1)), (i >> 1) & 1u, 1);
+        if (!ok) c.ctl[0] = 1;
+        if (!agree(c)) return;  // (a barrier per instruction; it also separates the scratch's users)
+        const Desc& d = *reinterpret_cast<const Desc*>(c.gb + sm.desc + (i & 1) * kDescBytes);
+        const MkbhLayer& L = d.L;
+        const float* rowv = reinterpret_cast<const float*>(c.gb + sm.rows + (i & 1) * kRowVecBytes + max(d.row_off, 0));
+        const uint8_t* vec = c.gb + sm.vec + d.vec_off;
+        const int op = c.opcode = d.op;
+        int* stamp = g.timings != nullptr && tid == 0 ? g.timings + ((size_t)blockIdx.x * g.queue_len + i) * MKBH_TIMING_SLOTS : nullptr;
+        auto rec = [&](int k) {
+            if (stamp) stamp[k] = (int)(uint32_t)globaltimer_ns();
+        };
+        if (op == MKBH_OP_NOOP) {
+            csync();
+            if (tid == 0) mbar_arrive(c.bar(kDescEmpty + (i & 1)));
+            continue;
+        }
+        rec(0);
+        // ---- what does not depend on the producers ----
+        StateCol state;
+        if (op == MKBH_OP_DELTA_STEP)
+            state.load(L.state + (((size_t)g.slot * L.heads + d.a0) * L.dim + d.a1 + warp) * L.dim, L.dim,
+                       c.pos > 0 && d.a1 + warp < d.a2);
+        if (op == MKBH_OP_ATTENTION) {
+            const AttnView<T> A(p, c, d, act);
+            A.stage(0, min(p.attn_chunk, A.count));
+        }
+        if (d.has_vec) {
+            ok = bar_wait(p, c, c.bar(kVecFull), vecs & 1u, 1);
+            if (!ok) c.ctl[0] = 1;
+            ++vecs;
+        }
+        // ---- the producers ----
+        if (tid == 0 && d.wait_idx >= 0)
+            poll_counter(counters + d.wait_idx, d.wait_thr, c.ctl, g.status, p.timeout_ns, i, op);
+        if (!agree(c)) return;
+        rec(1);
+        bool signal = true;
+        if (op == MKBH_OP_DELTA_STEP) {
+            delta_step<T>(p, c, d, act, vec, rowv, state);
+            csync();
+            if (tid == 0) mbar_arrive(c.bar(kVecEmpty));
+        } else if (op == MKBH_OP_ATTENTION) {
+            const AttnView<T> A(p, c, d, act);
+            const int need = (A.nq + kConsumers / A.E - 1) / (kConsumers / A.E);
+            if (need <= 2) attend<T, 2>(p, A, d);
+            else if (need <= 4) attend<T, 4>(p, A, d);
+            else attend<T, 16>(p, A, d);
+            csync();
+            if (tid == 0) {
+                int old;
+                int* cnt = counters + (g.num_layers + 1) * MKBH_BARRIERS_PER_LAYER + d.layer * g.max_kv_heads + d.a0;
+                asm volatile("atom.acq_rel.gpu.global.add.s32 %0, [%1], 1;" : "=r"(old) : "l"(cnt) : "memory");
+                c.ctl[1] = old == d.a2 - 1;
             }
-        } break;
-        case MKBH_OP_NORM_UP: {
-            if (!wait_phase(c, layer, MKBH_OP_OUT_PROJ)) return false;
-            rec(c, 1);
-            norm_activation<T>(c, L.norm2, false, false);
-            rec(c, 2);
-            if (!matvec<T>(c, b, groups)) return false;
-            // (the stacked projection is no longer needed: its buffer takes the feed-forward's input)
-            for (int i = tid; i < b.r1 - b.r0; i += kConsumers) g.proj[b.r0 + i] = row_sum(c, i, groups);
-        } break;
-        default: {  // MKBH_OP_HEAD
-            const int last = g.num_layers - 1;
-            if (!wait_phase(c, last, last_phase(g.layers_device[last]))) return false;
-            rec(c, 1);
-            norm_activation<T>(c, g.final_norm, false, false);
-            rec(c, 2);
-            if (!matvec<T>(c, b, groups)) return false;
+            csync();
+            signal = c.ctl[1] != 0;
+            if (signal) merge_splits(p, d, act);
+            csync();
+        } else if (op >= MKBH_OP_NORM_PROJ && op <= MKBH_OP_HEAD) {
+            const int rows = d.a1 - d.a0, K = d.row_bytes / (int)sizeof(T);
+            const bool adds = op == MKBH_OP_OUT_PROJ || op == MKBH_OP_DOWN;
+            // this instruction is the only writer of its rows of the residual stream
+            const float old = adds && tid < rows ? ld_cg_f32(g.x + d.a0 + tid) : 0.f;
+            if (op == MKBH_OP_OUT_PROJ) {
+                if (L.mixer == MKBH_DELTA_RULE) delta_activation(p, L, reinterpret_cast<const float*>(vec), act);
+                else if (K <= 8192) plain_activation<16>(g.mixed, L.heads * L.vdim, act);
+                else plain_activation<32>(g.mixed, L.heads * L.vdim, act);
+            } else if (op == MKBH_OP_DOWN) {
+                if (K <= 8192) poly_activation<16>(p, L, act, red, turn);
+                else poly_activation<32>(p, L, act, red, turn);
+            } else {
+                const float* w = reinterpret_cast<const float*>(vec);
+                const bool first = op == MKBH_OP_NORM_PROJ && d.layer == 0, publish = first && d.a0 == 0;
+                if (K <= 2048) norm_activation<T, 4>(p, c, w, act, red, turn, first, publish);
+                else if (K <= 8192) norm_activation<T, 16>(p, c, w, act, red, turn, first, publish);
+                else norm_activation<T, 32>(p, c, w, act, red, turn, first, publish);
+            }
+            csync();
+            if (tid == 0 && d.has_vec) mbar_arrive(c.bar(kVecEmpty));
+            rec(2);
+            const int chunks = d.row_bytes / 16;
+            if (chunks <= d.groups * 32) ok = matvec_rows<T, 1>(p, c, d, act, slot, phase);
+            else if (chunks <= d.groups * 64) ok = matvec_rows<T, 2>(p, c, d, act, slot, phase);
+            else ok = matvec_rows<T, 4>(p, c, d, act, slot, phase);
+            if (!ok) return;
+            rec(3);
             unsigned long long best = 0;
-            for (int i = tid; i < b.r1 - b.r0; i += kConsumers) {
-                const float y = row_sum(c, i, groups);
-                g.logits[b.r0 + i] = y;
-                const unsigned long long k = argmax_key(y, b.r0 + i);
-                best = k > best ? k : best;
+            if (tid < rows) {
+                float y = 0.f;
+                for (int k = 0; k < d.groups; ++k) y += act[tid * d.groups + k];
+                const int row = d.a0 + tid;
+                if (adds) {
+                    g.x[row] = fmaf(rowv[tid], y, old);
+                } else if (op == MKBH_OP_HEAD) {
+                    g.logits[row] = y;
+                    best = argmax_key(y, row);
+                } else {
+                    // (NORM_UP: the stacked projection is no longer needed, its buffer takes the
+                    // feed-forward's input)
+                    g.proj[row] = y + (d.row_off >= 0 ? rowv[tid] : 0.f);
+                }
             }
-            if (g.argmax_out != nullptr) {
+            if (op == MKBH_OP_HEAD && g.argmax_out != nullptr) {
+                signal = false;
 #pragma unroll
                 for (int o = 16; o; o >>= 1) {
                     const unsigned long long k = __shfl_xor_sync(0xffffffffu, best, o);
@@ -878,70 +1129,61 @@ __device__ bool run_instruction(Ctx& c, const int* w) {
                 if ((tid & 31) == 0 && best) atomicMax(total, best);
                 csync();
                 if (tid == 0) {
-                    int old;
+                    int before;
                     asm volatile("atom.acq_rel.gpu.global.add.s32 %0, [%1], 1;"
-                                 : "=r"(old)
-                                 : "l"(counter(c, g.num_layers, MKBH_OP_HEAD))
+                                 : "=r"(before)
+                                 : "l"(counters + d.arrive_idx)
                                  : "memory");
-                    if (old == threshold(c, g.num_layers, MKBH_OP_HEAD) - 1)
+                    if (before == d.arrive_thr - 1)
                         *g.argmax_out = (int)(0xffffffffu - (uint32_t)(atomicMax(total, 0ull) & 0xffffffffull));
                 }
-                return true;
             }
-        } break;
+            csync();
+        } else {
+            if (tid == 0) report(g.status, c.ctl, MKBH_ERR_BAD_OPCODE, 1, i, op, 0, 0, 0);
+            return;
+        }
+        if (tid == 0) {
+            if (signal) red_release_gpu_add(counters + d.arrive_idx, 1);
+            mbar_arrive(c.bar(kDescEmpty + (i & 1)));
+        }
+        rec(4);
     }
-    signal_phase(c, op == MKBH_OP_HEAD ? g.num_layers : layer, op);
-    return true;
 }
 
 template <typename T>
 __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_constant__ Params p) {
     extern __shared__ uint8_t raw[];
     const uint32_t raw32 = smem_u32(raw), base = (raw32 + 127u) & ~127u;
-    uint8_t* gb = raw + (base - raw32);
-    const Smem sm(p.stages, p.act_bytes);
-    Ctx c;
-    c.p = &p;
-    c.g = &p.g;
+    const Smem sm(p.stages, p.act_bytes, p.vec_bytes);
+    Cta c;
     c.base = base;
-    c.act = reinterpret_cast<float*>(gb + sm.act);
-    c.part = reinterpret_cast<float*>(gb + sm.part);
-    c.red = reinterpret_cast<float*>(gb + sm.red);
+    c.gb = raw + (base - raw32);
     c.bars = base + sm.bars;
-    c.ctl = reinterpret_cast<volatile int*>(gb + sm.ctl);
+    c.ctl = reinterpret_cast<volatile int*>(c.gb + sm.ctl);
     c.instr = -1;
     c.opcode = -1;
-    c.slot = 0;
-    c.phase = 0;
+    c.turn = 0;
     c.pos = p.g.pos_device ? __ldg(p.g.pos_device) : p.g.pos0;
     if (threadIdx.x == 0) {
         for (int s = 0; s < p.stages; ++s) {
             mbar_init(c.full(s), 1);
             mbar_init(c.empty(s), kConsumerWarps);
         }
+        for (int s = 0; s < kRing; ++s) mbar_init(c.bar(s), 1);
         c.ctl[0] = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     __syncthreads();
     if (c.pos < 0 || c.pos >= p.g.max_positions) {  // uniform over the grid
-        if (threadIdx.x == 0) report(c, MKBH_ERR_INVALID_ARGUMENT, 1, c.pos, p.g.max_positions, 0);
+        if (threadIdx.x == 0) report(p.g.status, c.ctl, MKBH_ERR_INVALID_ARGUMENT, 1, -1, -1, c.pos, p.g.max_positions, 0);
         return;
     }
-    if (threadIdx.x < kConsumers) {
-        const int* queue = p.g.instructions + (size_t)blockIdx.x * p.g.queue_len * MKBH_INTS_PER_INSTRUCTION;
-        for (int i = 0; i < p.g.queue_len; ++i) {
-            const int* w = queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION;
-            c.instr = i;
-            c.opcode = __ldg(w);
-            if (c.opcode == MKBH_OP_NOOP) continue;
-            rec(c, 0);
-            if (!run_instruction<T>(c, w)) break;
-            rec(c, 4);
-        }
-    } else if (threadIdx.x == kConsumers) {
-        loader_main<T>(c);
-    }
+    const int warp = threadIdx.x >> 5;
+    if (warp < kConsumerWarps) consumer_main<T>(p, c, sm);
+    else if (warp == kOperandWarp) operand_main<T>(p, c, sm);
+    else if ((threadIdx.x & 31) == 0) loader_main<T>(p, c);
     __syncthreads();
 }
 
@@ -951,33 +1193,39 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     p.g = g;
     p.timeout_ns = (g.wait_timeout_ms ? g.wait_timeout_ms : 2000u) * 1000000ull;
     if (!(g.flags & MKBH_FLAG_RECORD_TIMINGS)) p.g.timings = nullptr;
-    int act = 4 * pad8(g.width);
+    int act = max(kScratchMin, 4 * pad8(g.width)), vec = 4 * g.width;
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
         const bool delta = L.mixer == MKBH_DELTA_RULE;
-        int need = 4 * pad8(L.heads * (delta ? L.dim : L.vdim));
-        if (delta) need = max(need, 4 * delta_scratch_floats(L.dim, L.rank));
-        if (L.ff) need = max(need, 4 * pad8(L.ff));
-        act = max(act, need);
+        act = max(act, 4 * pad8(L.heads * (delta ? L.dim : L.vdim)));
+        if (delta) {
+            act = max(act, 4 * (L.rank + 4 + L.dim));
+            vec = max(vec, max(4 * L.heads * L.dim, L.dim * L.rank * (int)sizeof(T)));
+        }
+        if (L.ff) act = max(act, 4 * pad8(L.ff));
     }
-    act = max(act, kScratchMin);
     // keys staged at a time: 64, fewer when a tile of wide heads would not fit
     p.attn_chunk = 64;
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
         if (L.mixer != MKBH_DIFF_ATTENTION) continue;
-        const int nq = 2 * (L.heads / L.kv_heads);
-        act = max(act, 4 * kConsumerWarps * L.vdim);  // merged rows
-        act = max(act, attn_scratch_bytes<T>(nq, L.dim, L.vdim, 8));
-        while (p.attn_chunk > 8 && attn_scratch_bytes<T>(nq, L.dim, L.vdim, p.attn_chunk) > act) p.attn_chunk -= 8;
+        const int per = L.heads / L.kv_heads, nq = 2 * per;
+        act = max(act, max(4 * merge_scratch_floats(nq, g.max_splits, per, L.vdim), attn_scratch_bytes<T>(nq, L.dim, L.vdim, 8)));
+    }
+    for (int i = 0; i < g.num_layers; ++i) {
+        const MkbhLayer& L = g.layers_host[i];
+        if (L.mixer != MKBH_DIFF_ATTENTION) continue;
+        while (p.attn_chunk > 8 && attn_scratch_bytes<T>(2 * (L.heads / L.kv_heads), L.dim, L.vdim, p.attn_chunk) > act)
+            p.attn_chunk -= 8;
     }
     p.act_bytes = (act + 127) & ~127;
-    const int fixed = Smem(0, p.act_bytes).total + 128;
+    p.vec_bytes = (vec + 32 + 127) & ~127;
+    const int fixed = Smem(0, p.act_bytes, p.vec_bytes).total + 128;
     p.stages = (kSmemLimit - fixed) / kStage;
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     if (p.stages < 2) return cudaErrorInvalidValue;
-    p.l2_window = p.stages + 8;
-    const int smem = Smem(p.stages, p.act_bytes).total + 128;
+    p.l2_window = p.stages + 12;
+    const int smem = Smem(p.stages, p.act_bytes, p.vec_bytes).total + 128;
     static int set[64] = {};
     int dev = 0;
     cudaError_t e = cudaGetDevice(&dev);

@@ -201,15 +201,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant
                     float* o = e.out + (size_t)m0 * e.ld + n;
                     if (e.scale) {
                         const float f = __ldg(e.scale + n);
-                        for (int i = 0; i < rows; i += 8) {
-                            float old[8];
-#pragma unroll
-                            for (int j = 0; j < 8; ++j)
-                                if (i + j < rows) old[j] = o[(size_t)(i + j) * e.ld];
-#pragma unroll
-                            for (int j = 0; j < 8; ++j)
-                                if (i + j < rows) o[(size_t)(i + j) * e.ld] = fmaf(f, tr[(i + j) * kEpiStride + lane], old[j]);
-                        }
+                        // (this tile is the only writer of these elements: one addition each, in L2)
+                        for (int i = 0; i < rows; ++i)
+                            asm volatile("red.global.add.f32 [%0], %1;" ::"l"(o + (size_t)i * e.ld), "f"(f * tr[i * kEpiStride + lane])
+                                         : "memory");
                     } else {
                         const float b = e.bias ? __ldg(e.bias + n) : 0.f;
                         for (int i = 0; i < rows; ++i) o[(size_t)i * e.ld] = tr[i * kEpiStride + lane] + b;

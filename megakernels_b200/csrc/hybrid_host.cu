@@ -43,7 +43,8 @@ int check_layer(const MkbhGlobals& g, int i) {
     REQUIRE(L.in_w && L.out_w && L.norm1 && L.ls1, "layer %d: missing weights", i);
     if (delta) {
         REQUIRE(L.dim <= 256, "layer %d: recurrence head size %d > 256", i, L.dim);
-        REQUIRE(L.rank > 0 && L.decay_w2 && L.decay_w0 && L.out_norm && L.state, "layer %d: incomplete recurrence", i);
+        REQUIRE(L.rank > 0 && L.rank <= 256, "layer %d: decay rank %d outside 1..256", i, L.rank);
+        REQUIRE(L.decay_w2 && L.decay_w0 && L.out_norm && L.state, "layer %d: incomplete recurrence", i);
         REQUIRE(L.in_rows == 5 * L.heads * L.dim + L.rank, "layer %d: %d projection rows", i, L.in_rows);
     } else {
         REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0, "layer %d: %d heads over %d KV heads", i, L.heads, L.kv_heads);
@@ -129,17 +130,19 @@ int mkb_hybrid_prefill(const MkbhGlobals* gp, void* stream) {
     REQUIRE(n > 0 && n <= g.portion_capacity, "a portion of %d tokens (capacity %d)", n, g.portion_capacity);
     REQUIRE(g.pos0 >= 0 && g.pos0 + n <= g.max_positions, "positions %d..%d of %d", g.pos0, g.pos0 + n - 1, g.max_positions);
     REQUIRE(g.num_want >= 0 && g.num_want <= n && (g.num_want == 0 || (g.want_rows && g.logits)), "bad list of wanted rows");
-    int64_t proj = 0, mixed = 0, act = pad8(g.width);
+    int64_t proj = 0, mixed = 0, decay = 0, act = pad8(g.width);
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
         const int64_t out = pad8(out_features(L));
         if (pad8(L.in_rows) > proj) proj = pad8(L.in_rows);
         if (pad8(L.ff) > proj) proj = pad8(L.ff);
         if (out > mixed) mixed = out;
+        if (L.mixer == MKBH_DELTA_RULE && L.heads * (L.dim + 2) > decay) decay = L.heads * (L.dim + 2);
         if (out > act) act = out;
         if (pad8(L.ff) > act) act = pad8(L.ff);
     }
-    REQUIRE(g.x_elems >= (int64_t)n * g.width && g.proj_elems >= n * proj && g.mixed_elems >= n * mixed && g.act_elems >= n * act,
+    REQUIRE(g.x_elems >= (int64_t)n * g.width && g.proj_elems >= n * proj && g.mixed_elems >= n * mixed && g.act_elems >= n * act &&
+                g.decay_elems >= n * decay,
             "activation buffers are too small for %d tokens", n);
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     return g.dtype == MKBH_F32 ? prefill<float>(g, s) : prefill<bf16>(g, s);
@@ -180,8 +183,6 @@ int mkb_hybrid_validate(const MkbhGlobals* gp, const int32_t* ins) {
             if (op == MKBH_OP_DELTA_STEP) {
                 REQUIRE(L.mixer == MKBH_DELTA_RULE && w[2] >= 0 && w[2] < L.heads && w[3] >= 0 && w[3] < w[4] && w[4] <= L.dim,
                         "queue %d, instruction %d: head %d, columns %d..%d", q, k, w[2], w[3], w[4]);
-                const int cols = w[4] - w[3], parts = 512 / cols < 16 ? 512 / cols : 16;
-                REQUIRE(cols <= 512 && parts * 16 >= L.dim, "queue %d, instruction %d: %d columns of %d channels", q, k, cols, L.dim);
             } else if (op == MKBH_OP_ATTENTION) {
                 REQUIRE(L.mixer == MKBH_DIFF_ATTENTION && w[2] >= 0 && w[2] < L.kv_heads && w[3] >= 0 && w[3] < w[4] && w[4] <= g.max_splits,
                         "queue %d, instruction %d: KV head %d, split %d of %d", q, k, w[2], w[3], w[4]);
@@ -198,7 +199,7 @@ int mkb_hybrid_validate(const MkbhGlobals* gp, const int32_t* ins) {
                 const int chunks = pad8(K) * elem_bytes(g) / 16;
                 int groups = 1;
                 while (groups < 16 && groups * 32 < chunks) groups *= 2;
-                REQUIRE(w[2] >= 0 && w[2] < w[3] && w[3] <= rows && (w[3] - w[2]) * groups <= 4096,
+                REQUIRE(w[2] >= 0 && w[2] < w[3] && w[3] <= rows && w[3] - w[2] <= 512 && (w[3] - w[2]) * groups <= 4096,
                         "queue %d, instruction %d: rows %d..%d of %d", q, k, w[2], w[3], rows);
             }
         }

@@ -32,6 +32,11 @@ struct Prefill {
     static cudaError_t attention(const MkbhGlobals& g, const MkbhLayer& L, T* out, int64_t ld, cudaStream_t s);
 };
 
+// bf16 prefill attention on tensor cores, for head sizes it supports; writes columns [0, heads * vdim)
+bool flash_supported(const MkbhLayer& L);
+cudaError_t flash_attention(const MkbhGlobals& g, const MkbhLayer& L, const bf16* kc, const bf16* vc, bf16* out,
+                            int64_t ldo, cudaStream_t s);
+
 // decode: one persistent kernel
 cudaError_t decode_launch(const MkbhGlobals& g, cudaStream_t s);
 

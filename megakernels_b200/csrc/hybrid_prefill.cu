@@ -83,40 +83,84 @@ __global__ void __launch_bounds__(kThreads) poly_norm_kernel(const float* __rest
 
 // ---- generalized delta rule ----------------------------------------------------------------- //
 // The stacked projection of a token is [r | k | v | a | g | w1], heads * dim each but for w1.
-// Replaces a by  c = sigmoid(a) / |k|^2  and writes the decays  w = exp(-decay_scale *
-// sigmoid(w2 tanh(w1) + w0)), so that with q = k^T S the step is
+// With c = sigmoid(a) / |k|^2 and q = k^T S (old state) a step is
 //   S <- diag(w) S - (c k) q + k v^T.
-constexpr int kPrepTokens = 16;
-__global__ void __launch_bounds__(kThreads) delta_prep_kernel(float* __restrict__ proj, int64_t ld, int n, int HD,
-                                                              int dim, int rank, const float* __restrict__ w2,
-                                                              const float* __restrict__ w0, float decay_scale,
-                                                              float unit_eps, float* __restrict__ decay) {
-    extern __shared__ float sm[];  // [kPrepTokens][rank] tanh(w1), [kPrepTokens] 1 / |k|^2
-    float* inner = sm;
-    float* inv = sm + kPrepTokens * rank;
-    const int head = blockIdx.y, t0 = blockIdx.x * kPrepTokens;
-    const int nt = min(kPrepTokens, n - t0);
-    for (int i = threadIdx.x; i < nt * rank; i += kThreads)
-        inner[i] = tanhf(proj[(size_t)(t0 + i / rank) * ld + 5 * HD + i % rank]);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int t = warp; t < nt; t += kThreads / 32) {
-        const float* k = proj + (size_t)(t0 + t) * ld + HD + head * dim;
-        float s = 0.f;
-        for (int i = lane; i < dim; i += 32) s += k[i] * k[i];
-        s = warp_sum(s);
-        if (lane == 0) inv[t] = 1.f / (s + unit_eps);
+// One warp per (token, head): replaces a by c, and writes what the scan's look-ahead needs,
+//   alpha_t = k_(t+1) . (c_t k_t),  beta_t = k_(t+1) . k_t   (0 for the portion's last token).
+__global__ void __launch_bounds__(kThreads) delta_keys_kernel(float* __restrict__ proj, int64_t ld, int n, int heads,
+                                                              int dim, float unit_eps, float* __restrict__ ab) {
+    const int HD = heads * dim, lane = threadIdx.x & 31;
+    const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+    if (item >= (int64_t)n * heads) return;
+    const int t = (int)(item / heads), h = (int)(item % heads);
+    const float* k = proj + (size_t)t * ld + HD + h * dim;
+    float* a = proj + (size_t)t * ld + 3 * HD + h * dim;
+    const bool more = t + 1 < n;
+    constexpr int R = 8;  // dim <= 256
+    float av[R], kk = 0.f, beta = 0.f, alpha = 0.f;
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+        const int i = lane + 32 * j;
+        av[j] = 0.f;
+        if (i < dim) {
+            const float x = k[i], y = more ? k[ld + i] : 0.f;
+            av[j] = sigmoid_f(a[i]);
+            kk = fmaf(x, x, kk);
+            beta = fmaf(x, y, beta);
+            alpha = fmaf(x * y, av[j], alpha);
+        }
+    }
+    const float inv = 1.f / (warp_sum(kk) + unit_eps);
+    alpha = warp_sum(alpha) * inv;
+    beta = warp_sum(beta);
+#pragma unroll
+    for (int j = 0; j < R; ++j)
+        if (lane + 32 * j < dim) a[lane + 32 * j] = av[j] * inv;
+    if (lane == 0) {
+        ab[2 * item] = alpha;
+        ab[2 * item + 1] = beta;
+    }
+}
+
+// Decays w = exp(-decay_scale * sigmoid(w2 tanh(w1) + w0)): a tile of 64 tokens x 64 channels of one head.
+constexpr int kDecayTile = 64;
+__host__ __device__ inline int decay_smem(int rank) { return (kDecayTile * (rank | 1) + rank * kDecayTile) * 4 + 16; }
+template <typename T>
+__global__ void __launch_bounds__(kThreads) delta_decay_kernel(const float* __restrict__ proj, int64_t ld, int n, int HD,
+                                                               int dim, int rank, const T* __restrict__ w2,
+                                                               const float* __restrict__ w0, float decay_scale,
+                                                               float* __restrict__ decay) {
+    extern __shared__ __align__(16) float sm[];
+    float* inner = sm;                         // [rank][64 tokens]
+    float* wt = sm + rank * kDecayTile;        // [64 channels][rank | 1]
+    const int t0 = blockIdx.x * kDecayTile, nt = min(kDecayTile, n - t0), ws = rank | 1;
+    const int c0 = blockIdx.z * kDecayTile, nc = min(kDecayTile, dim - c0), col0 = blockIdx.y * dim + c0;
+    for (int i = threadIdx.x; i < kDecayTile * rank; i += kThreads) {
+        const int t = i / rank, r = i % rank;
+        inner[r * kDecayTile + t] = t < nt ? tanhf(proj[(size_t)(t0 + t) * ld + 5 * HD + r]) : 0.f;
+        wt[t * ws + r] = t < nc ? to_f(w2[(size_t)(col0 + t) * rank + r]) : 0.f;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < nt * dim; i += kThreads) {
-        const int t = i / dim, col = head * dim + i % dim;
-        const float* row = w2 + (size_t)col * rank;
-        const float* in = inner + t * rank;
-        float s = w0[col];
-        for (int r = 0; r < rank; ++r) s += row[r] * in[r];
-        decay[(size_t)(t0 + t) * HD + col] = expf(-decay_scale * sigmoid_f(s));
-        float* a = proj + (size_t)(t0 + t) * ld + 3 * HD + col;
-        *a = sigmoid_f(*a) * inv[t];
+    const int ch = threadIdx.x & 63, tg = (threadIdx.x >> 6) * 16;
+    float acc[16];
+#pragma unroll
+    for (int j = 0; j < 16; ++j) acc[j] = 0.f;
+    for (int r = 0; r < rank; ++r) {
+        const float w = wt[ch * ws + r];
+#pragma unroll
+        for (int j = 0; j < 16; j += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(inner + r * kDecayTile + tg + j);
+            acc[j] = fmaf(w, f.x, acc[j]);
+            acc[j + 1] = fmaf(w, f.y, acc[j + 1]);
+            acc[j + 2] = fmaf(w, f.z, acc[j + 2]);
+            acc[j + 3] = fmaf(w, f.w, acc[j + 3]);
+        }
     }
+    if (ch >= nc) return;
+    const float bias = w0[col0 + ch];
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+        if (tg + j < nt) decay[(size_t)(t0 + tg + j) * HD + col0 + ch] = expf(-decay_scale * sigmoid_f(acc[j] + bias));
 }
 
 __device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
@@ -134,64 +178,88 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 // state matrix are independent of each other.  A warp holds 4 columns, 8 lanes per column; lane
 // group j of a column owns the key channels 32 m + 4 j + {0..3}, so that the broadcast reads of
 // a token's vectors are conflict-free.
+//
+// The chain of a token is  q_t = k_t^T S_(t-1)  (a reduction over lanes)  ->  S_t.  One token of
+// look-ahead halves it: with
+//   q_(t+1) = (w_t k_(t+1))^T S_(t-1) - alpha_t q_t + beta_t v_t
+// the reduction for token t + 1 starts from the state before token t.  Outputs are reduced for
+// eight tokens at a time.
 constexpr int kScanCols = 16;
 constexpr int kScanThreads = 128;
 template <int M>
 __host__ __device__ constexpr int scan_tokens() { return M <= 2 ? 16 : 8; }
 template <int M>
-__host__ __device__ constexpr int scan_smem() { return 2 * scan_tokens<M>() * (4 * 32 * M + kScanCols) * 4; }
+__host__ __device__ constexpr int scan_buf() {  // floats of one buffer
+    return (scan_tokens<M>() + 1) * 4 * 32 * M + scan_tokens<M>() * (kScanCols + 2);
+}
+template <int M>
+__host__ __device__ constexpr int scan_smem() { return 2 * scan_buf<M>() * 4; }
+
+template <int M>
+__device__ __forceinline__ void lds_rows(float (&v)[4 * M], const float4* base) {
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+        const float4 f = base[8 * m];
+        v[4 * m] = f.x; v[4 * m + 1] = f.y; v[4 * m + 2] = f.z; v[4 * m + 3] = f.w;
+    }
+}
 
 template <int M>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* __restrict__ proj, int64_t ld, int n,
-                                                                  int HD, int dim, const float* __restrict__ decay,
+                                                                  int heads, int dim, const float* __restrict__ decay,
+                                                                  const float* __restrict__ ab,
                                                                   float* __restrict__ state, int fresh,
                                                                   float* __restrict__ out) {
-    constexpr int DP = 32 * M, TC = scan_tokens<M>();
-    extern __shared__ __align__(16) float sm[];  // [2][TC][r k c w][DP], [2][TC][kScanCols]
-    float* vec = sm;
-    float* val = sm + 2 * TC * 4 * DP;
-    const int head = blockIdx.y, col0 = blockIdx.x * kScanCols;
+    constexpr int DP = 32 * M, TC = scan_tokens<M>(), BUF = scan_buf<M>();
+    extern __shared__ __align__(16) float sm[];  // two of: [TC + 1][r k c w][DP], [TC][kScanCols], [TC][alpha beta]
+    const int head = blockIdx.y, col0 = blockIdx.x * kScanCols, HD = heads * dim;
     const int tid = threadIdx.x, lane = tid & 31, grp = lane & 7;
     const int lcol = (tid >> 5) * 4 + (lane >> 3), col = col0 + lcol;
     const bool live = col < dim;
-    for (int i = tid; i < 2 * TC * (4 * DP + kScanCols); i += kScanThreads) sm[i] = 0.f;  // padding channels stay zero
-    float* S0 = state + (size_t)head * dim * dim;
+    for (int i = tid; i < 2 * BUF; i += kScanThreads) sm[i] = 0.f;  // padding channels stay zero
+    float* S0 = state + ((size_t)head * dim + (live ? col : 0)) * dim;
     float S[4 * M];
 #pragma unroll
-    for (int m = 0; m < M; ++m)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = 32 * m + 4 * grp + e;
-            S[4 * m + e] = (!fresh && live && i < dim) ? S0[(size_t)i * dim + col] : 0.f;
-        }
+    for (int i = 0; i < 4 * M; ++i) {
+        const int ch = 32 * (i >> 2) + 4 * grp + (i & 3);
+        S[i] = (!fresh && live && ch < dim) ? S0[ch] : 0.f;
+    }
     __syncthreads();
 
-    const float* src[4] = {proj + head * dim, proj + HD + head * dim, proj + 3 * HD + head * dim, decay + head * dim};
+    const float* hp = proj + head * dim;
+    const float* hd = decay + head * dim;
     const bool wide = (dim % 4 == 0) && (HD % 4 == 0) && (ld % 4 == 0);
     auto fetch = [&](int t0, int buf) {
-        const int nt = min(TC, n - t0);
-        const uint32_t dst = mkb::smem_u32(vec + buf * TC * 4 * DP);
-        if (wide) {
-            const int per = dim / 4;
-            for (int i = tid; i < nt * 4 * per; i += kScanThreads) {
-                const int t = i / (4 * per), q = i / per % 4, c = i % per;
-                cp_async16(dst + ((t * 4 + q) * DP + c * 4) * 4, src[q] + (size_t)(t0 + t) * (q == 3 ? HD : ld) + c * 4);
-            }
-        } else {
-            for (int i = tid; i < nt * 4 * dim; i += kScanThreads) {
-                const int t = i / (4 * dim), q = i / dim % 4, c = i % dim;
-                cp_async4(dst + ((t * 4 + q) * DP + c) * 4, src[q] + (size_t)(t0 + t) * (q == 3 ? HD : ld) + c);
+        float* b = sm + buf * BUF;
+        const int nt = min(TC, n - t0), nk = min(TC + 1, n - t0);  // the next chunk's first key as well
+        const int unit = wide ? 4 : 1, per = dim / unit;
+        for (int i = tid; i < (TC + 1) * 4 * per; i += kScanThreads) {
+            const int c = i % per, q = i / per % 4, t = i / (4 * per);
+            float* dst = b + (t * 4 + q) * DP + c * unit;
+            if (t < nt || (q == 1 && t < nk)) {
+                const float* src = (q == 3 ? hd + (size_t)(t0 + t) * HD : hp + (size_t)(t0 + t) * ld + (q == 2 ? 3 : q) * HD) + c * unit;
+                if (wide) cp_async16(mkb::smem_u32(dst), src);
+                else cp_async4(mkb::smem_u32(dst), src);
+            } else {  // beyond the portion: a step that changes nothing
+                for (int u = 0; u < unit; ++u) dst[u] = q == 3 ? 1.f : 0.f;
             }
         }
-        const uint32_t vdst = mkb::smem_u32(val + buf * TC * kScanCols);
+        float *vals = b + (TC + 1) * 4 * DP, *abs_ = vals + TC * kScanCols;
         const int nc = min(kScanCols, dim - col0);
-        for (int i = tid; i < nt * nc; i += kScanThreads)
-            cp_async4(vdst + ((i / nc) * kScanCols + i % nc) * 4,
-                      proj + (size_t)(t0 + i / nc) * ld + 2 * HD + head * dim + col0 + i % nc);
+        for (int i = tid; i < TC * kScanCols; i += kScanThreads) {
+            const int t = i / kScanCols, c = i % kScanCols;
+            if (t < nt && c < nc) cp_async4(mkb::smem_u32(vals + i), hp + (size_t)(t0 + t) * ld + 2 * HD + col0 + c);
+            else vals[i] = 0.f;
+        }
+        for (int i = tid; i < TC * 2; i += kScanThreads) {
+            if (i / 2 < nt) cp_async4(mkb::smem_u32(abs_ + i), ab + ((size_t)(t0 + i / 2) * heads + head) * 2 + (i & 1));
+            else abs_[i] = 0.f;
+        }
         cp_async_commit();
     };
 
     fetch(0, 0);
+    float k[4 * M], q = 0.f;
     for (int t0 = 0, buf = 0; t0 < n; t0 += TC, buf ^= 1) {
         if (t0 + TC < n) {
             fetch(t0 + TC, buf ^ 1);
@@ -200,73 +268,103 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* _
             cp_async_wait<0>();
         }
         __syncthreads();
-        const int nt = min(TC, n - t0);
-        for (int t = 0; t < nt; ++t) {
-            const float4* base = reinterpret_cast<const float4*>(vec + (size_t)((buf * TC + t) * 4) * DP) + grp;
-            float k[4 * M];
-            float q0 = 0.f, q1 = 0.f;
+        const float* b = sm + buf * BUF;
+        const float4* vecs = reinterpret_cast<const float4*>(b) + grp;
+        const float *vals = b + (TC + 1) * 4 * DP + lcol, *abs_ = b + (TC + 1) * 4 * DP + TC * kScanCols;
+        if (t0 == 0) {
+            lds_rows<M>(k, vecs + DP / 4);
 #pragma unroll
-            for (int m = 0; m < M; ++m) {
-                const float4 f = base[DP / 4 + 8 * m];
-                k[4 * m] = f.x; k[4 * m + 1] = f.y; k[4 * m + 2] = f.z; k[4 * m + 3] = f.w;
-                q0 = fmaf(f.x, S[4 * m], q0);
-                q1 = fmaf(f.y, S[4 * m + 1], q1);
-                q0 = fmaf(f.z, S[4 * m + 2], q0);
-                q1 = fmaf(f.w, S[4 * m + 3], q1);
-            }
-            float q = q0 + q1;
+            for (int i = 0; i < 4 * M; ++i) q = fmaf(k[i], S[i], q);
 #pragma unroll
             for (int o = 1; o < 8; o <<= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
-            const float v = val[(buf * TC + t) * kScanCols + lcol];
-            float o0 = 0.f, o1 = 0.f;
+        }
+#pragma unroll 1
+        for (int t8 = 0; t8 < TC; t8 += 8) {
+            float op[8];
 #pragma unroll
-            for (int m = 0; m < M; ++m) {
-                const float4 c = base[2 * (DP / 4) + 8 * m], w = base[3 * (DP / 4) + 8 * m], r = base[8 * m];
-                const float cc[4] = {c.x, c.y, c.z, c.w}, ww[4] = {w.x, w.y, w.z, w.w}, rr[4] = {r.x, r.y, r.z, r.w};
+            for (int j = 0; j < 8; ++j) {
+                const int t = t8 + j;
+                const float4* base = vecs + (size_t)t * DP;  // 4 vectors of DP / 4
+                float w[4 * M], kn[4 * M], c[4 * M], r[4 * M];
+                lds_rows<M>(w, base + 3 * (DP / 4));
+                lds_rows<M>(kn, base + DP + DP / 4);
+                lds_rows<M>(c, base + 2 * (DP / 4));
+                lds_rows<M>(r, base);
+                const float v = vals[t * kScanCols];
+                const float2 al = *reinterpret_cast<const float2*>(abs_ + 2 * t);
+                float d0 = 0.f, d1 = 0.f;
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int i = 4 * m + e;
-                    S[i] = fmaf(k[i], fmaf(-cc[e], q, v), ww[e] * S[i]);
-                    if (e & 1) o1 = fmaf(rr[e], S[i], o1);
-                    else o0 = fmaf(rr[e], S[i], o0);
+                for (int i = 0; i < 4 * M; i += 2) {
+                    S[i] *= w[i];
+                    S[i + 1] *= w[i + 1];
+                    d0 = fmaf(kn[i], S[i], d0);
+                    d1 = fmaf(kn[i + 1], S[i + 1], d1);
                 }
-            }
-            float o = o0 + o1;
+                float d = d0 + d1;
 #pragma unroll
-            for (int d = 1; d < 8; d <<= 1) o += __shfl_xor_sync(0xffffffffu, o, d);
-            if (grp == 0 && live) out[(size_t)(t0 + t) * HD + head * dim + col] = o;
+                for (int o = 1; o < 8; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+                float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+                for (int i = 0; i < 4 * M; i += 2) {
+                    S[i] = fmaf(k[i], fmaf(-c[i], q, v), S[i]);
+                    S[i + 1] = fmaf(k[i + 1], fmaf(-c[i + 1], q, v), S[i + 1]);
+                    o0 = fmaf(r[i], S[i], o0);
+                    o1 = fmaf(r[i + 1], S[i + 1], o1);
+                }
+                op[j] = o0 + o1;
+                q = fmaf(al.y, v, fmaf(-al.x, q, d));
+#pragma unroll
+                for (int i = 0; i < 4 * M; ++i) k[i] = kn[i];
+            }
+            // eight sums over eight lanes in seven shuffles: lane group j ends up with token j
+#pragma unroll
+            for (int h = 4; h; h >>= 1)
+#pragma unroll
+                for (int j = 0; j < h; ++j) {
+                    const bool up = grp & h;
+                    const float keep = up ? op[j + h] : op[j], send = up ? op[j] : op[j + h];
+                    op[j] = keep + __shfl_xor_sync(0xffffffffu, send, h);
+                }
+            const int t = t0 + t8 + grp;
+            if (live && t < n) out[(size_t)t * HD + head * dim + col] = op[0];
         }
         __syncthreads();
     }
 #pragma unroll
-    for (int m = 0; m < M; ++m)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = 32 * m + 4 * grp + e;
-            if (live && i < dim) S0[(size_t)i * dim + col] = S[4 * m + e];
-        }
+    for (int i = 0; i < 4 * M; ++i) {
+        const int ch = 32 * (i >> 2) + 4 * grp + (i & 3);
+        if (live && ch < dim) S0[ch] = S[i];
+    }
 }
 
-// o of each head / its root mean square, times the norm weight, times sigmoid(g)
+// o of each head / its root mean square, times the norm weight, times sigmoid(g): one warp per (token, head)
 template <typename T>
 __global__ void __launch_bounds__(kThreads) delta_gate_kernel(const float* __restrict__ o, const float* __restrict__ proj,
-                                                              int64_t ld, int heads, int dim,
+                                                              int64_t ld, int n, int heads, int dim,
                                                               const float* __restrict__ w, float eps,
                                                               T* __restrict__ out, int64_t ldo) {
-    const int HD = heads * dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const float* row = o + (size_t)blockIdx.x * HD;
-    const float* g = proj + (size_t)blockIdx.x * ld + 4 * HD;
-    T* dst = out + (size_t)blockIdx.x * ldo;
-    for (int h = warp; h < heads; h += kThreads / 32) {
-        float s = 0.f;
-        for (int i = lane; i < dim; i += 32) s += row[h * dim + i] * row[h * dim + i];
-        const float inv = 1.f / sqrtf(warp_sum(s) / dim + eps);
-        for (int i = lane; i < dim; i += 32) {
-            const int c = h * dim + i;
-            dst[c] = from_f<T>(row[c] * inv * w[c] * sigmoid_f(g[c]));
-        }
+    const int HD = heads * dim, lane = threadIdx.x & 31;
+    const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+    if (item >= (int64_t)n * heads) return;
+    const int t = (int)(item / heads), h = (int)(item % heads);
+    const float *row = o + (size_t)t * HD + h * dim, *g = proj + (size_t)t * ld + 4 * HD + h * dim;
+    T* dst = out + (size_t)t * ldo + h * dim;
+    constexpr int R = 8;  // dim <= 256
+    float v[R], x[R], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+        const int i = lane + 32 * j;
+        v[j] = i < dim ? row[i] : 0.f;
+        x[j] = i < dim ? g[i] : 0.f;
+        s = fmaf(v[j], v[j], s);
     }
-    for (int i = HD + threadIdx.x; i < pad8(HD); i += kThreads) dst[i] = from_f<T>(0.f);
+    const float inv = 1.f / sqrtf(warp_sum(s) / dim + eps);
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+        const int i = lane + 32 * j;
+        if (i < dim) dst[i] = from_f<T>(v[j] * inv * w[h * dim + i] * sigmoid_f(x[j]));
+    }
+    if (h == heads - 1 && lane < pad8(HD) - HD) dst[dim + lane] = from_f<T>(0.f);
 }
 
 // ---- windowed differential attention ---------------------------------------------------------- //
@@ -282,7 +380,8 @@ __global__ void kv_append_kernel(const float* __restrict__ proj, int64_t ld, int
     }
 }
 
-// One CTA per (token, query head): scores of 128 keys at a time, both maps, online softmax.
+// One CTA per (token, query head): scores of 128 keys at a time, both maps, online softmax.  The
+// float build's attention, and the bf16 build's for head sizes hybrid_attention.cu does not take.
 constexpr int kAttnThreads = 128;
 constexpr int kAttnMaxE = 4;  // vdim <= 512
 template <typename T>
@@ -375,8 +474,9 @@ cudaError_t launch_scan(const MkbhGlobals& g, const MkbhLayer& L, int64_t ld, fl
         set[dev & 63] = true;
     }
     dim3 grid((L.dim + kScanCols - 1) / kScanCols, L.heads);
-    delta_scan_kernel<M><<<grid, kScanThreads, scan_smem<M>(), s>>>(g.proj, ld, g.num_tokens, L.heads * L.dim, L.dim,
-                                                                   g.decay, state, g.pos0 == 0, g.mixed);
+    delta_scan_kernel<M><<<grid, kScanThreads, scan_smem<M>(), s>>>(
+        g.proj, ld, g.num_tokens, L.heads, L.dim, g.decay, g.decay + (size_t)g.num_tokens * L.heads * L.dim, state,
+        g.pos0 == 0, g.mixed);
     return cudaGetLastError();
 }
 
@@ -404,11 +504,19 @@ template <typename T>
 cudaError_t Prefill<T>::delta(const MkbhGlobals& g, const MkbhLayer& L, T* out, int64_t ldo, cudaStream_t s) {
     const int n = g.num_tokens, HD = L.heads * L.dim;
     const int64_t ld = pad8(L.in_rows);
-    const int smem = kPrepTokens * (L.rank + 1) * 4;
-    delta_prep_kernel<<<dim3((n + kPrepTokens - 1) / kPrepTokens, L.heads), kThreads, smem, s>>>(
-        g.proj, ld, n, HD, L.dim, L.rank, L.decay_w2, L.decay_w0, L.decay_scale, L.unit_eps, g.decay);
+    const int warps = kThreads / 32, pairs = (int)(((int64_t)n * L.heads + warps - 1) / warps);
+    delta_keys_kernel<<<pairs, kThreads, 0, s>>>(g.proj, ld, n, L.heads, L.dim, L.unit_eps, g.decay + (size_t)n * HD);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
+    const int smem = decay_smem(L.rank);
+    if (smem > 48 * 1024) {
+        e = cudaFuncSetAttribute(delta_decay_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return e;
+    }
+    delta_decay_kernel<T><<<dim3((n + kDecayTile - 1) / kDecayTile, L.heads, (L.dim + kDecayTile - 1) / kDecayTile), kThreads,
+                            smem, s>>>(g.proj, ld, n, HD, L.dim, L.rank, static_cast<const T*>(L.decay_w2), L.decay_w0,
+                                       L.decay_scale, g.decay);
+    if ((e = cudaGetLastError()) != cudaSuccess) return e;
     float* state = L.state + (size_t)g.slot * HD * L.dim;
     switch ((L.dim + 31) / 32) {
         case 1: e = launch_scan<1>(g, L, ld, state, s); break;
@@ -420,7 +528,7 @@ cudaError_t Prefill<T>::delta(const MkbhGlobals& g, const MkbhLayer& L, T* out, 
         default: return cudaErrorInvalidValue;
     }
     if (e != cudaSuccess) return e;
-    delta_gate_kernel<T><<<n, kThreads, 0, s>>>(g.mixed, g.proj, ld, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
+    delta_gate_kernel<T><<<pairs, kThreads, 0, s>>>(g.mixed, g.proj, ld, n, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
     return cudaGetLastError();
 }
 template <typename T>
@@ -436,6 +544,8 @@ cudaError_t Prefill<T>::attention(const MkbhGlobals& g, const MkbhLayer& L, T* o
         cudaError_t e = cudaGetLastError();
         if (e != cudaSuccess) return e;
     }
+    if constexpr (sizeof(T) == 2)
+        if (flash_supported(L)) return flash_attention(g, L, kc, vc, out, ldo, s);
     attention_kernel<T><<<dim3(n, L.heads), kAttnThreads, (2 * L.dim + 2 * kAttnThreads) * 4, s>>>(
         g.proj, ld, g.pos0, L, kc, vc, g.eps, out, ldo);
     return cudaGetLastError();

@@ -17,6 +17,7 @@ from megakernels_b200.instructions import Instruction
 from megakernels_b200.utils import get_sm_count
 
 COUNTERS_PER_LAYER = 8  # MKBH_BARRIERS_PER_LAYER
+MAX_ROWS = 512  # output rows of an instruction
 PARTIAL_SUMS = 4096  # per-row, per-column-group sums an instruction may hold
 
 

@@ -12,6 +12,7 @@ import torch
 
 from megakernels_b200.demos.hybrid.instructions import (
     COUNTERS_PER_LAYER,
+    MAX_ROWS,
     PARTIAL_SUMS,
     DeltaStep,
     Down,
@@ -45,21 +46,18 @@ def column_groups(in_features: int, elem_bytes: int) -> int:
 def row_ranges(rows: int, in_features: int, elem_bytes: int, sm_count: int) -> list[tuple[int, int]]:
     """Contiguous runs of rows, as even as possible: one per SM, or the fewest equal waves whose
     runs fit the partial-sum buffer."""
-    most = PARTIAL_SUMS // column_groups(in_features, elem_bytes)
+    most = min(MAX_ROWS, PARTIAL_SUMS // column_groups(in_features, elem_bytes))
     count = min(rows, sm_count * -(-rows // (sm_count * most)))
     return [(rows * i // count, rows * (i + 1) // count) for i in range(count)]
 
 
 def state_columns(heads: int, dim: int, sm_count: int) -> int:
-    """Columns per recurrence instruction: the narrowest block that fits one wave of SMs.
-
-    A block of c columns gives a column min(16, 512 // c) threads of 16 channels each.
-    """
-    fits = [c for c in (16, 32, 64) if min(16, 512 // c) * 16 >= dim]
-    for c in fits:
-        if heads * -(-dim // c) <= sm_count:
-            return c
-    return fits[-1]
+    """Columns per recurrence instruction (a warp carries one at a time, 16 side by side): the
+    narrowest block that fits one wave of SMs."""
+    c = 16
+    while c < dim and heads * -(-dim // c) > sm_count:
+        c += 16
+    return c
 
 
 def make_globals(model, options: HybridScheduleOptions) -> HybridGlobals:
@@ -83,7 +81,7 @@ def make_globals(model, options: HybridScheduleOptions) -> HybridGlobals:
     return HybridGlobals(
         model=model, device=device, portion=n,
         tokens=i32(n), want_rows=i32(n), x=f32(n, cfg.width), proj=f32(n, proj), mixed=f32(n, mixed),
-        decay=f32(n, max([d.inner for d in delta], default=1)),
+        decay=f32(n, max([d.inner + 2 * d.heads for d in delta], default=1)),
         act=torch.zeros(n, act, device=device, dtype=model.dtype),
         logits=f32(cfg.vocab_size), argmax_out=i32(1),
         counters=i32((2 + (L + 1) * COUNTERS_PER_LAYER + L * kv_heads + 1) // 2 * 2),

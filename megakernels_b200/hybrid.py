@@ -7,7 +7,7 @@ container owns what the kernels' globals are built from (padded, stacked weights
 
 Weight layout the kernels read: matrices row-major ``[out, in]`` in the model dtype with ``in``
 padded with zeros to a multiple of 8; the projections that read the same input are stacked into one
-matrix; vectors, biases and the low-rank decay factor are float32.
+matrix; vectors and biases are float32.
 """
 
 from __future__ import annotations
@@ -232,7 +232,7 @@ class HybridForCausalLM:
                 bias[3 * m.inner : 4 * m.inner] = vec(get(p + "mix.a.b"))
                 kw = dict(
                     in_w=mat(torch.cat(mix("r", "k", "v", "a", "g", "w1"))), in_bias=bias,
-                    decay_w2=vec(get(p + "mix.w2")), decay_w0=vec(get(p + "mix.w0")), out_norm=vec(get(p + "mix.norm")),
+                    decay_w2=get(p + "mix.w2").to(device=device, dtype=dtype).contiguous(), decay_w0=vec(get(p + "mix.w0")), out_norm=vec(get(p + "mix.norm")),
                 )
             else:
                 own = ("k", "v") if m.kv_from is None else ()

@@ -50,7 +50,7 @@ class MkbhGlobals(ctypes.Structure):
         ("instructions", _ptr), ("timings", _ptr), ("num_sms", _i32), ("queue_len", _i32),
         ("arrivals", _ptr), ("attn_part", _ptr), ("max_splits", _i32), ("part_vdim", _i32),
         *[(n, _ptr) for n in ("x", "proj", "mixed", "decay", "act")],
-        *[(n, _i64) for n in ("x_elems", "proj_elems", "mixed_elems", "act_elems")],
+        *[(n, _i64) for n in ("x_elems", "proj_elems", "mixed_elems", "act_elems", "decay_elems")],
         ("portion_capacity", _i32),
         ("flags", _u32), ("wait_timeout_ms", _u32), ("status", _ptr),
     ]
@@ -153,7 +153,7 @@ class Call:
                      "decay", "act", "status"):
             setattr(g, name, _p(getattr(globs, name)))
         g.num_counters = globs.counters.numel()
-        for name in ("x", "proj", "mixed", "act"):
+        for name in ("x", "proj", "mixed", "act", "decay"):
             setattr(g, f"{name}_elems", getattr(globs, name).numel())
         g.portion_capacity = globs.portion
         self._validated = None

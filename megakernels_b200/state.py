@@ -6,7 +6,7 @@ A slot is one sequence's share of every cache.  ``SlotPool`` hands slots out and
 * attention layers that project their own keys and values hold ``keep + ring`` rows per slot: the
   first ``keep`` positions for good, later positions modulo ``ring``.  Layers that read another
   layer's rows own nothing; ``keep`` and ``ring`` cover the widest reader;
-* recurrent layers hold one 32-bit matrix per head and slot.
+* recurrent layers hold one 32-bit matrix per head and slot, value column by value column.
 
 Nothing has to be cleared between owners of a slot: a sequence starts at position 0, where the
 kernels take the recurrent state as zero, and no query looks at a position that its own sequence

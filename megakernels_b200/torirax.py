@@ -91,6 +91,6 @@ def preset(width: int, heads: int, dim: int, kv_heads: int, ff: int, vocab: int,
 
 PRESETS = {
     # 1B / 8B class: the widths, feed-forward sizes and vocabulary of the Llama presets
-    "torirax-1b": lambda groups=4: preset(2048, 16, 64, 4, 8192, 128256, groups, 1024, 64),
+    "torirax-1b": lambda groups=5: preset(2048, 16, 64, 4, 8192, 128256, groups, 1024, 64),
     "torirax-8b": lambda groups=6: preset(4096, 16, 128, 4, 14336, 128256, groups, 2048, 128),
 }

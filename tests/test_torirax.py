@@ -242,10 +242,10 @@ def test_row_ranges_fit_the_partial_sums():
         r = row_ranges(rows, k, size, 148)
         assert r[0][0] == 0 and r[-1][1] == rows and all(a[1] == b[0] for a, b in zip(r, r[1:]))
         assert max(b - a for a, b in r) * column_groups(k, size) <= I.PARTIAL_SUMS
+        assert max(b - a for a, b in r) <= I.MAX_ROWS
         assert len(r) <= 148 or len(r) % 148 == 0
-    for heads, dim in ((1, 8), (32, 64), (64, 128), (100, 256), (6, 100)):
-        c = state_columns(heads, dim, 148)
-        assert min(16, 512 // c) * 16 >= dim
+    for heads, dim, want in ((1, 8, 16), (32, 64, 16), (64, 128, 64), (100, 256, 256), (6, 100, 16)):
+        assert state_columns(heads, dim, 148) == want
 
 
 def test_split_counts_and_options():
