@@ -14,6 +14,11 @@ constexpr int kFlashThreads = 256;
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
 }
+__device__ __forceinline__ float fast_exp2(float x) {  // arguments <= 0; tiny results flush to zero
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
@@ -60,7 +65,7 @@ struct FlashSmem {  // bf16 element offsets; row strides are odd multiples of 16
 };
 
 template <int EP>
-__global__ void __launch_bounds__(kFlashThreads) flash_kernel(const FlashArgs a) {
+__global__ void __launch_bounds__(kFlashThreads, EP <= 128 ? 2 : 1) flash_kernel(const FlashArgs a) {
     extern __shared__ __align__(128) bf16 sm[];
     const MkbhLayer& L = a.L;
     const int D = L.dim, E = L.vdim, G = L.kv_heads, dp = a.dp;
@@ -73,6 +78,13 @@ __global__ void __launch_bounds__(kFlashThreads) flash_kernel(const FlashArgs a)
     const int lo = max(0, p0 - L.window + 1), sinks = min(L.keep_first, lo);
     const int total = sinks + p1 - lo + 1;
     auto key_of = [&](int t) { return t < sinks ? t : lo + t - sinks; };
+    // row of a key: the window is shorter than the ring, so it wraps at most once
+    const int keep = L.cache_keep, ring = L.cache_ring, ring_lo = max(lo, keep), ring_row = (ring_lo - keep) % ring;
+    auto row_of = [&](int j) {
+        if (j < keep) return j;
+        const int r = ring_row + (j - ring_lo);
+        return keep + (r >= ring ? r - ring : r);
+    };
 
     for (int i = tid; i < S.total / 8; i += kFlashThreads) reinterpret_cast<uint4*>(sm)[i] = make_uint4(0, 0, 0, 0);
     __syncthreads();  // padding columns stay zero
@@ -86,7 +98,7 @@ __global__ void __launch_bounds__(kFlashThreads) flash_kernel(const FlashArgs a)
         for (int t = warp; t < kBKeys; t += kFlashThreads / 32) {  // one warp per key
             const int idx = tile * kBKeys + t;
             const bool live = idx < total;
-            const size_t row = cache_row(key_of(live ? idx : 0), L.cache_keep, L.cache_ring);
+            const size_t row = row_of(key_of(live ? idx : 0));
             const bf16 *ks = a.kc + (row * G + g) * 2 * D, *vs = a.vc + (row * G + g) * E;
             for (int u = lane; u < 2 * kunits + vunits; u += 32) {
                 if (u < 2 * kunits) {
@@ -164,13 +176,13 @@ __global__ void __launch_bounds__(kFlashThreads) flash_kernel(const FlashArgs a)
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
             const float base = mx == -INFINITY ? 0.f : mx;
-            f[r] = exp2f(m_[r] - base);
+            f[r] = fast_exp2(m_[r] - base);
             m_[r] = mx;
             float sum = 0.f;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                s[i][2 * r] = exp2f(fmaf(s[i][2 * r], scale, -base));
-                s[i][2 * r + 1] = exp2f(fmaf(s[i][2 * r + 1], scale, -base));
+                s[i][2 * r] = fast_exp2(fmaf(s[i][2 * r], scale, -base));
+                s[i][2 * r + 1] = fast_exp2(fmaf(s[i][2 * r + 1], scale, -base));
                 sum += s[i][2 * r] + s[i][2 * r + 1];
             }
             l_[r] = l_[r] * f[r] + sum;
@@ -241,14 +253,14 @@ __global__ void __launch_bounds__(kFlashThreads) flash_kernel(const FlashArgs a)
         sq += __shfl_xor_sync(0xffffffffu, sq, 2);
         if (row >= nq) continue;  // (after the shuffles)
         const float fin = (1.f - L.diff) / sqrtf(sq / E + a.eps);
-        const float* gate = a.proj + (size_t)(t0 + row) * a.ld + L.heads * 2 * D + h * E;
-        bf16* dst = a.out + (size_t)(t0 + row) * a.ldo + h * E;
+        const float* __restrict__ gate = a.proj + (size_t)(t0 + row) * a.ld + L.heads * 2 * D + h * E;
+        bf16* __restrict__ dst = a.out + (size_t)(t0 + row) * a.ldo + h * E;
 #pragma unroll
         for (int i = 0; i < EP / 8; ++i) {
             const int e = i * 8 + (lane & 3) * 2;
             if (e < E)  // E is a multiple of 8
                 *reinterpret_cast<uint32_t*>(dst + e) =
-                    mkb::pack_bf16x2(o[i][2 * r] * fin * sigmoid_f(gate[e]), o[i][2 * r + 1] * fin * sigmoid_f(gate[e + 1]));
+                    mkb::pack_bf16x2(o[i][2 * r] * fin * sigmoid_f(__ldg(gate + e)), o[i][2 * r + 1] * fin * sigmoid_f(__ldg(gate + e + 1)));
         }
     }
 }

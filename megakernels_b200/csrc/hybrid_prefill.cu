@@ -85,46 +85,60 @@ __global__ void __launch_bounds__(kThreads) poly_norm_kernel(const float* __rest
 // The stacked projection of a token is [r | k | v | a | g | w1], heads * dim each but for w1.
 // With c = sigmoid(a) / |k|^2 and q = k^T S (old state) a step is
 //   S <- diag(w) S - (c k) q + k v^T.
-// One warp per (token, head): replaces a by c, and writes what the scan's look-ahead needs,
+// Per (token, head), one warp: replaces a by c, and writes what the scan's look-ahead needs,
 //   alpha_t = k_(t+1) . (c_t k_t),  beta_t = k_(t+1) . k_t   (0 for the portion's last token).
+// A warp takes 8 / R pairs at a time, R channels of each per lane (dim <= 32 R).
+template <int R>
 __global__ void __launch_bounds__(kThreads) delta_keys_kernel(float* __restrict__ proj, int64_t ld, int n, int heads,
                                                               int dim, float unit_eps, float* __restrict__ ab) {
+    constexpr int P = 8 / R;
     const int HD = heads * dim, lane = threadIdx.x & 31;
-    const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-    if (item >= (int64_t)n * heads) return;
-    const int t = (int)(item / heads), h = (int)(item % heads);
-    const float* k = proj + (size_t)t * ld + HD + h * dim;
-    float* a = proj + (size_t)t * ld + 3 * HD + h * dim;
-    const bool more = t + 1 < n;
-    constexpr int R = 8;  // dim <= 256
-    float av[R], kk = 0.f, beta = 0.f, alpha = 0.f;
+    const int64_t first = ((int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5)) * P, total = (int64_t)n * heads;
+    float x[P][R], y[P][R], av[P][R];
 #pragma unroll
-    for (int j = 0; j < R; ++j) {
-        const int i = lane + 32 * j;
-        av[j] = 0.f;
-        if (i < dim) {
-            const float x = k[i], y = more ? k[ld + i] : 0.f;
-            av[j] = sigmoid_f(a[i]);
-            kk = fmaf(x, x, kk);
-            beta = fmaf(x, y, beta);
-            alpha = fmaf(x * y, av[j], alpha);
+    for (int u = 0; u < P; ++u) {
+        const int64_t item = first + u < total ? first + u : total - 1;
+        const int t = (int)(item / heads), h = (int)(item % heads);
+        const float* k = proj + (size_t)t * ld + HD + h * dim;
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+            const int i = lane + 32 * j;
+            const bool live = i < dim;
+            x[u][j] = live ? k[i] : 0.f;
+            y[u][j] = live && t + 1 < n ? k[ld + i] : 0.f;
+            av[u][j] = live ? k[2 * HD + i] : 0.f;
         }
     }
-    const float inv = 1.f / (warp_sum(kk) + unit_eps);
-    alpha = warp_sum(alpha) * inv;
-    beta = warp_sum(beta);
 #pragma unroll
-    for (int j = 0; j < R; ++j)
-        if (lane + 32 * j < dim) a[lane + 32 * j] = av[j] * inv;
-    if (lane == 0) {
-        ab[2 * item] = alpha;
-        ab[2 * item + 1] = beta;
+    for (int u = 0; u < P; ++u) {
+        const int64_t item = first + u;
+        if (item >= total) break;  // uniform over the warp
+        float kk = 0.f, beta = 0.f, alpha = 0.f;
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+            const float s = sigmoid_f(av[u][j]);
+            kk = fmaf(x[u][j], x[u][j], kk);
+            beta = fmaf(x[u][j], y[u][j], beta);
+            alpha = fmaf(x[u][j] * y[u][j], s, alpha);
+            av[u][j] = s;
+        }
+        const float inv = 1.f / (warp_sum(kk) + unit_eps);
+        alpha = warp_sum(alpha) * inv;
+        beta = warp_sum(beta);
+        float* a = proj + (size_t)(item / heads) * ld + 3 * HD + (item % heads) * dim;
+#pragma unroll
+        for (int j = 0; j < R; ++j)
+            if (lane + 32 * j < dim) a[lane + 32 * j] = av[u][j] * inv;
+        if (lane == 0) {
+            ab[2 * item] = alpha;
+            ab[2 * item + 1] = beta;
+        }
     }
 }
 
 // Decays w = exp(-decay_scale * sigmoid(w2 tanh(w1) + w0)): a tile of 64 tokens x 64 channels of one head.
-constexpr int kDecayTile = 64;
-__host__ __device__ inline int decay_smem(int rank) { return (kDecayTile * (rank | 1) + rank * kDecayTile) * 4 + 16; }
+constexpr int kDecayTile = 64, kDecayStride = kDecayTile + 4;
+__host__ __device__ inline int decay_smem(int rank) { return (kDecayTile * (rank | 1) + rank * kDecayStride) * 4; }
 template <typename T>
 __global__ void __launch_bounds__(kThreads) delta_decay_kernel(const float* __restrict__ proj, int64_t ld, int n, int HD,
                                                                int dim, int rank, const T* __restrict__ w2,
@@ -132,12 +146,12 @@ __global__ void __launch_bounds__(kThreads) delta_decay_kernel(const float* __re
                                                                float* __restrict__ decay) {
     extern __shared__ __align__(16) float sm[];
     float* inner = sm;                         // [rank][64 tokens]
-    float* wt = sm + rank * kDecayTile;        // [64 channels][rank | 1]
+    float* wt = sm + rank * kDecayStride;      // [64 channels][rank | 1]
     const int t0 = blockIdx.x * kDecayTile, nt = min(kDecayTile, n - t0), ws = rank | 1;
     const int c0 = blockIdx.z * kDecayTile, nc = min(kDecayTile, dim - c0), col0 = blockIdx.y * dim + c0;
     for (int i = threadIdx.x; i < kDecayTile * rank; i += kThreads) {
         const int t = i / rank, r = i % rank;
-        inner[r * kDecayTile + t] = t < nt ? tanhf(proj[(size_t)(t0 + t) * ld + 5 * HD + r]) : 0.f;
+        inner[r * kDecayStride + t] = t < nt ? tanhf(proj[(size_t)(t0 + t) * ld + 5 * HD + r]) : 0.f;
         wt[t * ws + r] = t < nc ? to_f(w2[(size_t)(col0 + t) * rank + r]) : 0.f;
     }
     __syncthreads();
@@ -149,7 +163,7 @@ __global__ void __launch_bounds__(kThreads) delta_decay_kernel(const float* __re
         const float w = wt[ch * ws + r];
 #pragma unroll
         for (int j = 0; j < 16; j += 4) {
-            const float4 f = *reinterpret_cast<const float4*>(inner + r * kDecayTile + tg + j);
+            const float4 f = *reinterpret_cast<const float4*>(inner + r * kDecayStride + tg + j);
             acc[j] = fmaf(w, f.x, acc[j]);
             acc[j + 1] = fmaf(w, f.y, acc[j + 1]);
             acc[j + 2] = fmaf(w, f.z, acc[j + 2]);
@@ -175,9 +189,9 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 }
 
 // One CTA carries kScanCols value columns of one head through the portion: the columns of the
-// state matrix are independent of each other.  A warp holds 4 columns, 8 lanes per column; lane
-// group j of a column owns the key channels 32 m + 4 j + {0..3}, so that the broadcast reads of
-// a token's vectors are conflict-free.
+// state matrix are independent of each other.  Four warps compute: a warp holds 4 columns, 8 lanes
+// per column; lane j of a column owns the key channels 32 m + 4 j + {0..3}, so that the broadcast
+// reads of a token's vectors are conflict-free.  Four more warps keep the next chunk of tokens coming.
 //
 // The chain of a token is  q_t = k_t^T S_(t-1)  (a reduction over lanes)  ->  S_t.  One token of
 // look-ahead halves it: with
@@ -185,9 +199,9 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 // the reduction for token t + 1 starts from the state before token t.  Outputs are reduced for
 // eight tokens at a time.
 constexpr int kScanCols = 16;
-constexpr int kScanThreads = 128;
+constexpr int kScanThreads = 256;
 template <int M>
-__host__ __device__ constexpr int scan_tokens() { return M <= 2 ? 16 : 8; }
+__host__ __device__ constexpr int scan_tokens() { return M <= 2 ? 32 : M <= 4 ? 16 : 8; }
 template <int M>
 __host__ __device__ constexpr int scan_buf() {  // floats of one buffer
     return (scan_tokens<M>() + 1) * 4 * 32 * M + scan_tokens<M>() * (kScanCols + 2);
@@ -195,28 +209,84 @@ __host__ __device__ constexpr int scan_buf() {  // floats of one buffer
 template <int M>
 __host__ __device__ constexpr int scan_smem() { return 2 * scan_buf<M>() * 4; }
 
+// A token's vectors as one lane needs them: decay, the NEXT token's key, removal rate, read vector.
 template <int M>
-__device__ __forceinline__ void lds_rows(float (&v)[4 * M], const float4* base) {
+struct ScanToken {
+    float w[4 * M], kn[4 * M], c[4 * M], r[4 * M], v;
+    float2 ab;
+    __device__ __forceinline__ static void rows(float (&x)[4 * M], const float4* base) {
 #pragma unroll
-    for (int m = 0; m < M; ++m) {
-        const float4 f = base[8 * m];
-        v[4 * m] = f.x; v[4 * m + 1] = f.y; v[4 * m + 2] = f.z; v[4 * m + 3] = f.w;
+        for (int m = 0; m < M; ++m) {
+            const float4 f = base[8 * m];
+            x[4 * m] = f.x; x[4 * m + 1] = f.y; x[4 * m + 2] = f.z; x[4 * m + 3] = f.w;
+        }
     }
-}
+    __device__ __forceinline__ void load(const float4* base, const float* vals, const float* abs_) {
+        constexpr int Q = 8 * M;  // float4 per vector
+        rows(w, base + 3 * Q);
+        rows(kn, base + 5 * Q);
+        rows(c, base + 2 * Q);
+        rows(r, base);
+        v = *vals;
+        ab = *reinterpret_cast<const float2*>(abs_);
+    }
+};
 
 template <int M>
-__global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* __restrict__ proj, int64_t ld, int n,
-                                                                  int heads, int dim, const float* __restrict__ decay,
-                                                                  const float* __restrict__ ab,
-                                                                  float* __restrict__ state, int fresh,
-                                                                  float* __restrict__ out) {
+__global__ void __launch_bounds__(kScanThreads, 1)
+delta_scan_kernel(const float* __restrict__ proj, int64_t ld, int n, int heads, int dim, const float* __restrict__ decay,
+                  const float* __restrict__ ab, float* __restrict__ state, int fresh, float* __restrict__ out) {
     constexpr int DP = 32 * M, TC = scan_tokens<M>(), BUF = scan_buf<M>();
     extern __shared__ __align__(16) float sm[];  // two of: [TC + 1][r k c w][DP], [TC][kScanCols], [TC][alpha beta]
     const int head = blockIdx.y, col0 = blockIdx.x * kScanCols, HD = heads * dim;
-    const int tid = threadIdx.x, lane = tid & 31, grp = lane & 7;
-    const int lcol = (tid >> 5) * 4 + (lane >> 3), col = col0 + lcol;
-    const bool live = col < dim;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     for (int i = tid; i < 2 * BUF; i += kScanThreads) sm[i] = 0.f;  // padding channels stay zero
+    __syncthreads();
+
+    if (warp >= 4) {  // producers: warp 4 + q copies vector q of every token
+        const int q = warp - 4, ptid = tid - 128;
+        const float* src = q == 3 ? decay + head * dim : proj + head * dim + (q == 2 ? 3 : q) * HD;
+        const int64_t stride = q == 3 ? HD : ld;
+        const float *vsrc = proj + 2 * HD + head * dim + col0, *asrc = ab + head * 2;
+        const bool wide = (dim % 4 == 0) && (HD % 4 == 0) && (ld % 4 == 0);
+        const int units = wide ? dim / 4 : dim;               // copies per vector
+        const int side = units < 32 ? 32 / units : 1;         // tokens side by side in a warp
+        const int first = units < 32 ? lane / units : 0, u0 = units < 32 ? lane % units : lane;
+        const int nc = min(kScanCols, dim - col0);
+        for (int t0 = 0, buf = 0; t0 < n; t0 += TC, buf ^= 1) {
+            if (t0 >= 2 * TC) __syncthreads();  // the buffer has been consumed
+            float* b = sm + buf * BUF;
+            const int nt = min(TC, n - t0), lim = q == 1 ? min(TC + 1, n - t0) : nt;  // keys: the next chunk's first as well
+            if (first < side)
+                for (int t = first; t < lim; t += side)
+                    for (int u = u0; u < units; u += 32) {
+                        const uint32_t dst = mkb::smem_u32(b + (t * 4 + q) * DP + u * (wide ? 4 : 1));
+                        if (wide) cp_async16(dst, src + (t0 + t) * stride + u * 4);
+                        else cp_async4(dst, src + (t0 + t) * stride + u);
+                    }
+            for (int t = lim; t < TC + (q == 1); ++t)  // beyond the portion: steps that change nothing
+                for (int c = lane; c < dim; c += 32) b[(t * 4 + q) * DP + c] = q == 3 ? 1.f : 0.f;
+            float *vals = b + (TC + 1) * 4 * DP, *abs_ = vals + TC * kScanCols;
+            for (int i = ptid; i < TC * kScanCols; i += 128) {
+                const int t = i / kScanCols, c = i % kScanCols;
+                if (t < nt && c < nc) cp_async4(mkb::smem_u32(vals + i), vsrc + (t0 + t) * ld + c);
+                else vals[i] = 0.f;
+            }
+            for (int i = ptid; i < TC * 2; i += 128) {
+                if (i / 2 < nt) cp_async4(mkb::smem_u32(abs_ + i), asrc + (size_t)(t0 + i / 2) * heads * 2 + (i & 1));
+                else abs_[i] = 0.f;
+            }
+            cp_async_commit();
+            cp_async_wait<0>();
+            __syncthreads();  // the chunk is there
+        }
+        return;
+    }
+
+    // Barriers of both sides, in order: chunk 0 there, chunk 1 there, chunk 0 consumed, chunk 2 there,
+    // chunk 1 consumed, ...
+    const int grp = lane & 7, lcol = warp * 4 + (lane >> 3), col = col0 + lcol, chunks = (n + TC - 1) / TC;
+    const bool live = col < dim;
     float* S0 = state + ((size_t)head * dim + (live ? col : 0)) * dim;
     float S[4 * M];
 #pragma unroll
@@ -224,99 +294,51 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* _
         const int ch = 32 * (i >> 2) + 4 * grp + (i & 3);
         S[i] = (!fresh && live && ch < dim) ? S0[ch] : 0.f;
     }
-    __syncthreads();
-
-    const float* hp = proj + head * dim;
-    const float* hd = decay + head * dim;
-    const bool wide = (dim % 4 == 0) && (HD % 4 == 0) && (ld % 4 == 0);
-    auto fetch = [&](int t0, int buf) {
-        float* b = sm + buf * BUF;
-        const int nt = min(TC, n - t0), nk = min(TC + 1, n - t0);  // the next chunk's first key as well
-        const int unit = wide ? 4 : 1, per = dim / unit;
-        for (int i = tid; i < (TC + 1) * 4 * per; i += kScanThreads) {
-            const int c = i % per, q = i / per % 4, t = i / (4 * per);
-            float* dst = b + (t * 4 + q) * DP + c * unit;
-            if (t < nt || (q == 1 && t < nk)) {
-                const float* src = (q == 3 ? hd + (size_t)(t0 + t) * HD : hp + (size_t)(t0 + t) * ld + (q == 2 ? 3 : q) * HD) + c * unit;
-                if (wide) cp_async16(mkb::smem_u32(dst), src);
-                else cp_async4(mkb::smem_u32(dst), src);
-            } else {  // beyond the portion: a step that changes nothing
-                for (int u = 0; u < unit; ++u) dst[u] = q == 3 ? 1.f : 0.f;
-            }
-        }
-        float *vals = b + (TC + 1) * 4 * DP, *abs_ = vals + TC * kScanCols;
-        const int nc = min(kScanCols, dim - col0);
-        for (int i = tid; i < TC * kScanCols; i += kScanThreads) {
-            const int t = i / kScanCols, c = i % kScanCols;
-            if (t < nt && c < nc) cp_async4(mkb::smem_u32(vals + i), hp + (size_t)(t0 + t) * ld + 2 * HD + col0 + c);
-            else vals[i] = 0.f;
-        }
-        for (int i = tid; i < TC * 2; i += kScanThreads) {
-            if (i / 2 < nt) cp_async4(mkb::smem_u32(abs_ + i), ab + ((size_t)(t0 + i / 2) * heads + head) * 2 + (i & 1));
-            else abs_[i] = 0.f;
-        }
-        cp_async_commit();
-    };
-
-    fetch(0, 0);
     float k[4 * M], q = 0.f;
-    for (int t0 = 0, buf = 0; t0 < n; t0 += TC, buf ^= 1) {
-        if (t0 + TC < n) {
-            fetch(t0 + TC, buf ^ 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
-        const float* b = sm + buf * BUF;
+    __syncthreads();  // chunk 0 is there
+    for (int ci = 0; ci < chunks; ++ci) {
+        const float* b = sm + (ci & 1) * BUF;
         const float4* vecs = reinterpret_cast<const float4*>(b) + grp;
         const float *vals = b + (TC + 1) * 4 * DP + lcol, *abs_ = b + (TC + 1) * 4 * DP + TC * kScanCols;
-        if (t0 == 0) {
-            lds_rows<M>(k, vecs + DP / 4);
+        if (ci == 0) {
+            ScanToken<M>::rows(k, vecs + 8 * M);
 #pragma unroll
             for (int i = 0; i < 4 * M; ++i) q = fmaf(k[i], S[i], q);
 #pragma unroll
             for (int o = 1; o < 8; o <<= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
         }
+        ScanToken<M> now, next;
+        now.load(vecs, vals, abs_);
 #pragma unroll 1
         for (int t8 = 0; t8 < TC; t8 += 8) {
             float op[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                const int t = t8 + j;
-                const float4* base = vecs + (size_t)t * DP;  // 4 vectors of DP / 4
-                float w[4 * M], kn[4 * M], c[4 * M], r[4 * M];
-                lds_rows<M>(w, base + 3 * (DP / 4));
-                lds_rows<M>(kn, base + DP + DP / 4);
-                lds_rows<M>(c, base + 2 * (DP / 4));
-                lds_rows<M>(r, base);
-                const float v = vals[t * kScanCols];
-                const float2 al = *reinterpret_cast<const float2*>(abs_ + 2 * t);
-                float d0 = 0.f, d1 = 0.f;
+                const int tn = j < 7 || t8 + 8 < TC ? t8 + j + 1 : 0;  // (the chunk's last token loads a dummy)
+                next.load(vecs + tn * DP, vals + tn * kScanCols, abs_ + 2 * tn);
+                float d[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f}, x[4 * M];
 #pragma unroll
-                for (int i = 0; i < 4 * M; i += 2) {
-                    S[i] *= w[i];
-                    S[i + 1] *= w[i + 1];
-                    d0 = fmaf(kn[i], S[i], d0);
-                    d1 = fmaf(kn[i + 1], S[i + 1], d1);
+                for (int i = 0; i < 4 * M; ++i) {
+                    S[i] *= now.w[i];
+                    d[i & 3] = fmaf(now.kn[i], S[i], d[i & 3]);
                 }
-                float d = d0 + d1;
+                float dd = (d[0] + d[1]) + (d[2] + d[3]);
+                dd += __shfl_xor_sync(0xffffffffu, dd, 1);
 #pragma unroll
-                for (int o = 1; o < 8; o <<= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-                float o0 = 0.f, o1 = 0.f;
+                for (int i = 0; i < 4 * M; ++i) x[i] = fmaf(-now.c[i], q, now.v);
+                dd += __shfl_xor_sync(0xffffffffu, dd, 2);
 #pragma unroll
-                for (int i = 0; i < 4 * M; i += 2) {
-                    S[i] = fmaf(k[i], fmaf(-c[i], q, v), S[i]);
-                    S[i + 1] = fmaf(k[i + 1], fmaf(-c[i + 1], q, v), S[i + 1]);
-                    o0 = fmaf(r[i], S[i], o0);
-                    o1 = fmaf(r[i + 1], S[i + 1], o1);
-                }
-                op[j] = o0 + o1;
-                q = fmaf(al.y, v, fmaf(-al.x, q, d));
+                for (int i = 0; i < 4 * M; ++i) S[i] = fmaf(k[i], x[i], S[i]);
+                dd += __shfl_xor_sync(0xffffffffu, dd, 4);
 #pragma unroll
-                for (int i = 0; i < 4 * M; ++i) k[i] = kn[i];
+                for (int i = 0; i < 4 * M; ++i) o[i & 3] = fmaf(now.r[i], S[i], o[i & 3]);
+                op[j] = (o[0] + o[1]) + (o[2] + o[3]);
+                q = fmaf(now.ab.y, now.v, fmaf(-now.ab.x, q, dd));
+#pragma unroll
+                for (int i = 0; i < 4 * M; ++i) k[i] = now.kn[i];
+                now = next;
             }
-            // eight sums over eight lanes in seven shuffles: lane group j ends up with token j
+            // eight sums over eight lanes in seven shuffles: lane j of a column ends up with token j
 #pragma unroll
             for (int h = 4; h; h >>= 1)
 #pragma unroll
@@ -325,10 +347,11 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* _
                     const float keep = up ? op[j + h] : op[j], send = up ? op[j] : op[j + h];
                     op[j] = keep + __shfl_xor_sync(0xffffffffu, send, h);
                 }
-            const int t = t0 + t8 + grp;
+            const int t = ci * TC + t8 + grp;
             if (live && t < n) out[(size_t)t * HD + head * dim + col] = op[0];
         }
-        __syncthreads();
+        if (ci + 1 < chunks) __syncthreads();  // chunk ci + 1 is there
+        if (ci + 2 < chunks) __syncthreads();  // chunk ci has been consumed
     }
 #pragma unroll
     for (int i = 0; i < 4 * M; ++i) {
@@ -337,34 +360,46 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const float* _
     }
 }
 
-// o of each head / its root mean square, times the norm weight, times sigmoid(g): one warp per (token, head)
-template <typename T>
+// o of each head / its root mean square, times the norm weight, times sigmoid(g): one warp per
+// (token, head), 8 / R of them at a time
+template <typename T, int R>
 __global__ void __launch_bounds__(kThreads) delta_gate_kernel(const float* __restrict__ o, const float* __restrict__ proj,
                                                               int64_t ld, int n, int heads, int dim,
                                                               const float* __restrict__ w, float eps,
                                                               T* __restrict__ out, int64_t ldo) {
+    constexpr int P = 8 / R;
     const int HD = heads * dim, lane = threadIdx.x & 31;
-    const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-    if (item >= (int64_t)n * heads) return;
-    const int t = (int)(item / heads), h = (int)(item % heads);
-    const float *row = o + (size_t)t * HD + h * dim, *g = proj + (size_t)t * ld + 4 * HD + h * dim;
-    T* dst = out + (size_t)t * ldo + h * dim;
-    constexpr int R = 8;  // dim <= 256
-    float v[R], x[R], s = 0.f;
+    const int64_t first = ((int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5)) * P, total = (int64_t)n * heads;
+    float v[P][R], x[P][R];
 #pragma unroll
-    for (int j = 0; j < R; ++j) {
-        const int i = lane + 32 * j;
-        v[j] = i < dim ? row[i] : 0.f;
-        x[j] = i < dim ? g[i] : 0.f;
-        s = fmaf(v[j], v[j], s);
-    }
-    const float inv = 1.f / sqrtf(warp_sum(s) / dim + eps);
+    for (int u = 0; u < P; ++u) {
+        const int64_t item = first + u < total ? first + u : total - 1;
+        const int t = (int)(item / heads), h = (int)(item % heads);
+        const float *row = o + (size_t)t * HD + h * dim, *g = proj + (size_t)t * ld + 4 * HD + h * dim;
 #pragma unroll
-    for (int j = 0; j < R; ++j) {
-        const int i = lane + 32 * j;
-        if (i < dim) dst[i] = from_f<T>(v[j] * inv * w[h * dim + i] * sigmoid_f(x[j]));
+        for (int j = 0; j < R; ++j) {
+            const int i = lane + 32 * j;
+            v[u][j] = i < dim ? row[i] : 0.f;
+            x[u][j] = i < dim ? g[i] : 0.f;
+        }
     }
-    if (h == heads - 1 && lane < pad8(HD) - HD) dst[dim + lane] = from_f<T>(0.f);
+#pragma unroll
+    for (int u = 0; u < P; ++u) {
+        const int64_t item = first + u;
+        if (item >= total) break;  // uniform over the warp
+        const int t = (int)(item / heads), h = (int)(item % heads);
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < R; ++j) s = fmaf(v[u][j], v[u][j], s);
+        const float inv = 1.f / sqrtf(warp_sum(s) / dim + eps);
+        T* dst = out + (size_t)t * ldo + h * dim;
+#pragma unroll
+        for (int j = 0; j < R; ++j) {
+            const int i = lane + 32 * j;
+            if (i < dim) dst[i] = from_f<T>(v[u][j] * inv * w[h * dim + i] * sigmoid_f(x[u][j]));
+        }
+        if (h == heads - 1 && lane < pad8(HD) - HD) dst[dim + lane] = from_f<T>(0.f);
+    }
 }
 
 // ---- windowed differential attention ---------------------------------------------------------- //
@@ -504,8 +539,12 @@ template <typename T>
 cudaError_t Prefill<T>::delta(const MkbhGlobals& g, const MkbhLayer& L, T* out, int64_t ldo, cudaStream_t s) {
     const int n = g.num_tokens, HD = L.heads * L.dim;
     const int64_t ld = pad8(L.in_rows);
-    const int warps = kThreads / 32, pairs = (int)(((int64_t)n * L.heads + warps - 1) / warps);
-    delta_keys_kernel<<<pairs, kThreads, 0, s>>>(g.proj, ld, n, L.heads, L.dim, L.unit_eps, g.decay + (size_t)n * HD);
+    const int R = L.dim <= 64 ? 2 : L.dim <= 128 ? 4 : 8, per_block = kThreads / 32 * (8 / R);
+    const int pairs = (int)(((int64_t)n * L.heads + per_block - 1) / per_block);
+    float* ab = g.decay + (size_t)n * HD;
+    if (R == 2) delta_keys_kernel<2><<<pairs, kThreads, 0, s>>>(g.proj, ld, n, L.heads, L.dim, L.unit_eps, ab);
+    else if (R == 4) delta_keys_kernel<4><<<pairs, kThreads, 0, s>>>(g.proj, ld, n, L.heads, L.dim, L.unit_eps, ab);
+    else delta_keys_kernel<8><<<pairs, kThreads, 0, s>>>(g.proj, ld, n, L.heads, L.dim, L.unit_eps, ab);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
     const int smem = decay_smem(L.rank);
@@ -528,7 +567,9 @@ cudaError_t Prefill<T>::delta(const MkbhGlobals& g, const MkbhLayer& L, T* out, 
         default: return cudaErrorInvalidValue;
     }
     if (e != cudaSuccess) return e;
-    delta_gate_kernel<T><<<pairs, kThreads, 0, s>>>(g.mixed, g.proj, ld, n, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
+    if (R == 2) delta_gate_kernel<T, 2><<<pairs, kThreads, 0, s>>>(g.mixed, g.proj, ld, n, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
+    else if (R == 4) delta_gate_kernel<T, 4><<<pairs, kThreads, 0, s>>>(g.mixed, g.proj, ld, n, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
+    else delta_gate_kernel<T, 8><<<pairs, kThreads, 0, s>>>(g.mixed, g.proj, ld, n, L.heads, L.dim, L.out_norm, g.eps, out, ldo);
     return cudaGetLastError();
 }
 template <typename T>

@@ -80,7 +80,7 @@ def test_token_by_token_equals_the_prompt(bench, name, dtype, tol):
 
 
 @pytest.mark.parametrize("cuts", [[2] * 75, [3, 2, 5, 2, 7, 11, 2, 13, 1, 1, 17, 2], [1, 149], [149, 1], [64, 64, 22], [33] * 5])
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "ragged"])
 def test_portions_of_several_sizes(bench, name, cuts):
     raw, w, path, toks, want = bench(name)
     assert rel(run_cut(load(path), toks, cuts), want) < F32_TOL

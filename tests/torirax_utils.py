@@ -51,7 +51,14 @@ EVEN = model_config([
 ], width=192, vocab=260)
 WIDE = model_config([delta(1, 256), attention(2, 1, 128, 256, size=90, keep_first=2, ff=1100), delta(2, 160)],
                     width=520, vocab=1031)
-MODELS = {"odd": ODD, "even": EVEN, "wide": WIDE}
+# an attention layer first, a width that is no multiple of 4, one kept position, KV heads of their own
+RAGGED = model_config([
+    attention(3, 3, 12, 40, size=21, keep_first=1, diff=0.7, ff=45),
+    attention(3, 3, 12, 40, size=4, keep_first=6, diff=0.25, scale=0.5, kv_from=0),
+    delta(5, 12),
+    delta(1, 33, ff=66),
+], width=71, vocab=97, eps=1e-4, scale=0.8)
+MODELS = {"odd": ODD, "even": EVEN, "wide": WIDE, "ragged": RAGGED}
 
 
 def rank_of(i: int) -> int:
