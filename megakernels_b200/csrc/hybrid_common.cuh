@@ -13,6 +13,8 @@ namespace mkbh {
 
 using bf16 = __nv_bfloat16;
 
+constexpr int kMaxRowBytes = 32768;  // longest row of a weight matrix (checked on the host)
+
 __host__ __device__ inline int pad8(int n) { return (n + 7) & ~7; }
 
 template <typename T> __device__ __forceinline__ float to_f(T v);

@@ -40,6 +40,7 @@ constexpr int kConsumers = kConsumerWarps * 32;
 constexpr int kOperandWarp = kConsumerWarps + 1;  // (warp 16 is the loader)
 constexpr int kBlock = kConsumers + 64;
 constexpr int kStage = 32768;
+static_assert(kStage >= kMaxRowBytes, "a stage holds whole rows");
 constexpr int kMaxStages = 6;
 constexpr int kPartFloats = 4096;      // per-row, per-column-group partial sums of an instruction
 constexpr int kMaxRows = 512;          // output rows of an instruction
@@ -53,7 +54,6 @@ struct Params {
     MkbhGlobals g;
     int stages, act_bytes, vec_bytes;
     int attn_chunk;        // keys staged at a time
-    int l2_window;         // stages the loader may prefetch into L2, ring included
     unsigned long long timeout_ns;
 };
 
@@ -227,35 +227,14 @@ __device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
     const MkbhGlobals& g = p.g;
     const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
     const uint64_t policy = mkb::l2_policy_evict_first();
-    Cursor<T> cur, pre;
-    uint32_t issued = 0, ahead = 0;  // stages copied, stages prefetched or copied
+    Cursor<T> cur;
+    uint32_t issued = 0;
     const uint8_t* src;
     uint32_t bytes;
-    bool more = true;
     const int S = p.stages;
     while (cur.next(g, queue, src, bytes)) {
         const int slot = issued % S;
-        const uint32_t parity = ((issued / S) & 1u) ^ 1u;
-        if (ahead <= issued && more) {  // keep the look-ahead cursor in front of the ring
-            const uint8_t* s2;
-            uint32_t b2;
-            more = pre.next(g, queue, s2, b2);
-            ++ahead;
-        }
-        bool ok = true;
-        while (!mbar_try_wait(c.empty(slot), parity)) {
-            if (more && ahead < issued + (uint32_t)p.l2_window) {
-                const uint8_t* s2;
-                uint32_t b2;
-                more = pre.next(g, queue, s2, b2);
-                if (more) asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(s2), "r"(b2) : "memory");
-                ++ahead;
-                continue;
-            }
-            ok = bar_wait(p, c, c.empty(slot), parity, 0);
-            break;
-        }
-        if (!ok) break;
+        if (!bar_wait(p, c, c.empty(slot), ((issued / S) & 1u) ^ 1u, 0)) break;
         mbar_expect_tx(c.full(slot), bytes);
         mkb::tma_bulk_g2s(c.base + slot * kStage, src, bytes, c.full(slot), policy);
         ++issued;
@@ -1224,7 +1203,6 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     p.stages = (kSmemLimit - fixed) / kStage;
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     if (p.stages < 2) return cudaErrorInvalidValue;
-    p.l2_window = p.stages + 12;
     const int smem = Smem(p.stages, p.act_bytes, p.vec_bytes).total + 128;
     static int set[64] = {};
     int dev = 0;

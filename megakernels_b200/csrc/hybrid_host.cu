@@ -60,8 +60,8 @@ int check_layer(const MkbhGlobals& g, int i) {
     }
     if (L.ff) REQUIRE(L.ff > 0 && L.up_w && L.down_w && L.norm2 && L.ls2, "layer %d: incomplete feed-forward", i);
     const int widest = pad8(L.ff > out_features(L) ? L.ff : out_features(L));
-    REQUIRE((widest > pad8(g.width) ? widest : pad8(g.width)) * elem_bytes(g) <= 32768,
-            "layer %d: a weight row is longer than 32768 bytes", i);
+    REQUIRE((widest > pad8(g.width) ? widest : pad8(g.width)) * elem_bytes(g) <= kMaxRowBytes,
+            "layer %d: a weight row is longer than %d bytes", i, kMaxRowBytes);
     return MKBH_OK;
 }
 
