@@ -51,7 +51,6 @@ class HybridGlobals:
     pos_id_device: Tensor | None = None  # int32 [1]; overrides pos_id in decode launches
     instructions: Tensor | None = None
     timings: Tensor | None = None
-    batch_size: int = 1
     hooks: dict = field(default_factory=dict)
 
     def sm_count(self) -> int:

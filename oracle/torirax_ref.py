@@ -1,6 +1,6 @@
 """Plain restatement of the Torirax decoder, one function per mechanism.
 
-Checker only: it shares no code with the product path, keeps no cache and computes every
+Test infrastructure only: it shares no code with the product path, keeps no cache and computes every
 sequence from its first token.  Everything runs in the dtype of the tensors it is given
 (the tests use float64).  ``weights`` maps tensor names to tensors, ``config`` is the parsed
 ``config.json``.
