@@ -66,16 +66,33 @@ __host__ __device__ inline int cache_row(int j, int keep, int ring) {
 }
 
 // Keys that the query at `pos` sees: the first `sinks` positions, then `count - sinks` positions
-// from `start` on (the window, which ends at the query itself).
+// from `start` on, up to the query itself: its window, or its chunk (chunks count from position 0).
 struct KeyRange {
     int sinks, start, count;
-    __host__ __device__ KeyRange(int pos, int window, int keep_first) {
-        const int n = pos + 1 < window ? pos + 1 : window;
+    __host__ __device__ KeyRange(int pos, int window, int keep_first, int chunk) {
+        const int n = chunk > 0 ? pos % chunk + 1 : pos + 1 < window ? pos + 1 : window;
         start = pos + 1 - n;
-        sinks = keep_first < start ? keep_first : start;
+        sinks = chunk > 0 ? 0 : keep_first < start ? keep_first : start;
         count = sinks + n;
     }
     __host__ __device__ int key(int t) const { return t < sinks ? t : start + (t - sinks); }
 };
+
+// Sizes of a layer's mixer.
+__host__ __device__ inline bool is_attention(const MkbhLayer& L) { return L.mixer != MKBH_DELTA_RULE; }
+__host__ __device__ inline int mixer_out(const MkbhLayer& L) { return L.heads * (L.mixer == MKBH_DELTA_RULE ? L.dim : L.vdim); }
+__host__ __device__ inline int latent_row(const MkbhLayer& L) { return pad8(L.rank) + pad8(L.rot_dim); }
+__host__ __device__ inline int up_rows(const MkbhLayer& L) { return L.ff_kind == MKBH_CLAMPED_GLU ? 2 * L.ff : L.ff; }
+// Phase whose end makes the mixer's output complete.
+__host__ __device__ inline int mixer_phase(int mixer) {
+    return mixer == MKBH_DELTA_RULE ? MKBH_OP_DELTA_STEP : mixer == MKBH_LATENT_ATTENTION ? MKBH_OP_EXPAND : MKBH_OP_ATTENTION;
+}
+
+// Gated unit with clamped halves: g' sigmoid(alpha g') (u' + 1).
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f(alpha * g) * (u + 1.f);
+}
 
 }  // namespace mkbh

@@ -2,8 +2,8 @@
 //
 // The scheme of megakernel.cu - one CTA per SM, an instruction queue per CTA, a ring of weight
 // stages in shared memory that a loader thread keeps full across instruction boundaries, counters
-// in HBM that order the phases - for layers that are listed one by one (delta-rule recurrence or
-// windowed differential attention, optional PolyNorm feed-forward) and for any sizes:
+// in HBM that order the phases - for layers that are listed one by one (delta-rule recurrence,
+// windowed differential, rotary or latent attention, optional feed-forward) and for any sizes:
 //   * a weight block is a run of whole rows, contiguous in memory, so a stage is ONE untiled bulk
 //     copy (no tensor maps, no divisibility rules beyond the zero padding of a row to 16 bytes);
 //   * 16 consumer warps multiply from shared memory with fp32 FMA (batch 1 is bandwidth-bound), the
@@ -48,12 +48,15 @@ static_assert(kPartFloats * 4 <= 40 * 1024, "");
 constexpr int kScratchMin = 40 * 1024; // activation / mixer scratch, at least
 constexpr int kRowVecBytes = kMaxRows * 4 + 32;
 constexpr int kSmemLimit = 226 * 1024;
+constexpr int kMaxStash = 512;         // channels whose normalised input an instruction publishes
 constexpr int kMaxChannels = 8;        // key channels of one column a lane carries (dim <= 256)
 
 struct Params {
     MkbhGlobals g;
     int stages, act_bytes, vec_bytes;
     int attn_chunk;        // keys staged at a time
+    int last_buf;          // residual buffer of the last layer
+    int part_base;         // where the second vector of an instruction lies in the vector buffer
     unsigned long long timeout_ns;
 };
 
@@ -64,7 +67,7 @@ struct Desc {
     int arrive_idx, arrive_thr;
     int row_bytes, per_stage, groups;
     int has_vec, vec_off, row_off;  // vector operands: present, byte offsets inside their buffers
-    int pad;
+    int part_off;                   // second vector (terms of earlier inputs), -1: none
     MkbhLayer L;
 };
 static_assert(sizeof(MkbhLayer) % 8 == 0, "");
@@ -73,14 +76,15 @@ constexpr int kDescBytes = (sizeof(Desc) + 127) & ~127;
 enum Bar { kDescFull = 0, kDescEmpty = 2, kVecFull = 4, kVecEmpty = 5, kRing = 6 };
 
 struct Smem {  // byte offsets from the 128-byte aligned base
-    int act, vec, rows, desc, red, bars, ctl, total;
+    int act, vec, rows, desc, red, stash, bars, ctl, total;
     __host__ __device__ Smem(int stages, int act_bytes, int vec_bytes) {
         act = stages * kStage;          // activations; partial sums once they are in registers
         vec = act + act_bytes;          // norm weights / decay factor
         rows = vec + vec_bytes;         // two slots: per-row vectors (bias, layer scale, decay bias)
         desc = rows + 2 * kRowVecBytes;
         red = (desc + 2 * kDescBytes + 127) & ~127;
-        bars = red + 2 * 3 * kConsumerWarps * 4;
+        stash = red + 2 * 3 * kConsumerWarps * 4;
+        bars = stash + kMaxStash * 4;
         ctl = bars + (kRing + 2 * kMaxStages) * 8;
         total = ctl + 16 * 4;
     }
@@ -167,6 +171,13 @@ __device__ __noinline__ void poll_counter(const int* addr, int thr, volatile int
 
 __device__ __forceinline__ int phase_index(int layer, int op) { return layer * MKBH_BARRIERS_PER_LAYER + op; }
 
+// Float buffers beside the stacked projection: feed-forward input and output of parallel layers,
+// absorbed queries and latent outputs.
+__device__ __forceinline__ float* side_in(const MkbhGlobals& g) { return g.side; }
+__device__ __forceinline__ float* side_out(const MkbhGlobals& g) { return g.side + g.side_ff; }
+__device__ __forceinline__ float* side_query(const MkbhGlobals& g) { return side_out(g) + pad8(g.width); }
+__device__ __forceinline__ float* side_latent(const MkbhGlobals& g) { return side_query(g) + g.side_rank; }
+
 // ---- loader: the weight stream ----------------------------------------------------------- //
 struct Block {  // rows [r0, r1) of a matrix of `row_bytes` rows
     const uint8_t* w;
@@ -181,11 +192,17 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, const int* w,
         case MKBH_OP_NORM_PROJ: b.w = (const uint8_t*)L->in_w; K = g.width; break;
         case MKBH_OP_OUT_PROJ:
             b.w = (const uint8_t*)L->out_w;
-            K = L->heads * (L->mixer == MKBH_DELTA_RULE ? L->dim : L->vdim);
+            K = mixer_out(*L);
             break;
         case MKBH_OP_NORM_UP: b.w = (const uint8_t*)L->up_w; K = g.width; break;
         case MKBH_OP_DOWN: b.w = (const uint8_t*)L->down_w; K = L->ff; break;
         case MKBH_OP_HEAD: b.w = (const uint8_t*)g.head; K = g.width; break;
+        case MKBH_OP_ENTER: b.w = (const uint8_t*)L->enter_w; K = 2 * g.width; break;
+        case MKBH_OP_ABSORB: b.w = (const uint8_t*)L->absorb_w; K = L->dim; break;
+        case MKBH_OP_EXPAND:  // (behind the keys' rows)
+            K = L->rank;
+            b.w = (const uint8_t*)L->expand_w + (size_t)L->heads * L->dim * pad8(K) * sizeof(T);
+            break;
         default: return false;
     }
     b.r0 = __ldg(w + 2);
@@ -252,7 +269,9 @@ __host__ __device__ inline int column_groups(int chunks) {
     return n;
 }
 // Phase that completes the residual stream a layer leaves.
-__device__ __forceinline__ int last_phase(int ff) { return ff ? MKBH_OP_DOWN : MKBH_OP_OUT_PROJ; }
+__device__ __forceinline__ int last_phase(const MkbhLayer* L) {
+    return __ldg(&L->ff) && !__ldg(&L->parallel) ? MKBH_OP_DOWN : MKBH_OP_OUT_PROJ;
+}
 
 __device__ __forceinline__ void copy_vec(uint32_t dst, const void* src, int bytes, uint32_t bar, uint64_t policy) {
     const uint64_t a = reinterpret_cast<uint64_t>(src) & ~15ull, e = (reinterpret_cast<uint64_t>(src) + bytes + 15) & ~15ull;
@@ -287,17 +306,30 @@ __device__ __forceinline__ void operand_main(const Params& p, Cta& c, const Smem
         const uint2* src = reinterpret_cast<const uint2*>(g.layers_device + layer);
         for (int k = lane; k < (int)sizeof(MkbhLayer) / 8; k += 32) reinterpret_cast<uint2*>(&d->L)[k] = __ldg(src + k);
         __syncwarp();
-        const void *vec = nullptr, *rows = nullptr;
+        const void *vec = nullptr, *rows = nullptr, *part = nullptr;
         int vec_n = 0, row_n = 0, K = 0;
         if (lane == 0) {
             const MkbhLayer& L = d->L;
             const bool delta = L.mixer == MKBH_DELTA_RULE;
             int wl = layer, wop = 0;
-            switch (op) {
-                case MKBH_OP_NORM_PROJ:
-                    K = g.width; vec = L.norm1; vec_n = K * 4; rows = L.in_bias;
+            const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
+            // phase that completes the layer's input stream
+            auto input_phase = [&](bool entered) {
+                if (L.enter_w != nullptr && entered) {
+                    wop = MKBH_OP_ENTER;
+                } else {
                     wl = layer - 1;
-                    wop = layer > 0 ? last_phase(__ldg(&g.layers_device[layer - 1].ff)) : -1;
+                    wop = layer > 0 ? last_phase(g.layers_device + wl) : -1;
+                }
+            };
+            switch (op) {
+                case MKBH_OP_ENTER: K = 2 * g.width; input_phase(false); break;
+                case MKBH_OP_NORM_PROJ:
+                    K = g.width; vec_n = K * 4;
+                    vec = L.canon_taps ? L.canon_gain : L.norm1;
+                    if (L.canon_taps > 1 && c.pos > 0) part = L.canon_part + ((size_t)g.slot * 2 + (c.pos & 1)) * g.width;
+                    rows = L.conv_taps ? L.conv_w + (size_t)(L.conv_taps - 1) * L.in_rows : L.in_bias;
+                    input_phase(true);
                     break;
                 case MKBH_OP_DELTA_STEP:
                     vec = (const uint8_t*)L.decay_w2 + (size_t)d->a0 * L.dim * L.rank * sizeof(T);
@@ -306,19 +338,25 @@ __device__ __forceinline__ void operand_main(const Params& p, Cta& c, const Smem
                     row_n = L.dim * 4;
                     wop = MKBH_OP_NORM_PROJ;
                     break;
-                case MKBH_OP_ATTENTION: wop = MKBH_OP_NORM_PROJ; break;
+                case MKBH_OP_ABSORB: K = L.dim; wop = MKBH_OP_NORM_PROJ; break;
+                case MKBH_OP_ATTENTION: wop = latent ? MKBH_OP_ABSORB : MKBH_OP_NORM_PROJ; break;
+                case MKBH_OP_EXPAND: K = L.rank; wop = MKBH_OP_ATTENTION; break;
                 case MKBH_OP_OUT_PROJ:
-                    K = L.heads * (delta ? L.dim : L.vdim);
+                    K = mixer_out(L);
                     rows = L.ls1;
                     if (delta) vec = L.out_norm, vec_n = K * 4;
-                    wop = delta ? MKBH_OP_DELTA_STEP : MKBH_OP_ATTENTION;
+                    wop = mixer_phase(L.mixer);
                     break;
-                case MKBH_OP_NORM_UP: K = g.width; vec = L.norm2; vec_n = K * 4; wop = MKBH_OP_OUT_PROJ; break;
-                case MKBH_OP_DOWN: K = L.ff; rows = L.ls2; wop = MKBH_OP_NORM_UP; break;
+                case MKBH_OP_NORM_UP:
+                    K = g.width; vec = L.norm2; vec_n = K * 4;
+                    if (L.parallel) input_phase(true);
+                    else wop = MKBH_OP_OUT_PROJ;
+                    break;
+                case MKBH_OP_DOWN: K = L.ff; rows = L.parallel ? nullptr : L.ls2; wop = MKBH_OP_NORM_UP; break;
                 case MKBH_OP_HEAD:
                     K = g.width; vec = g.final_norm; vec_n = K * 4;
                     wl = g.num_layers - 1;
-                    wop = last_phase(__ldg(&g.layers_device[wl].ff));
+                    wop = last_phase(g.layers_device + wl);
                     break;
                 default: wop = -1; break;
             }
@@ -328,13 +366,16 @@ __device__ __forceinline__ void operand_main(const Params& p, Cta& c, const Smem
             }
             d->wait_idx = wop < 0 ? -1 : phase_index(wl, wop);
             d->wait_thr = wop < 0 ? 0 : __ldg(g.arrivals + phase_index(wl, wop));
-            d->arrive_idx = phase_index(op == MKBH_OP_HEAD ? g.num_layers : layer, op);
+            // (a feed-forward beside a mixer counts into the phase that the output projection waits for)
+            d->arrive_idx = phase_index(op == MKBH_OP_HEAD ? g.num_layers : layer,
+                                        op == MKBH_OP_DOWN && L.parallel ? mixer_phase(L.mixer) : op);
             d->arrive_thr = op == MKBH_OP_HEAD ? __ldg(g.arrivals + d->arrive_idx) : 0;
             d->row_bytes = pad8(K) * (int)sizeof(T);
             d->per_stage = K > 0 ? kStage / d->row_bytes : 0;
             d->groups = column_groups(d->row_bytes / 16);
             d->has_vec = vec != nullptr;
             d->vec_off = (int)(reinterpret_cast<uint64_t>(vec) & 15);
+            d->part_off = part != nullptr ? p.part_base + (int)(reinterpret_cast<uint64_t>(part) & 15) : -1;
             d->row_off = rows != nullptr && row_n > 0 ? (int)(reinterpret_cast<uint64_t>(rows) & 15) : -1;
         }
         __syncwarp();
@@ -349,8 +390,9 @@ __device__ __forceinline__ void operand_main(const Params& p, Cta& c, const Smem
             if (vec != nullptr) {
                 flag = bar_wait(p, c, c.bar(kVecEmpty), (vecs & 1u) ^ 1u, 2);
                 if (flag) {
-                    mbar_expect_tx(c.bar(kVecFull), vec_span(vec, vec_n));
+                    mbar_expect_tx(c.bar(kVecFull), vec_span(vec, vec_n) + (part != nullptr ? vec_span(part, vec_n) : 0u));
                     copy_vec(c.base + sm.vec, vec, vec_n, c.bar(kVecFull), policy);
+                    if (part != nullptr) copy_vec(c.base + sm.vec + p.part_base, part, vec_n, c.bar(kVecFull), policy);
                     ++vecs;
                 }
             }
@@ -528,45 +570,71 @@ struct Spread {
     }
 };
 
-// Layer norm of the residual stream (or of the token's embedding, which `publish` also writes out).
+__device__ __forceinline__ int token_id(const MkbhGlobals& g) {
+    const int tok = __ldg(g.tokens);
+    return tok < 0 ? 0 : tok >= g.vocab ? g.vocab - 1 : tok;
+}
+
+// Norm of the residual stream `src` (NULL: of the token's embedding, which goes to `publish` as
+// well).  `part`: what earlier inputs add through the input convolution; `stash` receives the
+// unweighted channels [c0, c1) for it.
 template <typename T, int kSlots>
-__device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, const float* w, float* act, float* red,
-                                                int& turn, bool embedding, bool publish) {
+__device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, const float* src, const float* w, const float* part,
+                                                float* act, float* red, int& turn, float* publish, float* stash, int c0, int c1) {
     const MkbhGlobals& g = p.g;
     Spread<kSlots> x;
     x.K = g.width;
     x.wide = g.width % 4 == 0;
-    if (embedding) {
-        int tok = __ldg(g.tokens);
-        tok = tok < 0 ? 0 : tok >= g.vocab ? g.vocab - 1 : tok;
-        const T* e = static_cast<const T*>(g.embed) + (size_t)tok * x.K;
-        const T* q = static_cast<const T*>(g.pos) + (size_t)c.pos * x.K;
+    if (src == nullptr) {
+        const T* e = static_cast<const T*>(g.embed) + (size_t)token_id(g) * x.K;
+        const T* q = g.pos != nullptr ? static_cast<const T*>(g.pos) + (size_t)c.pos * x.K : nullptr;
 #pragma unroll
         for (int s = 0; s < kSlots; ++s) {
             const int i = x.index(s);
-            x.v[s] = i < x.K ? to_f(e[i]) * g.embed_scale + to_f(q[i]) : 0.f;
-            if (publish && i < x.K) g.x[i] = x.v[s];
+            x.v[s] = i < x.K ? to_f(e[i]) * g.embed_scale + (q != nullptr ? to_f(q[i]) : 0.f) : 0.f;
+            if (publish != nullptr && i < x.K) publish[i] = x.v[s];
         }
     } else {
-        x.load_cg(g.x);
+        x.load_cg(src);
     }
     float sum[1] = {0.f};
+    if (g.norm_kind == MKBH_LAYER_NORM) {
 #pragma unroll
-    for (int s = 0; s < kSlots; ++s) sum[0] += x.v[s];
-    csum<1>(red, turn, sum);
-    const float mean = sum[0] / x.K;
+        for (int s = 0; s < kSlots; ++s) sum[0] += x.v[s];
+        csum<1>(red, turn, sum);
+        const float mean = sum[0] / x.K;
+#pragma unroll
+        for (int s = 0; s < kSlots; ++s) x.v[s] = x.has(s) ? x.v[s] - mean : 0.f;
+    }
     sum[0] = 0.f;
 #pragma unroll
-    for (int s = 0; s < kSlots; ++s) {
-        x.v[s] = x.has(s) ? x.v[s] - mean : 0.f;
-        sum[0] = fmaf(x.v[s], x.v[s], sum[0]);
-    }
+    for (int s = 0; s < kSlots; ++s) sum[0] = fmaf(x.v[s], x.v[s], sum[0]);
     csum<1>(red, turn, sum);
     const float inv = 1.f / sqrtf(sum[0] / x.K + g.eps);
 #pragma unroll
     for (int s = 0; s < kSlots; ++s)
-        if (x.has(s)) x.v[s] *= inv * w[x.index(s)];
+        if (x.has(s)) {
+            const int i = x.index(s);
+            x.v[s] *= inv;
+            if (i >= c0 && i < c1) stash[i - c0] = x.v[s];
+            x.v[s] = part != nullptr ? fmaf(x.v[s], w[i], part[i]) : x.v[s] * w[i];
+        }
     x.store(act);
+}
+
+// The residual stream next to the token's embedding.
+template <typename T>
+__device__ __forceinline__ void enter_activation(const MkbhGlobals& g, const float* src, float* act) {
+    const int W = g.width;
+    const T* e = static_cast<const T*>(g.embed) + (size_t)token_id(g) * W;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < W; i += kConsumers) {
+        const float x0 = to_f(e[i]) * g.embed_scale;
+        act[i] = src != nullptr ? ld_cg_f32(src + i) : x0;
+        act[W + i] = x0;
+    }
+    const int z = 2 * W + (int)threadIdx.x;
+    if (z < pad8(2 * W)) act[z] = 0.f;
 }
 
 template <int kSlots>
@@ -596,7 +664,7 @@ template <int kSlots>
 __device__ __forceinline__ void plain_activation(const float* src, int K, float* act) {
     Spread<kSlots> v;
     v.K = K;
-    v.wide = K % 4 == 0;
+    v.wide = K % 4 == 0 && (reinterpret_cast<uint64_t>(src) & 15) == 0;
     v.load_cg(src);
     v.store(act);
 }
@@ -723,27 +791,36 @@ __device__ __forceinline__ void delta_step(const Params& p, const Cta& c, const 
     }
 }
 
-// ---- windowed differential attention: one split of the keys of one KV head -------------------- //
+// ---- attention: one split of the keys of one KV head ----------------------------------------- //
+// `maps` query vectors per head against as many keys per position (differential: 2).  Latent
+// attention is one key per position, the latent with its rotated part, whose first `rank` entries
+// are the value too; a "KV head" is then a group of heads.
+__host__ __device__ inline int attn_maps(const MkbhLayer& L) { return L.mixer == MKBH_DIFF_ATTENTION ? 2 : 1; }
+__host__ __device__ inline int attn_dim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? latent_row(L) : L.dim; }
+__host__ __device__ inline int attn_vdim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? L.rank : L.vdim; }
 struct AttnScratch {  // float offsets; the key and value tiles follow
-    int q, p, m, l, f, tile;
-    __host__ __device__ AttnScratch(int nq, int dim, int chunk) {
+    int q, p, m, l, f, own, tile;
+    __host__ __device__ AttnScratch(const MkbhLayer& L, int chunk) {
+        const int nq = attn_maps(L) * (L.heads / L.kv_heads), dim = attn_dim(L);
         q = 0;
         p = nq * dim;
         p = (p + 3) & ~3;
         m = p + nq * chunk;
         l = m + nq;
         f = l + nq;
-        tile = (f + nq + 3) & ~3;
+        own = (f + nq + 3) & ~3;  // this token's key and value as floats
+        tile = own + (L.mixer == MKBH_DIFF_ATTENTION ? 0 : (dim + attn_vdim(L) + 3) & ~3);
     }
 };
 template <typename T>
-__host__ __device__ inline int key_stride(int dim) {  // bytes; an odd number of 16-byte units
-    const int u = (2 * dim * (int)sizeof(T) + 15) / 16;
+__host__ __device__ inline int key_stride(int elems) {  // bytes; an odd number of 16-byte units
+    const int u = (elems * (int)sizeof(T) + 15) / 16;
     return (u | 1) * 16;
 }
 template <typename T>
-__host__ __device__ inline int attn_scratch_bytes(int nq, int dim, int vdim, int chunk) {
-    return AttnScratch(nq, dim, chunk).tile * 4 + chunk * (key_stride<T>(dim) + vdim * (int)sizeof(T)) + 16;
+__host__ __device__ inline int attn_scratch_bytes(const MkbhLayer& L, int chunk) {
+    const int value = L.mixer == MKBH_LATENT_ATTENTION ? 0 : L.vdim * (int)sizeof(T);
+    return AttnScratch(L, chunk).tile * 4 + chunk * (key_stride<T>(attn_maps(L) * attn_dim(L)) + value) + 16;
 }
 __host__ __device__ inline int merge_scratch_floats(int nq, int splits, int per, int vdim) {
     return nq * splits + per * (vdim + 1);
@@ -751,59 +828,152 @@ __host__ __device__ inline int merge_scratch_floats(int nq, int splits, int per,
 
 template <typename T>
 struct AttnView {
-    int D, E, G, per, nq, ks, t_lo, count, keep, ring, pos;
+    int D, KE, E, G, per, nq, ks, vs, t_lo, count, keep, ring, pos;
+    size_t krow, vrow;  // elements between positions
     KeyRange keys;
     T *kc, *vc, *kt, *vt;
-    float *q, *p, *m, *l, *f;
+    float *q, *p, *m, *l, *f, *own;
+    bool latent;
     __device__ __forceinline__ AttnView(const Params& pr, const Cta& c, const Desc& d, float* act)
-        : keys(c.pos, d.L.window, d.L.keep_first) {
+        : keys(c.pos, d.L.window, d.L.keep_first, d.L.chunk) {
         const MkbhLayer& L = d.L;
-        D = L.dim; E = L.vdim; G = L.kv_heads; per = L.heads / G; nq = 2 * per;
+        latent = L.mixer == MKBH_LATENT_ATTENTION;
+        D = attn_dim(L); KE = attn_maps(L) * D; E = attn_vdim(L); G = L.kv_heads; per = L.heads / G; nq = attn_maps(L) * per;
         keep = L.cache_keep; ring = L.cache_ring; pos = c.pos;
-        const AttnScratch a(nq, D, pr.attn_chunk);
-        q = act + a.q; p = act + a.p; m = act + a.m; l = act + a.l; f = act + a.f;
+        const AttnScratch a(L, pr.attn_chunk);
+        q = act + a.q; p = act + a.p; m = act + a.m; l = act + a.l; f = act + a.f; own = act + a.own;
         kt = reinterpret_cast<T*>(act + a.tile);
-        ks = key_stride<T>(D) / (int)sizeof(T);
-        vt = kt + (size_t)pr.attn_chunk * ks;
+        ks = key_stride<T>(KE) / (int)sizeof(T);
+        vt = latent ? kt : kt + (size_t)pr.attn_chunk * ks;
+        vs = latent ? ks : E;
         t_lo = (int)((long long)keys.count * d.a1 / d.a2);
         count = (int)((long long)keys.count * (d.a1 + 1) / d.a2) - t_lo;
         const size_t rows0 = (size_t)pr.g.slot * (keep + ring);
-        kc = static_cast<T*>(L.k_cache) + rows0 * G * 2 * D + (size_t)d.a0 * 2 * D;
-        vc = static_cast<T*>(L.v_cache) + rows0 * G * E + (size_t)d.a0 * E;
+        krow = latent ? (size_t)D : (size_t)G * KE;
+        vrow = (size_t)G * E;
+        kc = static_cast<T*>(L.k_cache) + rows0 * krow + (latent ? 0 : (size_t)d.a0 * KE);
+        vc = latent ? nullptr : static_cast<T*>(L.v_cache) + rows0 * vrow + (size_t)d.a0 * E;
     }
+    __device__ __forceinline__ bool has_own() const { return count > 0 && t_lo + count == keys.count; }
     // Start copying rows [c0, c0 + nk) of the split, except this token's own: older rows do not
     // depend on this step (other layers' caches included).  One warp per key.
     __device__ __forceinline__ void stage(int c0, int nk) const {
         const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-        const bool wide = (D * sizeof(T)) % 16 == 0 && (E * sizeof(T)) % 16 == 0;
+        const int VE = latent ? 0 : E;
+        const bool wide = (KE * sizeof(T)) % 16 == 0 && (VE * sizeof(T)) % 16 == 0;
         for (int t = warp; t < nk; t += kConsumerWarps) {
             const int j = keys.key(t_lo + c0 + t);
             if (j == pos) continue;
             const size_t row = cache_row(j, keep, ring);
-            const T *ksrc = kc + row * G * 2 * D, *vsrc = vc + row * G * E;
-            T *kd = kt + t * ks, *vd = vt + t * E;
+            const T *ksrc = kc + row * krow, *vsrc = vc + row * vrow;
+            T *kd = kt + t * ks, *vd = vt + t * vs;
             if (wide) {
-                const int U = 16 / (int)sizeof(T), kn = 2 * D / U, n = kn + E / U;
+                const int U = 16 / (int)sizeof(T), kn = KE / U, n = kn + VE / U;
                 for (int u = lane; u < n; u += 32) {
                     const void* s = u < kn ? (const void*)(ksrc + u * U) : (const void*)(vsrc + (u - kn) * U);
                     const uint32_t dst = u < kn ? smem_u32(kd + u * U) : smem_u32(vd + (u - kn) * U);
                     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(s) : "memory");
                 }
             } else {
-                for (int u = lane; u < 2 * D; u += 32) kd[u] = __ldcg(ksrc + u);
-                for (int u = lane; u < E; u += 32) vd[u] = __ldcg(vsrc + u);
+                for (int u = lane; u < KE; u += 32) kd[u] = __ldcg(ksrc + u);
+                for (int u = lane; u < VE; u += 32) vd[u] = __ldcg(vsrc + u);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     }
 };
 
+// One head's vector, by one warp: optional norm (weight w), rotation of the first `rot` elements
+// (neighbours by the angles of `rope`), factor `mul`.
+__device__ __noinline__ void head_vector(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
+                                         float mul, float* dst) {
+    constexpr int J = 4;  // pairs per lane kept in registers
+    const int lane = threadIdx.x & 31;
+    float a[J], b[J], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < J; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        a[j] = i < n ? ld_cg_f32(src + i) : 0.f;
+        b[j] = i + 1 < n ? ld_cg_f32(src + i + 1) : 0.f;
+        s = fmaf(a[j], a[j], fmaf(b[j], b[j], s));
+    }
+    if (w != nullptr) {
+        for (int i = 64 * J + lane; i < n; i += 32) {
+            const float x = ld_cg_f32(src + i);
+            s = fmaf(x, x, s);
+        }
+        s = 1.f / sqrtf(warp_sum(s) / n + eps);
+    }
+    for (int j = 0; 64 * j < n; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        if (i >= n) break;
+        float x = 0.f, y = 0.f;
+#pragma unroll
+        for (int k = 0; k < J; ++k)
+            if (k == j) x = a[k], y = b[k];
+        if (j >= J) {
+            x = ld_cg_f32(src + i);
+            y = i + 1 < n ? ld_cg_f32(src + i + 1) : 0.f;
+        }
+        if (w != nullptr) {
+            x *= s * __ldg(w + i);
+            if (i + 1 < n) y *= s * __ldg(w + i + 1);
+        }
+        if (i < rot) {
+            const float2 r = __ldg(rope + (i >> 1));
+            const float z = x * r.x - y * r.y;
+            y = y * r.x + x * r.y;
+            x = z;
+        }
+        dst[i] = x * mul;
+        if (i + 1 < n) dst[i + 1] = y * mul;
+    }
+}
+
+// Queries of the KV head's heads, normalised, rotated and scaled, and, in the split that holds it,
+// this token's key and value.  Ends with a barrier.
+template <typename T>
+__device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView<T>& A, const MkbhLayer& L, int kvh) {
+    const MkbhGlobals& g = pr.g;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tasks = A.nq + (A.has_own() ? 2 : 0);
+    const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)A.pos * (L.rope_dims / 2);
+    for (int t = warp; t < tasks; t += kConsumerWarps) {
+        const int h = kvh * A.per + t;
+        if (A.latent) {
+            const int hd = L.dim + L.rot_dim, lead = pad8(L.rank);
+            const float* down = g.proj + (size_t)L.heads * hd;
+            float* dst = t < A.nq ? A.q + t * A.D : A.own;
+            if (t < A.nq) {
+                for (int i = lane; i < L.rank; i += 32) dst[i] = ld_cg_f32(side_query(g) + (size_t)h * L.rank + i) * L.scale;
+                head_vector(g.proj + (size_t)h * hd + L.dim, L.rot_dim, nullptr, 0.f, rope, L.rope_dims, L.scale, dst + lead);
+            } else if (t == A.nq) {
+                head_vector(down, L.rank, L.k_norm, g.eps, nullptr, 0, 1.f, dst);
+            } else {
+                head_vector(down + L.rank, L.rot_dim, nullptr, 0.f, rope, L.rope_dims, 1.f, dst + lead);
+            }
+            if (t <= A.nq) {  // padding
+                for (int i = L.rank + lane; i < lead; i += 32) dst[i] = 0.f;
+                for (int i = lead + L.rot_dim + lane; i < A.D; i += 32) dst[i] = 0.f;
+            }
+        } else if (t < A.nq) {
+            head_vector(g.proj + (size_t)h * A.D, A.D, L.q_norm, g.eps, rope, L.rope_dims, L.scale * __ldg(L.temp + h), A.q + t * A.D);
+        } else if (t == A.nq) {
+            head_vector(g.proj + (size_t)(L.heads + kvh) * A.D, A.D, L.k_norm, g.eps, rope, L.rope_dims, 1.f, A.own);
+        } else {
+            const float2* turn = L.value_rope == nullptr ? nullptr : reinterpret_cast<const float2*>(L.value_rope) + (size_t)A.pos * (A.E / 2);
+            head_vector(g.proj + (size_t)(L.heads + A.G) * A.D + (size_t)kvh * A.E, A.E, nullptr, 0.f, turn, turn ? A.E : 0, 1.f, A.own + A.D);
+        }
+    }
+    csync();
+}
+
 template <typename T, int kAcc>
 __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, const Desc& d) {
     const MkbhGlobals& g = pr.g;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, KC = pr.attn_chunk;
     const int D = A.D, E = A.E, nq = A.nq, kvh = d.a0;
-    const float scale = d.L.scale;
+    const bool diff = d.L.mixer == MKBH_DIFF_ATTENTION;
+    const float scale = diff ? d.L.scale : 1.f;
     const bool owns = d.L.owns_kv != 0;
     const int kv_off = d.L.heads * (2 * D + E);
     const int lanes_e = kConsumers / E;  // query vectors served side by side (E <= 512)
@@ -813,7 +983,10 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
     float acc[kAcc];
 #pragma unroll
     for (int i = 0; i < kAcc; ++i) acc[i] = 0.f;
-    for (int i = tid; i < nq * D; i += kConsumers) A.q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
+    if (diff)
+        for (int i = tid; i < nq * D; i += kConsumers) A.q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
+    else
+        rotary_operands<T>(pr, A, d.L, kvh);
 
     for (int c0 = 0; c0 < A.count; c0 += KC) {
         const int nk = min(KC, A.count - c0);
@@ -821,18 +994,22 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
         if (A.keys.key(A.t_lo + c0 + nk - 1) == A.pos) {  // this token's own row (always the last key)
             const int t = nk - 1;
             const size_t row = cache_row(A.pos, A.keep, A.ring);
-            for (int i = tid; i < 2 * D + E; i += kConsumers) {
-                const bool is_k = i < 2 * D;
-                T* cell = is_k ? A.kc + row * A.G * 2 * D + i : A.vc + row * A.G * E + (i - 2 * D);
+            const int KE = A.KE;
+            for (int i = tid; i < KE + (A.latent ? 0 : E); i += kConsumers) {
+                const bool is_k = i < KE;
+                T* cell = is_k ? A.kc + row * A.krow + i : A.vc + row * A.vrow + (i - KE);
                 T x;
-                if (owns) {
-                    x = from_f<T>(ld_cg_f32(g.proj + kv_off + (is_k ? kvh * 2 * D + i : A.G * 2 * D + kvh * E + (i - 2 * D))));
+                if (!diff) {
+                    x = from_f<T>(A.own[i]);
+                    if (!A.latent || kvh == 0) *cell = x;  // (every group of heads has the same latent)
+                } else if (owns) {
+                    x = from_f<T>(ld_cg_f32(g.proj + kv_off + (is_k ? kvh * KE + i : A.G * KE + kvh * E + (i - KE))));
                     *cell = x;
                 } else {
                     x = __ldcg(cell);
                 }
                 if (is_k) A.kt[t * A.ks + i] = x;
-                else A.vt[t * E + (i - 2 * D)] = x;
+                else A.vt[t * A.vs + (i - KE)] = x;
             }
         }
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -842,7 +1019,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
             const int t = i % KC, qv = i / KC;
             float s = -INFINITY;
             if (t < nk) {
-                const T* k = A.kt + t * A.ks + (qv & 1) * D;
+                const T* k = A.kt + t * A.ks + (diff ? (qv & 1) * D : 0);
                 const float* qq = A.q + qv * D;
                 s = 0.f;
                 if (dot16) {
@@ -894,7 +1071,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
             for (int t = 0; t < nk; t += 4) {  // weights beyond nk are zero
                 float v[4];
 #pragma unroll
-                for (int j = 0; j < 4; ++j) v[j] = t + j < nk ? to_f(A.vt[(t + j) * E + e]) : 0.f;
+                for (int j = 0; j < 4; ++j) v[j] = t + j < nk ? to_f(A.vt[(t + j) * A.vs + e]) : 0.f;
 #pragma unroll
                 for (int i = 0; i < kAcc; ++i) {
                     const int qv = qv0 + i * lanes_e;
@@ -907,7 +1084,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
         }
         csync();
     }
-    // partial rows [head][map][split][m, l, acc...]
+    // partial rows [head and map][split][m, l, acc...]
     const int PE = g.part_vdim + 2, split = d.a1;
     float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
     if (has_e) {
@@ -926,44 +1103,59 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
     }
 }
 
-// The split of a KV head that arrives last merges the partial rows, combines the maps, normalises
-// and gates.
-__device__ __forceinline__ void merge_splits(const Params& pr, const Desc& d, float* act) {
+// The split of a KV head that arrives last merges the partial rows.  Differential: combines the
+// maps, normalises and gates.  Rotary: turns the outputs back.
+__device__ __forceinline__ void merge_splits(const Params& pr, const Cta& c, const Desc& d, float* act) {
     const MkbhGlobals& g = pr.g;
     const MkbhLayer& L = d.L;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int E = L.vdim, per = L.heads / L.kv_heads, nq = 2 * per, kvh = d.a0, splits = d.a2, PE = g.part_vdim + 2;
+    const bool diff = L.mixer == MKBH_DIFF_ATTENTION;
+    const int E = attn_vdim(L), per = L.heads / L.kv_heads, maps = attn_maps(L), nq = maps * per, kvh = d.a0, splits = d.a2, PE = g.part_vdim + 2;
     const float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
     float *fac = act, *o = act + nq * splits, *norm = o + per * E;
     for (int qv = warp; qv < nq; qv += kConsumerWarps) {
         const float* row = part + ((size_t)qv * g.max_splits + lane) * PE;
         const float m = lane < splits ? ld_cg_f32(row) : -INFINITY, l = lane < splits ? ld_cg_f32(row + 1) : 0.f;
-        const float f = expf(m - warp_max(m)), total = warp_sum(l * f);
+        const float sink = L.sink != nullptr ? __ldg(L.sink + kvh * per + qv) : -INFINITY;  // (one map)
+        const float top = fmaxf(warp_max(m), sink), f = expf(m - top), total = warp_sum(l * f) + expf(sink - top);
         if (lane < splits) fac[qv * splits + lane] = f / total;
     }
     csync();
     for (int i = tid; i < per * E; i += kConsumers) {
         const int hh = i / E, e = i % E;
-        const float *s1 = part + (size_t)(2 * hh) * g.max_splits * PE + 2 + e, *s2 = s1 + (size_t)g.max_splits * PE;
-        const float *f1 = fac + 2 * hh * splits, *f2 = f1 + splits;
+        const float *s1 = part + (size_t)(maps * hh) * g.max_splits * PE + 2 + e, *s2 = s1 + (size_t)g.max_splits * PE;
+        const float *f1 = fac + maps * hh * splits, *f2 = f1 + splits;
         float a1 = 0.f, a2 = 0.f;
         for (int s = 0; s < splits; s += 8) {
             float x[8], y[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 x[j] = s + j < splits ? ld_cg_f32(s1 + (size_t)(s + j) * PE) : 0.f;
-                y[j] = s + j < splits ? ld_cg_f32(s2 + (size_t)(s + j) * PE) : 0.f;
+                y[j] = diff && s + j < splits ? ld_cg_f32(s2 + (size_t)(s + j) * PE) : 0.f;
             }
 #pragma unroll
             for (int j = 0; j < 8; ++j)
                 if (s + j < splits) {
                     a1 = fmaf(f1[s + j], x[j], a1);
-                    a2 = fmaf(f2[s + j], y[j], a2);
+                    if (diff) a2 = fmaf(f2[s + j], y[j], a2);
                 }
         }
-        o[i] = a1 - L.lambda * a2;
+        o[i] = diff ? a1 - L.lambda * a2 : a1;
     }
     csync();
+    if (!diff) {
+        float* dst = (L.mixer == MKBH_LATENT_ATTENTION ? side_latent(g) : g.mixed) + (size_t)kvh * per * E;
+        const float2* turn = L.value_rope == nullptr ? nullptr : reinterpret_cast<const float2*>(L.value_rope) + (size_t)c.pos * (E / 2);
+        for (int i = tid; i < per * E; i += kConsumers) {
+            float y = o[i];
+            if (turn != nullptr) {  // (an even number of elements per head)
+                const float2 r = __ldg(turn + (i % E >> 1));
+                y = y * r.x + (i & 1 ? -r.y : r.y) * o[i ^ 1];
+            }
+            dst[i] = y;
+        }
+        return;
+    }
     for (int hh = warp; hh < per; hh += kConsumerWarps) {
         float s = 0.f;
         for (int e = lane; e < E; e += 32) s = fmaf(o[hh * E + e], o[hh * E + e], s);
@@ -974,6 +1166,32 @@ __device__ __forceinline__ void merge_splits(const Params& pr, const Desc& d, fl
     const float* gate = g.proj + L.heads * 2 * L.dim + (size_t)kvh * per * E;
     for (int i = tid; i < per * E; i += kConsumers)
         g.mixed[(size_t)kvh * per * E + i] = o[i] * norm[i / E] * sigmoid_f(ld_cg_f32(gate + i));
+}
+
+// Short convolutions over time: keep this token's inputs and sum up the terms of the next token's
+// earlier inputs.  `stash` holds the normalised channels of the instruction's share of the mixer's
+// input, `u` is this thread's row of the stacked projection before its convolution.
+__device__ __forceinline__ void keep_input(float now, const float* w, float* hist, float* next, int taps, size_t ld, int pos) {
+    float s = __ldg(w + (taps - 2) * ld) * now;
+    for (int i = 1; i <= taps - 2 && i <= pos; ++i) s = fmaf(__ldg(w + (taps - 2 - i) * ld), hist[((pos - i) % (taps - 1)) * ld], s);
+    hist[(pos % (taps - 1)) * ld] = now;
+    *next = s;
+}
+__device__ __forceinline__ void publish_convolutions(const Params& p, const Cta& c, const Desc& d, const float* stash, float u) {
+    const MkbhGlobals& g = p.g;
+    const MkbhLayer& L = d.L;
+    const int tid = threadIdx.x, lo = (int)((long long)g.width * d.a0 / L.in_rows), hi = (int)((long long)g.width * d.a1 / L.in_rows);
+    if (L.canon_taps > 1 && tid < hi - lo) {
+        const int ch = lo + tid;
+        keep_input(stash[tid] * __ldg(L.norm1 + ch), L.canon_w + ch,
+                   L.canon_hist + (size_t)g.slot * (L.canon_taps - 1) * g.width + ch,
+                   L.canon_part + ((size_t)g.slot * 2 + ((c.pos + 1) & 1)) * g.width + ch, L.canon_taps, g.width, c.pos);
+    }
+    if (L.conv_taps > 1 && tid < d.a1 - d.a0) {
+        const int row = d.a0 + tid;
+        keep_input(u, L.conv_w + row, L.conv_hist + (size_t)g.slot * (L.conv_taps - 1) * L.in_rows + row,
+                   L.conv_part + (size_t)g.slot * L.in_rows + row, L.conv_taps, L.in_rows, c.pos);
+    }
 }
 
 __device__ __forceinline__ unsigned long long argmax_key(float v, int i) {
@@ -988,6 +1206,7 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
     const int tid = threadIdx.x, warp = tid >> 5;
     float* act = reinterpret_cast<float*>(c.gb + sm.act);
     float* red = reinterpret_cast<float*>(c.gb + sm.red);
+    float* stash = reinterpret_cast<float*>(c.gb + sm.stash);
     int* counters = g.counters + 2;
     uint32_t slot = 0, phase = 0, vecs = 0;
     int turn = 0;
@@ -1026,12 +1245,16 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             if (!ok) c.ctl[0] = 1;
             ++vecs;
         }
+        const bool conv = op == MKBH_OP_NORM_PROJ && L.conv_taps > 0;
+        float* conv_part = conv ? L.conv_part + (size_t)g.slot * L.in_rows + d.a0 + tid : nullptr;
+        const float earlier = conv && c.pos > 0 && tid < d.a1 - d.a0 ? *conv_part : 0.f;  // earlier inputs' terms
         // ---- the producers ----
         if (tid == 0 && d.wait_idx >= 0)
             poll_counter(counters + d.wait_idx, d.wait_thr, c.ctl, g.status, p.timeout_ns, i, op);
         if (!agree(c)) return;
         rec(1);
         bool signal = true;
+        float kept = 0.f;  // this thread's row before the convolution
         if (op == MKBH_OP_DELTA_STEP) {
             delta_step<T>(p, c, d, act, vec, rowv, state);
             csync();
@@ -1051,26 +1274,47 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             }
             csync();
             signal = c.ctl[1] != 0;
-            if (signal) merge_splits(p, d, act);
+            if (signal) merge_splits(p, c, d, act);
             csync();
-        } else if (op >= MKBH_OP_NORM_PROJ && op <= MKBH_OP_HEAD) {
+        } else if (op >= MKBH_OP_NORM_PROJ && op <= MKBH_OP_EXPAND) {
             const int rows = d.a1 - d.a0, K = d.row_bytes / (int)sizeof(T);
-            const bool adds = op == MKBH_OP_OUT_PROJ || op == MKBH_OP_DOWN;
+            // channels whose input this instruction keeps for the convolution of later tokens
+            const bool canon = op == MKBH_OP_NORM_PROJ && L.canon_taps > 1;
+            const int stash_lo = canon ? (int)((long long)g.width * d.a0 / L.in_rows) : 0;
+            const int stash_hi = canon ? (int)((long long)g.width * d.a1 / L.in_rows) : 0;
+            const bool aside = op == MKBH_OP_DOWN && L.parallel;  // the output projection adds it
+            const bool adds = op == MKBH_OP_OUT_PROJ || (op == MKBH_OP_DOWN && !L.parallel);
+            float* x = g.x + (size_t)L.x_buf * g.width;
+            const bool first = d.layer == 0 && (op == MKBH_OP_ENTER || L.enter_w == nullptr);  // the stream is the embedding
             // this instruction is the only writer of its rows of the residual stream
-            const float old = adds && tid < rows ? ld_cg_f32(g.x + d.a0 + tid) : 0.f;
+            float old = adds && tid < rows ? ld_cg_f32(x + d.a0 + tid) : 0.f;
+            if (op == MKBH_OP_OUT_PROJ && L.parallel && L.ff && tid < rows) old += ld_cg_f32(side_out(g) + d.a0 + tid);
             if (op == MKBH_OP_OUT_PROJ) {
                 if (L.mixer == MKBH_DELTA_RULE) delta_activation(p, L, reinterpret_cast<const float*>(vec), act);
                 else if (K <= 8192) plain_activation<16>(g.mixed, L.heads * L.vdim, act);
                 else plain_activation<32>(g.mixed, L.heads * L.vdim, act);
+            } else if (op == MKBH_OP_DOWN && L.ff_kind == MKBH_CLAMPED_GLU) {
+                if (K <= 8192) plain_activation<16>(side_in(g), L.ff, act);
+                else plain_activation<32>(side_in(g), L.ff, act);
             } else if (op == MKBH_OP_DOWN) {
                 if (K <= 8192) poly_activation<16>(p, L, act, red, turn);
                 else poly_activation<32>(p, L, act, red, turn);
+            } else if (op == MKBH_OP_ABSORB) {
+                plain_activation<4>(g.proj + (size_t)(d.a0 / L.rank) * (L.dim + L.rot_dim), L.dim, act);
+            } else if (op == MKBH_OP_EXPAND) {
+                plain_activation<4>(side_latent(g) + (size_t)(d.a0 / L.vdim) * L.rank, L.rank, act);
+            } else if (op == MKBH_OP_ENTER) {
+                enter_activation<T>(g, first ? nullptr : g.x + (size_t)(L.x_buf ^ 1) * g.width, act);
             } else {
                 const float* w = reinterpret_cast<const float*>(vec);
-                const bool first = op == MKBH_OP_NORM_PROJ && d.layer == 0, publish = first && d.a0 == 0;
-                if (K <= 2048) norm_activation<T, 4>(p, c, w, act, red, turn, first, publish);
-                else if (K <= 8192) norm_activation<T, 16>(p, c, w, act, red, turn, first, publish);
-                else norm_activation<T, 32>(p, c, w, act, red, turn, first, publish);
+                const float* part = d.part_off >= 0 ? reinterpret_cast<const float*>(c.gb + sm.vec + d.part_off) : nullptr;
+                const bool in = op == MKBH_OP_NORM_PROJ;
+                const float* src = first && (in || (op == MKBH_OP_NORM_UP && L.parallel)) ? nullptr
+                                   : op == MKBH_OP_HEAD ? g.x + (size_t)p.last_buf * g.width : x;
+                float* publish = src == nullptr && in && d.a0 == 0 ? x : nullptr;
+                if (K <= 2048) norm_activation<T, 4>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
+                else if (K <= 8192) norm_activation<T, 16>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
+                else norm_activation<T, 32>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
             }
             csync();
             if (tid == 0 && d.has_vec) mbar_arrive(c.bar(kVecEmpty));
@@ -1086,8 +1330,25 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
                 float y = 0.f;
                 for (int k = 0; k < d.groups; ++k) y += act[tid * d.groups + k];
                 const int row = d.a0 + tid;
+                kept = y;
                 if (adds) {
-                    g.x[row] = fmaf(rowv[tid], y, old);
+                    x[row] = fmaf(d.row_off >= 0 ? rowv[tid] : 1.f, y, old);
+                } else if (conv) {
+                    g.proj[row] = fmaf(rowv[tid], y, earlier);
+                } else if (op == MKBH_OP_ENTER) {
+                    x[row] = y;
+                } else if (aside) {
+                    side_out(g)[row] = y;
+                } else if (op == MKBH_OP_ABSORB) {
+                    side_query(g)[row] = y;
+                } else if (op == MKBH_OP_EXPAND) {
+                    g.mixed[row] = y;
+                } else if (op == MKBH_OP_NORM_UP && L.ff_kind == MKBH_CLAMPED_GLU) {  // rows alternate gate, up
+                    if ((tid & 1) == 0) {
+                        float up = 0.f;
+                        for (int k = 0; k < d.groups; ++k) up += act[(tid + 1) * d.groups + k];
+                        side_in(g)[row >> 1] = clamped_glu(y, up, L.glu_limit, L.glu_alpha);
+                    }
                 } else if (op == MKBH_OP_HEAD) {
                     g.logits[row] = y;
                     best = argmax_key(y, row);
@@ -1122,10 +1383,12 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             if (tid == 0) report(g.status, c.ctl, MKBH_ERR_BAD_OPCODE, 1, i, op, 0, 0, 0);
             return;
         }
-        if (tid == 0) {
-            if (signal) red_release_gpu_add(counters + d.arrive_idx, 1);
-            mbar_arrive(c.bar(kDescEmpty + (i & 1)));
+        if (tid == 0 && signal) red_release_gpu_add(counters + d.arrive_idx, 1);
+        if (op == MKBH_OP_NORM_PROJ && (L.canon_taps > 1 || L.conv_taps > 1)) {  // for later tokens only
+            publish_convolutions(p, c, d, stash, kept);
+            csync();
         }
+        if (tid == 0) mbar_arrive(c.bar(kDescEmpty + (i & 1)));
         rec(4);
     }
 }
@@ -1173,32 +1436,37 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     p.timeout_ns = (g.wait_timeout_ms ? g.wait_timeout_ms : 2000u) * 1000000ull;
     if (!(g.flags & MKBH_FLAG_RECORD_TIMINGS)) p.g.timings = nullptr;
     int act = max(kScratchMin, 4 * pad8(g.width)), vec = 4 * g.width;
+    bool part = false;
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
         const bool delta = L.mixer == MKBH_DELTA_RULE;
-        act = max(act, 4 * pad8(L.heads * (delta ? L.dim : L.vdim)));
+        act = max(act, 4 * pad8(mixer_out(L)));
         if (delta) {
             act = max(act, 4 * (L.rank + 4 + L.dim));
             vec = max(vec, max(4 * L.heads * L.dim, L.dim * L.rank * (int)sizeof(T)));
         }
         if (L.ff) act = max(act, 4 * pad8(L.ff));
+        if (L.enter_w) act = max(act, 4 * pad8(2 * g.width));
+        part |= L.canon_taps > 1;
     }
     // keys staged at a time: 64, fewer when a tile of wide heads would not fit
     p.attn_chunk = 64;
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
-        if (L.mixer != MKBH_DIFF_ATTENTION) continue;
-        const int per = L.heads / L.kv_heads, nq = 2 * per;
-        act = max(act, max(4 * merge_scratch_floats(nq, g.max_splits, per, L.vdim), attn_scratch_bytes<T>(nq, L.dim, L.vdim, 8)));
+        if (!is_attention(L)) continue;
+        const int per = L.heads / L.kv_heads, nq = attn_maps(L) * per;
+        act = max(act, max(4 * merge_scratch_floats(nq, g.max_splits, per, attn_vdim(L)),
+                           attn_scratch_bytes<T>(L, L.mixer == MKBH_LATENT_ATTENTION && sizeof(T) == 2 ? 32 : 8)));
     }
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
-        if (L.mixer != MKBH_DIFF_ATTENTION) continue;
-        while (p.attn_chunk > 8 && attn_scratch_bytes<T>(2 * (L.heads / L.kv_heads), L.dim, L.vdim, p.attn_chunk) > act)
-            p.attn_chunk -= 8;
+        if (!is_attention(L)) continue;
+        while (p.attn_chunk > 8 && attn_scratch_bytes<T>(L, p.attn_chunk) > act) p.attn_chunk -= 8;
     }
+    p.last_buf = g.layers_host[g.num_layers - 1].x_buf;
     p.act_bytes = (act + 127) & ~127;
-    p.vec_bytes = (vec + 32 + 127) & ~127;
+    p.part_base = (vec + 32 + 127) & ~127;
+    p.vec_bytes = p.part_base + (part ? (4 * g.width + 32 + 127) & ~127 : 0);
     const int fixed = Smem(0, p.act_bytes, p.vec_bytes).total + 128;
     p.stages = (kSmemLimit - fixed) / kStage;
     if (p.stages > kMaxStages) p.stages = kMaxStages;

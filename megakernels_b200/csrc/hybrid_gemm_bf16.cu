@@ -4,8 +4,8 @@
 // Persistent, warp-specialised: one producer thread (TMA, 128-byte swizzle), one MMA thread
 // (tcgen05.mma, M = 128 tokens, N = kBN features), four epilogue warps that read one of two
 // accumulators back while the other is being filled.  The epilogue goes through shared memory so
-// that every store is a full 128-byte row segment, adds the bias or applies the layer scale and
-// adds to the 32-bit residual stream.
+// that stores are row segments: plus the bias, times the layer scale into the 32-bit residual stream,
+// in bf16, or the gated unit of neighbouring columns in bf16.
 #include "hybrid_kernels.h"
 
 #include <cuda.h>
@@ -196,11 +196,28 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant
 #pragma unroll
                 for (int j = 0; j < 32; ++j) tr[lane * kEpiStride + j] = __uint_as_float(r[j]);
                 __syncwarp();
+                if (e.what == Result::kCast) {  // two rows at a time, two columns per lane
+                    const int col = 2 * (lane & 15), n = n0 + c0 + col;
+                    bf16* o = static_cast<bf16*>(e.cast) + (size_t)m0 * e.ld + n;
+                    for (int i = lane >> 4; i < rows; i += 2) {
+                        const float *v = tr + i * kEpiStride + col;
+                        if (n + 1 < s.N) *reinterpret_cast<uint32_t*>(o + (size_t)i * e.ld) = mkb::pack_bf16x2(v[0], v[1]);
+                        else if (n < s.N) o[(size_t)i * e.ld] = __float2bfloat16_rn(v[0]);
+                    }
+                } else if (e.what == Result::kGlu) {  // 16 units of a row per half warp
+                    const int col = 2 * (lane & 15), n = n0 + c0 + col;
+                    bf16* o = static_cast<bf16*>(e.cast) + (size_t)m0 * e.ld + n / 2;
+                    if (n < s.N)  // (N is even)
+                        for (int i = lane >> 4; i < rows; i += 2) {
+                            const float* v = tr + i * kEpiStride + col;
+                            o[(size_t)i * e.ld] = __float2bfloat16_rn(clamped_glu(v[0], v[1], e.limit, e.alpha));
+                        }
+                }
                 const int n = n0 + c0 + lane;
-                if (n < s.N) {
+                if (n < s.N && e.what <= Result::kAdd) {
                     float* o = e.out + (size_t)m0 * e.ld + n;
-                    if (e.scale) {
-                        const float f = __ldg(e.scale + n);
+                    if (e.what == Result::kAdd) {
+                        const float f = e.scale ? __ldg(e.scale + n) : 1.f;
                         // (this tile is the only writer of these elements: one addition each, in L2)
                         for (int i = 0; i < rows; ++i)
                             asm volatile("red.global.add.f32 [%0], %1;" ::"l"(o + (size_t)i * e.ld), "f"(f * tr[i * kEpiStride + lane])

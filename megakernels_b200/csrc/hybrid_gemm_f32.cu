@@ -17,9 +17,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     float acc[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += kDepth) {
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f), w = a;
-        if (k0 + lc < K) {  // K is a multiple of 8
+        if (k0 + lc < K) {  // (rows are padded to 8: what lies beyond K may be read, and is dropped)
             if (t0 + lr < T) a = *reinterpret_cast<const float4*>(A + (size_t)(t0 + lr) * lda + k0 + lc);
             if (n0 + lr < N) w = *reinterpret_cast<const float4*>(W + (size_t)(n0 + lr) * ldw + k0 + lc);
+            if (k0 + lc + 1 >= K) a.y = 0.f;
+            if (k0 + lc + 2 >= K) a.z = 0.f;
+            if (k0 + lc + 3 >= K) a.w = 0.f;
         }
         sa[lc][lr] = a.x; sa[lc + 1][lr] = a.y; sa[lc + 2][lr] = a.z; sa[lc + 3][lr] = a.w;
         sw[lc][lr] = w.x; sw[lc + 1][lr] = w.y; sw[lc + 2][lr] = w.z; sw[lc + 3][lr] = w.w;
@@ -42,8 +45,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
         for (int j = 0; j < 4; ++j) {
             const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
             if (t >= T || n >= N) continue;
-            float* o = e.out + (size_t)t * e.ld + n;
-            if (e.scale) *o += e.scale[n] * acc[i][j];
+            if (e.what == Result::kGlu) {  // (N is even: both columns are there)
+                if ((j & 1) == 0)
+                    static_cast<float*>(e.cast)[(size_t)t * e.ld + n / 2] = clamped_glu(acc[i][j], acc[i][j | 1], e.limit, e.alpha);
+                continue;
+            }
+            float* o = (e.what == Result::kCast ? static_cast<float*>(e.cast) : e.out) + (size_t)t * e.ld + n;
+            if (e.what == Result::kAdd) *o += (e.scale ? e.scale[n] : 1.f) * acc[i][j];
             else *o = acc[i][j] + (e.bias ? e.bias[n] : 0.f);
         }
 }

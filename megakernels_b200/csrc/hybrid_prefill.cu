@@ -1,5 +1,5 @@
-// Prefill kernels of the hybrid models other than the matrix products: embedding, layer norm,
-// PolyNorm, the recurrence over a portion of tokens, and windowed differential attention.
+// Prefill kernels of the hybrid models other than the matrix products: embedding, norms, short
+// convolutions, PolyNorm, the recurrence over a portion of tokens, and attention.
 // Norms, scores, softmax weights, decays and the recurrent state are 32-bit in both builds.
 #include "hybrid_kernels.h"
 
@@ -17,13 +17,27 @@ __global__ void embed_kernel(const int32_t* __restrict__ tokens, int pos0, int v
     tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;  // ids are checked on the host; never read outside the table
     for (int i = threadIdx.x; i < width; i += blockDim.x)
         x[(size_t)t * width + i] =
-            to_f(embed[(size_t)tok * width + i]) * scale + to_f(pos[(size_t)(pos0 + t) * width + i]);
+            to_f(embed[(size_t)tok * width + i]) * scale + (pos != nullptr ? to_f(pos[(size_t)(pos0 + t) * width + i]) : 0.f);
 }
 
-// ---- layer norm --------------------------------------------------------------------------- //
+// [residual stream | embedding] of every token
+template <typename T>
+__global__ void enter_kernel(const int32_t* __restrict__ tokens, int vocab, int width, float scale, const T* __restrict__ embed,
+                             const float* __restrict__ x, T* __restrict__ out, int64_t ld) {
+    const int t = blockIdx.x;
+    int tok = tokens[t];
+    tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;
+    T* o = out + (size_t)t * ld;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        o[i] = from_f<T>(x[(size_t)t * width + i]);
+        o[width + i] = from_f<T>(to_f(embed[(size_t)tok * width + i]) * scale);
+    }
+}
+
+// ---- norms --------------------------------------------------------------------------- //
 template <typename T>
 __global__ void __launch_bounds__(kThreads) norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows,
-                                                        int width, const float* __restrict__ w, float eps,
+                                                        int width, const float* __restrict__ w, float eps, bool centre,
                                                         T* __restrict__ out, int64_t ld) {
     __shared__ float red[kThreads / 32];
     const float* row = x + (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * width;
@@ -37,8 +51,11 @@ __global__ void __launch_bounds__(kThreads) norm_kernel(const float* __restrict_
         s[0] += v[k];
     }
     for (int i = threadIdx.x + R * kThreads; i < width; i += kThreads) s[0] += row[i];
-    block_sum<1, kThreads>(s, red);
-    const float mean = s[0] / width;
+    float mean = 0.f;
+    if (centre) {
+        block_sum<1, kThreads>(s, red);
+        mean = s[0] / width;
+    }
     s[0] = 0.f;
 #pragma unroll
     for (int k = 0; k < R; ++k) {
@@ -55,6 +72,85 @@ __global__ void __launch_bounds__(kThreads) norm_kernel(const float* __restrict_
     }
     for (int i = threadIdx.x + R * kThreads; i < width; i += kThreads) o[i] = from_f<T>((row[i] - mean) * inv * w[i]);
     for (int i = width + threadIdx.x; i < pad8(width); i += kThreads) o[i] = from_f<T>(0.f);
+}
+
+// The mixer's input h = N(x) w1, plus a causal convolution over time of its channels, and the input
+// N(x) w2 of a feed-forward beside the mixer.  A block takes kNormTokens tokens and, before them,
+// the inputs their convolution reaches back to (from the tokens of this portion, else from `hist`).
+// The portion's last taps - 1 inputs go to `tail`, latest first.
+constexpr int kNormTokens = 8;
+template <typename T>
+__global__ void __launch_bounds__(kThreads) canon_norm_kernel(const float* __restrict__ x, int n, int pos0, int width,
+                                                              const float* __restrict__ w1, const float* __restrict__ w2,
+                                                              float eps, bool centre, const float* __restrict__ taps_w, int taps,
+                                                              const float* __restrict__ hist, float* __restrict__ tail,
+                                                              T* __restrict__ out, T* __restrict__ out2, int64_t ld) {
+    extern __shared__ __align__(16) float ring[];  // [taps][width]
+    __shared__ float red[kThreads / 32];
+    const int t0 = blockIdx.x * kNormTokens, t1 = min(n, t0 + kNormTokens), back = taps > 1 ? taps - 1 : 0;
+    for (int t = t0 - back; t < t1; ++t) {
+        float* h = ring + (taps > 0 ? (t + back) % taps : 0) * width;
+        if (t < 0) {  // (every thread reads back only what it wrote itself)
+            const int pos = pos0 + t;
+            for (int i = threadIdx.x; i < width; i += kThreads) h[i] = pos >= 0 ? hist[(size_t)(pos % back) * width + i] : 0.f;
+            continue;
+        }
+        const float* row = x + (size_t)t * width;
+        float mean = 0.f, s[1] = {0.f};
+        if (centre) {
+            for (int i = threadIdx.x; i < width; i += kThreads) s[0] += row[i];
+            block_sum<1, kThreads>(s, red);
+            mean = s[0] / width;
+            s[0] = 0.f;
+        }
+        for (int i = threadIdx.x; i < width; i += kThreads) s[0] += (row[i] - mean) * (row[i] - mean);
+        block_sum<1, kThreads>(s, red);
+        const float inv = 1.f / sqrtf(s[0] / width + eps);
+        const bool live = t >= t0;
+        for (int i = threadIdx.x; i < width; i += kThreads) {
+            const float y = (row[i] - mean) * inv;
+            float v = y * w1[i];
+            if (taps > 0) {
+                h[i] = v;
+                if (live) {
+                    float c = v;
+                    for (int j = 0; j < taps; ++j) c = fmaf(taps_w[(size_t)j * width + i], ring[((t + back - (taps - 1) + j) % taps) * width + i], c);
+                    if (n - 1 - t < back) tail[(size_t)(n - 1 - t) * width + i] = v;
+                    v = c;
+                }
+            }
+            if (live) {
+                out[(size_t)t * ld + i] = from_f<T>(v);
+                if (out2 != nullptr) out2[(size_t)t * ld + i] = from_f<T>(y * w2[i]);
+            }
+        }
+    }
+}
+
+// After a portion: the last taps - 1 inputs of a convolution by position, and the sum of the next
+// position's terms of earlier inputs.  `back(i)` is the input i tokens before the portion's end.
+template <typename Back>
+__device__ __forceinline__ void keep_channel(const float* w, float* hist, float* next, int taps, size_t ld, int n, int end, Back back) {
+    // end: position of the portion's last token
+    float s = 0.f;
+    for (int i = 0; i < taps - 1 && i <= end; ++i) {
+        const float v = i < n ? back(i) : hist[((end - i) % (taps - 1)) * ld];
+        s = fmaf(w[(taps - 2 - i) * ld], v, s);
+    }
+    for (int i = 0; i < taps - 1 && i < n; ++i) hist[((end - i) % (taps - 1)) * ld] = back(i);
+    *next = s;
+}
+__global__ void __launch_bounds__(kThreads) keep_inputs_kernel(const MkbhLayer L, int slot, int n, int pos0, int width,
+                                                               const float* __restrict__ tail, const float* __restrict__ proj, int64_t ld) {
+    const int ch = blockIdx.x * kThreads + threadIdx.x, end = pos0 + n - 1;
+    if (L.canon_taps > 1 && ch < width)
+        keep_channel(L.canon_w + ch, L.canon_hist + (size_t)slot * (L.canon_taps - 1) * width + ch,
+                     L.canon_part + ((size_t)slot * 2 + ((end + 1) & 1)) * width + ch, L.canon_taps, width, n, end,
+                     [&](int i) { return tail[(size_t)i * width + ch]; });
+    if (L.conv_taps > 1 && ch < L.in_rows)
+        keep_channel(L.conv_w + ch, L.conv_hist + (size_t)slot * (L.conv_taps - 1) * L.in_rows + ch,
+                     L.conv_part + (size_t)slot * L.in_rows + ch, L.conv_taps, L.in_rows, n, end,
+                     [&](int i) { return proj[(size_t)(n - 1 - i) * ld + ch]; });
 }
 
 // ---- PolyNorm ----------------------------------------------------------------------------- //
@@ -434,7 +530,7 @@ __global__ void __launch_bounds__(kAttnThreads) attention_kernel(const float* __
     // (q takes the precision of the activations it would have had as a stored tensor)
     for (int i = tid; i < 2 * D; i += kAttnThreads) q[i] = to_f(from_f<T>(row[h * 2 * D + i]));
     __syncthreads();
-    const KeyRange keys(pos0 + t, L.window, L.keep_first);
+    const KeyRange keys(pos0 + t, L.window, L.keep_first, L.chunk);
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, acc[2][kAttnMaxE] = {};
     for (int c0 = 0; c0 < keys.count; c0 += kAttnThreads) {
         const int nk = min(kAttnThreads, keys.count - c0);
@@ -497,6 +593,166 @@ __global__ void __launch_bounds__(kAttnThreads) attention_kernel(const float* __
         for (int i = H * E + tid; i < pad8(H * E); i += kAttnThreads) out[(size_t)t * ldo + i] = from_f<T>(0.f);
 }
 
+// ---- rotary and latent attention ------------------------------------------------------------- //
+// Operands of a portion.  A warp takes one vector (a query, key or value head; the latent, its
+// rotated part) of kOpTokens tokens: convolution over time, norm, rotation of neighbours, and
+// stores it as an element of the query buffer or as a cache row.
+constexpr int kOpTokens = 8;
+struct OperandArgs {
+    const float* proj;
+    int64_t ld, ldq;
+    int n, pos0;
+    MkbhLayer L;
+    const float* hist;  // of the projection's convolution, this slot
+    float eps;
+    void *query, *kc, *vc;  // (cache bases of the slot)
+};
+template <typename T, int J>
+__device__ __forceinline__ void operand_vector(const OperandArgs& a, int t, int col, int len, const float* w, const float2* rope,
+                                               int rot, T* dst) {
+    const MkbhLayer& L = a.L;
+    const int lane = threadIdx.x & 31, taps = L.conv_taps, pos = a.pos0 + t;
+    float u[J][2], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < J; ++j)
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+            const int i = 2 * (lane + 32 * j) + b, ch = col + i;
+            float v = 0.f;
+            if (i < len) {
+                v = a.proj[(size_t)t * a.ld + ch];
+                if (taps > 0) {
+                    v *= L.conv_w[(size_t)(taps - 1) * L.in_rows + ch];
+                    for (int k = 1; k < taps && k <= pos; ++k)  // k tokens ago
+                        v = fmaf(L.conv_w[(size_t)(taps - 1 - k) * L.in_rows + ch],
+                                 k <= t ? a.proj[(size_t)(t - k) * a.ld + ch] : a.hist[(size_t)((pos - k) % (taps - 1)) * L.in_rows + ch], v);
+                }
+            }
+            u[j][b] = v;
+            s = fmaf(v, v, s);
+        }
+    const float inv = w != nullptr ? 1.f / sqrtf(warp_sum(s) / len + a.eps) : 1.f;
+#pragma unroll
+    for (int j = 0; j < J; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        if (i >= len) break;
+        float x = u[j][0], y = u[j][1];
+        if (w != nullptr) {
+            x *= inv * w[i];
+            if (i + 1 < len) y *= inv * w[i + 1];
+        }
+        if (i < rot) {
+            const float2 r = rope[i >> 1];
+            const float z = x * r.x - y * r.y;
+            y = y * r.x + x * r.y;
+            x = z;
+        }
+        dst[i] = from_f<T>(x);
+        if (i + 1 < len) dst[i + 1] = from_f<T>(y);
+    }
+}
+template <typename T, int J>
+__global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const OperandArgs a) {
+    const MkbhLayer& L = a.L;
+    const int task = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5), H = L.heads, G = L.kv_heads;
+    const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
+    if (task >= (latent ? H + 1 : H + 2 * G)) return;
+    const int t1 = min(a.n, ((int)blockIdx.x + 1) * kOpTokens);
+    for (int t = blockIdx.x * kOpTokens; t < t1; ++t) {
+        const int pos = a.pos0 + t;
+        const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)pos * (L.rope_dims / 2);
+        const size_t row = cache_row(pos, L.cache_keep, L.cache_ring);
+        T* q = static_cast<T*>(a.query) + (size_t)t * a.ldq;
+        if (latent) {
+            const int hd = L.dim + L.rot_dim;
+            if (task < H) {
+                operand_vector<T, J>(a, t, task * hd, L.dim, nullptr, nullptr, 0, q + task * hd);
+                operand_vector<T, J>(a, t, task * hd + L.dim, L.rot_dim, nullptr, rope, L.rope_dims, q + task * hd + L.dim);
+            } else {
+                T* kc = static_cast<T*>(a.kc) + row * latent_row(L);
+                operand_vector<T, J>(a, t, H * hd, L.rank, L.k_norm, nullptr, 0, kc);
+                operand_vector<T, J>(a, t, H * hd + L.rank, L.rot_dim, nullptr, rope, L.rope_dims, kc + pad8(L.rank));
+            }
+        } else if (task < H) {
+            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.q_norm, rope, L.rope_dims, q + task * L.dim);
+        } else if (task < H + G) {
+            const int g = task - H;
+            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.k_norm, rope, L.rope_dims, static_cast<T*>(a.kc) + (row * G + g) * L.dim);
+        } else {
+            const int g = task - H - G;
+            const float2* turn = L.value_rope ? reinterpret_cast<const float2*>(L.value_rope) + (size_t)pos * (L.vdim / 2) : nullptr;
+            operand_vector<T, J>(a, t, (H + G) * L.dim + g * L.vdim, L.vdim, nullptr, turn, turn ? L.vdim : 0,
+                                 static_cast<T*>(a.vc) + (row * G + g) * L.vdim);
+        }
+    }
+}
+
+// One CTA per (token, query head), 128 keys at a time, online softmax.  The float build's
+// attention, and the bf16 build's for head sizes hybrid_attention.cu does not take.
+template <typename T>
+__global__ void __launch_bounds__(kAttnThreads) rotary_attention_kernel(const T* __restrict__ query, int64_t ldq, int pos0, const MkbhLayer L,
+                                                                        const KeySource<T> src, T* __restrict__ out, int64_t ldo) {
+    extern __shared__ float sm[];  // q [split + rest], p [128], o [vdim]
+    __shared__ float red[kAttnThreads / 32];
+    const int A = src.split, B = src.rest, E = L.vdim, H = L.heads;
+    const int t = blockIdx.x, h = blockIdx.y, g = h / src.per, tid = threadIdx.x, pos = pos0 + t;
+    float *q = sm, *p = sm + A + B, *o = p + kAttnThreads;
+    for (int i = tid; i < A + B; i += kAttnThreads) q[i] = to_f(query[(size_t)t * ldq + h * (A + B) + i]);
+    __syncthreads();
+    const KeyRange keys(pos, L.window, L.keep_first, L.chunk);
+    const float scale = L.scale * (L.temp ? L.temp[h] : 1.f);
+    float m = L.sink ? L.sink[h] : -INFINITY, l = L.sink ? 1.f : 0.f, acc[kAttnMaxE] = {};
+    for (int c0 = 0; c0 < keys.count; c0 += kAttnThreads) {
+        const int nk = min(kAttnThreads, keys.count - c0);
+        float s = -INFINITY;
+        if (tid < nk) {
+            const size_t row = cache_row(keys.key(c0 + tid), src.keep, src.ring);
+            const T *k = src.keys + row * src.key_ld + g * A, *r = src.shared + row * src.shared_ld;
+            float d = 0.f;
+            for (int i = 0; i < A; ++i) d = fmaf(q[i], to_f(k[i]), d);
+            for (int i = 0; i < B; ++i) d = fmaf(q[A + i], to_f(r[i]), d);
+            s = d * scale;
+        }
+        float x = warp_max(s);
+        if ((tid & 31) == 0) red[tid >> 5] = x;
+        __syncthreads();
+        x = m;
+        for (int w = 0; w < kAttnThreads / 32; ++w) x = fmaxf(x, red[w]);
+        const float f = expf(m - x);
+        m = x;
+        s = tid < nk ? expf(s - x) : 0.f;
+        p[tid] = s;
+        __syncthreads();
+        float ps[1] = {s};
+        block_sum<1, kAttnThreads>(ps, red);
+        l = l * f + ps[0];
+        for (int ei = 0; ei < kAttnMaxE; ++ei) {
+            const int e = tid + ei * kAttnThreads;
+            if (e >= E) break;
+            float y = acc[ei] * f;
+            for (int j = 0; j < nk; ++j)
+                y = fmaf(p[j], to_f(src.values[(size_t)cache_row(keys.key(c0 + j), src.keep, src.ring) * src.value_ld + g * E + e]), y);
+            acc[ei] = y;
+        }
+        __syncthreads();
+    }
+    for (int ei = 0; ei < kAttnMaxE; ++ei)
+        if (tid + ei * kAttnThreads < E) o[tid + ei * kAttnThreads] = acc[ei] / l;
+    __syncthreads();
+    const float2* turn = L.value_rope ? reinterpret_cast<const float2*>(L.value_rope) + (size_t)pos * (E / 2) : nullptr;
+    T* dst = out + (size_t)t * ldo + h * E;
+    for (int e = tid; e < E; e += kAttnThreads) {
+        float y = o[e];
+        if (turn != nullptr) {  // back by the query's angle
+            const float2 r = turn[e >> 1];
+            y = y * r.x + (e & 1 ? -r.y : r.y) * o[e ^ 1];
+        }
+        dst[e] = from_f<T>(y);
+    }
+    if (h == 0)
+        for (int i = H * E + tid; i < pad8(H * E); i += kAttnThreads) out[(size_t)t * ldo + i] = from_f<T>(0.f);
+}
+
 template <int M>
 cudaError_t launch_scan(const MkbhGlobals& g, const MkbhLayer& L, int64_t ld, float* state, cudaStream_t s) {
     static bool set[64] = {};
@@ -524,9 +780,64 @@ cudaError_t Prefill<T>::embed(const MkbhGlobals& g, cudaStream_t s) {
     return cudaGetLastError();
 }
 template <typename T>
-cudaError_t Prefill<T>::norm(const float* x, const int32_t* rows, int n, int width, const float* w, float eps, T* out,
-                             int64_t ld, cudaStream_t s) {
-    norm_kernel<T><<<n, kThreads, 0, s>>>(x, rows, width, w, eps, out, ld);
+cudaError_t Prefill<T>::enter(const MkbhGlobals& g, T* out, int64_t ld, cudaStream_t s) {
+    enter_kernel<T><<<g.num_tokens, 256, 0, s>>>(g.tokens, g.vocab, g.width, g.embed_scale, static_cast<const T*>(g.embed), g.x, out, ld);
+    return cudaGetLastError();
+}
+template <typename T>
+cudaError_t Prefill<T>::norm(const MkbhGlobals& g, const int32_t* rows, int n, const float* w, T* out, int64_t ld, cudaStream_t s) {
+    norm_kernel<T><<<n, kThreads, 0, s>>>(g.x, rows, g.width, w, g.eps, g.norm_kind == MKBH_LAYER_NORM, out, ld);
+    return cudaGetLastError();
+}
+template <typename T>
+cudaError_t Prefill<T>::canon_norm(const MkbhGlobals& g, const MkbhLayer& L, T* out, T* out2, int64_t ld, cudaStream_t s) {
+    static int set[64] = {};
+    const int n = g.num_tokens, smem = max(1, L.canon_taps) * g.width * 4;
+    int dev = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e != cudaSuccess) return e;
+    if (smem > 48 * 1024 && set[dev & 63] < smem) {
+        e = cudaFuncSetAttribute(canon_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return e;
+        set[dev & 63] = smem;
+    }
+    const float* hist = L.canon_hist + (L.canon_taps > 1 ? (size_t)g.slot * (L.canon_taps - 1) * g.width : 0);
+    canon_norm_kernel<T><<<(n + kNormTokens - 1) / kNormTokens, kThreads, smem, s>>>(
+        g.x, n, g.pos0, g.width, L.norm1, L.norm2, g.eps, g.norm_kind == MKBH_LAYER_NORM, L.canon_w, L.canon_taps, hist, g.tail, out, out2, ld);
+    return cudaGetLastError();
+}
+template <typename T>
+cudaError_t Prefill<T>::keep_inputs(const MkbhGlobals& g, const MkbhLayer& L, cudaStream_t s) {
+    const int channels = max(L.canon_taps > 1 ? g.width : 0, L.conv_taps > 1 ? L.in_rows : 0);
+    keep_inputs_kernel<<<(channels + kThreads - 1) / kThreads, kThreads, 0, s>>>(L, g.slot, g.num_tokens, g.pos0, g.width, g.tail, g.proj,
+                                                                                pad8(L.in_rows));
+    return cudaGetLastError();
+}
+template <typename T>
+cudaError_t Prefill<T>::rotary_operands(const MkbhGlobals& g, const MkbhLayer& L, cudaStream_t s) {
+    const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
+    const int n = g.num_tokens, tasks = latent ? L.heads + 1 : L.heads + 2 * L.kv_heads;
+    const int widest = latent ? max(max(L.dim, L.rot_dim), L.rank) : max(L.dim, L.vdim);
+    const size_t rows = (size_t)g.slot * (L.cache_keep + L.cache_ring);
+    OperandArgs a{g.proj, pad8(L.in_rows), latent ? (int64_t)pad8(L.heads * (L.dim + L.rot_dim)) : (int64_t)pad8(L.heads * L.dim), n, g.pos0, L,
+                  L.conv_hist + (L.conv_taps > 1 ? (size_t)g.slot * (L.conv_taps - 1) * L.in_rows : 0), g.eps, g.query,
+                  static_cast<T*>(L.k_cache) + rows * (latent ? latent_row(L) : L.kv_heads * L.dim),
+                  latent ? nullptr : static_cast<T*>(L.v_cache) + rows * L.kv_heads * L.vdim};
+    const dim3 grid((n + kOpTokens - 1) / kOpTokens, (tasks + kThreads / 32 - 1) / (kThreads / 32));
+    if (widest <= 64) rotary_operands_kernel<T, 1><<<grid, kThreads, 0, s>>>(a);
+    else if (widest <= 128) rotary_operands_kernel<T, 2><<<grid, kThreads, 0, s>>>(a);
+    else if (widest <= 256) rotary_operands_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
+    else rotary_operands_kernel<T, 8><<<grid, kThreads, 0, s>>>(a);
+    return cudaGetLastError();
+}
+template <typename T>
+cudaError_t Prefill<T>::rotary_attention(const MkbhGlobals& g, const MkbhLayer& L, T* out, int64_t ldo, cudaStream_t s) {
+    if constexpr (sizeof(T) == 2)
+        if (rotary_flash_supported(L)) return rotary_flash(g, L, out, ldo, s);
+    const KeySource<T> src = key_source<T>(g, L);
+    const int q = src.split + src.rest;
+    rotary_attention_kernel<T><<<dim3(g.num_tokens, L.heads), kAttnThreads, (q + kAttnThreads + L.vdim) * 4, s>>>(
+        static_cast<const T*>(g.query), pad8(L.heads * q), g.pos0, L, src, out, ldo);
     return cudaGetLastError();
 }
 template <typename T>

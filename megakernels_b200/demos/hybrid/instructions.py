@@ -16,7 +16,7 @@ from torch import Tensor
 from megakernels_b200.instructions import Instruction
 from megakernels_b200.utils import get_sm_count
 
-COUNTERS_PER_LAYER = 8  # MKBH_BARRIERS_PER_LAYER
+COUNTERS_PER_LAYER = 12  # MKBH_BARRIERS_PER_LAYER
 MAX_ROWS = 512  # output rows of an instruction
 PARTIAL_SUMS = 4096  # per-row, per-column-group sums an instruction may hold
 
@@ -31,7 +31,7 @@ class HybridGlobals:
 
     tokens: Tensor  # int32 [portion]
     want_rows: Tensor  # int32 [portion]
-    x: Tensor  # fp32 [portion, width]: the residual stream
+    x: Tensor  # fp32 [portion (decode: 2), width]: the residual stream
     proj: Tensor  # fp32 [portion, stacked projection rows or ff]
     mixed: Tensor  # fp32 [portion, mixer output]
     decay: Tensor  # fp32 [portion, recurrence channels]
@@ -39,12 +39,20 @@ class HybridGlobals:
     logits: Tensor  # fp32 [vocab]
     argmax_out: Tensor  # int32 [1]
     counters: Tensor  # int32, zeroed by every decode launch
-    arrivals: Tensor  # int32 [layers + 1, COUNTERS_PER_LAYER]
+    arrivals: Tensor  # int32 [layer runs + 1, COUNTERS_PER_LAYER]
     attn_part: Tensor  # fp32 [max heads, 2, max_splits, max vdim + 2]
     status: Tensor  # int32 [16]
     max_splits: int
     max_kv_heads: int
     part_vdim: int
+    query: Tensor  # model dtype [portion, heads * query/key size]: rotated queries
+    act2: Tensor  # model dtype [portion, width]: input of a feed-forward beside a mixer
+    ffn: Tensor  # model dtype [portion, ff]: gated units
+    keys: Tensor  # model dtype [positions, heads * (dim + vdim)]: keys and values expanded from latents
+    tail: Tensor  # fp32 [taps, width]: the portion's last inputs of the input convolution
+    side: Tensor  # fp32 [side_ff + width + 2 * side_rank]: decode vectors beside the stacked projection
+    side_ff: int
+    side_rank: int
 
     slot: int = 0
     pos_id: int = 0
@@ -66,12 +74,19 @@ def matrix_shape(globs: HybridGlobals, opcode: int, layer: int) -> tuple[int, in
     cfg = globs.model.config
     if opcode == Head.opcode():
         return cfg.vocab_size, cfg.width
-    spec = cfg.layers[layer]
+    spec = cfg.run_layers[layer]
+    m, mlp = spec.mixer, spec.mlp
+    if opcode == Enter.opcode():
+        return cfg.width, 2 * cfg.width
+    if opcode == Absorb.opcode():
+        return m.heads * m.rank, m.dim
+    if opcode == Expand.opcode():
+        return m.out_features, m.rank
     return {
-        NormProj.opcode(): (spec.mixer.in_rows, cfg.width),
-        OutProj.opcode(): (cfg.width, spec.mixer.out_features),
-        NormUp.opcode(): (spec.mlp.ff if spec.mlp else 0, cfg.width),
-        Down.opcode(): (cfg.width, spec.mlp.ff if spec.mlp else 0),
+        NormProj.opcode(): (m.in_rows, cfg.width),
+        OutProj.opcode(): (cfg.width, m.out_features),
+        NormUp.opcode(): (mlp.up_rows if mlp else 0, cfg.width),
+        Down.opcode(): (cfg.width, mlp.ff if mlp else 0),
     }[opcode]
 
 
@@ -91,7 +106,7 @@ class RowRange(Instruction):
 
 @dataclass
 class NormProj(RowRange):
-    """Layer norm of the residual stream, stacked input projection of the mixer."""
+    """Norm of the residual stream, input convolution, stacked input projection of the mixer."""
 
     @classmethod
     def opcode(cls) -> int:
@@ -116,12 +131,12 @@ class DeltaStep(Instruction):
         return {"pool": "compute"}
 
     def cost(self, globs) -> float:
-        m = globs.model.config.layers[self.layer_idx].mixer
+        m = globs.model.config.run_layers[self.layer_idx].mixer
         return (self.col_end - self.col_start) * m.dim * 4
 
 
 @dataclass
-class WindowAttention(Instruction):
+class KeyAttention(Instruction):
     """One split of the keys a KV head's queries see; the last split to arrive merges them."""
 
     layer_idx: int
@@ -138,8 +153,8 @@ class WindowAttention(Instruction):
         return {"pool": "compute"}
 
     def cost(self, globs) -> float:
-        m = globs.model.config.layers[self.layer_idx].mixer
-        return (m.window + m.keep_first) * (2 * m.dim + m.vdim) / self.num_splits
+        m = globs.model.config.run_layers[self.layer_idx].mixer
+        return min(m.window + m.keep_first, globs.model.max_len()) * m.key_elems / m.key_groups / self.num_splits
 
 
 @dataclass
@@ -153,7 +168,7 @@ class OutProj(RowRange):
 
 @dataclass
 class NormUp(RowRange):
-    """Layer norm, up projection of the feed-forward."""
+    """Norm, up projection of the feed-forward (with a gate: the gated unit)."""
 
     @classmethod
     def opcode(cls) -> int:
@@ -162,7 +177,7 @@ class NormUp(RowRange):
 
 @dataclass
 class Down(RowRange):
-    """PolyNorm, down projection, layer scale, residual add."""
+    """Activation, down projection, layer scale, residual add (beside a mixer: left to ``OutProj``)."""
 
     @classmethod
     def opcode(cls) -> int:
@@ -171,8 +186,35 @@ class Down(RowRange):
 
 @dataclass
 class Head(RowRange):
-    """Final layer norm, logits and their running argmax."""
+    """Final norm, logits and their running argmax."""
 
     @classmethod
     def opcode(cls) -> int:
         return 7
+
+
+@dataclass
+class Enter(RowRange):
+    """Start of a pass of the loop: the residual stream and the embedding, projected to one stream."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 8
+
+
+@dataclass
+class Absorb(RowRange):
+    """Latent attention: a head's query times the key expansion (rows of one head)."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 9
+
+
+@dataclass
+class Expand(RowRange):
+    """Latent attention: a head's output from latent to value space (rows of one head)."""
+
+    @classmethod
+    def opcode(cls) -> int:
+        return 10

@@ -324,7 +324,7 @@ class Hybrid_Generator(MK_Generator):
                 logits = torch.empty(len(here), V, device=globs.device, dtype=torch.float32)
             trace = None
             if layers_out is not None:
-                trace = torch.empty(len(model.layers), count, model.config.width, device=globs.device)
+                trace = torch.empty(len(model.config.runs), count, model.config.width, device=globs.device)
                 layers_out.append(trace)
             self.last_call = self.interpreter.prefill(globs, count, len(here), logits, trace)
             if here:

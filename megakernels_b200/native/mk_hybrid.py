@@ -11,17 +11,21 @@ from pathlib import Path
 
 import torch
 
+from megakernels_b200.hybrid import RopeSpec
+
 _HERE = Path(__file__).resolve().parent
 LIB_PATH = _HERE / "libmkb200_hybrid.so"
 
-MKBH_ABI_VERSION = 1
+MKBH_ABI_VERSION = 2
 STATUS_WORDS = 16
 FLAG_RECORD_TIMINGS = 1
 ERROR_NAMES = {
     0: "MKBH_OK", 1: "MKBH_ERR_INVALID_ARGUMENT", 2: "MKBH_ERR_CUDA", 3: "MKBH_ERR_DEVICE_TIMEOUT",
     4: "MKBH_ERR_BAD_OPCODE", 5: "MKBH_ERR_UNSUPPORTED",
 }
-MIXERS = {"delta_rule": 0, "diff_attention": 1}
+MIXERS = {"delta_rule": 0, "diff_attention": 1, "attention": 2, "latent_attention": 3}
+NORMS = {"layer_norm": 0, "rms_norm": 1}
+FEED_FORWARDS = {"poly_norm": 0, "clamped_glu": 1}
 
 _i32, _f32, _ptr, _i64, _u32 = ctypes.c_int32, ctypes.c_float, ctypes.c_void_p, ctypes.c_int64, ctypes.c_uint32
 
@@ -29,11 +33,15 @@ _i32, _f32, _ptr, _i64, _u32 = ctypes.c_int32, ctypes.c_float, ctypes.c_void_p, 
 class MkbhLayer(ctypes.Structure):
     _fields_ = [
         *[(n, _i32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "rank", "window", "keep_first", "owns_kv",
-                              "cache_keep", "cache_ring", "ff", "in_rows")],
+                              "cache_keep", "cache_ring", "ff", "in_rows", "chunk", "ff_kind", "parallel", "x_buf", "canon_taps",
+                              "conv_taps", "rot_dim", "rope_dims")],
         *[(n, _f32) for n in ("scale", "diff", "diff_lambda", "decay_scale", "unit_eps")],
         ("act", _f32 * 4),
+        ("glu_limit", _f32), ("glu_alpha", _f32),
         *[(n, _ptr) for n in ("in_w", "out_w", "up_w", "down_w", "in_bias", "norm1", "norm2", "ls1", "ls2", "decay_w2",
-                              "decay_w0", "out_norm", "k_cache", "v_cache", "state")],
+                              "decay_w0", "out_norm", "k_cache", "v_cache", "state", "enter_w", "canon_w", "canon_gain", "canon_hist",
+                              "canon_part", "conv_w", "conv_hist", "conv_part", "q_norm", "k_norm", "temp", "sink", "rope",
+                              "value_rope", "absorb_w", "expand_w")],
     ]
 
 
@@ -41,6 +49,7 @@ class MkbhGlobals(ctypes.Structure):
     _fields_ = [
         ("abi_version", _u32), ("struct_bytes", _u32),
         *[(n, _i32) for n in ("dtype", "num_layers", "width", "vocab", "max_positions", "slots")],
+        ("norm_kind", _i32), ("reserved", _i32),
         ("eps", _f32), ("embed_scale", _f32),
         *[(n, _ptr) for n in ("embed", "pos", "head", "final_norm", "layers_host", "layers_device", "tokens")],
         ("num_tokens", _i32), ("slot", _i32), ("pos0", _i32),
@@ -51,7 +60,10 @@ class MkbhGlobals(ctypes.Structure):
         ("arrivals", _ptr), ("attn_part", _ptr), ("max_splits", _i32), ("part_vdim", _i32),
         *[(n, _ptr) for n in ("x", "proj", "mixed", "decay", "act")],
         *[(n, _i64) for n in ("x_elems", "proj_elems", "mixed_elems", "act_elems", "decay_elems")],
-        ("portion_capacity", _i32),
+        *[(n, _ptr) for n in ("query", "act2", "ffn", "keys", "tail", "side")],
+        *[(n, _i64) for n in ("query_elems", "act2_elems", "ffn_elems", "keys_elems", "tail_elems", "side_elems")],
+        ("side_ff", _i32), ("side_rank", _i32),
+        ("portion_capacity", _i32), ("reserved2", _i32),
         ("flags", _u32), ("wait_timeout_ms", _u32), ("status", _ptr),
     ]
 
@@ -103,26 +115,48 @@ def _p(t) -> int | None:
 
 
 def layer_structs(model):
-    """Host array of layer descriptors."""
-    out = (MkbhLayer * len(model.layers))()
-    state = model.state
-    for i, (spec, w) in enumerate(zip(model.config.layers, model.layers)):
-        m, s = spec.mixer, out[i]
+    """Host array of layer descriptors, one per run."""
+    runs, state, buf = model.config.runs, model.state, 0
+    out = (MkbhLayer * len(runs))()
+    for i, (layer, enters) in enumerate(runs):
+        spec, w, s = model.config.layers[layer], model.layers[layer], out[i]
+        m = spec.mixer
         s.mixer, s.heads, s.dim, s.in_rows = MIXERS[m.kind], m.heads, m.dim, m.in_rows
+        if enters:  # (reads one residual buffer and writes the other)
+            buf ^= 1
+            s.enter_w = _p(model.enter)
+        s.x_buf, s.parallel, s.canon_taps = buf, int(spec.parallel), spec.canon_taps
         if m.kind == "delta_rule":
             s.rank, s.decay_scale, s.unit_eps = m.rank, m.decay_scale, m.unit_eps
             s.decay_w2, s.decay_w0, s.out_norm = _p(w.decay_w2), _p(w.decay_w0), _p(w.out_norm)
             s.state = _p(state.matrices[i])
         else:
             src = i if m.kv_from is None else m.kv_from
-            s.kv_heads, s.vdim, s.scale, s.diff, s.diff_lambda = m.kv_heads, m.vdim, m.scale, m.diff, w.diff_lambda
+            s.kv_heads, s.vdim, s.scale = m.key_groups, m.vdim, m.scale
             s.window, s.keep_first, s.owns_kv = m.window, min(m.keep_first, model.max_len()), int(m.kv_from is None)
             s.cache_keep, s.cache_ring = state.rows[src].keep, state.rows[src].ring
-            s.k_cache, s.v_cache = _p(state.keys[src]), _p(state.values[src])
-        for name in ("in_w", "out_w", "up_w", "down_w", "in_bias", "norm1", "norm2", "ls1", "ls2"):
+            s.k_cache, s.v_cache = _p(state.keys[src]), _p(state.values.get(src))
+        if m.kind == "diff_attention":
+            s.diff, s.diff_lambda = m.diff, w.diff_lambda
+        elif m.kind == "attention":
+            s.chunk, s.conv_taps = m.chunk, m.conv_taps
+            if m.turn_values:
+                s.value_rope = _p(model.rope_table(RopeSpec(m.vdim, m.rope.base)))
+            if m.conv_taps:
+                s.conv_hist, s.conv_part = _p(state.projected[i]), _p(state.projected_terms[i])
+        elif m.kind == "latent_attention":
+            s.rank, s.rot_dim = m.rank, m.rot_dim
+        if m.kind in ("attention", "latent_attention"):
+            s.rope, s.rope_dims = _p(model.rope_table(m.rope)), m.rope.dims
+        if spec.canon_taps:
+            s.canon_hist, s.canon_part = _p(state.inputs[i]), _p(state.input_terms[i])
+        for name in ("in_w", "out_w", "up_w", "down_w", "in_bias", "norm1", "norm2", "ls1", "ls2", "canon_w", "canon_gain", "conv_w",
+                     "q_norm", "k_norm", "temp", "sink", "absorb_w", "expand_w"):
             setattr(s, name, _p(getattr(w, name)))
         if spec.mlp is not None:
-            s.ff, s.act = spec.mlp.ff, (_f32 * 4)(*w.act)
+            s.ff, s.ff_kind, s.act = spec.mlp.ff, FEED_FORWARDS[spec.mlp.kind], (_f32 * 4)(*w.act)
+            if spec.mlp.kind == "clamped_glu":
+                s.glu_limit, s.glu_alpha = spec.mlp.limit, spec.mlp.alpha
     return out
 
 
@@ -142,7 +176,8 @@ class Call:
         g.abi_version, g.struct_bytes = MKBH_ABI_VERSION, ctypes.sizeof(MkbhGlobals)
         cfg = model.config
         g.dtype = 1 if model.dtype == torch.float32 else 0
-        g.num_layers, g.width, g.vocab = len(model.layers), cfg.width, cfg.vocab_size
+        g.num_layers, g.width, g.vocab = len(cfg.runs), cfg.width, cfg.vocab_size
+        g.norm_kind = NORMS[cfg.norm]
         g.max_positions, g.slots = model.max_len(), model.state.pool.count
         g.eps, g.embed_scale = cfg.eps, cfg.embed_scale
         g.embed, g.pos, g.head, g.final_norm = _p(model.embed), _p(model.positions), _p(model.head), _p(model.final_norm)
@@ -150,11 +185,12 @@ class Call:
         g.layers_device = _p(self.layers_device)
         g.max_kv_heads, g.max_splits, g.part_vdim = globs.max_kv_heads, globs.max_splits, globs.part_vdim
         for name in ("tokens", "want_rows", "argmax_out", "counters", "arrivals", "attn_part", "x", "proj", "mixed",
-                     "decay", "act", "status"):
+                     "decay", "act", "query", "act2", "ffn", "keys", "tail", "side", "status"):
             setattr(g, name, _p(getattr(globs, name)))
         g.num_counters = globs.counters.numel()
-        for name in ("x", "proj", "mixed", "act", "decay"):
+        for name in ("x", "proj", "mixed", "act", "decay", "query", "act2", "ffn", "keys", "tail", "side"):
             setattr(g, f"{name}_elems", getattr(globs, name).numel())
+        g.side_ff, g.side_rank = globs.side_ff, globs.side_rank
         g.portion_capacity = globs.portion
         self._validated = None
 

@@ -9,7 +9,7 @@ from typing import Any, Callable
 
 import torch
 
-from megakernels_b200 import torirax
+from megakernels_b200 import dumalix, torirax
 from megakernels_b200.llama import LlamaConfig, LlamaForCausalLM
 from megakernels_b200.model_types import ExtraModelConfig
 
@@ -28,6 +28,10 @@ FAMILIES = (
     ModelFamily(
         "torirax", torirax.ToriraxForCausalLM, "hybrid", (torch.bfloat16, torch.float32),
         lambda raw: raw.get("architecture") == "Torirax", dict(torirax.PRESETS),
+    ),
+    ModelFamily(
+        "dumalix", dumalix.DumalixForCausalLM, "hybrid", (torch.bfloat16, torch.float32),
+        lambda raw: raw.get("architecture") == "Dumalix", dict(dumalix.PRESETS),
     ),
     ModelFamily(
         "llama", LlamaForCausalLM, "llama", (torch.bfloat16,),

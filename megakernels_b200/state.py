@@ -5,12 +5,16 @@ A slot is one sequence's share of every cache.  ``SlotPool`` hands slots out and
 
 * attention layers that project their own keys and values hold ``keep + ring`` rows per slot: the
   first ``keep`` positions for good, later positions modulo ``ring``.  Layers that read another
-  layer's rows own nothing; ``keep`` and ``ring`` cover the widest reader;
-* recurrent layers hold one 32-bit matrix per head and slot, value column by value column.
+  layer's rows own nothing; ``keep`` and ``ring`` cover the widest reader.  A latent attention's row
+  is the latent and the rotated key part;
+* recurrent layers hold one 32-bit matrix per head and slot, value column by value column;
+* a convolution over time of ``taps`` holds its last ``taps - 1`` inputs in a ring by position, and
+  the sum of the terms that they add to the next position (32-bit).
 
-Nothing has to be cleared between owners of a slot: a sequence starts at position 0, where the
-kernels take the recurrent state as zero, and no query looks at a position that its own sequence
-has not written.
+Keys of the dictionaries are layer runs: each pass of a loop has its own.  Nothing has to be cleared
+between owners of a slot: a sequence starts at position 0, where the kernels take the recurrent
+state and earlier inputs as zero, and no query looks at a position that its own sequence has not
+written.
 """
 
 from __future__ import annotations
@@ -81,16 +85,31 @@ class HybridState:
         self.keys: dict[int, Tensor] = {}
         self.values: dict[int, Tensor] = {}
         self.matrices: dict[int, Tensor] = {}
-        for i, layer in enumerate(config.layers):
+        self.inputs: dict[int, Tensor] = {}  # input convolution: [slots, taps - 1, width]
+        self.input_terms: dict[int, Tensor] = {}  # [slots, 2, width], in turn by the position's parity
+        self.projected: dict[int, Tensor] = {}  # the projections' convolution: [slots, taps - 1, rows]
+        self.projected_terms: dict[int, Tensor] = {}  # [slots, rows]
+        layers = config.run_layers
+        f32 = lambda *shape: torch.zeros(slots, *shape, device=device, dtype=torch.float32)  # noqa: E731
+        for i, layer in enumerate(layers):
             m = layer.mixer
             if m.kind == "delta_rule":
-                self.matrices[i] = torch.zeros(slots, m.heads, m.dim, m.dim, device=device, dtype=torch.float32)
+                self.matrices[i] = f32(m.heads, m.dim, m.dim)
             elif m.kv_from is None:
-                readers = [m] + [o.mixer for o in config.layers if getattr(o.mixer, "kv_from", None) == i]
+                readers = [m] + [o.mixer for o in layers if getattr(o.mixer, "kv_from", None) == i]
                 rows = self.rows[i] = plan_cache_rows(readers, max_len, portion)
-                self.keys[i] = torch.zeros(slots, rows.total, m.kv_heads, 2, m.dim, device=device, dtype=dtype)
-                self.values[i] = torch.zeros(slots, rows.total, m.kv_heads, m.vdim, device=device, dtype=dtype)
+                cache = lambda *shape: torch.zeros(slots, rows.total, *shape, device=device, dtype=dtype)  # noqa: E731
+                if m.kind == "latent_attention":
+                    self.keys[i] = cache(m.row_elems)
+                else:
+                    maps = (2,) if m.kind == "diff_attention" else ()
+                    self.keys[i], self.values[i] = cache(m.kv_heads, *maps, m.dim), cache(m.kv_heads, m.vdim)
+            if layer.canon_taps:
+                self.inputs[i], self.input_terms[i] = f32(max(layer.canon_taps - 1, 1), config.width), f32(2, config.width)
+            if getattr(m, "conv_taps", 0):
+                self.projected[i], self.projected_terms[i] = f32(max(m.conv_taps - 1, 1), m.in_rows), f32(m.in_rows)
 
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size()
-                   for d in (self.keys, self.values, self.matrices) for t in d.values())
+                   for d in (self.keys, self.values, self.matrices, self.inputs, self.input_terms, self.projected, self.projected_terms)
+                   for t in d.values())

@@ -8,20 +8,14 @@ Reads a checkpoint directory (``config.json``, ``*.safetensors``) into the mecha
 
 from __future__ import annotations
 
-import json
-from pathlib import Path
-
-import torch
-
 from megakernels_b200.hybrid import (
+    CheckpointForCausalLM,
     DeltaRuleSpec,
     DiffAttentionSpec,
     HybridConfig,
-    HybridForCausalLM,
     LayerSpec,
     PolyNormSpec,
 )
-from megakernels_b200.model_types import DeviceType, ExtraModelConfig
 
 
 def read_layer(i: int, raw: dict, shape_of) -> LayerSpec:
@@ -41,35 +35,14 @@ def read_layer(i: int, raw: dict, shape_of) -> LayerSpec:
     return LayerSpec(mixer, None if mlp is None else PolyNormSpec(mlp["ff"]))
 
 
-def read_config(raw: dict, shape_of) -> HybridConfig:
-    """``shape_of(name)`` is a tensor's shape (the low-rank decay's inner size is only there)."""
-    return HybridConfig(
-        width=raw["width"], vocab_size=raw["vocab"], max_position_embeddings=raw["max_positions"],
-        eps=raw["norm"]["eps"], embed_scale=raw["embedding"]["scale"],
-        layers=tuple(read_layer(i, layer, shape_of) for i, layer in enumerate(raw["layers"])),
-    )
-
-
-class ToriraxForCausalLM(HybridForCausalLM):
+class ToriraxForCausalLM(CheckpointForCausalLM):
     @classmethod
-    def from_pretrained(
-        cls,
-        model_path: str | Path,
-        extra_config: ExtraModelConfig | None = None,
-        device: DeviceType = "cuda:0",
-        dtype: torch.dtype = torch.bfloat16,
-    ) -> "ToriraxForCausalLM":
-        from safetensors import safe_open
-
-        path = Path(model_path)
-        files = sorted(path.glob("*.safetensors"))
-        if not files:
-            raise FileNotFoundError(f"no safetensors files under {path}")
-        handles = [safe_open(f, framework="pt", device="cpu") for f in files]
-        where = {name: h for h in handles for name in h.keys()}
-        config = read_config(json.loads((path / "config.json").read_text()),
-                             lambda name: where[name].get_slice(name).get_shape())
-        return cls.assemble(config, extra_config, device, dtype, lambda name: where[name].get_tensor(name))
+    def read_config(cls, raw: dict, shape_of) -> HybridConfig:
+        return HybridConfig(
+            width=raw["width"], vocab_size=raw["vocab"], max_position_embeddings=raw["max_positions"],
+            eps=raw["norm"]["eps"], embed_scale=raw["embedding"]["scale"],
+            layers=tuple(read_layer(i, layer, shape_of) for i, layer in enumerate(raw["layers"])),
+        )
 
 
 # ---- random-weight shapes (layers of a real model's proportions) ---------------------------- #

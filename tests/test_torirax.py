@@ -14,7 +14,7 @@ import torch
 from megakernels_b200.demos.hybrid import instructions as I
 from megakernels_b200.demos.hybrid.scheduler import HybridScheduleOptions, column_groups, row_ranges, state_columns
 from megakernels_b200.dispatch import make_schedule_builder
-from megakernels_b200.hybrid import DiffAttentionSpec, HybridConfig, HybridForCausalLM, LayerSpec, tensor_shapes
+from megakernels_b200.hybrid import DiffAttentionSpec, HybridConfig, HybridForCausalLM, LayerSpec, key_splits, tensor_shapes
 from megakernels_b200.model_types import ExtraModelConfig
 from megakernels_b200.registry import family_of_checkpoint, load_model
 from megakernels_b200.scheduler import assign_to_sms, tensorize_instructions
@@ -196,9 +196,7 @@ def test_slot_pool():
 def build(raw, dtype=torch.bfloat16, options=None, **extra):
     w = make_weights(raw)
     cfg_shapes = {n: tuple(t.shape) for n, t in w.items()}
-    from megakernels_b200.torirax import read_config
-
-    m = HybridForCausalLM.assemble(read_config(raw, lambda n: cfg_shapes[n]), ExtraModelConfig(**extra), "cpu", dtype, w.get)
+    m = HybridForCausalLM.assemble(ToriraxForCausalLM.read_config(raw, lambda n: cfg_shapes[n]), ExtraModelConfig(**extra), "cpu", dtype, w.get)
     return make_schedule_builder("hybrid", options).build(m)
 
 
@@ -226,8 +224,8 @@ def test_schedule_covers_every_row_once_and_counts_its_arrivals(name, mode):
             assert sorted(cells) == [(h, c) for h in range(spec.mixer.heads) for c in range(spec.mixer.dim)]
             assert int(g.arrivals[i, 2]) == len(by[I.DeltaStep, i])
         else:
-            n = spec.mixer.num_splits(148)
-            assert sorted((x.kv_head_idx, x.split_idx) for x in by[I.WindowAttention, i]) == \
+            n = key_splits(spec.mixer, g.model.max_len(), 148)
+            assert sorted((x.kv_head_idx, x.split_idx) for x in by[I.KeyAttention, i]) == \
                 [(h, s) for h in range(spec.mixer.kv_heads) for s in range(n)]
             assert int(g.arrivals[i, 3]) == spec.mixer.kv_heads and n <= g.max_splits
     # a phase's instructions precede the next phase's in every queue
@@ -250,10 +248,10 @@ def test_row_ranges_fit_the_partial_sums():
 
 def test_split_counts_and_options():
     sched = build(EVEN, options=HybridScheduleOptions(keys_per_split=8, state_columns=32))
-    splits = [i for i in sched.get_linear_instructions() if isinstance(i, I.WindowAttention)]
+    splits = [i for i in sched.get_linear_instructions() if isinstance(i, I.KeyAttention)]
     assert max(i.num_splits for i in splits) == 10 and sched.globs.max_splits == 10
     assert {i.col_end - i.col_start for i in sched.get_linear_instructions() if isinstance(i, I.DeltaStep)} == {32}
-    assert DiffAttentionSpec(8, 8, 64, 64, 1.0, 10**6, 0, 0.1).num_splits(148) == 18
+    assert key_splits(DiffAttentionSpec(8, 8, 64, 64, 1.0, 10**6, 0, 0.1), 10**6, 148) == 18
 
 
 def test_presets_have_real_proportions():

@@ -7,7 +7,7 @@ import json
 import torch
 
 from megakernels_b200.hybrid import tensor_shapes
-from megakernels_b200.torirax import read_config
+from megakernels_b200.torirax import ToriraxForCausalLM
 from oracle import torirax_ref
 
 F32_TOL, BF16_TOL = 6e-5, 4e-2  # root mean square of the logits' difference over that of the logits
@@ -69,7 +69,7 @@ def make_weights(raw, seed=0, qk_gain=1.0):
     """Random bf16 tensors; ``qk_gain`` scales the query and key projections (peaked attention)."""
     gen = torch.Generator().manual_seed(seed)
     layer = lambda name: int(name.split(".")[0][1:])  # noqa: E731
-    config = read_config(raw, lambda name: (rank_of(layer(name)), raw["width"]))
+    config = ToriraxForCausalLM.read_config(raw, lambda name: (rank_of(layer(name)), raw["width"]))
     out = {}
     for name, shape in tensor_shapes(config).items():
         w = torch.randn(shape, generator=gen)
