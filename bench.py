@@ -85,9 +85,9 @@ def parse_args():
     ap.add_argument("--batch", type=int, default=1,
                     help="independent sequences decoded per launch (2..8: the batched kernel; 9..64: its tcgen05 "
                          "build; each sequence gets a seeded random KV length in [256, 4096] unless --prefill is given)")
-    ap.add_argument("--layer-list", default="", choices=["", "torirax-1b", "torirax-8b"],
-                    help="instead of the llama workload: prefill and decode of a layer-list model, beside the llama "
-                         "preset of its width (one GPU)")
+    ap.add_argument("--layer-list", default="", choices=["", "torirax-1b", "torirax-8b", "dumalix-1b", "dumalix-8b"],
+                    help="instead of the llama workload: prefill and decode of a layer-list model, beside the presets "
+                         "of its width that are closest to it (one GPU)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true")
     ap.add_argument("--no-e2e", action="store_true")

@@ -74,6 +74,6 @@ def preset(width: int, heads: int, kv_heads: int, dim: int, latent_heads: int, r
 
 PRESETS = {
     # 1B / 8B class: the widths, feed-forward sizes, vocabulary and layer runs of the Llama presets
-    "dumalix-1b": lambda: preset(2048, 32, 8, 64, 16, 512, 8192, 128256, 12, LoopSpec(4, 6, 3), 2048),
-    "dumalix-8b": lambda: preset(4096, 32, 8, 128, 32, 512, 14336, 128256, 24, LoopSpec(8, 12, 3), 4096),
+    "dumalix-1b": lambda: preset(2048, 32, 8, 64, 16, 512, 8192, 128256, 12, LoopSpec(4, 6, 3), 8192),
+    "dumalix-8b": lambda: preset(4096, 32, 8, 128, 32, 512, 14336, 128256, 24, LoopSpec(8, 12, 3), 8192),
 }

@@ -1,6 +1,7 @@
-"""Prefill and decode throughput of a layer-list model beside the llama preset of its width.
+"""Prefill and decode throughput of a layer-list model beside the presets of its width that are
+closest to it.
 
-Run through ``bench.py --layer-list torirax-1b``.  Random bf16 weights drawn on the device; the
+Run through ``bench.py --layer-list dumalix-1b``.  Random bf16 weights drawn on the device; the
 weights of one pass exceed L2, so no flush is needed between iterations.  Device times are CUDA
 events on the launching stream.
 """
@@ -19,43 +20,56 @@ from megakernels_b200.llama import LlamaForCausalLM
 from megakernels_b200.model_types import ExtraModelConfig
 from megakernels_b200.registry import family_of_preset
 
-CLOSEST = {"torirax-1b": "llama-1b", "torirax-8b": "llama-8b"}
+# the llama preset whose decode step is measured beside it, the layer-list preset whose prefill is
+CLOSEST = {"torirax-1b": ("llama-1b", None), "torirax-8b": ("llama-8b", None),
+           "dumalix-1b": ("llama-1b", "torirax-1b"), "dumalix-8b": ("llama-8b", "torirax-8b")}
 ATTENDED = 4096  # position of the first decoded token
 
 
 def matrix_params(cfg: HybridConfig, head: bool = True) -> int:
+    """Entries of the matrices a token meets (once per run of its layer)."""
     n = cfg.vocab_size * cfg.width if head else 0
-    for s in cfg.layers:
-        m = s.mixer
-        n += (m.in_rows + m.out_features) * cfg.width
-        if s.mlp is not None:
-            n += 2 * s.mlp.ff * cfg.width
+    for i, enters in cfg.runs:
+        m, mlp = cfg.layers[i].mixer, cfg.layers[i].mlp
+        n += (m.in_rows + m.out_features) * cfg.width + 2 * cfg.width**2 * enters
+        if m.kind == "latent_attention":
+            n += m.heads * (m.dim + m.vdim) * m.rank
+        if mlp is not None:
+            n += (mlp.up_rows + mlp.ff) * cfg.width
     return n
+
+
+def visible_keys(m, position: int) -> int:
+    if m.kind == "attention":
+        return position % m.chunk + 1
+    return min(position + 1, m.window + m.keep_first)
 
 
 def decode_bytes(cfg: HybridConfig, position: int) -> int:
     """Weights once, the visible keys and values, the recurrent matrices read and written."""
     n = 2 * matrix_params(cfg)
-    for s in cfg.layers:
+    for s in cfg.run_layers:
         m = s.mixer
         if m.kind == "delta_rule":
             n += 8 * m.heads * m.dim * m.dim + 4 * m.inner * m.rank
         else:
-            keys = min(position + 1, m.window + m.keep_first)
-            n += 2 * keys * m.kv_heads * (2 * m.dim + m.vdim)
+            n += 2 * visible_keys(m, position) * m.key_elems
     return n
 
 
-def prefill_flops(cfg: HybridConfig, tokens: int) -> float:
-    """Matrix products of the layers plus the attention inside its window (long prompts)."""
+def prefill_flops(cfg: HybridConfig, tokens: int, portion: int = 2048) -> float:
+    """Matrix products of the layers plus the attention over the keys that are seen."""
     f = 2.0 * tokens * matrix_params(cfg, head=False)
-    for s in cfg.layers:
+    at = range(0, tokens, 64)
+    for s in cfg.run_layers:
         m = s.mixer
         if m.kind == "delta_rule":
             f += tokens * m.heads * (10.0 * m.dim * m.dim)
-        else:
-            keys = sum(min(i + 1, m.window + m.keep_first) for i in range(0, tokens, 64)) / max(1, len(range(0, tokens, 64)))
-            f += tokens * keys * m.heads * 2 * (2 * m.dim + 2 * m.vdim)
+            continue
+        keys = sum(visible_keys(m, i) for i in at) / max(1, len(at))
+        pair = {"diff_attention": 2 * (2 * m.dim + 2 * m.vdim), "attention": 2 * (m.dim + m.vdim),
+                "latent_attention": 2 * (m.dim + getattr(m, "rot_dim", 0) + m.vdim)}[m.kind]
+        f += tokens * keys * m.heads * pair
     return f
 
 
@@ -117,32 +131,48 @@ def prefill_ms(gen, n: int, reps: int) -> float:
 
 
 def layer_parts(cfg: HybridConfig, tokens: int) -> dict:
-    """Milliseconds of one layer of each kind at ``tokens`` tokens: stacks of four, minus the shell
-    (embedding and head of one row)."""
-    delta = next(s for s in cfg.layers if s.mixer.kind == "delta_rule")
-    attn = next(s for s in cfg.layers if s.mixer.kind == "diff_attention")
-    stacks = {
-        "delta_rule": [replace(delta, mlp=None)] * 8,
-        "diff_attention": [replace(attn, mlp=None)] * 8,
-        "delta_rule+mlp": [delta] * 8,
-    }
+    """Milliseconds of one layer of each kind at ``tokens`` tokens: stacks of eight, minus stacks of
+    two (embedding, head of one row)."""
+    stacks = {}
+    for layer in cfg.layers:
+        stacks.setdefault(layer.mixer.kind, replace(layer, mlp=None))
+        if layer.mlp is not None:
+            stacks.setdefault(layer.mixer.kind + "+mlp", layer)
     out = {}
-    for name, layers in stacks.items():
+    for name, layer in stacks.items():
+        if getattr(layer.mixer, "kv_from", None) is not None:
+            continue
         both = []
         for k in (2, 8):
-            gen = hybrid_generator(replace(cfg, layers=tuple(layers[:k]), vocab_size=1024), tokens)
+            gen = hybrid_generator(replace(cfg, layers=(layer,) * k, loop=None, vocab_size=1024), tokens)
             both.append(prefill_ms(gen, tokens, 5))
             del gen
-        out[name] = (both[1] - both[0]) / 6
+        out[name] = round((both[1] - both[0]) / 6, 4)
     return out
+
+
+def prefill_table(gen, cfg, hbm: float, tflops: float) -> dict:
+    out = {}
+    for n in (64, 512, 2048, 8192):
+        ms = prefill_ms(gen, n, 5)
+        flops = prefill_flops(cfg, n)
+        floor = max(flops / (tflops * 1e9), 2e-6 * matrix_params(cfg, False) / hbm)
+        out[n] = {"ms": round(ms, 4), "tokens_per_s": round(n / ms * 1e3), "tflops": round(flops / ms * 1e-9, 1),
+                  "of_roofline": round(floor / ms, 3)}
+    return out
+
+
+def decode_row(kernel: float, step: float, nbytes: int, hbm: float) -> dict:
+    return {"kernel_ms": round(kernel, 4), "step_ms": round(step, 4), "bytes": nbytes, "gbs": round(nbytes / kernel * 1e-6),
+            "of_roofline": round(nbytes / kernel * 1e-6 / hbm, 3)}
 
 
 def run(args, sampler_cls, peaks: dict) -> None:
     hbm, tflops = peaks["hbm_gbs"], peaks["bf16_tflops_sustained"]
     torch.cuda.set_device(0)
     steps, warmup = min(args.steps, 128), max(3, args.warmup)
-    family = family_of_preset(args.layer_list)
-    cfg = family.presets[args.layer_list]()
+    cfg = family_of_preset(args.layer_list).presets[args.layer_list]()
+    close, close_list = CLOSEST[args.layer_list]
     max_len = ATTENDED + steps + warmup + 16
     sampler = sampler_cls(0)
     sampler.start()
@@ -150,27 +180,16 @@ def run(args, sampler_cls, peaks: dict) -> None:
         gen = hybrid_generator(cfg, max(max_len, 8192))
         line = {"metric": "layer_list_decode_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
                 "dtype": "bf16", "data": "synthetic (random weights)", "steps": steps, "warmup": warmup,
-                "config": {"model": args.layer_list, "layers": cfg.num_hidden_layers, "width": cfg.width,
+                "config": {"model": args.layer_list, "layers": cfg.num_hidden_layers, "layer_runs": len(cfg.runs), "width": cfg.width,
                            "position": ATTENDED, "l2": "weights of a pass exceed L2"}}
-        prefill = {}
-        for n in (64, 512, 2048, 8192):
-            ms = prefill_ms(gen, n, 5)
-            achieved = prefill_flops(cfg, n) / ms * 1e-9
-            floor = max(prefill_flops(cfg, n) / (tflops * 1e9), 2e-6 * matrix_params(cfg, False) / hbm)
-            prefill[n] = {"ms": round(ms, 4), "tokens_per_s": round(n / ms * 1e3), "tflops": round(achieved, 1),
-                          "of_roofline": round(floor / ms, 3)}
-        line["prefill"] = prefill
+        line["prefill"] = prefill_table(gen, cfg, hbm, tflops)
         kernel, step = decode_ms(gen, ATTENDED, steps, warmup)
-        nbytes = decode_bytes(cfg, ATTENDED)
-        line.update(value=1e3 / step, ms_per_step=step,
-                    decode={"kernel_ms": round(kernel, 4), "step_ms": round(step, 4), "bytes": nbytes,
-                            "gbs": round(nbytes / kernel * 1e-6), "of_roofline": round(nbytes / kernel * 1e-6 / hbm, 3)})
+        line.update(value=1e3 / step, ms_per_step=step, decode=decode_row(kernel, step, decode_bytes(cfg, ATTENDED), hbm))
         del gen
         torch.cuda.empty_cache()
-        line["prefill_ms_per_layer_2048"] = {k: round(v, 4) for k, v in layer_parts(cfg, 2048).items()}
+        line["prefill_ms_per_layer_2048"] = layer_parts(cfg, 2048)
         torch.cuda.empty_cache()
 
-        close = CLOSEST[args.layer_list]
         lcfg = family_of_preset(close).presets[close]()
         extra = ExtraModelConfig(interleave_rope=True, max_len_override=max_len)
         model = LlamaForCausalLM.from_random(lcfg, extra, draw_on="device")
@@ -181,12 +200,19 @@ def run(args, sampler_cls, peaks: dict) -> None:
         H, I, D = lcfg.hidden_size, lcfg.intermediate_size, lcfg.head_dim
         Hq, Hk, L = lcfg.num_attention_heads, lcfg.num_key_value_heads, lcfg.num_hidden_layers
         nbytes = 2 * (L * ((Hq + 2 * Hk) * D * H + H * Hq * D + 3 * I * H) + lcfg.vocab_size * H) + 4 * ATTENDED * Hk * D * L
-        line["closest"] = {
-            "model": close, "layers": L,
-            "decode": {"kernel_ms": round(kernel, 4), "step_ms": round(step, 4), "bytes": nbytes,
-                       "gbs": round(nbytes / kernel * 1e-6), "of_roofline": round(nbytes / kernel * 1e-6 / hbm, 3)},
-            # its prompts go through the decode kernel token by token
-            "prefill_tokens_per_s": round(1e3 / step),
-        }
+        line["closest"] = {"model": close, "layers": L, "decode": decode_row(kernel, step, nbytes, hbm),
+                           "prefill_tokens_per_s": round(1e3 / step)}  # its prompts go through the decode kernel token by token
+        if close_list:
+            del gen, model
+            torch.cuda.empty_cache()
+            tcfg = family_of_preset(close_list).presets[close_list]()
+            gen = hybrid_generator(tcfg, max(max_len, 8192))
+            line["closest_layer_list"] = {"model": close_list, "layers": tcfg.num_hidden_layers,
+                                          "prefill": prefill_table(gen, tcfg, hbm, tflops)}
+            kernel, step = decode_ms(gen, ATTENDED, steps, warmup)
+            line["closest_layer_list"]["decode"] = decode_row(kernel, step, decode_bytes(tcfg, ATTENDED), hbm)
+            del gen
+            torch.cuda.empty_cache()
+            line["closest_layer_list"]["prefill_ms_per_layer_2048"] = layer_parts(tcfg, 2048)
     line["clocks"] = sampler.stop()
     print(json.dumps(line), flush=True)
