@@ -53,7 +53,7 @@ enum MkbhOpcode {
     MKBH_OP_HEAD = 7,        /* row_start, row_end: final norm, logits, argmax */
     MKBH_OP_ENTER = 8,       /* row_start, row_end: x <- W [x; embedding] before a pass of the loop */
     MKBH_OP_ABSORB = 9,      /* row_start, row_end (of one head): query times the key up-projection */
-    MKBH_OP_EXPAND = 10      /* row_start, row_end (of one head): latent output to value space */
+    MKBH_OP_EXPAND = 10      /* row_start, row_end (of one head), num_splits: latent output to value space */
 };
 
 #define MKBH_INTS_PER_INSTRUCTION 32
@@ -151,7 +151,7 @@ typedef struct MkbhGlobals {
     int32_t *timings;          /* [num_sms, queue_len, 128] or NULL */
     int32_t num_sms, queue_len;
     const int32_t *arrivals;   /* device [num_layers + 1, MKBH_BARRIERS_PER_LAYER]: instructions per phase */
-    float *attn_part;          /* [max heads, 2, max_splits, part_vdim + 2] */
+    float *attn_part;          /* [max heads, 2, max_splits, 4 + part_vdim rounded up to 4] */
     int32_t max_splits, part_vdim; /* largest split count and vdim of any attention layer */
 
     /* activations: x [rows, width]; proj [rows, max in_rows, ff]; act [rows, ld] in the model dtype;
@@ -162,11 +162,11 @@ typedef struct MkbhGlobals {
     /* parallel layers, convolutions, rotary and latent attention (NULL without them).
      * Prefill, model dtype: query [rows, widest heads * (dim + rot_dim)], act2 [rows, width],
      * ffn [rows, ff], keys [max_positions, widest heads * (dim + vdim)]; tail: float [taps, width].
-     * Decode, float: side [ff | width | heads * rank | heads * rank]. */
+     * Decode, float: side [ff | width | heads * rank]. */
     void *query, *act2, *ffn, *keys;
     float *tail, *side;
     int64_t query_elems, act2_elems, ffn_elems, keys_elems, tail_elems, side_elems;
-    int32_t side_ff, side_rank;  /* room of the first, third and fourth part of `side` */
+    int32_t side_ff, side_rank;  /* room of the first and the third part of `side` */
     int32_t portion_capacity, reserved2;
 
     uint32_t flags;

@@ -51,6 +51,13 @@ constexpr int kSmemLimit = 226 * 1024;
 constexpr int kMaxStash = 512;         // channels whose normalised input an instruction publishes
 constexpr int kMaxChannels = 8;        // key channels of one column a lane carries (dim <= 256)
 
+// Which mechanisms a build of the kernel has; a launch takes the smallest build that serves its
+// layers, so that one family's code and registers do not weigh on the other's.
+enum Features {
+    kClassic = 1,  // delta rule, differential attention, PolyNorm, layer norms
+    kRotary = 2,   // rotary and latent attention, gated units, feed-forwards beside mixers, convolutions, loops
+};
+
 struct Params {
     MkbhGlobals g;
     int stages, act_bytes, vec_bytes;
@@ -172,11 +179,10 @@ __device__ __noinline__ void poll_counter(const int* addr, int thr, volatile int
 __device__ __forceinline__ int phase_index(int layer, int op) { return layer * MKBH_BARRIERS_PER_LAYER + op; }
 
 // Float buffers beside the stacked projection: feed-forward input and output of parallel layers,
-// absorbed queries and latent outputs.
+// absorbed queries.
 __device__ __forceinline__ float* side_in(const MkbhGlobals& g) { return g.side; }
 __device__ __forceinline__ float* side_out(const MkbhGlobals& g) { return g.side + g.side_ff; }
 __device__ __forceinline__ float* side_query(const MkbhGlobals& g) { return side_out(g) + pad8(g.width); }
-__device__ __forceinline__ float* side_latent(const MkbhGlobals& g) { return side_query(g) + g.side_rank; }
 
 // ---- loader: the weight stream ----------------------------------------------------------- //
 struct Block {  // rows [r0, r1) of a matrix of `row_bytes` rows
@@ -578,7 +584,7 @@ __device__ __forceinline__ int token_id(const MkbhGlobals& g) {
 // Norm of the residual stream `src` (NULL: of the token's embedding, which goes to `publish` as
 // well).  `part`: what earlier inputs add through the input convolution; `stash` receives the
 // unweighted channels [c0, c1) for it.
-template <typename T, int kSlots>
+template <typename T, int F, int kSlots>
 __device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, const float* src, const float* w, const float* part,
                                                 float* act, float* red, int& turn, float* publish, float* stash, int c0, int c1) {
     const MkbhGlobals& g = p.g;
@@ -598,7 +604,7 @@ __device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, c
         x.load_cg(src);
     }
     float sum[1] = {0.f};
-    if (g.norm_kind == MKBH_LAYER_NORM) {
+    if (F == kClassic || ((F & kClassic) && g.norm_kind == MKBH_LAYER_NORM)) {
 #pragma unroll
         for (int s = 0; s < kSlots; ++s) sum[0] += x.v[s];
         csum<1>(red, turn, sum);
@@ -616,8 +622,8 @@ __device__ __forceinline__ void norm_activation(const Params& p, const Cta& c, c
         if (x.has(s)) {
             const int i = x.index(s);
             x.v[s] *= inv;
-            if (i >= c0 && i < c1) stash[i - c0] = x.v[s];
-            x.v[s] = part != nullptr ? fmaf(x.v[s], w[i], part[i]) : x.v[s] * w[i];
+            if ((F & kRotary) && i >= c0 && i < c1) stash[i - c0] = x.v[s];
+            x.v[s] = (F & kRotary) && part != nullptr ? fmaf(x.v[s], w[i], part[i]) : x.v[s] * w[i];
         }
     x.store(act);
 }
@@ -798,6 +804,9 @@ __device__ __forceinline__ void delta_step(const Params& p, const Cta& c, const 
 __host__ __device__ inline int attn_maps(const MkbhLayer& L) { return L.mixer == MKBH_DIFF_ATTENTION ? 2 : 1; }
 __host__ __device__ inline int attn_dim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? latent_row(L) : L.dim; }
 __host__ __device__ inline int attn_vdim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? L.rank : L.vdim; }
+// Partial rows of the splits: [m, l, -, -, sums ...], 16-byte aligned.
+constexpr int kPartLead = 4;
+__host__ __device__ inline int part_row(int vdim) { return ((vdim + 3) & ~3) + kPartLead; }
 struct AttnScratch {  // float offsets; the key and value tiles follow
     int q, p, m, l, f, own, tile;
     __host__ __device__ AttnScratch(const MkbhLayer& L, int chunk) {
@@ -826,22 +835,62 @@ __host__ __device__ inline int merge_scratch_floats(int nq, int splits, int per,
     return nq * splits + per * (vdim + 1);
 }
 
+// Tensor-core variant of the one-map mixers (bf16): what it keeps in shared memory, in floats.
+constexpr int kMmaKeys = 256;  // keys per pass
+constexpr int kMmaCols = kMmaKeys + 8;  // scores of a head; column kMmaKeys is this token's own key
 template <typename T>
+__host__ __device__ inline bool mma_attention(const MkbhLayer& L) {
+    return sizeof(T) == 2 && (L.mixer == MKBH_ATTENTION || L.mixer == MKBH_LATENT_ATTENTION) && attn_dim(L) % 8 == 0 &&
+           attn_vdim(L) % 8 == 0 && L.heads / L.kv_heads <= 16;
+}
+struct MmaScratch {
+    int q, qs, frag, planes, p, m, l, f, own, rows, red, slices, groups, total;
+    __host__ __device__ MmaScratch(const MkbhLayer& L) {
+        const int nq = L.heads / L.kv_heads, dim = attn_dim(L), e = attn_vdim(L);
+        slices = (e + 31) / 32;             // of the value columns, a warp each ...
+        groups = kConsumerWarps / slices;   // ... times groups of keys
+        planes = nq > 8 ? 2 : 1;
+        qs = (dim + 31) / 32 * 32;
+        q = 0;
+        frag = nq * qs;                     // queries as fragments: [plane][16 columns][lane][high 2, low 2]
+        p = frag + planes * (qs / 16) * 32 * 4;
+        m = p + nq * kMmaCols;
+        l = m + nq;
+        f = l + nq;
+        own = (f + nq + 3) & ~3;
+        rows = own + ((dim + e + 3) & ~3);  // cache rows of a pass
+        red = rows + kMmaKeys;
+        total = red + (groups > 1 ? groups * nq * e : 0);
+    }
+};
+
+template <typename T, int F>
 struct AttnView {
-    int D, KE, E, G, per, nq, ks, vs, t_lo, count, keep, ring, pos;
+    int D, KE, E, G, per, nq, qs, ks, vs, t_lo, count, keep, ring, pos;
     size_t krow, vrow;  // elements between positions
     KeyRange keys;
     T *kc, *vc, *kt, *vt;
     float *q, *p, *m, *l, *f, *own;
-    bool latent;
-    __device__ __forceinline__ AttnView(const Params& pr, const Cta& c, const Desc& d, float* act)
-        : keys(c.pos, d.L.window, d.L.keep_first, d.L.chunk) {
+    int* rows;  // cache rows of the pass's keys
+    bool latent, diff;
+    __device__ __forceinline__ AttnView(const Params& pr, int at, const Desc& d, float* act)
+        : keys(at, d.L.window, d.L.keep_first, d.L.chunk) {
         const MkbhLayer& L = d.L;
-        latent = L.mixer == MKBH_LATENT_ATTENTION;
-        D = attn_dim(L); KE = attn_maps(L) * D; E = attn_vdim(L); G = L.kv_heads; per = L.heads / G; nq = attn_maps(L) * per;
-        keep = L.cache_keep; ring = L.cache_ring; pos = c.pos;
+        latent = (F & kRotary) && L.mixer == MKBH_LATENT_ATTENTION;
+        diff = F == kClassic || ((F & kClassic) && L.mixer == MKBH_DIFF_ATTENTION);
+        D = latent ? latent_row(L) : L.dim; KE = diff ? 2 * D : D; E = latent ? L.rank : L.vdim;
+        G = L.kv_heads; per = L.heads / G; nq = diff ? 2 * per : per;
+        keep = L.cache_keep; ring = L.cache_ring; pos = at;
         const AttnScratch a(L, pr.attn_chunk);
         q = act + a.q; p = act + a.p; m = act + a.m; l = act + a.l; f = act + a.f; own = act + a.own;
+        qs = D;
+        rows = nullptr;
+        if ((F & kRotary) && mma_attention<T>(L)) {
+            const MmaScratch b(L);
+            rows = reinterpret_cast<int*>(act + b.rows);
+            q = act + b.q; p = act + b.p; m = act + b.m; l = act + b.l; f = act + b.f; own = act + b.own;
+            qs = b.qs;
+        }
         kt = reinterpret_cast<T*>(act + a.tile);
         ks = key_stride<T>(KE) / (int)sizeof(T);
         vt = latent ? kt : kt + (size_t)pr.attn_chunk * ks;
@@ -853,6 +902,24 @@ struct AttnView {
         vrow = (size_t)G * E;
         kc = static_cast<T*>(L.k_cache) + rows0 * krow + (latent ? 0 : (size_t)d.a0 * KE);
         vc = latent ? nullptr : static_cast<T*>(L.v_cache) + rows0 * vrow + (size_t)d.a0 * E;
+    }
+    // Cache rows of the keys of a pass.
+    __device__ __forceinline__ void list_rows(int c0, int n) const {
+        for (int i = threadIdx.x; i < n; i += kConsumers) rows[i] = cache_row(keys.key(t_lo + c0 + i), keep, ring);
+    }
+    // Bring the split's rows and the position's rotations into L2 (they do not depend on this step).
+    __device__ __forceinline__ void prefetch(const MkbhLayer& L) const {
+        const int n = count - (has_own() ? 1 : 0), klines = (KE * (int)sizeof(T) + 127) / 128, vlines = latent ? 0 : (E * (int)sizeof(T) + 127) / 128;
+        list_rows(0, min(n, kMmaKeys));
+        auto line = [](const void* a) { asm volatile("prefetch.global.L2 [%0];" ::"l"(a)); };
+        for (int i = threadIdx.x; i < n * (klines + vlines); i += kConsumers) {
+            const int t = i / (klines + vlines), u = i % (klines + vlines);
+            const size_t row = cache_row(keys.key(t_lo + t), keep, ring);
+            line(u < klines ? kc + row * krow + u * (128 / sizeof(T)) : vc + row * vrow + (u - klines) * (128 / sizeof(T)));
+        }
+        const int lane = threadIdx.x & 31;
+        if (threadIdx.x < 32 && lane * 32 < L.rope_dims) line(L.rope + (size_t)pos * L.rope_dims + lane * 32);
+        if (threadIdx.x < 32 && L.value_rope != nullptr && lane * 32 < L.vdim) line(L.value_rope + (size_t)pos * L.vdim + lane * 32);
     }
     __device__ __forceinline__ bool has_own() const { return count > 0 && t_lo + count == keys.count; }
     // Start copying rows [c0, c0 + nk) of the split, except this token's own: older rows do not
@@ -883,96 +950,127 @@ struct AttnView {
     }
 };
 
+// What an attention instruction fetches before its producers are done.
+template <typename T, int F>
+__device__ __forceinline__ void attend_ahead(const Params& pr, int pos, const Desc& d, float* act) {
+    const AttnView<T, F> A(pr, pos, d, act);
+    if ((F & kRotary) && mma_attention<T>(d.L)) A.prefetch(d.L);
+    else A.stage(0, min(pr.attn_chunk, A.count));
+}
+
 // One head's vector, by one warp: optional norm (weight w), rotation of the first `rot` elements
-// (neighbours by the angles of `rope`), factor `mul`.
-__device__ __noinline__ void head_vector(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
-                                         float mul, float* dst) {
-    constexpr int J = 4;  // pairs per lane kept in registers
+// (neighbours by the angles of `rope`), factor `mul`.  All of it is read before anything is used;
+// n <= 64 J.
+template <int J>
+__device__ __forceinline__ void head_vector(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
+                                            float mul, float* dst) {
     const int lane = threadIdx.x & 31;
-    float a[J], b[J], s = 0.f;
+    float a[J], b[J], wa[J], wb[J], s = 0.f;
+    float2 r[J];
 #pragma unroll
     for (int j = 0; j < J; ++j) {
         const int i = 2 * (lane + 32 * j);
         a[j] = i < n ? ld_cg_f32(src + i) : 0.f;
         b[j] = i + 1 < n ? ld_cg_f32(src + i + 1) : 0.f;
-        s = fmaf(a[j], a[j], fmaf(b[j], b[j], s));
+        wa[j] = w != nullptr && i < n ? __ldg(w + i) : 1.f;
+        wb[j] = w != nullptr && i + 1 < n ? __ldg(w + i + 1) : 1.f;
+        r[j] = i < rot ? __ldg(rope + (i >> 1)) : make_float2(1.f, 0.f);
     }
     if (w != nullptr) {
-        for (int i = 64 * J + lane; i < n; i += 32) {
-            const float x = ld_cg_f32(src + i);
-            s = fmaf(x, x, s);
-        }
-        s = 1.f / sqrtf(warp_sum(s) / n + eps);
-    }
-    for (int j = 0; 64 * j < n; ++j) {
-        const int i = 2 * (lane + 32 * j);
-        if (i >= n) break;
-        float x = 0.f, y = 0.f;
 #pragma unroll
-        for (int k = 0; k < J; ++k)
-            if (k == j) x = a[k], y = b[k];
-        if (j >= J) {
-            x = ld_cg_f32(src + i);
-            y = i + 1 < n ? ld_cg_f32(src + i + 1) : 0.f;
-        }
-        if (w != nullptr) {
-            x *= s * __ldg(w + i);
-            if (i + 1 < n) y *= s * __ldg(w + i + 1);
-        }
-        if (i < rot) {
-            const float2 r = __ldg(rope + (i >> 1));
-            const float z = x * r.x - y * r.y;
-            y = y * r.x + x * r.y;
-            x = z;
-        }
-        dst[i] = x * mul;
-        if (i + 1 < n) dst[i + 1] = y * mul;
+        for (int j = 0; j < J; ++j) s = fmaf(a[j], a[j], fmaf(b[j], b[j], s));
+        s = 1.f / sqrtf(warp_sum(s) / n + eps);
+    } else {
+        s = 1.f;
     }
+#pragma unroll
+    for (int j = 0; j < J; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        const float x = a[j] * s * wa[j], y = b[j] * s * wb[j];
+        if (i < n) dst[i] = (x * r[j].x - y * r[j].y) * mul;
+        if (i + 1 < n) dst[i + 1] = (y * r[j].x + x * r[j].y) * mul;
+    }
+}
+// (by size: one call site each for up to 64, 128 and 512 elements)
+__device__ __noinline__ void head_vector_any(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
+                                             float mul, float* dst) {
+    if (n <= 64) head_vector<1>(src, n, w, eps, rope, rot, mul, dst);
+    else if (n <= 128) head_vector<2>(src, n, w, eps, rope, rot, mul, dst);
+    else head_vector<8>(src, n, w, eps, rope, rot, mul, dst);
 }
 
 // Queries of the KV head's heads, normalised, rotated and scaled, and, in the split that holds it,
 // this token's key and value.  Ends with a barrier.
-template <typename T>
-__device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView<T>& A, const MkbhLayer& L, int kvh) {
+template <typename T, int F>
+__device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView<T, F>& A, const MkbhLayer& L, int kvh) {
     const MkbhGlobals& g = pr.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tasks = A.nq + (A.has_own() ? 2 : 0);
     const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)A.pos * (L.rope_dims / 2);
     for (int t = warp; t < tasks; t += kConsumerWarps) {
         const int h = kvh * A.per + t;
+        const bool query = t < A.nq, first = t == A.nq;
+        const float *src, *w = nullptr;
+        const float2* angles = rope;
+        int n, rot = L.rope_dims;
+        float mul = 1.f;
+        float* dst = query ? A.q + t * A.qs : A.own;
         if (A.latent) {
             const int hd = L.dim + L.rot_dim, lead = pad8(L.rank);
             const float* down = g.proj + (size_t)L.heads * hd;
-            float* dst = t < A.nq ? A.q + t * A.D : A.own;
-            if (t < A.nq) {
-                for (int i = lane; i < L.rank; i += 32) dst[i] = ld_cg_f32(side_query(g) + (size_t)h * L.rank + i) * L.scale;
-                head_vector(g.proj + (size_t)h * hd + L.dim, L.rot_dim, nullptr, 0.f, rope, L.rope_dims, L.scale, dst + lead);
-            } else if (t == A.nq) {
-                head_vector(down, L.rank, L.k_norm, g.eps, nullptr, 0, 1.f, dst);
+            if (query) {
+                const float* absorbed = side_query(g) + (size_t)h * L.rank;
+                const float scale = L.scale;
+                mul = scale;
+                for (int i0 = 0; i0 < L.rank; i0 += 256) {
+                    float x[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) x[j] = i0 + lane + 32 * j < L.rank ? ld_cg_f32(absorbed + i0 + lane + 32 * j) : 0.f;
+#pragma unroll
+                    for (int j = 0; j < 8; ++j)
+                        if (i0 + lane + 32 * j < L.rank) dst[i0 + lane + 32 * j] = x[j] * scale;
+                }
+            }
+            if (!first) {  // rotated part
+                src = query ? g.proj + (size_t)h * hd + L.dim : down + L.rank;
+                n = L.rot_dim;
+                dst += lead;
+                for (int i = n + lane; i < (query ? A.qs : A.D) - lead; i += 32) dst[i] = 0.f;
             } else {
-                head_vector(down + L.rank, L.rot_dim, nullptr, 0.f, rope, L.rope_dims, 1.f, dst + lead);
+                src = down;
+                n = L.rank;
+                w = L.k_norm;
+                rot = 0;
             }
-            if (t <= A.nq) {  // padding
-                for (int i = L.rank + lane; i < lead; i += 32) dst[i] = 0.f;
-                for (int i = lead + L.rot_dim + lane; i < A.D; i += 32) dst[i] = 0.f;
-            }
-        } else if (t < A.nq) {
-            head_vector(g.proj + (size_t)h * A.D, A.D, L.q_norm, g.eps, rope, L.rope_dims, L.scale * __ldg(L.temp + h), A.q + t * A.D);
-        } else if (t == A.nq) {
-            head_vector(g.proj + (size_t)(L.heads + kvh) * A.D, A.D, L.k_norm, g.eps, rope, L.rope_dims, 1.f, A.own);
+            if (query || first)
+                for (int i = L.rank + lane; i < lead; i += 32) dst[i - (query ? lead : 0)] = 0.f;
+        } else if (query) {
+            src = g.proj + (size_t)h * A.D;
+            n = A.D;
+            w = L.q_norm;
+            mul = L.scale * __ldg(L.temp + h);
+            for (int i = A.D + lane; i < A.qs; i += 32) dst[i] = 0.f;
+        } else if (first) {
+            src = g.proj + (size_t)(L.heads + kvh) * A.D;
+            n = A.D;
+            w = L.k_norm;
         } else {
-            const float2* turn = L.value_rope == nullptr ? nullptr : reinterpret_cast<const float2*>(L.value_rope) + (size_t)A.pos * (A.E / 2);
-            head_vector(g.proj + (size_t)(L.heads + A.G) * A.D + (size_t)kvh * A.E, A.E, nullptr, 0.f, turn, turn ? A.E : 0, 1.f, A.own + A.D);
+            src = g.proj + (size_t)(L.heads + A.G) * A.D + (size_t)kvh * A.E;
+            n = A.E;
+            angles = reinterpret_cast<const float2*>(L.value_rope) + (size_t)A.pos * (A.E / 2);
+            rot = L.value_rope != nullptr ? A.E : 0;
+            dst += A.D;
         }
+        head_vector_any(src, n, w, g.eps, angles, rot, mul, dst);
     }
     csync();
 }
 
-template <typename T, int kAcc>
-__device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, const Desc& d) {
+template <typename T, int F, int kAcc>
+__device__ __forceinline__ void attend(const Params& pr, const AttnView<T, F>& A, const Desc& d) {
     const MkbhGlobals& g = pr.g;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, KC = pr.attn_chunk;
     const int D = A.D, E = A.E, nq = A.nq, kvh = d.a0;
-    const bool diff = d.L.mixer == MKBH_DIFF_ATTENTION;
+    const bool diff = A.diff;
     const float scale = diff ? d.L.scale : 1.f;
     const bool owns = d.L.owns_kv != 0;
     const int kv_off = d.L.heads * (2 * D + E);
@@ -985,8 +1083,8 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
     for (int i = 0; i < kAcc; ++i) acc[i] = 0.f;
     if (diff)
         for (int i = tid; i < nq * D; i += kConsumers) A.q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
-    else
-        rotary_operands<T>(pr, A, d.L, kvh);
+    else if constexpr (F & kRotary)
+        rotary_operands<T, F>(pr, A, d.L, kvh);
 
     for (int c0 = 0; c0 < A.count; c0 += KC) {
         const int nk = min(KC, A.count - c0);
@@ -1085,7 +1183,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
         csync();
     }
     // partial rows [head and map][split][m, l, acc...]
-    const int PE = g.part_vdim + 2, split = d.a1;
+    const int PE = part_row(g.part_vdim), split = d.a1;
     float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
     if (has_e) {
 #pragma unroll
@@ -1093,7 +1191,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
             const int qv = qv0 + i * lanes_e;
             if (qv < nq) {
                 float* row = part + ((size_t)qv * g.max_splits + split) * PE;
-                row[2 + e] = acc[i];
+                row[kPartLead + e] = acc[i];
                 if (e == 0) {
                     row[0] = A.count > 0 ? A.m[qv] : -INFINITY;
                     row[1] = A.count > 0 ? A.l[qv] : 0.f;
@@ -1103,69 +1201,315 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T>& A, c
     }
 }
 
+template <typename T, int F>
+__device__ __forceinline__ void attend_fma(const Params& pr, int pos, const Desc& d, float* act) {
+    const AttnView<T, F> A(pr, pos, d, act);
+    const int need = (A.nq + kConsumers / A.E - 1) / (kConsumers / A.E);
+    if (need <= 2) attend<T, F, 2>(pr, A, d);
+    else if (need <= 4) attend<T, F, 4>(pr, A, d);
+    else attend<T, F, 16>(pr, A, d);
+}
+
+__device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = mkb::pack_bf16x2(x, y);
+    lo = mkb::pack_bf16x2(x - mkb::bf16_lo(hi), y - mkb::bf16_hi(hi));
+}
+
+// One split on mma.sync, straight from the cache rows: the M side of both products are the heads of
+// the group (queries and softmax weights enter as a high and a low bf16 part), the N side keys, then
+// value columns.  The index of a contraction may be permuted as long as both operands agree, so a
+// lane's share of a fragment is a run of neighbours in memory.
+template <typename T, int F>
+__device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc& d, float* act) {
+    const MkbhGlobals& g = pr.g;
+    const AttnView<T, F> A(pr, pos, d, act);
+    const MmaScratch S(d.L);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c = lane & 3;
+    const int D = A.D, E = A.E, nq = A.nq, kvh = d.a0;
+    const bool own = A.has_own(), latent = A.latent;
+    float *const p = A.p, *const red = act + S.red;
+    const uint4* const frag = reinterpret_cast<const uint4*>(act + S.frag);
+    const float* const own_v = latent ? A.own : A.own + D;
+    const int slice = warp % S.slices, group = warp / S.slices, e0 = slice * 32 + r * 4;
+    const T *const kbase = A.kc, *const vbase = latent ? A.kc : A.vc;
+    const size_t krow = A.krow, vrow = latent ? A.krow : A.vrow;
+    const int* const rows = A.rows;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    rotary_operands<T, F>(pr, A, d.L, kvh);
+    const int blocks = S.qs / 32;
+    for (int i = tid; i < S.planes * blocks * 64; i += kConsumers) {  // queries in fragment order
+        const int l = i & 31, col = (i >> 6) % blocks * 32 + (l & 3) * 8 + (i >> 5 & 1) * 4, head = (l >> 2) + 8 * (i / (blocks * 64));
+        uint4 f = make_uint4(0, 0, 0, 0);
+        if (head < nq) {
+            const float4 x = *reinterpret_cast<const float4*>(A.q + head * S.qs + col);
+            split_bf16(x.x, x.y, f.x, f.z);
+            split_bf16(x.z, x.w, f.y, f.w);
+        }
+        reinterpret_cast<uint4*>(act + S.frag)[i] = f;
+    }
+    if (own) {  // this token's row
+        const size_t row = cache_row(pos, A.keep, A.ring);
+        if (!latent || kvh == 0)  // (every group of heads has the same latent)
+            for (int i = tid; i < D + (latent ? 0 : E); i += kConsumers)
+                (i < D ? A.kc[row * krow + i] : A.vc[row * vrow + (i - D)]) = from_f<T>(A.own[i]);
+    }
+    csync();
+    const int old = A.count - (own ? 1 : 0);
+    for (int c0 = 0; c0 == 0 || c0 < old; c0 += kMmaKeys) {
+        const int n = min(kMmaKeys, old - c0);
+        const bool last = c0 + kMmaKeys >= old, with_own = last && own;
+        // scores: a warp takes tiles of 8 keys; lane (r, c) holds eight neighbours of key r's row per 32
+        for (int t = warp; t * 8 < n; t += kConsumerWarps) {
+            const bool live = t * 8 + r < n;
+            const T* k = kbase + (size_t)rows[live ? t * 8 + r : 0] * krow + c * 8;
+            float s[2][4] = {};
+            for (int b0 = 0; b0 < blocks; b0 += 6) {
+                uint4 kv[6];
+#pragma unroll
+                for (int i = 0; i < 6; ++i)
+                    kv[i] = live && (b0 + i) * 32 + c * 8 < D ? mkb::ld_nc_v4(k + (b0 + i) * 32) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                for (int i = 0; i < 6; ++i) {
+                    if (b0 + i >= blocks) break;
+#pragma unroll
+                    for (int h = 0; h < 2; ++h) {
+                        const uint4 x = frag[((b0 + i) * 2 + h) * 32 + lane];
+                        uint4 y = make_uint4(0, 0, 0, 0);
+                        if (S.planes > 1) y = frag[((blocks + b0 + i) * 2 + h) * 32 + lane];
+                        const uint32_t hi[4] = {x.x, y.x, x.y, y.y}, lo[4] = {x.z, y.z, x.w, y.w};
+                        const uint32_t k0 = h ? kv[i].z : kv[i].x, k1 = h ? kv[i].w : kv[i].y;
+                        mma_16816(s[0], hi, k0, k1);
+                        mma_16816(s[1], lo, k0, k1);
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int head = r + 8 * (j >> 1), key = t * 8 + 2 * c + (j & 1);
+                if (head < nq) p[head * kMmaCols + key] = key < n ? s[0][j] + s[1][j] : -INFINITY;
+            }
+        }
+        if (with_own)
+            for (int h = kConsumerWarps - 1 - warp; h < nq; h += kConsumerWarps) {
+                float s = 0.f;
+                for (int i = lane; i < D; i += 32) s = fmaf(A.q[h * S.qs + i], to_f(from_f<T>(A.own[i])), s);
+                s = warp_sum(s);
+                if (lane == 0) p[h * kMmaCols + kMmaKeys] = s;
+            }
+        csync();
+        const int padded = (n + 15) & ~15;
+        for (int h = warp; h < nq; h += kConsumerWarps) {
+            float* row = p + h * kMmaCols;
+            const float before = c0 > 0 ? A.m[h] : -INFINITY;
+            float v[kMmaKeys / 32], x = with_own ? fmaxf(before, row[kMmaKeys]) : before;
+#pragma unroll
+            for (int j = 0; j < kMmaKeys / 32; ++j) {
+                v[j] = lane + 32 * j < n ? row[lane + 32 * j] : -INFINITY;
+                x = fmaxf(x, v[j]);
+            }
+            x = warp_max(x);
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < kMmaKeys / 32; ++j) {
+                const float y = x == -INFINITY ? 0.f : expf(v[j] - x);
+                if (lane + 32 * j < padded) row[lane + 32 * j] = y;
+                s += y;
+            }
+            s = warp_sum(s);
+            if (lane == 0) {
+                const float fac = x == -INFINITY ? 1.f : expf(before - x);
+                if (with_own) s += row[kMmaKeys] = expf(row[kMmaKeys] - x);
+                A.l[h] = (c0 > 0 ? A.l[h] * fac : 0.f) + s;
+                A.f[h] = fac;
+                A.m[h] = x;
+            }
+        }
+        csync();
+        if (group < S.groups) {
+            if (c0 > 0) {
+                const float f0 = r < nq ? A.f[r] : 0.f, f1 = r + 8 < nq ? A.f[r + 8] : 0.f;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    acc[i][0] *= f0;
+                    acc[i][1] *= f0;
+                    acc[i][2] *= f1;
+                    acc[i][3] *= f1;
+                }
+            }
+            // a warp takes 32 value columns and every groups-th run of 16 keys, four runs at a time
+            const int step = 16 * S.groups;
+            for (int k0 = group * 16; k0 < n; k0 += 4 * step) {
+                uint2 v[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const int key = k0 + u * step + 2 * c + (j & 1) + 8 * (j >> 1);
+                        v[u][j] = make_uint2(0, 0);
+                        if (key < n && e0 < E) v[u][j] = __ldg(reinterpret_cast<const uint2*>(vbase + (size_t)rows[key] * vrow + e0));
+                    }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const int k = k0 + u * step;
+                    if (k >= n) break;
+                    uint32_t hi[4] = {}, lo[4] = {};
+                    const float* row = p + r * kMmaCols + k + 2 * c;
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        if (r + 8 * (j & 1) >= nq) continue;
+                        const float2 y = *reinterpret_cast<const float2*>(row + (j & 1) * 8 * kMmaCols + 8 * (j >> 1));
+                        split_bf16(y.x, y.y, hi[j], lo[j]);
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const uint32_t a0 = j < 2 ? v[u][0].x : v[u][0].y, a1 = j < 2 ? v[u][1].x : v[u][1].y;
+                        const uint32_t a2 = j < 2 ? v[u][2].x : v[u][2].y, a3 = j < 2 ? v[u][3].x : v[u][3].y;
+                        const uint32_t sel = j & 1 ? 0x7632u : 0x5410u, b0 = __byte_perm(a0, a1, sel), b1 = __byte_perm(a2, a3, sel);
+                        mma_16816(acc[j], hi, b0, b1);
+                        mma_16816(acc[j], lo, b0, b1);
+                    }
+                }
+            }
+        }
+        if (!last) {
+            csync();  // the buffers of scores and rows are free
+            A.list_rows(c0 + kMmaKeys, min(kMmaKeys, old - c0 - kMmaKeys));
+            csync();
+        }
+    }
+    // this lane's sums: heads r and r + 8, four neighbouring columns for each of two indices
+    const int PE = part_row(g.part_vdim), max_splits = g.max_splits;
+    float* const part = g.attn_part + ((size_t)kvh * nq * max_splits + d.a1) * PE;
+    auto out = [&](float* dst, size_t ld, bool finish) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int head = r + 8 * (j >> 1), e = slice * 32 + (2 * c + (j & 1)) * 4;
+            if (head >= nq || e >= E) continue;  // (E is a multiple of 8)
+            float4 y = make_float4(acc[0][j], acc[1][j], acc[2][j], acc[3][j]);
+            if (finish && own) {
+                const float w = p[head * kMmaCols + kMmaKeys];
+                const float* v = own_v + e;
+                y.x = fmaf(w, to_f(from_f<T>(v[0])), y.x);
+                y.y = fmaf(w, to_f(from_f<T>(v[1])), y.y);
+                y.z = fmaf(w, to_f(from_f<T>(v[2])), y.z);
+                y.w = fmaf(w, to_f(from_f<T>(v[3])), y.w);
+            }
+            *reinterpret_cast<float4*>(dst + head * ld + e) = y;
+        }
+    };
+    if (S.groups == 1) {
+        if (group == 0) out(part + kPartLead, (size_t)max_splits * PE, true);
+    } else {
+        if (group < S.groups) out(red + group * nq * E, E, false);
+        csync();
+        for (int i = tid; i < nq * E; i += kConsumers) {
+            const int h = i / E, e = i - h * E;
+            float y = own ? p[h * kMmaCols + kMmaKeys] * to_f(from_f<T>(own_v[e])) : 0.f;
+            for (int k = 0; k < S.groups; ++k) y += red[k * nq * E + i];
+            part[(size_t)h * max_splits * PE + kPartLead + e] = y;
+        }
+    }
+    if (tid < nq) {
+        part[(size_t)tid * max_splits * PE] = A.m[tid];
+        part[(size_t)tid * max_splits * PE + 1] = A.l[tid];
+    }
+}
+
+// Output of a latent attention's head in latent space, merged over the splits: the input of its
+// expansion.  Every warp works out the splits' factors; the partial rows are on their way meanwhile.
+__device__ __forceinline__ void latent_activation(const Params& pr, const MkbhLayer& L, int head, int splits, float* act) {
+    const MkbhGlobals& g = pr.g;
+    const int lane = threadIdx.x & 31, PE = part_row(g.part_vdim), e = threadIdx.x;  // (rank <= 512)
+    const float* row = g.attn_part + (size_t)head * g.max_splits * PE;
+    const float m = lane < splits ? ld_cg_f32(row + (size_t)lane * PE) : -INFINITY;
+    const float l = lane < splits ? ld_cg_f32(row + (size_t)lane * PE + 1) : 0.f;
+    float x[16], y = 0.f, f = 0.f;
+    for (int s0 = 0; s0 < splits; s0 += 16) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) x[j] = e < L.rank && s0 + j < splits ? ld_cg_f32(row + (size_t)(s0 + j) * PE + kPartLead + e) : 0.f;
+        if (s0 == 0) {
+            f = expf(m - warp_max(m));
+            f /= warp_sum(l * f);
+        }
+#pragma unroll
+        for (int j = 0; j < 16; ++j) y = fmaf(__shfl_sync(0xffffffffu, f, (s0 + j) & 31), x[j], y);
+    }
+    if (e < pad8(L.rank)) act[e] = e < L.rank ? y : 0.f;
+}
+
 // The split of a KV head that arrives last merges the partial rows.  Differential: combines the
 // maps, normalises and gates.  Rotary: turns the outputs back.
-__device__ __forceinline__ void merge_splits(const Params& pr, const Cta& c, const Desc& d, float* act) {
+template <bool kDiff>
+__device__ __forceinline__ void merge_splits(const Params& pr, int pos, const Desc& d, float* act) {
     const MkbhGlobals& g = pr.g;
     const MkbhLayer& L = d.L;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const bool diff = L.mixer == MKBH_DIFF_ATTENTION;
-    const int E = attn_vdim(L), per = L.heads / L.kv_heads, maps = attn_maps(L), nq = maps * per, kvh = d.a0, splits = d.a2, PE = g.part_vdim + 2;
-    const float* part = g.attn_part + (size_t)kvh * nq * g.max_splits * PE;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, max_splits = g.max_splits;
+    const int E = L.vdim, per = L.heads / L.kv_heads, maps = kDiff ? 2 : 1, nq = maps * per, kvh = d.a0, splits = d.a2, PE = part_row(g.part_vdim);
+    const float* part = g.attn_part + (size_t)kvh * nq * max_splits * PE;
     float *fac = act, *o = act + nq * splits, *norm = o + per * E;
     for (int qv = warp; qv < nq; qv += kConsumerWarps) {
-        const float* row = part + ((size_t)qv * g.max_splits + lane) * PE;
+        const float* row = part + ((size_t)qv * max_splits + lane) * PE;
         const float m = lane < splits ? ld_cg_f32(row) : -INFINITY, l = lane < splits ? ld_cg_f32(row + 1) : 0.f;
-        const float sink = L.sink != nullptr ? __ldg(L.sink + kvh * per + qv) : -INFINITY;  // (one map)
-        const float top = fmaxf(warp_max(m), sink), f = expf(m - top), total = warp_sum(l * f) + expf(sink - top);
+        const float sink = !kDiff && L.sink != nullptr ? __ldg(L.sink + kvh * per + qv) : -INFINITY;
+        const float top = fmaxf(warp_max(m), sink), f = expf(m - top), total = warp_sum(l * f) + (kDiff ? 0.f : expf(sink - top));
         if (lane < splits) fac[qv * splits + lane] = f / total;
     }
     csync();
     for (int i = tid; i < per * E; i += kConsumers) {
         const int hh = i / E, e = i % E;
-        const float *s1 = part + (size_t)(maps * hh) * g.max_splits * PE + 2 + e, *s2 = s1 + (size_t)g.max_splits * PE;
+        const float *s1 = part + (size_t)(maps * hh) * max_splits * PE + kPartLead + e, *s2 = s1 + (size_t)max_splits * PE;
         const float *f1 = fac + maps * hh * splits, *f2 = f1 + splits;
+        constexpr int B = kDiff ? 8 : 16;  // splits in flight
         float a1 = 0.f, a2 = 0.f;
-        for (int s = 0; s < splits; s += 8) {
-            float x[8], y[8];
+        for (int s = 0; s < splits; s += B) {
+            float x[B], y[B];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < B; ++j) {
                 x[j] = s + j < splits ? ld_cg_f32(s1 + (size_t)(s + j) * PE) : 0.f;
-                y[j] = diff && s + j < splits ? ld_cg_f32(s2 + (size_t)(s + j) * PE) : 0.f;
+                if constexpr (kDiff) y[j] = s + j < splits ? ld_cg_f32(s2 + (size_t)(s + j) * PE) : 0.f;
             }
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+            for (int j = 0; j < B; ++j)
                 if (s + j < splits) {
                     a1 = fmaf(f1[s + j], x[j], a1);
-                    if (diff) a2 = fmaf(f2[s + j], y[j], a2);
+                    if constexpr (kDiff) a2 = fmaf(f2[s + j], y[j], a2);
                 }
         }
-        o[i] = diff ? a1 - L.lambda * a2 : a1;
+        o[i] = kDiff ? a1 - L.lambda * a2 : a1;
     }
     csync();
-    if (!diff) {
-        float* dst = (L.mixer == MKBH_LATENT_ATTENTION ? side_latent(g) : g.mixed) + (size_t)kvh * per * E;
-        const float2* turn = L.value_rope == nullptr ? nullptr : reinterpret_cast<const float2*>(L.value_rope) + (size_t)c.pos * (E / 2);
+    if constexpr (!kDiff) {
+        const float2* turn = L.value_rope == nullptr ? nullptr : reinterpret_cast<const float2*>(L.value_rope) + (size_t)pos * (E / 2);
         for (int i = tid; i < per * E; i += kConsumers) {
             float y = o[i];
             if (turn != nullptr) {  // (an even number of elements per head)
                 const float2 r = __ldg(turn + (i % E >> 1));
                 y = y * r.x + (i & 1 ? -r.y : r.y) * o[i ^ 1];
             }
-            dst[i] = y;
+            g.mixed[(size_t)kvh * per * E + i] = y;
         }
-        return;
+    } else {
+        for (int hh = warp; hh < per; hh += kConsumerWarps) {
+            float s = 0.f;
+            for (int e = lane; e < E; e += 32) s = fmaf(o[hh * E + e], o[hh * E + e], s);
+            s = warp_sum(s);
+            if (lane == 0) norm[hh] = (1.f - L.diff) / sqrtf(s / E + g.eps);
+        }
+        csync();
+        const float* gate = g.proj + L.heads * 2 * L.dim + (size_t)kvh * per * E;
+        for (int i = tid; i < per * E; i += kConsumers)
+            g.mixed[(size_t)kvh * per * E + i] = o[i] * norm[i / E] * sigmoid_f(ld_cg_f32(gate + i));
     }
-    for (int hh = warp; hh < per; hh += kConsumerWarps) {
-        float s = 0.f;
-        for (int e = lane; e < E; e += 32) s = fmaf(o[hh * E + e], o[hh * E + e], s);
-        s = warp_sum(s);
-        if (lane == 0) norm[hh] = (1.f - L.diff) / sqrtf(s / E + g.eps);
-    }
-    csync();
-    const float* gate = g.proj + L.heads * 2 * L.dim + (size_t)kvh * per * E;
-    for (int i = tid; i < per * E; i += kConsumers)
-        g.mixed[(size_t)kvh * per * E + i] = o[i] * norm[i / E] * sigmoid_f(ld_cg_f32(gate + i));
 }
 
 // Short convolutions over time: keep this token's inputs and sum up the terms of the next token's
@@ -1173,7 +1517,18 @@ __device__ __forceinline__ void merge_splits(const Params& pr, const Cta& c, con
 // input, `u` is this thread's row of the stacked projection before its convolution.
 __device__ __forceinline__ void keep_input(float now, const float* w, float* hist, float* next, int taps, size_t ld, int pos) {
     float s = __ldg(w + (taps - 2) * ld) * now;
-    for (int i = 1; i <= taps - 2 && i <= pos; ++i) s = fmaf(__ldg(w + (taps - 2 - i) * ld), hist[((pos - i) % (taps - 1)) * ld], s);
+    for (int i0 = 1; i0 <= taps - 2; i0 += 4) {
+        float a[4], b[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = i0 + j;
+            const bool live = i <= taps - 2 && i <= pos;
+            a[j] = live ? __ldg(w + (taps - 2 - i) * ld) : 0.f;
+            b[j] = live ? hist[((pos - i) % (taps - 1)) * ld] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s = fmaf(a[j], b[j], s);
+    }
     hist[(pos % (taps - 1)) * ld] = now;
     *next = s;
 }
@@ -1200,7 +1555,7 @@ __device__ __forceinline__ unsigned long long argmax_key(float v, int i) {
     return ((unsigned long long)u << 32) | (0xffffffffu - (uint32_t)i);
 }
 
-template <typename T>
+template <typename T, int F>
 __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Smem& sm) {
     const MkbhGlobals& g = p.g;
     const int tid = threadIdx.x, warp = tid >> 5;
@@ -1233,19 +1588,16 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
         rec(0);
         // ---- what does not depend on the producers ----
         StateCol state;
-        if (op == MKBH_OP_DELTA_STEP)
+        if ((F & kClassic) && op == MKBH_OP_DELTA_STEP)
             state.load(L.state + (((size_t)g.slot * L.heads + d.a0) * L.dim + d.a1 + warp) * L.dim, L.dim,
                        c.pos > 0 && d.a1 + warp < d.a2);
-        if (op == MKBH_OP_ATTENTION) {
-            const AttnView<T> A(p, c, d, act);
-            A.stage(0, min(p.attn_chunk, A.count));
-        }
+        if (op == MKBH_OP_ATTENTION) attend_ahead<T, F>(p, c.pos, d, act);
         if (d.has_vec) {
             ok = bar_wait(p, c, c.bar(kVecFull), vecs & 1u, 1);
             if (!ok) c.ctl[0] = 1;
             ++vecs;
         }
-        const bool conv = op == MKBH_OP_NORM_PROJ && L.conv_taps > 0;
+        const bool conv = (F & kRotary) && op == MKBH_OP_NORM_PROJ && L.conv_taps > 0;
         float* conv_part = conv ? L.conv_part + (size_t)g.slot * L.in_rows + d.a0 + tid : nullptr;
         const float earlier = conv && c.pos > 0 && tid < d.a1 - d.a0 ? *conv_part : 0.f;  // earlier inputs' terms
         // ---- the producers ----
@@ -1255,66 +1607,72 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
         rec(1);
         bool signal = true;
         float kept = 0.f;  // this thread's row before the convolution
-        if (op == MKBH_OP_DELTA_STEP) {
+        if ((F & kClassic) && op == MKBH_OP_DELTA_STEP) {
             delta_step<T>(p, c, d, act, vec, rowv, state);
             csync();
             if (tid == 0) mbar_arrive(c.bar(kVecEmpty));
         } else if (op == MKBH_OP_ATTENTION) {
-            const AttnView<T> A(p, c, d, act);
-            const int need = (A.nq + kConsumers / A.E - 1) / (kConsumers / A.E);
-            if (need <= 2) attend<T, 2>(p, A, d);
-            else if (need <= 4) attend<T, 4>(p, A, d);
-            else attend<T, 16>(p, A, d);
-            csync();
-            if (tid == 0) {
-                int old;
-                int* cnt = counters + (g.num_layers + 1) * MKBH_BARRIERS_PER_LAYER + d.layer * g.max_kv_heads + d.a0;
-                asm volatile("atom.acq_rel.gpu.global.add.s32 %0, [%1], 1;" : "=r"(old) : "l"(cnt) : "memory");
-                c.ctl[1] = old == d.a2 - 1;
+            bool done = false;
+            if constexpr (sizeof(T) == 2 && (F & kRotary)) {
+                done = mma_attention<T>(L);
+                if (done) attend_mma<T, F>(p, c.pos, d, act);
             }
+            if (!done) attend_fma<T, F>(p, c.pos, d, act);
             csync();
-            signal = c.ctl[1] != 0;
-            if (signal) merge_splits(p, c, d, act);
-            csync();
+            if (F == kClassic || L.mixer != MKBH_LATENT_ATTENTION) {  // (a latent's partial rows are merged by what expands them)
+                if (tid == 0) {
+                    int old;
+                    int* cnt = counters + (g.num_layers + 1) * MKBH_BARRIERS_PER_LAYER + d.layer * g.max_kv_heads + d.a0;
+                    asm volatile("atom.acq_rel.gpu.global.add.s32 %0, [%1], 1;" : "=r"(old) : "l"(cnt) : "memory");
+                    c.ctl[1] = old == d.a2 - 1;
+                }
+                csync();
+                signal = c.ctl[1] != 0;
+                if (signal) {
+                    if (F == kClassic || ((F & kClassic) && L.mixer == MKBH_DIFF_ATTENTION)) merge_splits<true>(p, c.pos, d, act);
+                    else merge_splits<false>(p, c.pos, d, act);
+                }
+                csync();
+            }
         } else if (op >= MKBH_OP_NORM_PROJ && op <= MKBH_OP_EXPAND) {
             const int rows = d.a1 - d.a0, K = d.row_bytes / (int)sizeof(T);
             // channels whose input this instruction keeps for the convolution of later tokens
-            const bool canon = op == MKBH_OP_NORM_PROJ && L.canon_taps > 1;
+            const bool canon = (F & kRotary) && op == MKBH_OP_NORM_PROJ && L.canon_taps > 1;
             const int stash_lo = canon ? (int)((long long)g.width * d.a0 / L.in_rows) : 0;
             const int stash_hi = canon ? (int)((long long)g.width * d.a1 / L.in_rows) : 0;
-            const bool aside = op == MKBH_OP_DOWN && L.parallel;  // the output projection adds it
-            const bool adds = op == MKBH_OP_OUT_PROJ || (op == MKBH_OP_DOWN && !L.parallel);
-            float* x = g.x + (size_t)L.x_buf * g.width;
-            const bool first = d.layer == 0 && (op == MKBH_OP_ENTER || L.enter_w == nullptr);  // the stream is the embedding
+            const bool beside = (F & kRotary) && L.parallel, aside = op == MKBH_OP_DOWN && beside;  // the output projection adds it
+            const bool adds = op == MKBH_OP_OUT_PROJ || (op == MKBH_OP_DOWN && !beside);
+            float* x = (F & kRotary) ? g.x + (size_t)L.x_buf * g.width : g.x;
+            const bool first = d.layer == 0 && (F == kClassic || op == MKBH_OP_ENTER || L.enter_w == nullptr);  // the stream is the embedding
             // this instruction is the only writer of its rows of the residual stream
             float old = adds && tid < rows ? ld_cg_f32(x + d.a0 + tid) : 0.f;
-            if (op == MKBH_OP_OUT_PROJ && L.parallel && L.ff && tid < rows) old += ld_cg_f32(side_out(g) + d.a0 + tid);
+            if (op == MKBH_OP_OUT_PROJ && beside && L.ff && tid < rows) old += ld_cg_f32(side_out(g) + d.a0 + tid);
             if (op == MKBH_OP_OUT_PROJ) {
-                if (L.mixer == MKBH_DELTA_RULE) delta_activation(p, L, reinterpret_cast<const float*>(vec), act);
+                if ((F & kClassic) && L.mixer == MKBH_DELTA_RULE) delta_activation(p, L, reinterpret_cast<const float*>(vec), act);
                 else if (K <= 8192) plain_activation<16>(g.mixed, L.heads * L.vdim, act);
                 else plain_activation<32>(g.mixed, L.heads * L.vdim, act);
-            } else if (op == MKBH_OP_DOWN && L.ff_kind == MKBH_CLAMPED_GLU) {
+            } else if ((F & kRotary) && op == MKBH_OP_DOWN && (F == kRotary || L.ff_kind == MKBH_CLAMPED_GLU)) {
                 if (K <= 8192) plain_activation<16>(side_in(g), L.ff, act);
                 else plain_activation<32>(side_in(g), L.ff, act);
-            } else if (op == MKBH_OP_DOWN) {
+            } else if ((F & kClassic) && op == MKBH_OP_DOWN) {
                 if (K <= 8192) poly_activation<16>(p, L, act, red, turn);
                 else poly_activation<32>(p, L, act, red, turn);
-            } else if (op == MKBH_OP_ABSORB) {
+            } else if ((F & kRotary) && op == MKBH_OP_ABSORB) {
                 plain_activation<4>(g.proj + (size_t)(d.a0 / L.rank) * (L.dim + L.rot_dim), L.dim, act);
-            } else if (op == MKBH_OP_EXPAND) {
-                plain_activation<4>(side_latent(g) + (size_t)(d.a0 / L.vdim) * L.rank, L.rank, act);
-            } else if (op == MKBH_OP_ENTER) {
+            } else if ((F & kRotary) && op == MKBH_OP_EXPAND) {
+                latent_activation(p, L, d.a0 / L.vdim, d.a2, act);
+            } else if ((F & kRotary) && op == MKBH_OP_ENTER) {
                 enter_activation<T>(g, first ? nullptr : g.x + (size_t)(L.x_buf ^ 1) * g.width, act);
             } else {
                 const float* w = reinterpret_cast<const float*>(vec);
-                const float* part = d.part_off >= 0 ? reinterpret_cast<const float*>(c.gb + sm.vec + d.part_off) : nullptr;
+                const float* part = (F & kRotary) && d.part_off >= 0 ? reinterpret_cast<const float*>(c.gb + sm.vec + d.part_off) : nullptr;
                 const bool in = op == MKBH_OP_NORM_PROJ;
-                const float* src = first && (in || (op == MKBH_OP_NORM_UP && L.parallel)) ? nullptr
-                                   : op == MKBH_OP_HEAD ? g.x + (size_t)p.last_buf * g.width : x;
+                const float* src = first && (in || (op == MKBH_OP_NORM_UP && beside)) ? nullptr
+                                   : (F & kRotary) && op == MKBH_OP_HEAD ? g.x + (size_t)p.last_buf * g.width : x;
                 float* publish = src == nullptr && in && d.a0 == 0 ? x : nullptr;
-                if (K <= 2048) norm_activation<T, 4>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
-                else if (K <= 8192) norm_activation<T, 16>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
-                else norm_activation<T, 32>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
+                if (K <= 2048) norm_activation<T, F, 4>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
+                else if (K <= 8192) norm_activation<T, F, 16>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
+                else norm_activation<T, F, 32>(p, c, src, w, part, act, red, turn, publish, stash, stash_lo, stash_hi);
             }
             csync();
             if (tid == 0 && d.has_vec) mbar_arrive(c.bar(kVecEmpty));
@@ -1335,15 +1693,15 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
                     x[row] = fmaf(d.row_off >= 0 ? rowv[tid] : 1.f, y, old);
                 } else if (conv) {
                     g.proj[row] = fmaf(rowv[tid], y, earlier);
-                } else if (op == MKBH_OP_ENTER) {
+                } else if ((F & kRotary) && op == MKBH_OP_ENTER) {
                     x[row] = y;
                 } else if (aside) {
                     side_out(g)[row] = y;
-                } else if (op == MKBH_OP_ABSORB) {
+                } else if ((F & kRotary) && op == MKBH_OP_ABSORB) {
                     side_query(g)[row] = y;
-                } else if (op == MKBH_OP_EXPAND) {
+                } else if ((F & kRotary) && op == MKBH_OP_EXPAND) {
                     g.mixed[row] = y;
-                } else if (op == MKBH_OP_NORM_UP && L.ff_kind == MKBH_CLAMPED_GLU) {  // rows alternate gate, up
+                } else if ((F & kRotary) && op == MKBH_OP_NORM_UP && (F == kRotary || L.ff_kind == MKBH_CLAMPED_GLU)) {  // rows alternate gate, up
                     if ((tid & 1) == 0) {
                         float up = 0.f;
                         for (int k = 0; k < d.groups; ++k) up += act[(tid + 1) * d.groups + k];
@@ -1384,7 +1742,7 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             return;
         }
         if (tid == 0 && signal) red_release_gpu_add(counters + d.arrive_idx, 1);
-        if (op == MKBH_OP_NORM_PROJ && (L.canon_taps > 1 || L.conv_taps > 1)) {  // for later tokens only
+        if ((F & kRotary) && op == MKBH_OP_NORM_PROJ && (L.canon_taps > 1 || L.conv_taps > 1)) {  // for later tokens only
             publish_convolutions(p, c, d, stash, kept);
             csync();
         }
@@ -1393,7 +1751,7 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
     }
 }
 
-template <typename T>
+template <typename T, int F>
 __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_constant__ Params p) {
     extern __shared__ uint8_t raw[];
     const uint32_t raw32 = smem_u32(raw), base = (raw32 + 127u) & ~127u;
@@ -1423,13 +1781,13 @@ __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_c
         return;
     }
     const int warp = threadIdx.x >> 5;
-    if (warp < kConsumerWarps) consumer_main<T>(p, c, sm);
+    if (warp < kConsumerWarps) consumer_main<T, F>(p, c, sm);
     else if (warp == kOperandWarp) operand_main<T>(p, c, sm);
     else if ((threadIdx.x & 31) == 0) loader_main<T>(p, c);
     __syncthreads();
 }
 
-template <typename T>
+template <typename T, int F>
 cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     Params p;
     p.g = g;
@@ -1456,11 +1814,11 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
         if (!is_attention(L)) continue;
         const int per = L.heads / L.kv_heads, nq = attn_maps(L) * per;
         act = max(act, max(4 * merge_scratch_floats(nq, g.max_splits, per, attn_vdim(L)),
-                           attn_scratch_bytes<T>(L, L.mixer == MKBH_LATENT_ATTENTION && sizeof(T) == 2 ? 32 : 8)));
+                           mma_attention<T>(L) ? 4 * MmaScratch(L).total : attn_scratch_bytes<T>(L, 8)));
     }
     for (int i = 0; i < g.num_layers; ++i) {
         const MkbhLayer& L = g.layers_host[i];
-        if (!is_attention(L)) continue;
+        if (!is_attention(L) || mma_attention<T>(L)) continue;
         while (p.attn_chunk > 8 && attn_scratch_bytes<T>(L, p.attn_chunk) > act) p.attn_chunk -= 8;
     }
     p.last_buf = g.layers_host[g.num_layers - 1].x_buf;
@@ -1477,7 +1835,7 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return e;
     if (set[dev & 63] < smem) {
-        e = cudaFuncSetAttribute(hybrid_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        e = cudaFuncSetAttribute(hybrid_decode_kernel<T, F>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return e;
         set[dev & 63] = smem;
     }
@@ -1485,14 +1843,24 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
     if (e != cudaSuccess) return e;
     // cooperative: the CTAs wait for one another, so all of them must be resident
     void* args[] = {&p};
-    return cudaLaunchCooperativeKernel((const void*)hybrid_decode_kernel<T>, dim3(g.num_sms), dim3(kBlock), args,
+    return cudaLaunchCooperativeKernel((const void*)hybrid_decode_kernel<T, F>, dim3(g.num_sms), dim3(kBlock), args,
                                        (size_t)smem, s);
 }
 
 }  // namespace
 
 cudaError_t decode_launch(const MkbhGlobals& g, cudaStream_t s) {
-    return g.dtype == MKBH_F32 ? launch<float>(g, s) : launch<bf16>(g, s);
+    int features = g.norm_kind == MKBH_LAYER_NORM ? kClassic : kRotary;
+    for (int i = 0; i < g.num_layers; ++i) {
+        const MkbhLayer& L = g.layers_host[i];
+        features |= L.mixer == MKBH_DELTA_RULE || L.mixer == MKBH_DIFF_ATTENTION ? kClassic : kRotary;
+        if (L.ff) features |= L.ff_kind == MKBH_POLY_NORM ? kClassic : kRotary;
+        if (L.parallel || L.canon_taps || L.conv_taps || L.enter_w) features |= kRotary;
+    }
+    const bool f32 = g.dtype == MKBH_F32;
+    if (features == kClassic) return f32 ? launch<float, kClassic>(g, s) : launch<bf16, kClassic>(g, s);
+    if (features == kRotary) return f32 ? launch<float, kRotary>(g, s) : launch<bf16, kRotary>(g, s);
+    return f32 ? launch<float, kClassic | kRotary>(g, s) : launch<bf16, kClassic | kRotary>(g, s);
 }
 
 }  // namespace mkbh

@@ -115,7 +115,7 @@ int check_globals(const MkbhGlobals* gp) {
             "missing pointers");
     REQUIRE(g.x && g.proj && g.mixed && g.decay && g.act, "missing activation buffers");
     REQUIRE(g.norm_kind == MKBH_LAYER_NORM || g.norm_kind == MKBH_RMS_NORM, "unknown norm %d", g.norm_kind);
-    REQUIRE(g.side_ff % 8 == 0 && g.side_rank % 8 == 0 && (!g.side || g.side_elems >= (int64_t)g.side_ff + pad8(g.width) + 2 * (int64_t)g.side_rank),
+    REQUIRE(g.side_ff % 8 == 0 && g.side_rank % 8 == 0 && (!g.side || g.side_elems >= (int64_t)g.side_ff + pad8(g.width) + (int64_t)g.side_rank),
             "side buffer too small");
     for (int i = 0; i < g.num_layers; ++i)
         if (int rc = check_layer(g, i)) return rc;
@@ -285,6 +285,8 @@ int mkb_hybrid_validate(const MkbhGlobals* gp, const int32_t* ins) {
                     REQUIRE(L.mixer == MKBH_LATENT_ATTENTION, "queue %d, instruction %d: layer %d has no latent", q, k, layer);
                     const int per = op == MKBH_OP_ABSORB ? L.rank : L.vdim;  // rows of a head
                     rows = L.heads * per, K = op == MKBH_OP_ABSORB ? L.dim : L.rank;
+                    if (op == MKBH_OP_EXPAND)
+                        REQUIRE(w[4] > 0 && w[4] <= g.max_splits, "queue %d, instruction %d: %d splits", q, k, w[4]);
                     REQUIRE(w[2] >= 0 && w[2] < w[3] && w[2] / per == (w[3] - 1) / per, "queue %d, instruction %d: rows %d..%d of several heads", q, k, w[2], w[3]);
                 } else {
                     REQUIRE(L.ff > 0, "queue %d, instruction %d: layer %d has no feed-forward", q, k, layer);

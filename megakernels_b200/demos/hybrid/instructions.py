@@ -40,7 +40,7 @@ class HybridGlobals:
     argmax_out: Tensor  # int32 [1]
     counters: Tensor  # int32, zeroed by every decode launch
     arrivals: Tensor  # int32 [layer runs + 1, COUNTERS_PER_LAYER]
-    attn_part: Tensor  # fp32 [max heads, 2, max_splits, max vdim + 2]
+    attn_part: Tensor  # fp32 [max heads, 2, max_splits, 4 + max vdim]
     status: Tensor  # int32 [16]
     max_splits: int
     max_kv_heads: int
@@ -50,7 +50,7 @@ class HybridGlobals:
     ffn: Tensor  # model dtype [portion, ff]: gated units
     keys: Tensor  # model dtype [positions, heads * (dim + vdim)]: keys and values expanded from latents
     tail: Tensor  # fp32 [taps, width]: the portion's last inputs of the input convolution
-    side: Tensor  # fp32 [side_ff + width + 2 * side_rank]: decode vectors beside the stacked projection
+    side: Tensor  # fp32 [side_ff + width + side_rank]: decode vectors beside the stacked projection
     side_ff: int
     side_rank: int
 
@@ -137,7 +137,8 @@ class DeltaStep(Instruction):
 
 @dataclass
 class KeyAttention(Instruction):
-    """One split of the keys a KV head's queries see; the last split to arrive merges them."""
+    """One split of the keys that a KV head's queries see; the last split to arrive merges them (of a
+    latent: ``Expand`` does)."""
 
     layer_idx: int
     kv_head_idx: int
@@ -213,7 +214,10 @@ class Absorb(RowRange):
 
 @dataclass
 class Expand(RowRange):
-    """Latent attention: a head's output from latent to value space (rows of one head)."""
+    """Latent attention: a head's output, merged over the splits of the keys, from latent to value
+    space (rows of one head)."""
+
+    num_splits: int
 
     @classmethod
     def opcode(cls) -> int:

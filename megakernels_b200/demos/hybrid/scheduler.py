@@ -103,12 +103,12 @@ def make_globals(model, options: HybridScheduleOptions) -> HybridGlobals:
         decay=f32(n, max([d.inner + 2 * d.heads for d in delta], default=1)), act=own(n, act),
         logits=f32(cfg.vocab_size), argmax_out=i32(1),
         counters=i32((2 + (R + 1) * COUNTERS_PER_LAYER + R * groups + 1) // 2 * 2),
-        arrivals=i32(R + 1, COUNTERS_PER_LAYER), attn_part=f32(heads, 2, splits, vdim + 2), status=i32(16),
+        arrivals=i32(R + 1, COUNTERS_PER_LAYER), attn_part=f32(heads, 2, splits, 4 + -(-vdim // 4) * 4), status=i32(16),
         max_splits=splits, max_kv_heads=groups, part_vdim=vdim,
         query=own(n, max(widest(m.heads * (m.dim + m.rot_dim) for m in latent), widest(m.heads * m.dim for m in rotary), 1)),
         act2=own(n, widest([cfg.width])), ffn=own(n, max(side_ff, 1)),
         keys=own(model.max_len(), widest(m.heads * (m.dim + m.vdim) for m in latent)) if latent else own(1),
-        tail=f32(max([s.canon_taps for s in layers] + [1]), cfg.width), side=f32(side_ff + pad8(cfg.width) + 2 * side_rank),
+        tail=f32(max([s.canon_taps for s in layers] + [1]), cfg.width), side=f32(side_ff + pad8(cfg.width) + side_rank),
         side_ff=side_ff, side_rank=side_rank,
     )
 
@@ -137,9 +137,9 @@ class HybridScheduleBuilder(ScheduleBuilder):
             n, k = matrix_shape(globs, cls.opcode(), layer)
             return [cls(layer, a, b) for a, b in row_ranges(n, k, globs.dtype_bytes, sms, unit)]
 
-        def head_rows(cls, layer, heads):
+        def head_rows(cls, layer, heads, *rest):
             n, k = matrix_shape(globs, cls.opcode(), layer)
-            return [cls(layer, a, b) for a, b in head_row_ranges(heads, n // heads, k, globs.dtype_bytes, sms)]
+            return [cls(layer, a, b, *rest) for a, b in head_row_ranges(heads, n // heads, k, globs.dtype_bytes, sms)]
 
         def up(i, spec, previous):
             return phase(rows(NormUp, i, unit=2 if spec.mlp.kind == "clamped_glu" else 1), previous, i)
@@ -162,10 +162,10 @@ class HybridScheduleBuilder(ScheduleBuilder):
                     last = phase(head_rows(Absorb, i, m.heads), last, i)
                 n = key_splits(m, globs.model.max_len(), sms, self.options.keys_per_split)
                 splits = [KeyAttention(i, g, s, n) for g in range(m.key_groups) for s in range(n)]
-                last = phase(splits, last, i, arrive=m.key_groups)
+                last = phase(splits, last, i, arrive=None if m.kind == "latent_attention" else m.key_groups)
             down = phase(rows(Down, i), inner, i) if beside else []
             if m.kind == "latent_attention":
-                last = phase(head_rows(Expand, i, m.heads), last, i)
+                last = phase(head_rows(Expand, i, m.heads, n), last, i)
             # (beside a mixer, ``Down`` counts into the phase that ``OutProj`` waits for)
             arrivals[i, last[0].instruction.opcode()] += len(down)
             last = phase(rows(OutProj, i), last + down, i)

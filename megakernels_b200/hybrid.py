@@ -185,7 +185,7 @@ class LatentAttentionSpec:
     @property
     def key_groups(self) -> int:
         """Groups of heads that share an attention instruction in a decode step."""
-        per = max(p for p in range(1, 5) if self.heads % p == 0)
+        per = max(p for p in range(1, 9) if self.heads % p == 0)
         return self.heads // per
 
 

@@ -300,7 +300,7 @@ def test_schedule_covers_everything_once_and_runs_to_its_end(name, mode):
                 if op == 3:
                     k = (i, ins.kv_head_idx)
                     heads_done[k] = heads_done.get(k, 0) + 1
-                    signal = heads_done[k] == ins.num_splits
+                    signal = heads_done[k] == ins.num_splits or cfg.run_layers[i].mixer.kind == "latent_attention"
                 else:
                     signal = True
                 mixer = cfg.run_layers[i].mixer.kind
