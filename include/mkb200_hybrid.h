@@ -96,9 +96,11 @@ typedef struct MkbhLayer {
     const void *decay_w2;      /* [heads*dim, rank], model dtype, not padded */
     const float *decay_w0;     /* [heads*dim] */
     const float *out_norm;     /* [heads*dim] */
-    void *k_cache;             /* [slots, cache_keep + cache_ring, kv_heads, maps, dim]; latent:
-                                  [slots, cache_ring, pad8(rank) + pad8(rot_dim)], latent then rotated key */
-    void *v_cache;             /* [slots, cache_keep + cache_ring, kv_heads, vdim] */
+    /* Rows are positions (cache_keep + cache_ring of them).  Differential: [slots, rows, kv_heads, 2, dim]
+     * and [slots, rows, kv_heads, vdim].  Rotary: [slots, kv_heads, rows, dim] and [slots, kv_heads, rows,
+     * vdim].  Latent: [slots, rows, pad8(rank) + pad8(rot_dim), plus 8 if that is an even number of
+     * eights], the latent, then the rotated key. */
+    void *k_cache, *v_cache;
     float *state;              /* [slots, heads, dim (value channel), dim (key channel)] */
     const void *enter_w;       /* [width, pad8(2 width)]: the run starts a pass of the loop; else NULL */
     /* Convolutions over time: inputs of the last taps-1 positions in a ring by position, and the

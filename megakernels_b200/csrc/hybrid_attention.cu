@@ -341,7 +341,7 @@ __global__ void __launch_bounds__(kFlashThreads, EP <= 128 ? 2 : 1) rotary_flash
             const int idx = tile * kBKeys + t;
             const bool live = idx < total;
             const size_t row = row_of(key_of(live ? idx : 0));
-            const bf16 *ks = a.src.keys + row * a.src.key_ld + g * A, *vs = a.src.values + row * a.src.value_ld + g * E;
+            const bf16 *ks = a.src.keys + row * a.src.key_ld + g * a.src.key_head, *vs = a.src.values + row * a.src.value_ld + g * a.src.value_head;
             for (int u = lane; u < kunits + vunits; u += 32) {
                 if (u < kunits) cp16(kd + (t * S.qs + u * 8) * 2, u < aunits ? ks + u * 8 : a.src.shared + row * a.src.shared_ld + (u - aunits) * 8, live);
                 else cp16(vd + (t * S.vs + (u - kunits) * 8) * 2, vs + (u - kunits) * 8, live);

@@ -81,7 +81,9 @@ struct KeyRange {
 // Sizes of a layer's mixer.
 __host__ __device__ inline bool is_attention(const MkbhLayer& L) { return L.mixer != MKBH_DELTA_RULE; }
 __host__ __device__ inline int mixer_out(const MkbhLayer& L) { return L.heads * (L.mixer == MKBH_DELTA_RULE ? L.dim : L.vdim); }
-__host__ __device__ inline int latent_row(const MkbhLayer& L) { return pad8(L.rank) + pad8(L.rot_dim); }
+__host__ __device__ inline int latent_dim(const MkbhLayer& L) { return pad8(L.rank) + pad8(L.rot_dim); }
+// Elements from one latent to the next: an odd number of eights (rows that start in different banks).
+__host__ __device__ inline int latent_row(const MkbhLayer& L) { return (latent_dim(L) / 8 | 1) * 8; }
 __host__ __device__ inline int up_rows(const MkbhLayer& L) { return L.ff_kind == MKBH_CLAMPED_GLU ? 2 * L.ff : L.ff; }
 // Phase whose end makes the mixer's output complete.
 __host__ __device__ inline int mixer_phase(int mixer) {

@@ -184,7 +184,7 @@ __device__ __forceinline__ float* side_in(const MkbhGlobals& g) { return g.side;
 __device__ __forceinline__ float* side_out(const MkbhGlobals& g) { return g.side + g.side_ff; }
 __device__ __forceinline__ float* side_query(const MkbhGlobals& g) { return side_out(g) + pad8(g.width); }
 
-// ---- loader: the weight stream ----------------------------------------------------------- //
+// ---- the weight stream --------------------------------------------------------------------- //
 struct Block {  // rows [r0, r1) of a matrix of `row_bytes` rows
     const uint8_t* w;
     int r0, r1, row_bytes;
@@ -215,56 +215,6 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, const int* w,
     b.r1 = __ldg(w + 3);
     b.row_bytes = pad8(K) * (int)sizeof(T);
     return true;
-}
-
-template <typename T>
-struct Cursor {  // the queue's weight blocks as a flat sequence of stages
-    int i = 0, row = 0, per = 1;
-    bool open = false;
-    Block b;
-    __device__ bool next(const MkbhGlobals& g, const int* queue, const uint8_t*& src, uint32_t& bytes) {
-        while (!open) {
-            if (i >= g.queue_len) return false;
-            if (weight_block<T>(g, queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION, b) && b.r1 > b.r0) {
-                open = true;
-                row = b.r0;
-                per = kStage / b.row_bytes;
-            } else {
-                ++i;
-            }
-        }
-        const int n = min(per, b.r1 - row);
-        src = b.w + (size_t)row * b.row_bytes;
-        bytes = (uint32_t)(n * b.row_bytes);
-        row += n;
-        if (row >= b.r1) {
-            open = false;
-            ++i;
-        }
-        return true;
-    }
-};
-
-template <typename T>
-__device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
-    const MkbhGlobals& g = p.g;
-    const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
-    const uint64_t policy = mkb::l2_policy_evict_first();
-    Cursor<T> cur;
-    uint32_t issued = 0;
-    const uint8_t* src;
-    uint32_t bytes;
-    const int S = p.stages;
-    while (cur.next(g, queue, src, bytes)) {
-        const int slot = issued % S;
-        if (!bar_wait(p, c, c.empty(slot), ((issued / S) & 1u) ^ 1u, 0)) break;
-        mbar_expect_tx(c.full(slot), bytes);
-        mkb::tma_bulk_g2s(c.base + slot * kStage, src, bytes, c.full(slot), policy);
-        ++issued;
-    }
-    // no copy may be in flight when the CTA's shared memory goes away
-    for (uint32_t s = issued > (uint32_t)S ? issued - S : 0u; s < issued; ++s)
-        bar_wait(p, c, c.full(s % S), (s / S) & 1u, 0, false);
 }
 
 // ---- operand warp ------------------------------------------------------------------------- //
@@ -802,7 +752,7 @@ __device__ __forceinline__ void delta_step(const Params& p, const Cta& c, const 
 // attention is one key per position, the latent with its rotated part, whose first `rank` entries
 // are the value too; a "KV head" is then a group of heads.
 __host__ __device__ inline int attn_maps(const MkbhLayer& L) { return L.mixer == MKBH_DIFF_ATTENTION ? 2 : 1; }
-__host__ __device__ inline int attn_dim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? latent_row(L) : L.dim; }
+__host__ __device__ inline int attn_dim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? latent_dim(L) : L.dim; }
 __host__ __device__ inline int attn_vdim(const MkbhLayer& L) { return L.mixer == MKBH_LATENT_ATTENTION ? L.rank : L.vdim; }
 // Partial rows of the splits: [m, l, -, -, sums ...], 16-byte aligned.
 constexpr int kPartLead = 4;
@@ -837,89 +787,81 @@ __host__ __device__ inline int merge_scratch_floats(int nq, int splits, int per,
 
 // Tensor-core variant of the one-map mixers (bf16): what it keeps in shared memory, in floats.
 constexpr int kMmaKeys = 256;  // keys per pass
-constexpr int kMmaCols = kMmaKeys + 8;  // scores of a head; column kMmaKeys is this token's own key
+constexpr int kMmaCols = kMmaKeys + 8;  // scores of a head
 template <typename T>
 __host__ __device__ inline bool mma_attention(const MkbhLayer& L) {
     return sizeof(T) == 2 && (L.mixer == MKBH_ATTENTION || L.mixer == MKBH_LATENT_ATTENTION) && attn_dim(L) % 8 == 0 &&
-           attn_vdim(L) % 8 == 0 && L.heads / L.kv_heads <= 16;
+           attn_vdim(L) % 8 == 0 && L.heads / L.kv_heads <= 16 && L.keep_first == 0;
 }
 struct MmaScratch {
-    int q, qs, frag, planes, p, m, l, f, own, rows, red, slices, groups, total;
+    int blocks, planes, frag, p, m, l, f, own, row, krows, vrows, red, slices, groups, total;
     __host__ __device__ MmaScratch(const MkbhLayer& L) {
         const int nq = L.heads / L.kv_heads, dim = attn_dim(L), e = attn_vdim(L);
         slices = (e + 31) / 32;             // of the value columns, a warp each ...
         groups = kConsumerWarps / slices;   // ... times groups of keys
         planes = nq > 8 ? 2 : 1;
-        qs = (dim + 31) / 32 * 32;
-        q = 0;
-        frag = nq * qs;                     // queries as fragments: [plane][16 columns][lane][high 2, low 2]
-        p = frag + planes * (qs / 16) * 32 * 4;
+        blocks = (dim + 31) / 32;
+        frag = 0;                           // queries as fragments: [plane][block][half][lane][high 2, low 2]
+        p = planes * blocks * 2 * 32 * 4;
         m = p + nq * kMmaCols;
         l = m + nq;
         f = l + nq;
-        own = (f + nq + 3) & ~3;
-        rows = own + ((dim + e + 3) & ~3);  // cache rows of a pass
-        red = rows + kMmaKeys;
+        own = (f + nq + 3) & ~3;            // this token's key and value: as floats ...
+        row = own + ((dim + e + 3) & ~3);   // ... and as rows of bf16
+        krows = row + ((dim + e + 7) / 8 * 4);  // where a pass's keys and values lie
+        vrows = krows + kMmaKeys;
+        red = vrows + kMmaKeys;
         total = red + (groups > 1 ? groups * nq * e : 0);
     }
 };
 
 template <typename T, int F>
 struct AttnView {
-    int D, KE, E, G, per, nq, qs, ks, vs, t_lo, count, keep, ring, pos;
+    int D, KE, E, G, per, nq, ks, vs, per_stage, t_lo, count, keep, ring, pos;
     size_t krow, vrow;  // elements between positions
     KeyRange keys;
     T *kc, *vc, *kt, *vt;
     float *q, *p, *m, *l, *f, *own;
-    int* rows;  // cache rows of the pass's keys
     bool latent, diff;
-    __device__ __forceinline__ AttnView(const Params& pr, int at, const Desc& d, float* act)
-        : keys(at, d.L.window, d.L.keep_first, d.L.chunk) {
-        const MkbhLayer& L = d.L;
+    __device__ __forceinline__ AttnView(const Params& pr, int at, const MkbhLayer& L, int kvh, int split, int splits, float* act)
+        : keys(at, L.window, L.keep_first, L.chunk) {
         latent = (F & kRotary) && L.mixer == MKBH_LATENT_ATTENTION;
         diff = F == kClassic || ((F & kClassic) && L.mixer == MKBH_DIFF_ATTENTION);
-        D = latent ? latent_row(L) : L.dim; KE = diff ? 2 * D : D; E = latent ? L.rank : L.vdim;
+        D = latent ? latent_dim(L) : L.dim; KE = diff ? 2 * D : D; E = latent ? L.rank : L.vdim;
         G = L.kv_heads; per = L.heads / G; nq = diff ? 2 * per : per;
         keep = L.cache_keep; ring = L.cache_ring; pos = at;
         const AttnScratch a(L, pr.attn_chunk);
         q = act + a.q; p = act + a.p; m = act + a.m; l = act + a.l; f = act + a.f; own = act + a.own;
-        qs = D;
-        rows = nullptr;
         if ((F & kRotary) && mma_attention<T>(L)) {
             const MmaScratch b(L);
-            rows = reinterpret_cast<int*>(act + b.rows);
-            q = act + b.q; p = act + b.p; m = act + b.m; l = act + b.l; f = act + b.f; own = act + b.own;
-            qs = b.qs;
+            p = act + b.p; m = act + b.m; l = act + b.l; f = act + b.f; own = act + b.own;
         }
         kt = reinterpret_cast<T*>(act + a.tile);
         ks = key_stride<T>(KE) / (int)sizeof(T);
         vt = latent ? kt : kt + (size_t)pr.attn_chunk * ks;
         vs = latent ? ks : E;
-        t_lo = (int)((long long)keys.count * d.a1 / d.a2);
-        count = (int)((long long)keys.count * (d.a1 + 1) / d.a2) - t_lo;
-        const size_t rows0 = (size_t)pr.g.slot * (keep + ring);
-        krow = latent ? (size_t)D : (size_t)G * KE;
-        vrow = (size_t)G * E;
-        kc = static_cast<T*>(L.k_cache) + rows0 * krow + (latent ? 0 : (size_t)d.a0 * KE);
-        vc = latent ? nullptr : static_cast<T*>(L.v_cache) + rows0 * vrow + (size_t)d.a0 * E;
-    }
-    // Cache rows of the keys of a pass.
-    __device__ __forceinline__ void list_rows(int c0, int n) const {
-        for (int i = threadIdx.x; i < n; i += kConsumers) rows[i] = cache_row(keys.key(t_lo + c0 + i), keep, ring);
-    }
-    // Bring the split's rows and the position's rotations into L2 (they do not depend on this step).
-    __device__ __forceinline__ void prefetch(const MkbhLayer& L) const {
-        const int n = count - (has_own() ? 1 : 0), klines = (KE * (int)sizeof(T) + 127) / 128, vlines = latent ? 0 : (E * (int)sizeof(T) + 127) / 128;
-        list_rows(0, min(n, kMmaKeys));
-        auto line = [](const void* a) { asm volatile("prefetch.global.L2 [%0];" ::"l"(a)); };
-        for (int i = threadIdx.x; i < n * (klines + vlines); i += kConsumers) {
-            const int t = i / (klines + vlines), u = i % (klines + vlines);
-            const size_t row = cache_row(keys.key(t_lo + t), keep, ring);
-            line(u < klines ? kc + row * krow + u * (128 / sizeof(T)) : vc + row * vrow + (u - klines) * (128 / sizeof(T)));
+        per_stage = 0;
+        if ((F & kRotary) && mma_attention<T>(L)) {
+            ks = latent ? latent_row(L) : D;
+            vs = latent ? ks : E;
+            per_stage = min(kMmaKeys - 8, kStage / ((ks + (latent ? 0 : vs)) * (int)sizeof(T)));
         }
-        const int lane = threadIdx.x & 31;
-        if (threadIdx.x < 32 && lane * 32 < L.rope_dims) line(L.rope + (size_t)pos * L.rope_dims + lane * 32);
-        if (threadIdx.x < 32 && L.value_rope != nullptr && lane * 32 < L.vdim) line(L.value_rope + (size_t)pos * L.vdim + lane * 32);
+        t_lo = (int)((long long)keys.count * split / splits);
+        count = (int)((long long)keys.count * (split + 1) / splits) - t_lo;
+        const size_t rows0 = (size_t)pr.g.slot * (keep + ring);
+        // (rotary attention keeps a KV head's rows together, differential attention a position's)
+        const size_t head = diff ? kvh : ((size_t)kvh * (keep + ring));
+        krow = latent ? (size_t)latent_row(L) : diff ? (size_t)G * KE : (size_t)KE;
+        vrow = diff ? (size_t)G * E : (size_t)E;
+        kc = static_cast<T*>(L.k_cache) + (latent ? rows0 * krow : rows0 * G * KE + head * KE);
+        vc = latent ? nullptr : static_cast<T*>(L.v_cache) + rows0 * G * E + head * E;
+    }
+    // Bring the position's rotations into L2 (they do not depend on this step).
+    __device__ __forceinline__ void prefetch(const MkbhLayer& L) const {
+        auto line = [](const void* a) { asm volatile("prefetch.global.L2 [%0];" ::"l"(a)); };
+        const int i = threadIdx.x * 32;
+        if (i < L.rope_dims) line(L.rope + (size_t)pos * L.rope_dims + i);
+        if (L.value_rope != nullptr && i < L.vdim) line(L.value_rope + (size_t)pos * L.vdim + i);
     }
     __device__ __forceinline__ bool has_own() const { return count > 0 && t_lo + count == keys.count; }
     // Start copying rows [c0, c0 + nk) of the split, except this token's own: older rows do not
@@ -950,10 +892,62 @@ struct AttnView {
     }
 };
 
+// ---- loader: weights, and the key/value rows of attention on tensor cores ---------------------- //
+// A key/value stage holds rows as they lie in the cache: keys, then values (none for latents).
+template <typename T, int F>
+__device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
+    const MkbhGlobals& g = p.g;
+    const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
+    const uint64_t policy = mkb::l2_policy_evict_first();
+    const int S = p.stages;
+    uint32_t issued = 0;
+    bool ok = true;
+    for (int i = 0; i < g.queue_len && ok; ++i) {
+        const int* w = queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION;
+        Block b;
+        if (weight_block<T>(g, w, b)) {
+            const int per = kStage / b.row_bytes;
+            for (int row = b.r0; row < b.r1; row += per) {
+                const int slot = issued % S;
+                ok = bar_wait(p, c, c.empty(slot), ((issued / S) & 1u) ^ 1u, 0);
+                if (!ok) break;
+                const uint32_t bytes = (uint32_t)(min(per, b.r1 - row) * b.row_bytes);
+                mbar_expect_tx(c.full(slot), bytes);
+                mkb::tma_bulk_g2s(c.base + slot * kStage, b.w + (size_t)row * b.row_bytes, bytes, c.full(slot), policy);
+                ++issued;
+            }
+        } else if constexpr (sizeof(T) == 2 && (F & kRotary)) {
+            if (__ldg(w) == MKBH_OP_ATTENTION && mma_attention<T>(g.layers_device[__ldg(w + 1)])) {
+                const AttnView<T, F> A(p, c.pos, g.layers_device[__ldg(w + 1)], __ldg(w + 2), __ldg(w + 3), __ldg(w + 4), nullptr);
+                const int old = A.count - (A.has_own() ? 1 : 0);
+                for (int k0 = 0; k0 < old; k0 += A.per_stage) {
+                    const int slot = issued % S, n = min(A.per_stage, old - k0);
+                    ok = bar_wait(p, c, c.empty(slot), ((issued / S) & 1u) ^ 1u, 0);
+                    if (!ok) break;
+                    const uint32_t kd = c.base + slot * kStage, vd = kd + A.per_stage * A.ks * (int)sizeof(T);
+                    const uint32_t kb = A.ks * (int)sizeof(T), vb = A.latent ? 0 : A.vs * (int)sizeof(T);
+                    mbar_expect_tx(c.full(slot), n * (kb + vb));
+                    // the rows are neighbours but where the ring ends
+                    for (int t = 0; t < n;) {
+                        const int row = cache_row(A.keys.key(A.t_lo + k0 + t), A.keep, A.ring), run = min(n - t, A.keep + A.ring - row);
+                        mkb::tma_bulk_g2s(kd + t * kb, A.kc + (size_t)row * A.krow, run * kb, c.full(slot), policy);
+                        if (vb) mkb::tma_bulk_g2s(vd + t * vb, A.vc + (size_t)row * A.vrow, run * vb, c.full(slot), policy);
+                        t += run;
+                    }
+                    ++issued;
+                }
+            }
+        }
+    }
+    // no copy may be in flight when the CTA's shared memory goes away
+    for (uint32_t s = issued > (uint32_t)S ? issued - S : 0u; s < issued; ++s)
+        bar_wait(p, c, c.full(s % S), (s / S) & 1u, 0, false);
+}
+
 // What an attention instruction fetches before its producers are done.
 template <typename T, int F>
 __device__ __forceinline__ void attend_ahead(const Params& pr, int pos, const Desc& d, float* act) {
-    const AttnView<T, F> A(pr, pos, d, act);
+    const AttnView<T, F> A(pr, pos, d.L, d.a0, d.a1, d.a2, act);
     if ((F & kRotary) && mma_attention<T>(d.L)) A.prefetch(d.L);
     else A.stage(0, min(pr.attn_chunk, A.count));
 }
@@ -961,9 +955,27 @@ __device__ __forceinline__ void attend_ahead(const Params& pr, int pos, const De
 // One head's vector, by one warp: optional norm (weight w), rotation of the first `rot` elements
 // (neighbours by the angles of `rope`), factor `mul`.  All of it is read before anything is used;
 // n <= 64 J.
+struct HeadOut {  // floats at dst, or (frag) the high and low bf16 parts in fragment order of row `head`
+    float* dst;
+    uint32_t* frag;
+    int head, col0;
+    __device__ __forceinline__ void put(int i, int n, float x, float y) const {  // columns i (even), i + 1
+        if (i >= n) return;
+        if (frag == nullptr) {
+            dst[i] = x;
+            if (i + 1 < n) dst[i + 1] = y;
+            return;
+        }
+        const int col = col0 + i;  // (heads of an odd size have no fragments)
+        uint32_t* f = frag + (((col >> 5) * 2 + (col >> 2 & 1)) * 32 + (head & 7) * 4 + (col >> 3 & 3)) * 4 + (col >> 1 & 1);
+        const uint32_t hi = mkb::pack_bf16x2(x, y);
+        f[0] = hi;
+        f[2] = mkb::pack_bf16x2(x - mkb::bf16_lo(hi), y - mkb::bf16_hi(hi));
+    }
+};
 template <int J>
 __device__ __forceinline__ void head_vector(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
-                                            float mul, float* dst) {
+                                            float mul, const HeadOut& out) {
     const int lane = threadIdx.x & 31;
     float a[J], b[J], wa[J], wb[J], s = 0.f;
     float2 r[J];
@@ -987,22 +999,22 @@ __device__ __forceinline__ void head_vector(const float* src, int n, const float
     for (int j = 0; j < J; ++j) {
         const int i = 2 * (lane + 32 * j);
         const float x = a[j] * s * wa[j], y = b[j] * s * wb[j];
-        if (i < n) dst[i] = (x * r[j].x - y * r[j].y) * mul;
-        if (i + 1 < n) dst[i + 1] = (y * r[j].x + x * r[j].y) * mul;
+        out.put(i, n, (x * r[j].x - y * r[j].y) * mul, (y * r[j].x + x * r[j].y) * mul);
     }
 }
 // (by size: one call site each for up to 64, 128 and 512 elements)
 __device__ __noinline__ void head_vector_any(const float* src, int n, const float* w, float eps, const float2* rope, int rot,
-                                             float mul, float* dst) {
-    if (n <= 64) head_vector<1>(src, n, w, eps, rope, rot, mul, dst);
-    else if (n <= 128) head_vector<2>(src, n, w, eps, rope, rot, mul, dst);
-    else head_vector<8>(src, n, w, eps, rope, rot, mul, dst);
+                                             float mul, const HeadOut out) {
+    if (n <= 64) head_vector<1>(src, n, w, eps, rope, rot, mul, out);
+    else if (n <= 128) head_vector<2>(src, n, w, eps, rope, rot, mul, out);
+    else head_vector<8>(src, n, w, eps, rope, rot, mul, out);
 }
 
 // Queries of the KV head's heads, normalised, rotated and scaled, and, in the split that holds it,
 // this token's key and value.  Ends with a barrier.
+// `frag`: where the queries go as fragments (NULL: floats at A.q).
 template <typename T, int F>
-__device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView<T, F>& A, const MkbhLayer& L, int kvh) {
+__device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView<T, F>& A, const MkbhLayer& L, int kvh, uint32_t* frag) {
     const MkbhGlobals& g = pr.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tasks = A.nq + (A.has_own() ? 2 : 0);
     const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)A.pos * (L.rope_dims / 2);
@@ -1013,42 +1025,44 @@ __device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView
         const float2* angles = rope;
         int n, rot = L.rope_dims;
         float mul = 1.f;
-        float* dst = query ? A.q + t * A.qs : A.own;
+        HeadOut out{query ? A.q + t * A.D : A.own, query && frag != nullptr ? frag + (t >> 3) * ((A.D + 31) / 32) * 256 : nullptr, t, 0};
         if (A.latent) {
             const int hd = L.dim + L.rot_dim, lead = pad8(L.rank);
             const float* down = g.proj + (size_t)L.heads * hd;
             if (query) {
                 const float* absorbed = side_query(g) + (size_t)h * L.rank;
-                const float scale = L.scale;
-                mul = scale;
-                for (int i0 = 0; i0 < L.rank; i0 += 256) {
-                    float x[8];
+                mul = L.scale;
+                for (int i0 = 0; i0 < lead; i0 += 512) {
+                    float x[8], y[8];
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) x[j] = i0 + lane + 32 * j < L.rank ? ld_cg_f32(absorbed + i0 + lane + 32 * j) : 0.f;
+                    for (int j = 0; j < 8; ++j) {
+                        const int i = i0 + 2 * (lane + 32 * j);
+                        x[j] = i < L.rank ? ld_cg_f32(absorbed + i) * mul : 0.f;
+                        y[j] = i + 1 < L.rank ? ld_cg_f32(absorbed + i + 1) * mul : 0.f;
+                    }
 #pragma unroll
-                    for (int j = 0; j < 8; ++j)
-                        if (i0 + lane + 32 * j < L.rank) dst[i0 + lane + 32 * j] = x[j] * scale;
+                    for (int j = 0; j < 8; ++j) out.put(i0 + 2 * (lane + 32 * j), lead, x[j], y[j]);
                 }
             }
             if (!first) {  // rotated part
                 src = query ? g.proj + (size_t)h * hd + L.dim : down + L.rank;
                 n = L.rot_dim;
-                dst += lead;
-                for (int i = n + lane; i < (query ? A.qs : A.D) - lead; i += 32) dst[i] = 0.f;
+                if (out.frag == nullptr) out.dst += lead;
+                else out.col0 = lead;
+                for (int i = (n & ~1) + 2 * lane; i < A.D - lead; i += 64) out.put(i, A.D - lead, 0.f, 0.f);
             } else {
                 src = down;
                 n = L.rank;
                 w = L.k_norm;
                 rot = 0;
+                for (int i = L.rank + lane; i < lead; i += 32) out.dst[i] = 0.f;
             }
-            if (query || first)
-                for (int i = L.rank + lane; i < lead; i += 32) dst[i - (query ? lead : 0)] = 0.f;
+            __syncwarp();
         } else if (query) {
             src = g.proj + (size_t)h * A.D;
             n = A.D;
             w = L.q_norm;
             mul = L.scale * __ldg(L.temp + h);
-            for (int i = A.D + lane; i < A.qs; i += 32) dst[i] = 0.f;
         } else if (first) {
             src = g.proj + (size_t)(L.heads + kvh) * A.D;
             n = A.D;
@@ -1058,9 +1072,9 @@ __device__ __forceinline__ void rotary_operands(const Params& pr, const AttnView
             n = A.E;
             angles = reinterpret_cast<const float2*>(L.value_rope) + (size_t)A.pos * (A.E / 2);
             rot = L.value_rope != nullptr ? A.E : 0;
-            dst += A.D;
+            out.dst += A.D;
         }
-        head_vector_any(src, n, w, g.eps, angles, rot, mul, dst);
+        head_vector_any(src, n, w, g.eps, angles, rot, mul, out);
     }
     csync();
 }
@@ -1084,7 +1098,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T, F>& A
     if (diff)
         for (int i = tid; i < nq * D; i += kConsumers) A.q[i] = ld_cg_f32(g.proj + (size_t)kvh * nq * D + i);
     else if constexpr (F & kRotary)
-        rotary_operands<T, F>(pr, A, d.L, kvh);
+        rotary_operands<T, F>(pr, A, d.L, kvh, nullptr);
 
     for (int c0 = 0; c0 < A.count; c0 += KC) {
         const int nk = min(KC, A.count - c0);
@@ -1203,7 +1217,7 @@ __device__ __forceinline__ void attend(const Params& pr, const AttnView<T, F>& A
 
 template <typename T, int F>
 __device__ __forceinline__ void attend_fma(const Params& pr, int pos, const Desc& d, float* act) {
-    const AttnView<T, F> A(pr, pos, d, act);
+    const AttnView<T, F> A(pr, pos, d.L, d.a0, d.a1, d.a2, act);
     const int need = (A.nq + kConsumers / A.E - 1) / (kConsumers / A.E);
     if (need <= 2) attend<T, F, 2>(pr, A, d);
     else if (need <= 4) attend<T, F, 4>(pr, A, d);
@@ -1221,63 +1235,77 @@ __device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint3
     lo = mkb::pack_bf16x2(x - mkb::bf16_lo(hi), y - mkb::bf16_hi(hi));
 }
 
-// One split on mma.sync, straight from the cache rows: the M side of both products are the heads of
+// One split on mma.sync, from the ring's key/value stages: the M side of both products are the heads of
 // the group (queries and softmax weights enter as a high and a low bf16 part), the N side keys, then
 // value columns.  The index of a contraction may be permuted as long as both operands agree, so a
 // lane's share of a fragment is a run of neighbours in memory.
 template <typename T, int F>
-__device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc& d, float* act) {
+__device__ __forceinline__ bool attend_mma(const Params& pr, Cta& cta, const Desc& d, float* act, uint32_t& ring_slot, uint32_t& ring_phase) {
     const MkbhGlobals& g = pr.g;
-    const AttnView<T, F> A(pr, pos, d, act);
+    const int pos = cta.pos;
+    const AttnView<T, F> A(pr, pos, d.L, d.a0, d.a1, d.a2, act);
     const MmaScratch S(d.L);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c = lane & 3;
     const int D = A.D, E = A.E, nq = A.nq, kvh = d.a0;
     const bool own = A.has_own(), latent = A.latent;
     float *const p = A.p, *const red = act + S.red;
     const uint4* const frag = reinterpret_cast<const uint4*>(act + S.frag);
-    const float* const own_v = latent ? A.own : A.own + D;
     const int slice = warp % S.slices, group = warp / S.slices, e0 = slice * 32 + r * 4;
-    const T *const kbase = A.kc, *const vbase = latent ? A.kc : A.vc;
-    const size_t krow = A.krow, vrow = latent ? A.krow : A.vrow;
-    const int* const rows = A.rows;
+    int *const krows = reinterpret_cast<int*>(act + S.krows), *const vrows = reinterpret_cast<int*>(act + S.vrows);
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    rotary_operands<T, F>(pr, A, d.L, kvh);
-    const int blocks = S.qs / 32;
-    for (int i = tid; i < S.planes * blocks * 64; i += kConsumers) {  // queries in fragment order
-        const int l = i & 31, col = (i >> 6) % blocks * 32 + (l & 3) * 8 + (i >> 5 & 1) * 4, head = (l >> 2) + 8 * (i / (blocks * 64));
-        uint4 f = make_uint4(0, 0, 0, 0);
-        if (head < nq) {
-            const float4 x = *reinterpret_cast<const float4*>(A.q + head * S.qs + col);
-            split_bf16(x.x, x.y, f.x, f.z);
-            split_bf16(x.z, x.w, f.y, f.w);
-        }
-        reinterpret_cast<uint4*>(act + S.frag)[i] = f;
-    }
+    // (columns beyond the heads' size and rows beyond their number are zero)
+    for (int i = tid; i < S.planes * S.blocks * 64; i += kConsumers) reinterpret_cast<uint4*>(act + S.frag)[i] = make_uint4(0, 0, 0, 0);
+    csync();
+    rotary_operands<T, F>(pr, A, d.L, kvh, reinterpret_cast<uint32_t*>(act + S.frag));
+    const int blocks = S.blocks;
+    T* const own_row = reinterpret_cast<T*>(act + S.row);
     if (own) {  // this token's row
         const size_t row = cache_row(pos, A.keep, A.ring);
-        if (!latent || kvh == 0)  // (every group of heads has the same latent)
-            for (int i = tid; i < D + (latent ? 0 : E); i += kConsumers)
-                (i < D ? A.kc[row * krow + i] : A.vc[row * vrow + (i - D)]) = from_f<T>(A.own[i]);
+        for (int i = tid; i < D + (latent ? 0 : E); i += kConsumers) {
+            const T x = from_f<T>(A.own[i]);
+            own_row[i] = x;
+            if (!latent || kvh == 0)  // (every group of heads has the same latent)
+                (i < D ? A.kc[row * A.krow + i] : A.vc[row * A.vrow + (i - D)]) = x;
+        }
     }
-    csync();
-    const int old = A.count - (own ? 1 : 0);
-    for (int c0 = 0; c0 == 0 || c0 < old; c0 += kMmaKeys) {
-        const int n = min(kMmaKeys, old - c0);
-        const bool last = c0 + kMmaKeys >= old, with_own = last && own;
+    const int old = A.count - (own ? 1 : 0), per_stage = A.per_stage;
+    const int most = max(1, min(pr.stages, (kMmaKeys - 1) / per_stage)), pass = most * per_stage;  // stages, keys of a pass
+    for (int c0 = 0; c0 == 0 || c0 < old; c0 += pass) {
+        const int staged = min(pass, old - c0), stages = (staged + per_stage - 1) / per_stage;
+        const bool last = c0 + pass >= old;
+        const int n = staged + (last && own ? 1 : 0);  // this token's own key comes last
+        if (c0 > 0) csync();  // the buffers are free
+        if (tid == 0 && n > staged) {
+            krows[staged] = (int)(smem_u32(own_row) - cta.base);
+            vrows[staged] = krows[staged] + (latent ? 0 : D * (int)sizeof(T));
+        }
+        for (int i = tid; i < staged; i += kConsumers) {
+            const int st = i / per_stage, j = i - st * per_stage, at = (int)((ring_slot + st) % pr.stages) * kStage;
+            krows[i] = at + j * A.ks * (int)sizeof(T);
+            vrows[i] = latent ? krows[i] : at + (per_stage * A.ks + j * A.vs) * (int)sizeof(T);
+        }
+        bool ok = true;
+        uint32_t slot = ring_slot, phase = ring_phase;
+        for (int i = 0; i < stages && ok; ++i) {
+            ok = bar_wait(pr, cta, cta.full(slot), phase, 1);
+            if (++slot == (uint32_t)pr.stages) slot = 0, phase ^= 1u;
+        }
+        if (!__all_sync(0xffffffffu, ok)) cta.ctl[0] = 1;
+        if (!agree(cta)) return false;
         // scores: a warp takes tiles of 8 keys; lane (r, c) holds eight neighbours of key r's row per 32
         for (int t = warp; t * 8 < n; t += kConsumerWarps) {
             const bool live = t * 8 + r < n;
-            const T* k = kbase + (size_t)rows[live ? t * 8 + r : 0] * krow + c * 8;
+            const uint32_t k = cta.base + krows[live ? t * 8 + r : 0] + c * 16;
             float s[2][4] = {};
             for (int b0 = 0; b0 < blocks; b0 += 6) {
                 uint4 kv[6];
 #pragma unroll
                 for (int i = 0; i < 6; ++i)
-                    kv[i] = live && (b0 + i) * 32 + c * 8 < D ? mkb::ld_nc_v4(k + (b0 + i) * 32) : make_uint4(0, 0, 0, 0);
+                    kv[i] = live && (b0 + i) * 32 + c * 8 < D ? lds_v4(k + (b0 + i) * 64) : make_uint4(0, 0, 0, 0);
 #pragma unroll
                 for (int i = 0; i < 6; ++i) {
                     if (b0 + i >= blocks) break;
@@ -1299,19 +1327,12 @@ __device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc
                 if (head < nq) p[head * kMmaCols + key] = key < n ? s[0][j] + s[1][j] : -INFINITY;
             }
         }
-        if (with_own)
-            for (int h = kConsumerWarps - 1 - warp; h < nq; h += kConsumerWarps) {
-                float s = 0.f;
-                for (int i = lane; i < D; i += 32) s = fmaf(A.q[h * S.qs + i], to_f(from_f<T>(A.own[i])), s);
-                s = warp_sum(s);
-                if (lane == 0) p[h * kMmaCols + kMmaKeys] = s;
-            }
         csync();
         const int padded = (n + 15) & ~15;
         for (int h = warp; h < nq; h += kConsumerWarps) {
             float* row = p + h * kMmaCols;
             const float before = c0 > 0 ? A.m[h] : -INFINITY;
-            float v[kMmaKeys / 32], x = with_own ? fmaxf(before, row[kMmaKeys]) : before;
+            float v[kMmaKeys / 32], x = before;
 #pragma unroll
             for (int j = 0; j < kMmaKeys / 32; ++j) {
                 v[j] = lane + 32 * j < n ? row[lane + 32 * j] : -INFINITY;
@@ -1328,7 +1349,6 @@ __device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc
             s = warp_sum(s);
             if (lane == 0) {
                 const float fac = x == -INFINITY ? 1.f : expf(before - x);
-                if (with_own) s += row[kMmaKeys] = expf(row[kMmaKeys] - x);
                 A.l[h] = (c0 > 0 ? A.l[h] * fac : 0.f) + s;
                 A.f[h] = fac;
                 A.m[h] = x;
@@ -1356,7 +1376,7 @@ __device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc
                     for (int j = 0; j < 4; ++j) {
                         const int key = k0 + u * step + 2 * c + (j & 1) + 8 * (j >> 1);
                         v[u][j] = make_uint2(0, 0);
-                        if (key < n && e0 < E) v[u][j] = __ldg(reinterpret_cast<const uint2*>(vbase + (size_t)rows[key] * vrow + e0));
+                        if (key < n && e0 < E) v[u][j] = mkb::lds_v2(cta.base + vrows[key] + e0 * 2);
                     }
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
@@ -1381,40 +1401,31 @@ __device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc
                 }
             }
         }
-        if (!last) {
-            csync();  // the buffers of scores and rows are free
-            A.list_rows(c0 + kMmaKeys, min(kMmaKeys, old - c0 - kMmaKeys));
-            csync();
+        __syncwarp();
+        for (int i = 0; i < stages; ++i) {
+            if (lane == 0) mbar_arrive(cta.empty(ring_slot));
+            if (++ring_slot == (uint32_t)pr.stages) ring_slot = 0, ring_phase ^= 1u;
         }
     }
     // this lane's sums: heads r and r + 8, four neighbouring columns for each of two indices
     const int PE = part_row(g.part_vdim), max_splits = g.max_splits;
     float* const part = g.attn_part + ((size_t)kvh * nq * max_splits + d.a1) * PE;
-    auto out = [&](float* dst, size_t ld, bool finish) {
+    auto out = [&](float* dst, size_t ld) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int head = r + 8 * (j >> 1), e = slice * 32 + (2 * c + (j & 1)) * 4;
-            if (head >= nq || e >= E) continue;  // (E is a multiple of 8)
-            float4 y = make_float4(acc[0][j], acc[1][j], acc[2][j], acc[3][j]);
-            if (finish && own) {
-                const float w = p[head * kMmaCols + kMmaKeys];
-                const float* v = own_v + e;
-                y.x = fmaf(w, to_f(from_f<T>(v[0])), y.x);
-                y.y = fmaf(w, to_f(from_f<T>(v[1])), y.y);
-                y.z = fmaf(w, to_f(from_f<T>(v[2])), y.z);
-                y.w = fmaf(w, to_f(from_f<T>(v[3])), y.w);
-            }
-            *reinterpret_cast<float4*>(dst + head * ld + e) = y;
+            if (head < nq && e < E)  // (E is a multiple of 8)
+                *reinterpret_cast<float4*>(dst + head * ld + e) = make_float4(acc[0][j], acc[1][j], acc[2][j], acc[3][j]);
         }
     };
     if (S.groups == 1) {
-        if (group == 0) out(part + kPartLead, (size_t)max_splits * PE, true);
+        if (group == 0) out(part + kPartLead, (size_t)max_splits * PE);
     } else {
-        if (group < S.groups) out(red + group * nq * E, E, false);
+        if (group < S.groups) out(red + group * nq * E, E);
         csync();
         for (int i = tid; i < nq * E; i += kConsumers) {
             const int h = i / E, e = i - h * E;
-            float y = own ? p[h * kMmaCols + kMmaKeys] * to_f(from_f<T>(own_v[e])) : 0.f;
+            float y = 0.f;
             for (int k = 0; k < S.groups; ++k) y += red[k * nq * E + i];
             part[(size_t)h * max_splits * PE + kPartLead + e] = y;
         }
@@ -1423,28 +1434,52 @@ __device__ __forceinline__ void attend_mma(const Params& pr, int pos, const Desc
         part[(size_t)tid * max_splits * PE] = A.m[tid];
         part[(size_t)tid * max_splits * PE + 1] = A.l[tid];
     }
+    return true;
 }
 
 // Output of a latent attention's head in latent space, merged over the splits: the input of its
-// expansion.  Every warp works out the splits' factors; the partial rows are on their way meanwhile.
+// expansion.  Every warp works out the splits' factors while the partial rows are on their way; a
+// quarter of the threads takes every fourth split.
 __device__ __forceinline__ void latent_activation(const Params& pr, const MkbhLayer& L, int head, int splits, float* act) {
     const MkbhGlobals& g = pr.g;
-    const int lane = threadIdx.x & 31, PE = part_row(g.part_vdim), e = threadIdx.x;  // (rank <= 512)
+    const int lane = threadIdx.x & 31, PE = part_row(g.part_vdim), e = 4 * (threadIdx.x & 127), quarter = threadIdx.x >> 7, rank = L.rank;
     const float* row = g.attn_part + (size_t)head * g.max_splits * PE;
-    const float m = lane < splits ? ld_cg_f32(row + (size_t)lane * PE) : -INFINITY;
-    const float l = lane < splits ? ld_cg_f32(row + (size_t)lane * PE + 1) : 0.f;
-    float x[16], y = 0.f, f = 0.f;
-    for (int s0 = 0; s0 < splits; s0 += 16) {
+    float m[2], l[2], f[2];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) x[j] = e < L.rank && s0 + j < splits ? ld_cg_f32(row + (size_t)(s0 + j) * PE + kPartLead + e) : 0.f;
-        if (s0 == 0) {
-            f = expf(m - warp_max(m));
-            f /= warp_sum(l * f);
+    for (int h = 0; h < 2; ++h) {
+        const bool live = lane + 32 * h < splits;
+        m[h] = live ? ld_cg_f32(row + (size_t)(lane + 32 * h) * PE) : -INFINITY;
+        l[h] = live ? ld_cg_f32(row + (size_t)(lane + 32 * h) * PE + 1) : 0.f;
+    }
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s0 = quarter; s0 < splits; s0 += 32) {
+        uint4 x[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            x[j] = e < rank && s0 + 4 * j < splits ? mkb::ld_cg_v4(row + (size_t)(s0 + 4 * j) * PE + kPartLead + e) : make_uint4(0, 0, 0, 0);
+        if (s0 == quarter) {
+            const float top = warp_max(fmaxf(m[0], m[1]));
+            f[0] = expf(m[0] - top);
+            f[1] = expf(m[1] - top);
+            const float inv = 1.f / warp_sum(l[0] * f[0] + l[1] * f[1]);
+            f[0] *= inv;
+            f[1] *= inv;
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) y = fmaf(__shfl_sync(0xffffffffu, f, (s0 + j) & 31), x[j], y);
+        for (int j = 0; j < 8; ++j) {
+            const int s = s0 + 4 * j;  // (uniform over the warp)
+            const float w = __shfl_sync(0xffffffffu, s & 32 ? f[1] : f[0], s & 31);
+            y.x = fmaf(w, __uint_as_float(x[j].x), y.x);
+            y.y = fmaf(w, __uint_as_float(x[j].y), y.y);
+            y.z = fmaf(w, __uint_as_float(x[j].z), y.z);
+            y.w = fmaf(w, __uint_as_float(x[j].w), y.w);
+        }
     }
-    if (e < pad8(L.rank)) act[e] = e < L.rank ? y : 0.f;
+    float* red = act + 512;
+    *reinterpret_cast<float4*>(red + quarter * 512 + e) = y;
+    csync();
+    const int i = threadIdx.x;
+    if (i < pad8(rank)) act[i] = i < rank ? (red[i] + red[512 + i]) + (red[1024 + i] + red[1536 + i]) : 0.f;
 }
 
 // The split of a KV head that arrives last merges the partial rows.  Differential: combines the
@@ -1615,7 +1650,7 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             bool done = false;
             if constexpr (sizeof(T) == 2 && (F & kRotary)) {
                 done = mma_attention<T>(L);
-                if (done) attend_mma<T, F>(p, c.pos, d, act);
+                if (done && !attend_mma<T, F>(p, c, d, act, slot, phase)) return;
             }
             if (!done) attend_fma<T, F>(p, c.pos, d, act);
             csync();
@@ -1783,7 +1818,7 @@ __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_c
     const int warp = threadIdx.x >> 5;
     if (warp < kConsumerWarps) consumer_main<T, F>(p, c, sm);
     else if (warp == kOperandWarp) operand_main<T>(p, c, sm);
-    else if ((threadIdx.x & 31) == 0) loader_main<T>(p, c);
+    else if ((threadIdx.x & 31) == 0) loader_main<T, F>(p, c);
     __syncthreads();
 }
 

@@ -246,7 +246,7 @@ int mkb_hybrid_decode(const MkbhGlobals* gp, void* stream) {
     for (int i = 0; i < g.num_layers; ++i)
         if (is_attention(g.layers_host[i])) {
             const MkbhLayer& L = g.layers_host[i];
-            REQUIRE(g.attn_part && g.max_splits >= 1 && g.max_splits <= 32 &&
+            REQUIRE(g.attn_part && g.max_splits >= 1 && g.max_splits <= 64 &&
                         g.part_vdim >= (L.mixer == MKBH_LATENT_ATTENTION ? L.rank : L.vdim) && L.kv_heads <= g.max_kv_heads,
                     "attention scratch too small");
         }
@@ -271,7 +271,8 @@ int mkb_hybrid_validate(const MkbhGlobals* gp, const int32_t* ins) {
                 REQUIRE(L.mixer == MKBH_DELTA_RULE && w[2] >= 0 && w[2] < L.heads && w[3] >= 0 && w[3] < w[4] && w[4] <= L.dim,
                         "queue %d, instruction %d: head %d, columns %d..%d", q, k, w[2], w[3], w[4]);
             } else if (op == MKBH_OP_ATTENTION) {
-                REQUIRE(is_attention(L) && w[2] >= 0 && w[2] < L.kv_heads && w[3] >= 0 && w[3] < w[4] && w[4] <= g.max_splits,
+                REQUIRE(is_attention(L) && w[2] >= 0 && w[2] < L.kv_heads && w[3] >= 0 && w[3] < w[4] && w[4] <= g.max_splits &&
+                            (w[4] <= 32 || L.mixer == MKBH_LATENT_ATTENTION),
                         "queue %d, instruction %d: KV head %d, split %d of %d", q, k, w[2], w[3], w[4]);
             } else {
                 int rows, K;

@@ -63,6 +63,7 @@ template <typename T>
 struct KeySource {
     const T *keys, *shared, *values;
     int64_t key_ld, shared_ld, value_ld;  // elements between rows
+    int64_t key_head, value_head;         // elements between key/value heads
     int split, rest, per;                 // query heads per key/value head
     int keep, ring;
 };
@@ -72,12 +73,12 @@ inline KeySource<T> key_source(const MkbhGlobals& g, const MkbhLayer& L) {
     if (L.mixer == MKBH_LATENT_ATTENTION) {
         const int64_t ld = pad8(L.heads * (L.dim + L.vdim)), lr = latent_row(L);
         const T* keys = static_cast<const T*>(g.keys);
-        return {keys, static_cast<const T*>(L.k_cache) + row0 * lr + pad8(L.rank), keys + L.heads * L.dim, ld, lr, ld,
+        return {keys, static_cast<const T*>(L.k_cache) + row0 * lr + pad8(L.rank), keys + L.heads * L.dim, ld, lr, ld, L.dim, L.vdim,
                 L.dim, L.rot_dim, 1, 0, L.cache_ring};
     }
-    const int64_t kw = L.kv_heads * L.dim, vw = L.kv_heads * L.vdim;
-    return {static_cast<const T*>(L.k_cache) + row0 * kw, nullptr, static_cast<const T*>(L.v_cache) + row0 * vw, kw, 0, vw,
-            L.dim, 0, L.heads / L.kv_heads, L.cache_keep, L.cache_ring};
+    const int64_t rows = L.cache_keep + L.cache_ring;
+    return {static_cast<const T*>(L.k_cache) + row0 * L.kv_heads * L.dim, nullptr, static_cast<const T*>(L.v_cache) + row0 * L.kv_heads * L.vdim,
+            L.dim, 0, L.vdim, rows * L.dim, rows * L.vdim, L.dim, 0, L.heads / L.kv_heads, L.cache_keep, L.cache_ring};
 }
 bool rotary_flash_supported(const MkbhLayer& L);
 cudaError_t rotary_flash(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_t ldo, cudaStream_t s);

@@ -661,7 +661,7 @@ __global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const Operand
     for (int t = blockIdx.x * kOpTokens; t < t1; ++t) {
         const int pos = a.pos0 + t;
         const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)pos * (L.rope_dims / 2);
-        const size_t row = cache_row(pos, L.cache_keep, L.cache_ring);
+        const size_t row = cache_row(pos, L.cache_keep, L.cache_ring), rows = L.cache_keep + L.cache_ring;
         T* q = static_cast<T*>(a.query) + (size_t)t * a.ldq;
         if (latent) {
             const int hd = L.dim + L.rot_dim;
@@ -677,12 +677,12 @@ __global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const Operand
             operand_vector<T, J>(a, t, task * L.dim, L.dim, L.q_norm, rope, L.rope_dims, q + task * L.dim);
         } else if (task < H + G) {
             const int g = task - H;
-            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.k_norm, rope, L.rope_dims, static_cast<T*>(a.kc) + (row * G + g) * L.dim);
+            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.k_norm, rope, L.rope_dims, static_cast<T*>(a.kc) + (g * rows + row) * L.dim);
         } else {
             const int g = task - H - G;
             const float2* turn = L.value_rope ? reinterpret_cast<const float2*>(L.value_rope) + (size_t)pos * (L.vdim / 2) : nullptr;
             operand_vector<T, J>(a, t, (H + G) * L.dim + g * L.vdim, L.vdim, nullptr, turn, turn ? L.vdim : 0,
-                                 static_cast<T*>(a.vc) + (row * G + g) * L.vdim);
+                                 static_cast<T*>(a.vc) + (g * rows + row) * L.vdim);
         }
     }
 }
@@ -707,7 +707,7 @@ __global__ void __launch_bounds__(kAttnThreads) rotary_attention_kernel(const T*
         float s = -INFINITY;
         if (tid < nk) {
             const size_t row = cache_row(keys.key(c0 + tid), src.keep, src.ring);
-            const T *k = src.keys + row * src.key_ld + g * A, *r = src.shared + row * src.shared_ld;
+            const T *k = src.keys + row * src.key_ld + g * src.key_head, *r = src.shared + row * src.shared_ld;
             float d = 0.f;
             for (int i = 0; i < A; ++i) d = fmaf(q[i], to_f(k[i]), d);
             for (int i = 0; i < B; ++i) d = fmaf(q[A + i], to_f(r[i]), d);
@@ -731,7 +731,7 @@ __global__ void __launch_bounds__(kAttnThreads) rotary_attention_kernel(const T*
             if (e >= E) break;
             float y = acc[ei] * f;
             for (int j = 0; j < nk; ++j)
-                y = fmaf(p[j], to_f(src.values[(size_t)cache_row(keys.key(c0 + j), src.keep, src.ring) * src.value_ld + g * E + e]), y);
+                y = fmaf(p[j], to_f(src.values[(size_t)cache_row(keys.key(c0 + j), src.keep, src.ring) * src.value_ld + g * src.value_head + e]), y);
             acc[ei] = y;
         }
         __syncthreads();

@@ -179,7 +179,7 @@ class LatentAttentionSpec:
 
     out_features = property(lambda self: self.heads * self.vdim)
     in_rows = property(lambda self: self.heads * (self.dim + self.rot_dim) + self.rank + self.rot_dim)
-    row_elems = property(lambda self: pad8(self.rank) + pad8(self.rot_dim))  # of the cache
+    row_elems = property(lambda self: ((pad8(self.rank) + pad8(self.rot_dim)) // 8 | 1) * 8)  # of the cache
     key_elems = row_elems
 
     @property
@@ -189,8 +189,9 @@ class LatentAttentionSpec:
         return self.heads // per
 
 
-def key_splits(m, max_len: int, sm_count: int, keys_per_split: int = 64, limit: int = 32) -> int:
+def key_splits(m, max_len: int, sm_count: int, keys_per_split: int = 64) -> int:
     """Splits of the visible keys per KV head in a decode step: at most one wave of SMs."""
+    limit = 64 if m.kind == "latent_attention" else 32  # (what the kernel merges)
     most = min(m.window + m.keep_first, max_len)
     return max(1, min(-(-most // keys_per_split), sm_count // m.key_groups or 1, limit))
 

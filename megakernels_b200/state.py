@@ -98,12 +98,14 @@ class HybridState:
             elif m.kv_from is None:
                 readers = [m] + [o.mixer for o in layers if getattr(o.mixer, "kv_from", None) == i]
                 rows = self.rows[i] = plan_cache_rows(readers, max_len, portion)
-                cache = lambda *shape: torch.zeros(slots, rows.total, *shape, device=device, dtype=dtype)  # noqa: E731
                 if m.kind == "latent_attention":
-                    self.keys[i] = cache(m.row_elems)
+                    self.keys[i] = torch.zeros(slots, rows.total, m.row_elems, device=device, dtype=dtype)
+                elif m.kind == "attention":  # (a head's rows together: its splits are runs of memory)
+                    cache = lambda n: torch.zeros(slots, m.kv_heads, rows.total, n, device=device, dtype=dtype)  # noqa: E731
+                    self.keys[i], self.values[i] = cache(m.dim), cache(m.vdim)
                 else:
-                    maps = (2,) if m.kind == "diff_attention" else ()
-                    self.keys[i], self.values[i] = cache(m.kv_heads, *maps, m.dim), cache(m.kv_heads, m.vdim)
+                    cache = lambda *shape: torch.zeros(slots, rows.total, m.kv_heads, *shape, device=device, dtype=dtype)  # noqa: E731
+                    self.keys[i], self.values[i] = cache(2, m.dim), cache(m.vdim)
             if layer.canon_taps:
                 self.inputs[i], self.input_terms[i] = f32(max(layer.canon_taps - 1, 1), config.width), f32(2, config.width)
             if getattr(m, "conv_taps", 0):

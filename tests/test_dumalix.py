@@ -196,8 +196,8 @@ def test_checkpoint_reading_stacks_and_folds(tmp_path):
     assert torch.equal(p.expand_w[:, :20], torch.cat([w["l1.mix.uk"], w["l1.mix.uv"]]).float())
     # every pass has its own rows and inputs
     assert m.config.runs[2] == (0, True) and m.state.rows[2] == CacheRows(keep=0, ring=90)
-    assert m.state.keys[0].shape == (2, 90, 3, 20) and m.state.keys[0].data_ptr() != m.state.keys[2].data_ptr()
-    assert m.state.keys[1].shape == (2, 90, 32) and 1 not in m.state.values
+    assert m.state.keys[0].shape == (2, 3, 90, 20) and m.state.keys[0].data_ptr() != m.state.keys[2].data_ptr()
+    assert m.state.keys[1].shape == (2, 90, 40) and 1 not in m.state.values
     assert m.state.inputs[3].shape == (2, 2, 72) and m.state.projected[2].shape == (2, 2, 6 * 20 + 3 * 48) and 1 not in m.state.projected
     b = load_model(path, ExtraModelConfig(max_len_override=90, prefill_portion=4), device="cpu")
     assert b.state.rows[0] == CacheRows(0, 11 + 4) and b.state.rows[1] == CacheRows(0, 90) and b.dtype == torch.bfloat16

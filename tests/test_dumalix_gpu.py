@@ -114,17 +114,18 @@ def test_portions_in_bf16(bench, name, cuts):
     assert rel(run_cut(start(path, torch.bfloat16), toks, cuts), want) < BF16_TOL
 
 
+@pytest.mark.parametrize("dtype,tol", DTYPES)
 @pytest.mark.parametrize("portion", [2, 5, 16, 50])
 @pytest.mark.parametrize("name", ["odd", "even"])
-def test_small_rings_wrap(bench, name, portion):
+def test_small_rings_wrap(bench, name, portion, dtype, tol):
     """Prompts longer than the portion limit are cut inside; with it the chunks' rings shrink to
     chunk + portion rows and wrap many times."""
     raw, w, path, toks, want = bench(name)
-    gen = start(path, portion=portion)
+    gen = start(path, dtype, portion=portion)
     assert min(r.ring for r in gen.model.state.rows.values()) < 150
-    assert rel(run_cut(gen, toks, [150]), want) < F32_TOL
-    assert rel(run_cut(gen, toks, [portion, 1, portion, 1, 1, 2 * portion + 1], slot=1), want) < F32_TOL
-    assert rel(run_cut(gen, toks, [100], slot=2), want) < F32_TOL
+    assert rel(run_cut(gen, toks, [150]), want) < tol
+    assert rel(run_cut(gen, toks, [portion, 1, portion, 1, 1, 2 * portion + 1], slot=1), want) < tol
+    assert rel(run_cut(gen, toks, [100], slot=2), want) < tol
 
 
 @pytest.mark.parametrize("name", ["odd", "even", "groups"])
