@@ -83,7 +83,7 @@ constexpr int kDescBytes = (sizeof(Desc) + 127) & ~127;
 enum Bar { kDescFull = 0, kDescEmpty = 2, kVecFull = 4, kVecEmpty = 5, kRing = 6 };
 
 struct Smem {  // byte offsets from the 128-byte aligned base
-    int act, vec, rows, desc, red, stash, bars, ctl, total;
+    int act, vec, rows, desc, red, stash, layer, bars, ctl, total;
     __host__ __device__ Smem(int stages, int act_bytes, int vec_bytes) {
         act = stages * kStage;          // activations; partial sums once they are in registers
         vec = act + act_bytes;          // norm weights / decay factor
@@ -91,7 +91,8 @@ struct Smem {  // byte offsets from the 128-byte aligned base
         desc = rows + 2 * kRowVecBytes;
         red = (desc + 2 * kDescBytes + 127) & ~127;
         stash = red + 2 * 3 * kConsumerWarps * 4;
-        bars = stash + kMaxStash * 4;
+        layer = stash + kMaxStash * 4;  // the loader's copy of a layer descriptor
+        bars = layer + (int)((sizeof(MkbhLayer) + 15) & ~15);
         ctl = bars + (kRing + 2 * kMaxStages) * 8;
         total = ctl + 16 * 4;
     }
@@ -190,9 +191,7 @@ struct Block {  // rows [r0, r1) of a matrix of `row_bytes` rows
     int r0, r1, row_bytes;
 };
 template <typename T>
-__device__ __forceinline__ bool weight_block(const MkbhGlobals& g, const int* w, Block& b) {
-    const int op = __ldg(w), layer = __ldg(w + 1);
-    const MkbhLayer* L = g.layers_device + layer;
+__device__ __forceinline__ bool weight_block(const MkbhGlobals& g, int op, const MkbhLayer* L, int r0, int r1, Block& b) {
     int K;
     switch (op) {
         case MKBH_OP_NORM_PROJ: b.w = (const uint8_t*)L->in_w; K = g.width; break;
@@ -211,8 +210,8 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, const int* w,
             break;
         default: return false;
     }
-    b.r0 = __ldg(w + 2);
-    b.r1 = __ldg(w + 3);
+    b.r0 = r0;
+    b.r1 = r1;
     b.row_bytes = pad8(K) * (int)sizeof(T);
     return true;
 }
@@ -894,18 +893,33 @@ struct AttnView {
 
 // ---- loader: weights, and the key/value rows of attention on tensor cores ---------------------- //
 // A key/value stage holds rows as they lie in the cache: keys, then values (none for latents).
+// The whole warp reads an instruction and its layer's descriptor; lane 0 waits and copies.
 template <typename T, int F>
-__device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
+__device__ __forceinline__ void loader_main(const Params& p, Cta& c, const Smem& sm) {
     const MkbhGlobals& g = p.g;
     const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
     const uint64_t policy = mkb::l2_policy_evict_first();
-    const int S = p.stages;
+    const int S = p.stages, lane = threadIdx.x & 31;
+    MkbhLayer* const L = reinterpret_cast<MkbhLayer*>(c.gb + sm.layer);
     uint32_t issued = 0;
+    int held = -1;  // layer whose descriptor is there
     bool ok = true;
     for (int i = 0; i < g.queue_len && ok; ++i) {
-        const int* w = queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION;
+        const int word = lane < 5 ? __ldg(queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION + lane) : 0;
+        int w[5];
+#pragma unroll
+        for (int k = 0; k < 5; ++k) w[k] = __shfl_sync(0xffffffffu, word, k);
+        if (w[0] == MKBH_OP_NOOP) continue;
+        if (w[1] != held) {
+            __syncwarp();
+            const uint2* src = reinterpret_cast<const uint2*>(g.layers_device + w[1]);
+            for (int k = lane; k < (int)sizeof(MkbhLayer) / 8; k += 32) reinterpret_cast<uint2*>(L)[k] = __ldg(src + k);
+            held = w[1];
+            __syncwarp();
+        }
         Block b;
-        if (weight_block<T>(g, w, b)) {
+        if (lane != 0) {
+        } else if (weight_block<T>(g, w[0], L, w[2], w[3], b)) {
             const int per = kStage / b.row_bytes;
             for (int row = b.r0; row < b.r1; row += per) {
                 const int slot = issued % S;
@@ -917,8 +931,8 @@ __device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
                 ++issued;
             }
         } else if constexpr (sizeof(T) == 2 && (F & kRotary)) {
-            if (__ldg(w) == MKBH_OP_ATTENTION && mma_attention<T>(g.layers_device[__ldg(w + 1)])) {
-                const AttnView<T, F> A(p, c.pos, g.layers_device[__ldg(w + 1)], __ldg(w + 2), __ldg(w + 3), __ldg(w + 4), nullptr);
+            if (w[0] == MKBH_OP_ATTENTION && mma_attention<T>(*L)) {
+                const AttnView<T, F> A(p, c.pos, *L, w[2], w[3], w[4], nullptr);
                 const int old = A.count - (A.has_own() ? 1 : 0);
                 for (int k0 = 0; k0 < old; k0 += A.per_stage) {
                     const int slot = issued % S, n = min(A.per_stage, old - k0);
@@ -938,7 +952,9 @@ __device__ __forceinline__ void loader_main(const Params& p, Cta& c) {
                 }
             }
         }
+        ok = __shfl_sync(0xffffffffu, ok, 0);
     }
+    if (lane != 0) return;
     // no copy may be in flight when the CTA's shared memory goes away
     for (uint32_t s = issued > (uint32_t)S ? issued - S : 0u; s < issued; ++s)
         bar_wait(p, c, c.full(s % S), (s / S) & 1u, 0, false);
@@ -1818,7 +1834,7 @@ __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_c
     const int warp = threadIdx.x >> 5;
     if (warp < kConsumerWarps) consumer_main<T, F>(p, c, sm);
     else if (warp == kOperandWarp) operand_main<T>(p, c, sm);
-    else if ((threadIdx.x & 31) == 0) loader_main<T, F>(p, c);
+    else loader_main<T, F>(p, c, sm);
     __syncthreads();
 }
 

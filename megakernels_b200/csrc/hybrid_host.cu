@@ -217,9 +217,9 @@ int mkb_hybrid_prefill(const MkbhGlobals* gp, void* stream) {
         if (L.mixer == MKBH_DELTA_RULE) most(decay, L.heads * (L.dim + 2));
         most(act, out);
         if (L.enter_w) most(act, pad8(2 * g.width));
-        if (L.mixer == MKBH_ATTENTION) most(query, pad8(L.heads * L.dim));
+        if (L.mixer == MKBH_ATTENTION || L.mixer == MKBH_LATENT_ATTENTION)
+            most(query, pad8(L.heads * (g.dtype == MKBH_F32 ? query_head<float>(L) : query_head<bf16>(L))));
         if (L.mixer == MKBH_LATENT_ATTENTION) {
-            most(query, pad8(L.heads * (L.dim + L.rot_dim)));
             most(keys, pad8(L.heads * (L.dim + L.vdim)));
         }
         if (L.canon_taps) most(tail, (int64_t)L.canon_taps * g.width);

@@ -80,6 +80,18 @@ inline KeySource<T> key_source(const MkbhGlobals& g, const MkbhLayer& L) {
     return {static_cast<const T*>(L.k_cache) + row0 * L.kv_heads * L.dim, nullptr, static_cast<const T*>(L.v_cache) + row0 * L.kv_heads * L.vdim,
             L.dim, 0, L.vdim, rows * L.dim, rows * L.vdim, L.dim, 0, L.heads / L.kv_heads, L.cache_keep, L.cache_ring};
 }
+// tcgen05 (sizes it supports), mma.sync (more sizes)
+bool flash_tc_supported(const MkbhLayer& L);
+// Entries of a query head, and where its rotated part (latent) starts: the tensor-core kernel reads
+// whole slabs of 64 columns, zero beyond either part.
+template <typename T>
+inline int query_rest(const MkbhLayer& L) { return sizeof(T) == 2 && flash_tc_supported(L) ? (L.dim + 63) / 64 * 64 : L.dim; }
+template <typename T>
+inline int query_head(const MkbhLayer& L) {
+    const int rest = L.mixer == MKBH_LATENT_ATTENTION ? L.rot_dim : 0;
+    return query_rest<T>(L) + (sizeof(T) == 2 && flash_tc_supported(L) ? (rest + 63) / 64 * 64 : rest);
+}
+cudaError_t flash_tc(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_t ldo, cudaStream_t s);
 bool rotary_flash_supported(const MkbhLayer& L);
 cudaError_t rotary_flash(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_t ldo, cudaStream_t s);
 

@@ -3,6 +3,8 @@
 // Norms, scores, softmax weights, decays and the recurrent state are 32-bit in both builds.
 #include "hybrid_kernels.h"
 
+#include <type_traits>
+
 namespace mkbh {
 namespace {
 
@@ -123,6 +125,83 @@ __global__ void __launch_bounds__(kThreads) canon_norm_kernel(const float* __res
                 out[(size_t)t * ld + i] = from_f<T>(v);
                 if (out2 != nullptr) out2[(size_t)t * ld + i] = from_f<T>(y * w2[i]);
             }
+        }
+    }
+}
+
+// The same for RMS norms, up to kTaps taps and widths that are multiples of 4: a warp per token for
+// the norm, then four channels per thread, the convolution's inputs in registers.
+template <typename T> struct Quad;
+template <> struct Quad<float> { static __device__ __forceinline__ void put(float* o, float4 v) { *reinterpret_cast<float4*>(o) = v; } };
+template <> struct Quad<bf16> {
+    static __device__ __forceinline__ void put(bf16* o, float4 v) {
+        *reinterpret_cast<uint2*>(o) = make_uint2(mkb::pack_bf16x2(v.x, v.y), mkb::pack_bf16x2(v.z, v.w));
+    }
+};
+constexpr int kCanonTaps = 4;
+template <typename T, int kT>
+__global__ void __launch_bounds__(kThreads) canon_norm4_kernel(const float* __restrict__ x, int n, int pos0, int width,
+                                                               const float* __restrict__ w1, const float* __restrict__ w2, float eps,
+                                                               const float* __restrict__ taps_w, const float* __restrict__ hist,
+                                                               float* __restrict__ tail, T* __restrict__ out, T* __restrict__ out2, int64_t ld) {
+    constexpr int kBack = kT > 1 ? kT - 1 : 0, kRowsHere = kNormTokens + kBack;
+    __shared__ float inv[kRowsHere];
+    const int t0 = blockIdx.x * kNormTokens, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = warp; i < kRowsHere; i += kThreads / 32) {
+        const int t = t0 - kBack + i;
+        if (t < 0 || t >= n) continue;
+        const float4* row = reinterpret_cast<const float4*>(x + (size_t)t * width);
+        float s = 0.f;
+#pragma unroll 8
+        for (int c = lane; c < width / 4; c += 32) {
+            const float4 v = row[c];
+            s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        s = warp_sum(s);
+        if (lane == 0) inv[i] = 1.f / sqrtf(s / width + eps);
+    }
+    __syncthreads();
+    for (int c = 4 * threadIdx.x; c < width; c += 4 * kThreads) {
+        const float4 a = *reinterpret_cast<const float4*>(w1 + c);
+        const float4 b = out2 != nullptr ? *reinterpret_cast<const float4*>(w2 + c) : a;
+        float4 tap[kT > 0 ? kT : 1], v[kRowsHere], h[kT > 0 ? kT : 1];  // h[k]: k tokens ago
+#pragma unroll
+        for (int k = 0; k < kT; ++k) {
+            tap[k] = *reinterpret_cast<const float4*>(taps_w + (size_t)(kT - 1 - k) * width + c);
+            h[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < kRowsHere; ++i) {
+            const int t = t0 - kBack + i;
+            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (t >= 0 && t < n) v[i] = *reinterpret_cast<const float4*>(x + (size_t)t * width + c);
+            else if (kBack > 0 && t < 0 && pos0 + t >= 0) v[i] = *reinterpret_cast<const float4*>(hist + (size_t)((pos0 + t) % (kBack > 0 ? kBack : 1)) * width + c);
+        }
+#pragma unroll
+        for (int i = 0; i < kRowsHere; ++i) {
+            const int t = t0 - kBack + i;
+            if (t >= n) break;
+            float4 y = v[i], in = y;  // (before the portion: the input itself)
+            if (t >= 0) {
+                const float f = inv[i];
+                y = make_float4(y.x * f, y.y * f, y.z * f, y.w * f);
+                in = make_float4(y.x * a.x, y.y * a.y, y.z * a.z, y.w * a.w);
+            }
+#pragma unroll
+            for (int k = kT - 1; k > 0; --k) h[k] = h[k - 1];
+            if (kT > 0) h[0] = in;
+            if (i < kBack) continue;
+            float4 o = in;
+#pragma unroll
+            for (int k = kT - 1; k >= 0; --k) {
+                o.x = fmaf(tap[k].x, h[k].x, o.x);
+                o.y = fmaf(tap[k].y, h[k].y, o.y);
+                o.z = fmaf(tap[k].z, h[k].z, o.z);
+                o.w = fmaf(tap[k].w, h[k].w, o.w);
+            }
+            if (kBack > 0 && n - 1 - t < kBack) *reinterpret_cast<float4*>(tail + (size_t)(n - 1 - t) * width + c) = in;
+            Quad<T>::put(out + (size_t)t * ld + c, o);
+            if (out2 != nullptr) Quad<T>::put(out2 + (size_t)t * ld + c, make_float4(y.x * b.x, y.y * b.y, y.z * b.z, y.w * b.w));
         }
     }
 }
@@ -606,6 +685,7 @@ struct OperandArgs {
     const float* hist;  // of the projection's convolution, this slot
     float eps;
     void *query, *kc, *vc;  // (cache bases of the slot)
+    int qhead, qrest;       // entries of a query head, start of its rotated part
 };
 template <typename T, int J>
 __device__ __forceinline__ void operand_vector(const OperandArgs& a, int t, int col, int len, const float* w, const float2* rope,
@@ -651,39 +731,128 @@ __device__ __forceinline__ void operand_vector(const OperandArgs& a, int t, int 
         if (i + 1 < len) dst[i + 1] = from_f<T>(y);
     }
 }
-template <typename T, int J>
+// The same for a run of tokens whose vector starts at an even column, with up to kTaps taps: every row
+// is read once, as pairs; `dst` gives a token's place.  Columns len .. end of the place become zero.
+constexpr int kTaps = 4;
+template <typename T> struct Pair;
+template <> struct Pair<float> { using type = float2; static __device__ __forceinline__ float2 make(float x, float y) { return make_float2(x, y); } };
+template <> struct Pair<bf16> {
+    using type = uint32_t;
+    static __device__ __forceinline__ uint32_t make(float x, float y) { return mkb::pack_bf16x2(x, y); }
+};
+template <typename T, int J, bool kConv, typename Dst>
+__device__ __forceinline__ void operand_run(const OperandArgs& a, int t0, int t1, int col, int len, const float* w, const float* rope, int rot,
+                                            int end, Dst dst) {
+    const MkbhLayer& L = a.L;
+    const int lane = threadIdx.x & 31, taps = L.conv_taps;
+    float2 tap[kConv ? kTaps : 1][J], norm[J], u[kConv ? kTaps : 1][J];  // tap k, u[k]: k tokens ago
+#pragma unroll
+    for (int j = 0; j < J; ++j) {
+        const int i = 2 * (lane + 32 * j);
+        const bool live = i < len;
+        norm[j] = w != nullptr && live ? make_float2(w[i], w[i + 1]) : make_float2(1.f, 1.f);
+        if constexpr (kConv) {
+#pragma unroll
+            for (int k = 0; k < kTaps; ++k) {
+                const float* c = L.conv_w + (size_t)(taps - 1 - k) * L.in_rows + col + i;
+                tap[k][j] = live && k < taps ? make_float2(c[0], c[1]) : make_float2(0.f, 0.f);
+                const int t = t0 - k, pos = a.pos0 + t;  // (k = 0 is read in the loop)
+                u[k][j] = make_float2(0.f, 0.f);
+                if (!live || k == 0 || k >= taps) continue;
+                if (t >= 0) u[k][j] = *reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i);
+                else if (pos >= 0) {
+                    const float* h = a.hist + (size_t)(pos % (taps - 1)) * L.in_rows + col + i;
+                    u[k][j] = make_float2(h[0], h[1]);
+                }
+            }
+        }
+    }
+#pragma unroll 4
+    for (int t = t0; t < t1; ++t) {
+        const float2* angles = reinterpret_cast<const float2*>(rope) + (size_t)(a.pos0 + t) * (rot / 2);
+        float2 v[J], r[J];
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+            const int i = 2 * (lane + 32 * j);
+            v[j] = i < len ? *reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i) : make_float2(0.f, 0.f);
+            r[j] = i < rot ? __ldg(angles + (i >> 1)) : make_float2(1.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+            if constexpr (kConv) {
+                u[0][j] = v[j];
+                float x = u[0][j].x * tap[0][j].x, y = u[0][j].y * tap[0][j].y;
+#pragma unroll
+                for (int k = 1; k < kTaps; ++k) x = fmaf(u[k][j].x, tap[k][j].x, x), y = fmaf(u[k][j].y, tap[k][j].y, y);
+                v[j] = make_float2(x, y);
+#pragma unroll
+                for (int k = kTaps - 1; k > 0; --k) u[k][j] = u[k - 1][j];
+            }
+            s = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, s));
+        }
+        const float inv = w != nullptr ? 1.f / sqrtf(warp_sum(s) / len + a.eps) : 1.f;
+        T* o = dst(t);
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+            const int i = 2 * (lane + 32 * j);
+            const float x = v[j].x * inv * norm[j].x, y = v[j].y * inv * norm[j].y;
+            if (i < end) *reinterpret_cast<typename Pair<T>::type*>(o + i) = Pair<T>::make(x * r[j].x - y * r[j].y, y * r[j].x + x * r[j].y);
+        }
+        for (int i = 64 * J + 2 * lane; i < end; i += 64) *reinterpret_cast<typename Pair<T>::type*>(o + i) = Pair<T>::make(0.f, 0.f);
+    }
+}
+// A vector of a run of tokens, by whatever path its size allows.
+template <typename T, bool kConv, typename Dst>
+__device__ __forceinline__ void operand_tokens(const OperandArgs& a, int t0, int t1, int col, int len, const float* w, const float* rope, int rot,
+                                               int end, Dst dst) {
+    const bool pairs = (col & 1) == 0 && (len & 1) == 0 && (rot == 0 || len >= rot) && (!kConv || a.L.conv_taps <= kTaps) &&
+                       (reinterpret_cast<uint64_t>(dst(t0)) & (2 * sizeof(T) - 1)) == 0 && (reinterpret_cast<uint64_t>(dst(t0 + 1)) & (2 * sizeof(T) - 1)) == 0;
+    if (pairs && len <= 64) return operand_run<T, 1, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+    if (pairs && len <= 128) return operand_run<T, 2, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+    if (pairs && len <= 256 && !kConv) return operand_run<T, 4, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+    for (int t = t0; t < t1; ++t) {
+        const float2* angles = reinterpret_cast<const float2*>(rope) + (size_t)(a.pos0 + t) * (rot / 2);
+        if (len <= 256) operand_vector<T, 4>(a, t, col, len, w, angles, rot, dst(t));
+        else operand_vector<T, 8>(a, t, col, len, w, angles, rot, dst(t));
+        for (int i = len + (threadIdx.x & 31); i < end; i += 32) dst(t)[i] = from_f<T>(0.f);
+    }
+}
+template <typename T, bool kLatent>
 __global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const OperandArgs a) {
     const MkbhLayer& L = a.L;
     const int task = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5), H = L.heads, G = L.kv_heads;
-    const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
-    if (task >= (latent ? H + 1 : H + 2 * G)) return;
-    const int t1 = min(a.n, ((int)blockIdx.x + 1) * kOpTokens);
-    for (int t = blockIdx.x * kOpTokens; t < t1; ++t) {
-        const int pos = a.pos0 + t;
-        const float2* rope = reinterpret_cast<const float2*>(L.rope) + (size_t)pos * (L.rope_dims / 2);
-        const size_t row = cache_row(pos, L.cache_keep, L.cache_ring), rows = L.cache_keep + L.cache_ring;
-        T* q = static_cast<T*>(a.query) + (size_t)t * a.ldq;
-        if (latent) {
-            const int hd = L.dim + L.rot_dim;
-            if (task < H) {
-                operand_vector<T, J>(a, t, task * hd, L.dim, nullptr, nullptr, 0, q + task * hd);
-                operand_vector<T, J>(a, t, task * hd + L.dim, L.rot_dim, nullptr, rope, L.rope_dims, q + task * hd + L.dim);
-            } else {
-                T* kc = static_cast<T*>(a.kc) + row * latent_row(L);
-                operand_vector<T, J>(a, t, H * hd, L.rank, L.k_norm, nullptr, 0, kc);
-                operand_vector<T, J>(a, t, H * hd + L.rank, L.rot_dim, nullptr, rope, L.rope_dims, kc + pad8(L.rank));
-            }
-        } else if (task < H) {
-            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.q_norm, rope, L.rope_dims, q + task * L.dim);
-        } else if (task < H + G) {
-            const int g = task - H;
-            operand_vector<T, J>(a, t, task * L.dim, L.dim, L.k_norm, rope, L.rope_dims, static_cast<T*>(a.kc) + (g * rows + row) * L.dim);
+    if (task >= (kLatent ? H + 1 : H + 2 * G)) return;
+    const int t0 = blockIdx.x * kOpTokens, t1 = min(a.n, t0 + kOpTokens);
+    const size_t rows = L.cache_keep + L.cache_ring;
+    auto query = [&](int h, int off) { return [=](int t) { return static_cast<T*>(a.query) + (size_t)t * a.ldq + h * a.qhead + off; }; };
+    auto cache = [&](void* base, size_t first, int len, int off) {
+        return [=](int t) { return static_cast<T*>(base) + (first + cache_row(a.pos0 + t, a.L.cache_keep, a.L.cache_ring)) * len + off; };
+    };
+    if constexpr (kLatent) {
+        const int hd = L.dim + L.rot_dim, lr = latent_row(L);
+        if (task < H) {
+            operand_tokens<T, false>(a, t0, t1, task * hd, L.dim, nullptr, nullptr, 0, a.qrest, query(task, 0));
+            operand_tokens<T, false>(a, t0, t1, task * hd + L.dim, L.rot_dim, nullptr, L.rope, L.rope_dims, a.qhead - a.qrest, query(task, a.qrest));
         } else {
-            const int g = task - H - G;
-            const float2* turn = L.value_rope ? reinterpret_cast<const float2*>(L.value_rope) + (size_t)pos * (L.vdim / 2) : nullptr;
-            operand_vector<T, J>(a, t, (H + G) * L.dim + g * L.vdim, L.vdim, nullptr, turn, turn ? L.vdim : 0,
-                                 static_cast<T*>(a.vc) + (g * rows + row) * L.vdim);
+            operand_tokens<T, false>(a, t0, t1, H * hd, L.rank, L.k_norm, nullptr, 0, L.rank, cache(a.kc, 0, lr, 0));
+            operand_tokens<T, false>(a, t0, t1, H * hd + L.rank, L.rot_dim, nullptr, L.rope, L.rope_dims, L.rot_dim, cache(a.kc, 0, lr, pad8(L.rank)));
         }
+    } else {
+        auto run = [&](auto conv) {
+            constexpr bool kConv = decltype(conv)::value;
+            if (task < H) {
+                operand_tokens<T, kConv>(a, t0, t1, task * L.dim, L.dim, L.q_norm, L.rope, L.rope_dims, a.qhead, query(task, 0));
+            } else if (task < H + G) {
+                operand_tokens<T, kConv>(a, t0, t1, task * L.dim, L.dim, L.k_norm, L.rope, L.rope_dims, L.dim, cache(a.kc, (task - H) * rows, L.dim, 0));
+            } else {
+                const int g = task - H - G;
+                operand_tokens<T, kConv>(a, t0, t1, (H + G) * L.dim + g * L.vdim, L.vdim, nullptr, L.value_rope, L.value_rope ? L.vdim : 0, L.vdim,
+                                         cache(a.vc, g * rows, L.vdim, 0));
+            }
+        };
+        if (L.conv_taps > 0) run(std::true_type{});
+        else run(std::false_type{});
     }
 }
 
@@ -793,6 +962,21 @@ template <typename T>
 cudaError_t Prefill<T>::canon_norm(const MkbhGlobals& g, const MkbhLayer& L, T* out, T* out2, int64_t ld, cudaStream_t s) {
     static int set[64] = {};
     const int n = g.num_tokens, smem = max(1, L.canon_taps) * g.width * 4;
+    const float* hist = L.canon_hist + (L.canon_taps > 1 ? (size_t)g.slot * (L.canon_taps - 1) * g.width : 0);
+    if (g.norm_kind == MKBH_RMS_NORM && g.width % 4 == 0 && L.canon_taps <= kCanonTaps) {
+        auto go = [&](auto taps) {
+            canon_norm4_kernel<T, decltype(taps)::value><<<(n + kNormTokens - 1) / kNormTokens, kThreads, 0, s>>>(
+                g.x, n, g.pos0, g.width, L.norm1, L.norm2, g.eps, L.canon_w, hist, g.tail, out, out2, ld);
+        };
+        switch (L.canon_taps) {
+            case 0: go(std::integral_constant<int, 0>{}); break;
+            case 1: go(std::integral_constant<int, 1>{}); break;
+            case 2: go(std::integral_constant<int, 2>{}); break;
+            case 3: go(std::integral_constant<int, 3>{}); break;
+            default: go(std::integral_constant<int, 4>{}); break;
+        }
+        return cudaGetLastError();
+    }
     int dev = 0;
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return e;
@@ -801,7 +985,6 @@ cudaError_t Prefill<T>::canon_norm(const MkbhGlobals& g, const MkbhLayer& L, T* 
         if (e != cudaSuccess) return e;
         set[dev & 63] = smem;
     }
-    const float* hist = L.canon_hist + (L.canon_taps > 1 ? (size_t)g.slot * (L.canon_taps - 1) * g.width : 0);
     canon_norm_kernel<T><<<(n + kNormTokens - 1) / kNormTokens, kThreads, smem, s>>>(
         g.x, n, g.pos0, g.width, L.norm1, L.norm2, g.eps, g.norm_kind == MKBH_LAYER_NORM, L.canon_w, L.canon_taps, hist, g.tail, out, out2, ld);
     return cudaGetLastError();
@@ -817,23 +1000,23 @@ template <typename T>
 cudaError_t Prefill<T>::rotary_operands(const MkbhGlobals& g, const MkbhLayer& L, cudaStream_t s) {
     const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
     const int n = g.num_tokens, tasks = latent ? L.heads + 1 : L.heads + 2 * L.kv_heads;
-    const int widest = latent ? max(max(L.dim, L.rot_dim), L.rank) : max(L.dim, L.vdim);
     const size_t rows = (size_t)g.slot * (L.cache_keep + L.cache_ring);
-    OperandArgs a{g.proj, pad8(L.in_rows), latent ? (int64_t)pad8(L.heads * (L.dim + L.rot_dim)) : (int64_t)pad8(L.heads * L.dim), n, g.pos0, L,
+    OperandArgs a{g.proj, pad8(L.in_rows), pad8(L.heads * query_head<T>(L)), n, g.pos0, L,
                   L.conv_hist + (L.conv_taps > 1 ? (size_t)g.slot * (L.conv_taps - 1) * L.in_rows : 0), g.eps, g.query,
                   static_cast<T*>(L.k_cache) + rows * (latent ? latent_row(L) : L.kv_heads * L.dim),
-                  latent ? nullptr : static_cast<T*>(L.v_cache) + rows * L.kv_heads * L.vdim};
+                  latent ? nullptr : static_cast<T*>(L.v_cache) + rows * L.kv_heads * L.vdim, query_head<T>(L), query_rest<T>(L)};
     const dim3 grid((n + kOpTokens - 1) / kOpTokens, (tasks + kThreads / 32 - 1) / (kThreads / 32));
-    if (widest <= 64) rotary_operands_kernel<T, 1><<<grid, kThreads, 0, s>>>(a);
-    else if (widest <= 128) rotary_operands_kernel<T, 2><<<grid, kThreads, 0, s>>>(a);
-    else if (widest <= 256) rotary_operands_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
-    else rotary_operands_kernel<T, 8><<<grid, kThreads, 0, s>>>(a);
+    if (latent) rotary_operands_kernel<T, true><<<grid, kThreads, 0, s>>>(a);
+    else rotary_operands_kernel<T, false><<<grid, kThreads, 0, s>>>(a);
     return cudaGetLastError();
 }
 template <typename T>
 cudaError_t Prefill<T>::rotary_attention(const MkbhGlobals& g, const MkbhLayer& L, T* out, int64_t ldo, cudaStream_t s) {
     if constexpr (sizeof(T) == 2)
+    {
+        if (flash_tc_supported(L)) return flash_tc(g, L, out, ldo, s);
         if (rotary_flash_supported(L)) return rotary_flash(g, L, out, ldo, s);
+    }
     const KeySource<T> src = key_source<T>(g, L);
     const int q = src.split + src.rest;
     rotary_attention_kernel<T><<<dim3(g.num_tokens, L.heads), kAttnThreads, (q + kAttnThreads + L.vdim) * 4, s>>>(

@@ -1,0 +1,128 @@
+// PTX wrappers of the 5th-generation tensor cores and of tiled TMA loads: bf16 operands, fp32
+// accumulators in tensor memory, 128-byte swizzled operand tiles.
+#pragma once
+
+#include <cuda.h>
+
+#include "hybrid_common.cuh"
+
+namespace mkbh {
+namespace {
+
+// Bounded wait; on expiry records the fault, marks the CTA as dead and returns false.
+__device__ __noinline__ bool tc_wait_slow(uint32_t bar, uint32_t parity, volatile int* dead, unsigned long long timeout_ns, int* status,
+                                          int role) {
+    const unsigned long long t0 = mkb::globaltimer_ns();
+    for (uint32_t spins = 1;; ++spins) {
+        if (mkb::mbar_try_wait(bar, parity)) return true;
+        if ((spins & 63u) == 0) {
+            if (dead != nullptr && *dead) return false;
+            if (mkb::globaltimer_ns() - t0 > timeout_ns) {
+                if (status != nullptr && atomicCAS(&status[0], 0, (int)MKBH_ERR_DEVICE_TIMEOUT) == 0) {
+                    status[1] = blockIdx.x;
+                    status[2] = -1;
+                    status[3] = -1;
+                    status[4] = role;
+                }
+                if (dead != nullptr) *dead = 1;
+                return false;
+            }
+        }
+    }
+}
+__device__ __forceinline__ bool tc_wait(uint32_t bar, uint32_t parity, volatile int* dead, unsigned long long timeout_ns, int* status, int role) {
+    return mkb::mbar_try_wait(bar, parity) || tc_wait_slow(bar, parity, dead, timeout_ns, status, role);
+}
+
+__device__ __forceinline__ void tc_tma_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
+            dst),
+        "l"(map), "r"(x), "r"(y), "r"(bar)
+        : "memory");
+}
+// K-major operand tile with the 128-byte swizzle: rows 128 bytes apart, groups of 8 rows 1024 bytes apart
+__device__ __forceinline__ uint64_t tc_desc(uint32_t addr) {
+    return (uint64_t)((addr & 0x3FFFFu) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) |
+           ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
+}
+// MN-major: a row holds 64 columns of one k, groups of 8 k are 1024 bytes apart, 64-column slabs `slab` bytes
+__device__ __forceinline__ uint64_t tc_desc_mn(uint32_t addr, uint32_t slab) {
+    return (uint64_t)((addr & 0x3FFFFu) >> 4) | ((uint64_t)(slab >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) |
+           ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
+}
+// bf16 x bf16 -> fp32, M x N; bit 16: B is MN-major
+__device__ __forceinline__ uint32_t tc_idesc(int m, int n, bool b_mn = false) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? 1u << 16 : 0u) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
+}
+__device__ __forceinline__ void tc_mma(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\tsetp.ne.u32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d),
+        "l"(a), "l"(b), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+// A from tensor memory
+__device__ __forceinline__ void tc_mma_ts(uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\tsetp.ne.u32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d),
+        "r"(a), "l"(b), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+__device__ __forceinline__ void tc_commit(uint32_t bar) {
+    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+__device__ __forceinline__ void tc_before_sync() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void tc_after_sync() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
+// 32 columns of the warp's 32 lanes (complete after tc_loaded)
+__device__ __forceinline__ void tc_load32_async(uint32_t addr, uint32_t* r) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,"
+        "%30,%31}, [%32];"
+        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+          "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
+          "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
+          "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+        : "r"(addr));
+}
+__device__ __forceinline__ void tc_loaded() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void tc_load32(uint32_t addr, uint32_t (&r)[32]) {
+    tc_load32_async(addr, r);
+    tc_loaded();
+}
+__device__ __forceinline__ void tc_store16(uint32_t addr, const uint32_t* r) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(addr),
+                 "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
+                 "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+                 : "memory");
+}
+__device__ __forceinline__ void tc_stored() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                             const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                             CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// Map of a row-major bf16 matrix; what lies outside it reads as zero.
+inline cudaError_t tc_map(CUtensorMap* map, const bf16* ptr, int cols, int rows, int64_t ld, int box_cols, int box_rows) {
+    static EncodeFn encode = nullptr;
+    if (encode == nullptr) {
+        void* fn = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q);
+        if (e != cudaSuccess) return e;
+        if (q != cudaDriverEntryPointSuccess || fn == nullptr) return cudaErrorNotSupported;
+        encode = reinterpret_cast<EncodeFn>(fn);
+    }
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows}, elem[2] = {1, 1};
+    const CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(ptr), dims, strides, box, elem,
+                              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? cudaSuccess : cudaErrorInvalidValue;
+}
+
+}  // namespace
+}  // namespace mkbh

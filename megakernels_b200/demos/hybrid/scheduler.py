@@ -82,6 +82,7 @@ def make_globals(model, options: HybridScheduleOptions) -> HybridGlobals:
     poly = [s.mlp.ff for s in layers if s.mlp is not None and s.mlp.kind == "poly_norm"]
     glu = [s.mlp.ff for s in layers if s.mlp is not None and s.mlp.kind == "clamped_glu"]
     widest = lambda sizes: max([pad8(x) for x in sizes], default=0)  # noqa: E731
+    pad64 = lambda x: -(-x // 64) * 64  # noqa: E731  (whole tensor-core slabs per query head)
     mixed = widest(s.mixer.out_features for s in layers)
     act = max(widest([cfg.width * (2 if cfg.loop else 1)]), mixed, widest(poly))
     from megakernels_b200.utils import get_sm_count
@@ -105,7 +106,7 @@ def make_globals(model, options: HybridScheduleOptions) -> HybridGlobals:
         counters=i32((2 + (R + 1) * COUNTERS_PER_LAYER + R * groups + 1) // 2 * 2),
         arrivals=i32(R + 1, COUNTERS_PER_LAYER), attn_part=f32(heads, 2, splits, 4 + -(-vdim // 4) * 4), status=i32(16),
         max_splits=splits, max_kv_heads=groups, part_vdim=vdim,
-        query=own(n, max(widest(m.heads * (m.dim + m.rot_dim) for m in latent), widest(m.heads * m.dim for m in rotary), 1)),
+        query=own(n, max([m.heads * (pad64(m.dim) + pad64(m.rot_dim)) for m in latent] + [m.heads * pad64(m.dim) for m in rotary] + [1])),
         act2=own(n, widest([cfg.width])), ffn=own(n, max(side_ff, 1)),
         keys=own(model.max_len(), widest(m.heads * (m.dim + m.vdim) for m in latent)) if latent else own(1),
         tail=f32(max([s.canon_taps for s in layers] + [1]), cfg.width), side=f32(side_ff + pad8(cfg.width) + side_rank),
