@@ -53,8 +53,9 @@ LIBRARIES = {
     ),
     "hybrid": Library(
         "libmkb200_hybrid.so",
-        ("hybrid_decode.cu", "hybrid_prefill.cu", "hybrid_attention.cu", "hybrid_flash.cu", "hybrid_gemm_bf16.cu", "hybrid_gemm_f32.cu", "hybrid_host.cu"),
-        ("hybrid_common.cuh", "hybrid_kernels.h", "hybrid_tcgen05.cuh", "mk_common.cuh", "../../include/mkb200.h",
+        ("hybrid_decode.cu", "hybrid_decode_rotary.cu", "hybrid_decode_mixed.cu", "hybrid_prefill.cu",
+         "hybrid_attention.cu", "hybrid_flash.cu", "hybrid_gemm_bf16.cu", "hybrid_gemm_f32.cu", "hybrid_host.cu"),
+        ("hybrid_common.cuh", "hybrid_kernels.h", "hybrid_decode.cu", "hybrid_tcgen05.cuh", "mk_common.cuh", "../../include/mkb200.h",
          "../../include/mkb200_hybrid.h"),
     ),
 }

@@ -17,9 +17,14 @@
 //   * what else does not depend on the token (recurrent state, older keys and values) is fetched
 //     before an instruction waits for its producers;
 //   * every wait is bounded and reports into the status record.
+//
+// Compiled once per set of mechanisms (MKBH_FEATURES, see Features): hybrid_decode_rotary.cu and
+// hybrid_decode_mixed.cu include this file.
 #include "hybrid_kernels.h"
 
-#include <cstring>
+#ifndef MKBH_FEATURES
+#define MKBH_FEATURES 1
+#endif
 
 namespace mkbh {
 namespace {
@@ -1900,6 +1905,12 @@ cudaError_t launch(const MkbhGlobals& g, cudaStream_t s) {
 
 }  // namespace
 
+template <>
+cudaError_t decode_build<MKBH_FEATURES>(const MkbhGlobals& g, cudaStream_t s) {
+    return g.dtype == MKBH_F32 ? launch<float, MKBH_FEATURES>(g, s) : launch<bf16, MKBH_FEATURES>(g, s);
+}
+
+#if MKBH_FEATURES == 1
 cudaError_t decode_launch(const MkbhGlobals& g, cudaStream_t s) {
     int features = g.norm_kind == MKBH_LAYER_NORM ? kClassic : kRotary;
     for (int i = 0; i < g.num_layers; ++i) {
@@ -1908,10 +1919,8 @@ cudaError_t decode_launch(const MkbhGlobals& g, cudaStream_t s) {
         if (L.ff) features |= L.ff_kind == MKBH_POLY_NORM ? kClassic : kRotary;
         if (L.parallel || L.canon_taps || L.conv_taps || L.enter_w) features |= kRotary;
     }
-    const bool f32 = g.dtype == MKBH_F32;
-    if (features == kClassic) return f32 ? launch<float, kClassic>(g, s) : launch<bf16, kClassic>(g, s);
-    if (features == kRotary) return f32 ? launch<float, kRotary>(g, s) : launch<bf16, kRotary>(g, s);
-    return f32 ? launch<float, kClassic | kRotary>(g, s) : launch<bf16, kClassic | kRotary>(g, s);
+    return features == kClassic ? decode_build<kClassic>(g, s) : features == kRotary ? decode_build<kRotary>(g, s) : decode_build<kClassic | kRotary>(g, s);
 }
+#endif
 
 }  // namespace mkbh

@@ -95,7 +95,12 @@ cudaError_t flash_tc(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_
 bool rotary_flash_supported(const MkbhLayer& L);
 cudaError_t rotary_flash(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_t ldo, cudaStream_t s);
 
-// decode: one persistent kernel
+// decode: one persistent kernel, built per set of mechanisms
+template <int kFeatures>
+cudaError_t decode_build(const MkbhGlobals& g, cudaStream_t s);
+template <> cudaError_t decode_build<1>(const MkbhGlobals& g, cudaStream_t s);
+template <> cudaError_t decode_build<2>(const MkbhGlobals& g, cudaStream_t s);
+template <> cudaError_t decode_build<3>(const MkbhGlobals& g, cudaStream_t s);
 cudaError_t decode_launch(const MkbhGlobals& g, cudaStream_t s);
 
 }  // namespace mkbh

@@ -759,7 +759,7 @@ __device__ __forceinline__ void operand_run(const OperandArgs& a, int t0, int t1
                 const int t = t0 - k, pos = a.pos0 + t;  // (k = 0 is read in the loop)
                 u[k][j] = make_float2(0.f, 0.f);
                 if (!live || k == 0 || k >= taps) continue;
-                if (t >= 0) u[k][j] = *reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i);
+                if (t >= 0) u[k][j] = __ldg(reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i));
                 else if (pos >= 0) {
                     const float* h = a.hist + (size_t)(pos % (taps - 1)) * L.in_rows + col + i;
                     u[k][j] = make_float2(h[0], h[1]);
@@ -775,7 +775,7 @@ __device__ __forceinline__ void operand_run(const OperandArgs& a, int t0, int t1
 #pragma unroll
         for (int j = 0; j < J; ++j) {
             const int i = 2 * (lane + 32 * j);
-            v[j] = i < len ? *reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i) : make_float2(0.f, 0.f);
+            v[j] = i < len ? __ldg(reinterpret_cast<const float2*>(a.proj + (size_t)t * a.ld + col + i)) : make_float2(0.f, 0.f);
             r[j] = i < rot ? __ldg(angles + (i >> 1)) : make_float2(1.f, 0.f);
         }
 #pragma unroll
@@ -810,7 +810,10 @@ __device__ __forceinline__ void operand_tokens(const OperandArgs& a, int t0, int
                        (reinterpret_cast<uint64_t>(dst(t0)) & (2 * sizeof(T) - 1)) == 0 && (reinterpret_cast<uint64_t>(dst(t0 + 1)) & (2 * sizeof(T) - 1)) == 0;
     if (pairs && len <= 64) return operand_run<T, 1, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
     if (pairs && len <= 128) return operand_run<T, 2, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
-    if (pairs && len <= 256 && !kConv) return operand_run<T, 4, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+    if constexpr (!kConv) {
+        if (pairs && len <= 256) return operand_run<T, 4, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+        if (pairs) return operand_run<T, 8, kConv>(a, t0, t1, col, len, w, rope, rot, end, dst);
+    }
     for (int t = t0; t < t1; ++t) {
         const float2* angles = reinterpret_cast<const float2*>(rope) + (size_t)(a.pos0 + t) * (rot / 2);
         if (len <= 256) operand_vector<T, 4>(a, t, col, len, w, angles, rot, dst(t));
@@ -822,7 +825,7 @@ template <typename T, bool kLatent>
 __global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const OperandArgs a) {
     const MkbhLayer& L = a.L;
     const int task = blockIdx.y * (kThreads / 32) + (threadIdx.x >> 5), H = L.heads, G = L.kv_heads;
-    if (task >= (kLatent ? H + 1 : H + 2 * G)) return;
+    if (task >= (kLatent ? H + 2 : H + 2 * G)) return;
     const int t0 = blockIdx.x * kOpTokens, t1 = min(a.n, t0 + kOpTokens);
     const size_t rows = L.cache_keep + L.cache_ring;
     auto query = [&](int h, int off) { return [=](int t) { return static_cast<T*>(a.query) + (size_t)t * a.ldq + h * a.qhead + off; }; };
@@ -834,8 +837,9 @@ __global__ void __launch_bounds__(kThreads) rotary_operands_kernel(const Operand
         if (task < H) {
             operand_tokens<T, false>(a, t0, t1, task * hd, L.dim, nullptr, nullptr, 0, a.qrest, query(task, 0));
             operand_tokens<T, false>(a, t0, t1, task * hd + L.dim, L.rot_dim, nullptr, L.rope, L.rope_dims, a.qhead - a.qrest, query(task, a.qrest));
-        } else {
+        } else if (task == H) {
             operand_tokens<T, false>(a, t0, t1, H * hd, L.rank, L.k_norm, nullptr, 0, L.rank, cache(a.kc, 0, lr, 0));
+        } else {
             operand_tokens<T, false>(a, t0, t1, H * hd + L.rank, L.rot_dim, nullptr, L.rope, L.rope_dims, L.rot_dim, cache(a.kc, 0, lr, pad8(L.rank)));
         }
     } else {
@@ -999,7 +1003,7 @@ cudaError_t Prefill<T>::keep_inputs(const MkbhGlobals& g, const MkbhLayer& L, cu
 template <typename T>
 cudaError_t Prefill<T>::rotary_operands(const MkbhGlobals& g, const MkbhLayer& L, cudaStream_t s) {
     const bool latent = L.mixer == MKBH_LATENT_ATTENTION;
-    const int n = g.num_tokens, tasks = latent ? L.heads + 1 : L.heads + 2 * L.kv_heads;
+    const int n = g.num_tokens, tasks = latent ? L.heads + 2 : L.heads + 2 * L.kv_heads;
     const size_t rows = (size_t)g.slot * (L.cache_keep + L.cache_ring);
     OperandArgs a{g.proj, pad8(L.in_rows), pad8(L.heads * query_head<T>(L)), n, g.pos0, L,
                   L.conv_hist + (L.conv_taps > 1 ? (size_t)g.slot * (L.conv_taps - 1) * L.in_rows : 0), g.eps, g.query,
