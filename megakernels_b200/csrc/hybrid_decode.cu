@@ -43,7 +43,12 @@ using mkb::smem_u32;
 constexpr int kConsumerWarps = 16;
 constexpr int kConsumers = kConsumerWarps * 32;
 constexpr int kOperandWarp = kConsumerWarps + 1;  // (warp 16 is the loader)
-constexpr int kBlock = kConsumers + 64;
+// The release of a counter waits until the CTA's stores are visible to the GPU.  Where an instruction's
+// successor in the queue is often independent of it (feed-forwards beside mixers), a warp of its own
+// does that, so that the consumers go on.
+constexpr bool kSignalWarp = (MKBH_FEATURES & 2) != 0;
+constexpr int kSignals = 4;  // signals in flight
+constexpr int kBlock = kConsumers + (kSignalWarp ? 96 : 64);
 constexpr int kStage = 32768;
 static_assert(kStage >= kMaxRowBytes, "a stage holds whole rows");
 constexpr int kMaxStages = 6;
@@ -85,7 +90,7 @@ struct Desc {
 static_assert(sizeof(MkbhLayer) % 8 == 0, "");
 constexpr int kDescBytes = (sizeof(Desc) + 127) & ~127;
 
-enum Bar { kDescFull = 0, kDescEmpty = 2, kVecFull = 4, kVecEmpty = 5, kRing = 6 };
+enum Bar { kDescFull = 0, kDescEmpty = 2, kVecFull = 4, kVecEmpty = 5, kSigFull = 6, kSigEmpty = kSigFull + kSignals, kRing = kSigEmpty + kSignals };
 
 struct Smem {  // byte offsets from the 128-byte aligned base
     int act, vec, rows, desc, red, stash, layer, bars, ctl, total;
@@ -99,7 +104,7 @@ struct Smem {  // byte offsets from the 128-byte aligned base
         layer = stash + kMaxStash * 4;  // the loader's copy of a layer descriptor
         bars = layer + (int)((sizeof(MkbhLayer) + 15) & ~15);
         ctl = bars + (kRing + 2 * kMaxStages) * 8;
-        total = ctl + 16 * 4;
+        total = ctl + 16 * 4;  // (words 8.. are the signals' counters)
     }
 };
 
@@ -107,7 +112,7 @@ struct Cta {  // small and passed by reference to inlined code only: stays in re
     uint32_t base, bars;
     uint8_t* gb;
     volatile int* ctl;  // [0] CTA abort, [1] last-arriver verdict, [2], [3] agreed abort
-    int instr, opcode, pos, turn;
+    int instr, opcode, pos, turn, signals;
     __device__ __forceinline__ uint32_t bar(int i) const { return bars + i * 8; }
     __device__ __forceinline__ uint32_t full(int s) const { return bars + (kRing + s) * 8; }
     __device__ __forceinline__ uint32_t empty(int s) const { return bars + (kRing + kMaxStages + s) * 8; }
@@ -182,6 +187,31 @@ __device__ __noinline__ void poll_counter(const int* addr, int thr, volatile int
     }
 }
 
+// Consumer thread 0, behind a consumer barrier: count an instruction's end into a phase counter
+// (-1: no more of them).
+__device__ __forceinline__ void post_signal(const Params& p, Cta& c, int* counters, int idx) {
+    if constexpr (kSignalWarp) {
+        const int slot = c.signals % kSignals;
+        bar_wait(p, c, c.bar(kSigEmpty + slot), ((c.signals / kSignals) & 1u) ^ 1u, 1);
+        c.ctl[8 + slot] = idx;
+        mbar_arrive(c.bar(kSigFull + slot));
+        ++c.signals;
+    } else if (idx >= 0) {
+        red_release_gpu_add(counters + idx, 1);
+    }
+}
+__device__ __forceinline__ void signal_main(const Params& p, Cta& c) {
+    int* counters = p.g.counters + 2;
+    for (;; ++c.signals) {
+        const int slot = c.signals % kSignals;
+        if (!bar_wait(p, c, c.bar(kSigFull + slot), (c.signals / kSignals) & 1u, 3)) return;
+        const int idx = c.ctl[8 + slot];
+        if (idx < 0) return;
+        red_release_gpu_add(counters + idx, 1);
+        mbar_arrive(c.bar(kSigEmpty + slot));
+    }
+}
+
 __device__ __forceinline__ int phase_index(int layer, int op) { return layer * MKBH_BARRIERS_PER_LAYER + op; }
 
 // Float buffers beside the stacked projection: feed-forward input and output of parallel layers,
@@ -207,12 +237,14 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, int op, const
         case MKBH_OP_NORM_UP: b.w = (const uint8_t*)L->up_w; K = g.width; break;
         case MKBH_OP_DOWN: b.w = (const uint8_t*)L->down_w; K = L->ff; break;
         case MKBH_OP_HEAD: b.w = (const uint8_t*)g.head; K = g.width; break;
+#if MKBH_FEATURES & 2
         case MKBH_OP_ENTER: b.w = (const uint8_t*)L->enter_w; K = 2 * g.width; break;
         case MKBH_OP_ABSORB: b.w = (const uint8_t*)L->absorb_w; K = L->dim; break;
         case MKBH_OP_EXPAND:  // (behind the keys' rows)
             K = L->rank;
             b.w = (const uint8_t*)L->expand_w + (size_t)L->heads * L->dim * pad8(K) * sizeof(T);
             break;
+#endif
         default: return false;
     }
     b.r0 = r0;
@@ -220,6 +252,36 @@ __device__ __forceinline__ bool weight_block(const MkbhGlobals& g, int op, const
     b.row_bytes = pad8(K) * (int)sizeof(T);
     return true;
 }
+
+template <typename T>
+struct Cursor {  // the queue's weight blocks as a flat sequence of stages
+    int i = 0, row = 0, per = 1;
+    bool open = false;
+    Block b;
+    __device__ bool next(const MkbhGlobals& g, const int* queue, const uint8_t*& src, uint32_t& bytes) {
+        while (!open) {
+            if (i >= g.queue_len) return false;
+            const int* w = queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION;
+            const int op = __ldg(w), layer = __ldg(w + 1);
+            if (weight_block<T>(g, op, g.layers_device + layer, __ldg(w + 2), __ldg(w + 3), b) && b.r1 > b.r0) {
+                open = true;
+                row = b.r0;
+                per = kStage / b.row_bytes;
+            } else {
+                ++i;
+            }
+        }
+        const int n = min(per, b.r1 - row);
+        src = b.w + (size_t)row * b.row_bytes;
+        bytes = (uint32_t)(n * b.row_bytes);
+        row += n;
+        if (row >= b.r1) {
+            open = false;
+            ++i;
+        }
+        return true;
+    }
+};
 
 // ---- operand warp ------------------------------------------------------------------------- //
 // Column groups of an input of `chunks` 16-byte chunks: warps that share a row.
@@ -822,7 +884,7 @@ struct MmaScratch {
 template <typename T, int F>
 struct AttnView {
     int D, KE, E, G, per, nq, ks, vs, per_stage, t_lo, count, keep, ring, pos;
-    size_t krow, vrow;  // elements between positions
+    int krow, vrow;  // elements between positions
     KeyRange keys;
     T *kc, *vc, *kt, *vt;
     float *q, *p, *m, *l, *f, *own;
@@ -855,8 +917,8 @@ struct AttnView {
         const size_t rows0 = (size_t)pr.g.slot * (keep + ring);
         // (rotary attention keeps a KV head's rows together, differential attention a position's)
         const size_t head = diff ? kvh : ((size_t)kvh * (keep + ring));
-        krow = latent ? (size_t)latent_row(L) : diff ? (size_t)G * KE : (size_t)KE;
-        vrow = diff ? (size_t)G * E : (size_t)E;
+        krow = latent ? latent_row(L) : diff ? G * KE : KE;
+        vrow = diff ? G * E : E;
         kc = static_cast<T*>(L.k_cache) + (latent ? rows0 * krow : rows0 * G * KE + head * KE);
         vc = latent ? nullptr : static_cast<T*>(L.v_cache) + rows0 * G * E + head * E;
     }
@@ -898,7 +960,31 @@ struct AttnView {
 
 // ---- loader: weights, and the key/value rows of attention on tensor cores ---------------------- //
 // A key/value stage holds rows as they lie in the cache: keys, then values (none for latents).
-// The whole warp reads an instruction and its layer's descriptor; lane 0 waits and copies.
+// Weights only, by one thread: a flat sequence of stages.
+template <typename T>
+__device__ __forceinline__ void weight_loader(const Params& p, Cta& c) {
+    const MkbhGlobals& g = p.g;
+    const int* queue = g.instructions + (size_t)blockIdx.x * g.queue_len * MKBH_INTS_PER_INSTRUCTION;
+    const uint64_t policy = mkb::l2_policy_evict_first();
+    Cursor<T> cur;
+    uint32_t issued = 0;
+    const uint8_t* src;
+    uint32_t bytes;
+    const int S = p.stages;
+    while (cur.next(g, queue, src, bytes)) {
+        const int slot = issued % S;
+        if (!bar_wait(p, c, c.empty(slot), ((issued / S) & 1u) ^ 1u, 0)) break;
+        mbar_expect_tx(c.full(slot), bytes);
+        mkb::tma_bulk_g2s(c.base + slot * kStage, src, bytes, c.full(slot), policy);
+        ++issued;
+    }
+    // no copy may be in flight when the CTA's shared memory goes away
+    for (uint32_t s = issued > (uint32_t)S ? issued - S : 0u; s < issued; ++s)
+        bar_wait(p, c, c.full(s % S), (s / S) & 1u, 0, false);
+}
+
+// The whole warp reads instructions (two ahead) and their layers' descriptors (one ahead), so that no
+// chain of loads stands between one instruction's copies and the next one's; lane 0 waits and copies.
 template <typename T, int F>
 __device__ __forceinline__ void loader_main(const Params& p, Cta& c, const Smem& sm) {
     const MkbhGlobals& g = p.g;
@@ -906,24 +992,38 @@ __device__ __forceinline__ void loader_main(const Params& p, Cta& c, const Smem&
     const uint64_t policy = mkb::l2_policy_evict_first();
     const int S = p.stages, lane = threadIdx.x & 31;
     MkbhLayer* const L = reinterpret_cast<MkbhLayer*>(c.gb + sm.layer);
+    constexpr int kWords = (int)sizeof(MkbhLayer) / 8, kPer = (kWords + 31) / 32;
+    auto words = [&](int i) { return lane < 5 && i < g.queue_len ? __ldg(queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION + lane) : 0; };
+    uint2 next[kPer];
+    auto fetch = [&](int layer) {
+        const uint2* src = reinterpret_cast<const uint2*>(g.layers_device + layer);
+#pragma unroll
+        for (int k = 0; k < kPer; ++k)
+            if (lane + 32 * k < kWords) next[k] = __ldg(src + lane + 32 * k);
+    };
+    auto keep = [&] {
+        __syncwarp();
+#pragma unroll
+        for (int k = 0; k < kPer; ++k)
+            if (lane + 32 * k < kWords) reinterpret_cast<uint2*>(L)[lane + 32 * k] = next[k];
+        __syncwarp();
+    };
     uint32_t issued = 0;
-    int held = -1;  // layer whose descriptor is there
+    int word = words(0), ahead = words(1);
+    int held = __shfl_sync(0xffffffffu, word, 1);  // layer whose descriptor is there
+    fetch(held);
+    keep();
     bool ok = true;
     for (int i = 0; i < g.queue_len && ok; ++i) {
-        const int word = lane < 5 ? __ldg(queue + (size_t)i * MKBH_INTS_PER_INSTRUCTION + lane) : 0;
         int w[5];
 #pragma unroll
         for (int k = 0; k < 5; ++k) w[k] = __shfl_sync(0xffffffffu, word, k);
-        if (w[0] == MKBH_OP_NOOP) continue;
-        if (w[1] != held) {
-            __syncwarp();
-            const uint2* src = reinterpret_cast<const uint2*>(g.layers_device + w[1]);
-            for (int k = lane; k < (int)sizeof(MkbhLayer) / 8; k += 32) reinterpret_cast<uint2*>(L)[k] = __ldg(src + k);
-            held = w[1];
-            __syncwarp();
-        }
+        const int layer = __shfl_sync(0xffffffffu, ahead, 1);
+        word = ahead;
+        ahead = words(i + 2);
+        if (layer != held) fetch(layer);
         Block b;
-        if (lane != 0) {
+        if (lane != 0 || w[0] == MKBH_OP_NOOP) {
         } else if (weight_block<T>(g, w[0], L, w[2], w[3], b)) {
             const int per = kStage / b.row_bytes;
             for (int row = b.r0; row < b.r1; row += per) {
@@ -958,6 +1058,10 @@ __device__ __forceinline__ void loader_main(const Params& p, Cta& c, const Smem&
             }
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);
+        if (layer != held) {
+            keep();
+            held = layer;
+        }
     }
     if (lane != 0) return;
     // no copy may be in flight when the CTA's shared memory goes away
@@ -1797,7 +1901,7 @@ __device__ __forceinline__ void consumer_main(const Params& p, Cta& c, const Sme
             if (tid == 0) report(g.status, c.ctl, MKBH_ERR_BAD_OPCODE, 1, i, op, 0, 0, 0);
             return;
         }
-        if (tid == 0 && signal) red_release_gpu_add(counters + d.arrive_idx, 1);
+        if (tid == 0 && signal) post_signal(p, c, counters, d.arrive_idx);
         if ((F & kRotary) && op == MKBH_OP_NORM_PROJ && (L.canon_taps > 1 || L.conv_taps > 1)) {  // for later tokens only
             publish_convolutions(p, c, d, stash, kept);
             csync();
@@ -1820,6 +1924,7 @@ __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_c
     c.instr = -1;
     c.opcode = -1;
     c.turn = 0;
+    c.signals = 0;
     c.pos = p.g.pos_device ? __ldg(p.g.pos_device) : p.g.pos0;
     if (threadIdx.x == 0) {
         for (int s = 0; s < p.stages; ++s) {
@@ -1837,9 +1942,15 @@ __global__ void __launch_bounds__(kBlock, 1) hybrid_decode_kernel(const __grid_c
         return;
     }
     const int warp = threadIdx.x >> 5;
-    if (warp < kConsumerWarps) consumer_main<T, F>(p, c, sm);
+    if (warp < kConsumerWarps) {
+        consumer_main<T, F>(p, c, sm);
+        if (kSignalWarp && threadIdx.x == 0) post_signal(p, c, nullptr, -1);
+    } else if (kSignalWarp && warp == kOperandWarp + 1) {
+        if ((threadIdx.x & 31) == 0) signal_main(p, c);
+    }
     else if (warp == kOperandWarp) operand_main<T>(p, c, sm);
-    else loader_main<T, F>(p, c, sm);
+    else if constexpr (F & kRotary) loader_main<T, F>(p, c, sm);
+    else if ((threadIdx.x & 31) == 0) weight_loader<T>(p, c);
     __syncthreads();
 }
 
