@@ -2,8 +2,9 @@
 // queries of one head x tiles of up to 128 keys.
 //
 // Warp roles: a TMA producer, an MMA thread, four softmax warps with one query row per thread.
-//   scores   S = Q K^T in tensor memory, two buffers: the next tile's scores are computed while this
-//            tile's go through the softmax;
+//   scores   S = Q K^T in tensor memory.  Two CTAs share an SM where shared and tensor memory allow, one
+//            of them in its softmax while the other multiplies; a CTA alone has two score buffers
+//            instead, and the next tile's scores are computed while this tile's are in the softmax;
 //   weights  overwrite their scores as bf16 in tensor memory and are the A operand of
 //   output   O += P V, V as it lies in the cache (MN-major), accumulated in tensor memory.
 // Scores, maxima, exponentials and sums are fp32.  O refers to a row maximum that is replaced only when
@@ -11,6 +12,8 @@
 // without a value that is there from the start.  Outputs of rotated values are turned back at the end.
 // Keys may come in two pieces (a latent's expanded part per head, its rotated part for all heads).
 // A tile never crosses the point where a ring of cache rows wraps.
+#include <type_traits>
+
 #include "hybrid_kernels.h"
 #include "hybrid_tcgen05.cuh"
 
@@ -22,7 +25,6 @@ namespace {
 // output columns that are not stored.
 constexpr int kRows = 128, kTile = 128, kSlab = kTile * 128;
 constexpr int kFlashThreads = 192;
-constexpr int kOut = 2 * kTile;  // tensor-memory column of the output, behind two score buffers
 constexpr float kSlack = 8.f;
 
 struct FlashShape {
@@ -59,8 +61,11 @@ struct Tiles {
     __device__ __forceinline__ int len(int j) const { return min(min(kTile, hi - j + 1), ring - row(j)); }
 };
 
-template <int kE>  // value columns, in whole slabs
-__global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid_constant__ FlashMaps maps, const FlashShape s) {
+// kE: value columns, in whole slabs.  kBufs: score buffers (1: two CTAs per SM).
+template <int kE, int kBufs>
+__global__ void __launch_bounds__(kFlashThreads, kBufs == 1 ? 2 : 1) flash_tc_kernel(const __grid_constant__ FlashMaps maps, const FlashShape s) {
+    constexpr int kOut = kBufs * kTile;  // tensor-memory column of the output, behind the scores
+    constexpr uint32_t kColumns = kOut + kE <= 256 ? 256 : 512;
     extern __shared__ uint8_t raw[];
     const uint32_t raw32 = mkb::smem_u32(raw), base = (raw32 + 1023u) & ~1023u;
     const int slabs = s.split_slabs + s.rest_slabs, S = s.stages;
@@ -98,7 +103,7 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     if (warp == 1) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(base + sm.ctl + 4), "r"(512u) : "memory");
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(base + sm.ctl + 4), "r"(kColumns) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     tc_before_sync();
@@ -151,28 +156,28 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
             for (int i = 0; i < slabs; ++i)
 #pragma unroll
                 for (int kk = 0; kk < 4; ++kk)
-                    tc_mma(tmem + (t & 1) * kTile, tc_desc(q + i * kSlab + kk * 32), tc_desc(k + i * kSlab + kk * 32), s_desc, (uint32_t)((i | kk) != 0));
+                    tc_mma(tmem + (t % kBufs) * kTile, tc_desc(q + i * kSlab + kk * 32), tc_desc(k + i * kSlab + kk * 32), s_desc, (uint32_t)((i | kk) != 0));
             tc_commit(k_empty(st));
-            tc_commit(s_full(t & 1));
+            tc_commit(s_full(t % kBufs));
             return true;
         };
         int count = 0;
         for (int j = tiles.lo; j <= tiles.hi; j += tiles.len(j)) ++count;
         bool ok = wait(q_full, 0, 1);
-        for (int t = 0; t < 2 && t < count && ok; ++t) ok = scores(t);
+        for (int t = 0; t < kBufs && t < count && ok; ++t) ok = scores(t);
         for (int t = 0; t < count && ok; ++t) {
             const int st = t % S;
-            ok = wait(p_full(t & 1), (uint32_t)(t >> 1), 1) && wait(v_full(st), (uint32_t)(t / S), 1);
+            ok = wait(p_full(t % kBufs), (uint32_t)(t / kBufs), 1) && wait(v_full(st), (uint32_t)(t / S), 1);
             if (!ok) break;
             tc_after_sync();
             const uint32_t v = base + sm.v + st * s.v_slabs * kSlab;
 #pragma unroll
             for (int kk = 0; kk < kTile / 16; ++kk)
-                tc_mma_ts(tmem + kOut, tmem + (t & 1) * kTile + kk * 8, tc_desc_mn(v + kk * 2048, kSlab), o_desc, (uint32_t)((t | kk) != 0));
+                tc_mma_ts(tmem + kOut, tmem + (t % kBufs) * kTile + kk * 8, tc_desc_mn(v + kk * 2048, kSlab), o_desc, (uint32_t)((t | kk) != 0));
             tc_commit(v_empty(st));
             tc_commit(o_done(t & 1));
             // (the weights have been read before their buffer takes scores again)
-            if (t + 2 < count) ok = wait(o_done(t & 1), (uint32_t)(t >> 1), 1) && scores(t + 2);
+            if (t + kBufs < count) ok = wait(o_done(t & 1), (uint32_t)(t >> 1), 1) && scores(t + kBufs);
         }
     } else if (warp >= 2) {
         const int quarter = warp & 3, r = quarter * 32 + lane;  // the tensor-memory lanes this warp may touch
@@ -185,35 +190,54 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
         int t = 0;
         for (int j = tiles.lo; j <= tiles.hi; j += tiles.len(j), ++t) {
             const int len = tiles.len(j);
-            ok = __all_sync(0xffffffffu, wait(s_full(t & 1), (uint32_t)(t >> 1), 2));
+            ok = __all_sync(0xffffffffu, wait(s_full(t % kBufs), (uint32_t)(t / kBufs), 2));
             if (!ok) break;
             tc_after_sync();
-            const uint32_t at = lanes + (t & 1) * kTile;
-            uint32_t x[kTile];
+            const uint32_t at = lanes + (t % kBufs) * kTile;
+            // a row in registers, or (two CTAs) a quarter of it at a time, read twice
+            constexpr bool kHold = kBufs > 1;
+            uint32_t x[kHold ? kTile : 64];
+            const bool whole = len == kTile && j >= warp_last_lo && j + kTile - 1 <= warp_p0;  // every row sees the whole tile
+            const int first = row_lo - j, last = min(pos - j, len - 1);
+            const float mul = whole || !kHold ? scale : 1.f;
+            float best, m4[4];
+            const bool low = whole && scale < 0.f;  // (then the smallest product is the largest score)
 #pragma unroll
-            for (int c = 0; c < kTile; c += 32) tc_load32_async(at + c, x + c);
-            tc_loaded();
-            float mul = scale, best = -INFINITY;
-            if (len == kTile && j >= warp_last_lo && j + kTile - 1 <= warp_p0) {  // every row sees the whole tile
-                if (scale >= 0.f) {
+            for (int i = 0; i < 4; ++i) m4[i] = low ? INFINITY : -INFINITY;
+            if constexpr (kHold) {
 #pragma unroll
-                    for (int c = 0; c < kTile; ++c) best = fmaxf(best, __uint_as_float(x[c]));
-                } else {
-                    best = INFINITY;
+                for (int c = 0; c < kTile; c += 32) tc_load32_async(at + c, x + c);
 #pragma unroll
-                    for (int c = 0; c < kTile; ++c) best = fminf(best, __uint_as_float(x[c]));
-                }
-                best *= scale;
+                for (int c = 0; c < kTile; c += 32) tc_loaded32(x + c);
             } else {
-                const int first = row_lo - j, last = min(pos - j, len - 1);
-#pragma unroll
-                for (int c = 0; c < kTile; ++c) {
-                    const float y = c >= first && c <= last ? __uint_as_float(x[c]) * scale : -INFINITY;
-                    best = fmaxf(best, y);
-                    x[c] = __float_as_uint(y);
-                }
-                mul = 1.f;
+                tc_load32_async(at, x);
             }
+#pragma unroll
+            for (int c = 0; c < kTile; c += 32) {
+                uint32_t* y = kHold ? x + c : x + (c & 32);
+                if constexpr (!kHold) {
+                    tc_loaded32(y);
+                    if (c + 32 < kTile) tc_load32_async(at + c + 32, x + ((c + 32) & 32));
+                    else tc_load32_async(at, x);  // (again, for the weights)
+                }
+                if (low) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) m4[i & 3] = fminf(m4[i & 3], __uint_as_float(y[i]));
+                } else if (whole) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(y[i]));
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) {
+                        const float z = c + i >= first && c + i <= last ? __uint_as_float(y[i]) * scale : -INFINITY;
+                        m4[i & 3] = fmaxf(m4[i & 3], z);
+                        if (kHold) y[i] = __float_as_uint(z);
+                    }
+                }
+            }
+            best = low ? fminf(fminf(m4[0], m4[1]), fminf(m4[2], m4[3])) : fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+            if (whole) best *= scale;
+            if constexpr (!kHold) tc_loaded32(x);
             const bool raise = best > top + kSlack;
             if (__any_sync(0xffffffffu, raise)) {
                 const float f = raise ? exp2f(top - best) : 1.f;  // (0 from minus infinity)
@@ -223,7 +247,7 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
                     ok = __all_sync(0xffffffffu, wait(o_done((t - 1) & 1), (uint32_t)((t - 1) >> 1), 2));
                     if (!ok) break;
                     tc_after_sync();
-#pragma unroll
+#pragma unroll 1
                     for (int c = 0; c < kE; c += 32) {
                         uint32_t o[32];
                         tc_load32(lanes + kOut + c, o);
@@ -236,24 +260,36 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
             }
             const float off = top == -INFINITY ? 0.f : top;
             float part[4] = {0.f, 0.f, 0.f, 0.f};
+            auto weights = [&](auto masked) {
 #pragma unroll
-            for (int c = 0; c < kTile; c += 32) {
-                uint32_t w[16];
+                for (int c = 0; c < kTile; c += 32) {
+                    uint32_t w[16], *y = kHold ? x + c : x + (c & 32);
+                    if constexpr (!kHold) {
+                        if (c > 0) tc_loaded32(y);
+                        if (c + 32 < kTile) tc_load32_async(at + c + 32, x + ((c + 32) & 32));
+                    }
 #pragma unroll
-                for (int i = 0; i < 16; ++i) {
-                    float a, b;
-                    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(a) : "f"(fmaf(__uint_as_float(x[c + 2 * i]), mul, -off)));
-                    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(b) : "f"(fmaf(__uint_as_float(x[c + 2 * i + 1]), mul, -off)));
-                    part[i & 3] += a + b;
-                    w[i] = mkb::pack_bf16x2(a, b);
+                    for (int i = 0; i < 16; ++i) {
+                        float z[2];
+#pragma unroll
+                        for (int k = 0; k < 2; ++k) {
+                            const float u = fmaf(__uint_as_float(y[2 * i + k]), mul, -off);
+                            asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(z[k]) : "f"(u));
+                            if constexpr (decltype(masked)::value) z[k] = c + 2 * i + k >= first && c + 2 * i + k <= last ? z[k] : 0.f;
+                        }
+                        part[i & 3] += z[0] + z[1];
+                        w[i] = mkb::pack_bf16x2(z[0], z[1]);
+                    }
+                    tc_store16(at + c / 2, w);
                 }
-                tc_store16(at + c / 2, w);
-            }
+            };
+            if (kHold || whole) weights(std::false_type{});
+            else weights(std::true_type{});
             sum += (part[0] + part[1]) + (part[2] + part[3]);
             tc_stored();
             tc_before_sync();
             __syncwarp();
-            if (lane == 0) mkb::mbar_arrive(p_full(t & 1));
+            if (lane == 0) mkb::mbar_arrive(p_full(t % kBufs));
         }
         if (ok) ok = __all_sync(0xffffffffu, wait(o_done((t - 1) & 1), (uint32_t)((t - 1) >> 1), 2));
         if (ok) {
@@ -288,30 +324,30 @@ __global__ void __launch_bounds__(kFlashThreads, 1) flash_tc_kernel(const __grid
     }
     tc_before_sync();
     __syncthreads();
-    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
 }
 
 int slabs_of(int n) { return (n + 63) / 64; }
-constexpr int kLimit = 227 * 1024 - 1024;
-int stages_for(int slabs, int v_slabs) {
+constexpr int kLimit = 227 * 1024 - 1024, kShared = 113 * 1024 - 1024;  // a CTA alone, two of them
+int stages_for(int slabs, int v_slabs, int limit) {
     for (int st = 4; st >= 2; --st)
-        if (FlashSmem(slabs, v_slabs, st).total <= kLimit) return st;
+        if (FlashSmem(slabs, v_slabs, st).total <= limit) return st;
     return 0;
 }
 
-template <int kE>
+template <int kE, int kBufs>
 cudaError_t launch(const FlashMaps& maps, const FlashShape& s, cudaStream_t stream) {
     static bool set[64] = {};
     int dev = 0;
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return e;
     if (!set[dev & 63]) {
-        e = cudaFuncSetAttribute(flash_tc_kernel<kE>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLimit + 1024);
+        e = cudaFuncSetAttribute(flash_tc_kernel<kE, kBufs>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLimit + 1024);
         if (e != cudaSuccess) return e;
         set[dev & 63] = true;
     }
     const int bytes = FlashSmem(s.split_slabs + s.rest_slabs, s.v_slabs, s.stages).total + 1024;
-    flash_tc_kernel<kE><<<dim3(s.heads, (s.n + kRows - 1) / kRows), kFlashThreads, bytes, stream>>>(maps, s);
+    flash_tc_kernel<kE, kBufs><<<dim3(s.heads, (s.n + kRows - 1) / kRows), kFlashThreads, bytes, stream>>>(maps, s);
     return cudaGetLastError();
 }
 
@@ -320,7 +356,7 @@ cudaError_t launch(const FlashMaps& maps, const FlashShape& s, cudaStream_t stre
 bool flash_tc_supported(const MkbhLayer& L) {
     const int rest = L.mixer == MKBH_LATENT_ATTENTION ? L.rot_dim : 0;
     return L.dim % 8 == 0 && rest % 8 == 0 && L.vdim % 8 == 0 && L.vdim <= 128 && L.cache_keep == 0 && L.keep_first == 0 &&
-           stages_for(slabs_of(L.dim) + slabs_of(rest), slabs_of(L.vdim)) >= 2;
+           stages_for(slabs_of(L.dim) + slabs_of(rest), slabs_of(L.vdim), kLimit) >= 2;
 }
 
 cudaError_t flash_tc(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_t ldo, cudaStream_t stream) {
@@ -341,8 +377,12 @@ cudaError_t flash_tc(const MkbhGlobals& g, const MkbhLayer& L, bf16* out, int64_
     FlashShape s{g.num_tokens, g.pos0, H, src.per, slabs_of(A), B > 0 ? slabs_of(B) : 0, slabs_of(L.vdim), 0,
                  latent ? A : 0, latent ? L.vdim : 0, latent ? H * A : 0, latent ? 0 : rows, latent ? 0 : rows,
                  L.window, L.chunk, rows, L.vdim, L.scale, L.temp, L.sink, L.value_rope, out, ldo, 2000000000ull, g.status};
-    s.stages = stages_for(s.split_slabs + s.rest_slabs, s.v_slabs);
-    return s.v_slabs == 1 ? launch<64>(m, s, stream) : launch<128>(m, s, stream);
+    const int all = s.split_slabs + s.rest_slabs;
+    s.stages = stages_for(all, s.v_slabs, kShared);
+    if (s.stages >= 2 && s.v_slabs == 1) return launch<64, 1>(m, s, stream);
+    if (s.stages >= 2) return launch<128, 1>(m, s, stream);
+    s.stages = stages_for(all, s.v_slabs, kLimit);
+    return s.v_slabs == 1 ? launch<64, 2>(m, s, stream) : launch<128, 2>(m, s, stream);
 }
 
 }  // namespace mkbh

@@ -75,7 +75,7 @@ __device__ __forceinline__ void tc_commit(uint32_t bar) {
 }
 __device__ __forceinline__ void tc_before_sync() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
 __device__ __forceinline__ void tc_after_sync() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-// 32 columns of the warp's 32 lanes (complete after tc_loaded)
+// 32 columns of the warp's 32 lanes (complete after tc_loaded32)
 __device__ __forceinline__ void tc_load32_async(uint32_t addr, uint32_t* r) {
     asm volatile(
         "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
@@ -87,10 +87,17 @@ __device__ __forceinline__ void tc_load32_async(uint32_t addr, uint32_t* r) {
           "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
         : "r"(addr));
 }
-__device__ __forceinline__ void tc_loaded() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+// (the registers pass through, so that nothing uses them before)
+__device__ __forceinline__ void tc_loaded32(uint32_t* r) {
+    asm volatile("tcgen05.wait::ld.sync.aligned;"
+                 : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]), "+r"(r[8]), "+r"(r[9]),
+                   "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]), "+r"(r[15]), "+r"(r[16]), "+r"(r[17]), "+r"(r[18]),
+                   "+r"(r[19]), "+r"(r[20]), "+r"(r[21]), "+r"(r[22]), "+r"(r[23]), "+r"(r[24]), "+r"(r[25]), "+r"(r[26]), "+r"(r[27]),
+                   "+r"(r[28]), "+r"(r[29]), "+r"(r[30]), "+r"(r[31])::"memory");
+}
 __device__ __forceinline__ void tc_load32(uint32_t addr, uint32_t (&r)[32]) {
     tc_load32_async(addr, r);
-    tc_loaded();
+    tc_loaded32(r);
 }
 __device__ __forceinline__ void tc_store16(uint32_t addr, const uint32_t* r) {
     asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(addr),
