@@ -4,8 +4,8 @@ Same ``key=value`` command line and timing method as the reference script
 (megakernels/scripts/generate.py:28-207): CUDA events around a whole
 generation of ``ntok - 1`` tokens, ``num_warmup`` + ``num_iters`` repeats.
 Differences: ``model=`` names an architecture preset (``llama-1b``,
-``llama-8b``, ``llama-70b``, ``torirax-1b``, ``torirax-8b``) initialised from
-``seed=`` or a local checkpoint directory of either family (``registry.py``), and the prompt is a list of token ids (``prompt_ids=1,2,3`` or
+``llama-8b``, ``llama-70b``, ``torirax-1b``, ``torirax-8b``, ``dumalix-1b``, ``dumalix-8b``) initialised
+from ``seed=`` or a local checkpoint directory of any family (``registry.py``), and the prompt is a list of token ids (``prompt_ids=1,2,3`` or
 ``prompt_len=32`` random ids) because no tokenizer ships with this package.
 Only ``mode=mk`` exists here.
 """
