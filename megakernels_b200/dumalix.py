@@ -31,7 +31,7 @@ def read_layer(i: int, raw: dict, canon_taps: int, shape_of) -> LayerSpec:
     if raw["type"] == "attention":
         mixer = RotaryAttentionSpec(
             heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=m["scale"], chunk=m["mask"]["size"],
-            rope=read_rope(m["rot"]), conv_taps=shape_of(f"l{i}.mix.q.conv")[1], turn_values=True,
+            rope=read_rope(m["rot"]), conv_taps=m["conv"] or 0 if "conv" in m else shape_of(f"l{i}.mix.q.conv")[1],
         )
     elif raw["type"] == "latent_attention":
         mixer = LatentAttentionSpec(

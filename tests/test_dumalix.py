@@ -10,7 +10,7 @@ import torch
 from megakernels_b200.demos.hybrid import instructions as I
 from megakernels_b200.demos.hybrid.scheduler import head_row_ranges, row_ranges
 from megakernels_b200.dispatch import make_schedule_builder
-from megakernels_b200.dumalix import PRESETS, DumalixForCausalLM
+from megakernels_b200.dumalix import PRESETS, DumalixForCausalLM, read_layer
 from megakernels_b200.hybrid import HybridConfig, HybridForCausalLM, LayerSpec, LoopSpec, PolyNormSpec, RopeSpec, YarnSpec, key_splits, tensor_shapes
 from megakernels_b200.model_types import ExtraModelConfig
 from megakernels_b200.registry import family_of_checkpoint, family_of_preset, load_model
@@ -200,6 +200,10 @@ def test_checkpoint_reading_stacks_and_folds(tmp_path):
     assert m.state.keys[1].shape == (2, 90, 40) and 1 not in m.state.values
     assert m.state.inputs[3].shape == (2, 2, 72) and m.state.projected[2].shape == (2, 2, 6 * 20 + 3 * 48) and 1 not in m.state.projected
     b = load_model(path, ExtraModelConfig(max_len_override=90, prefill_portion=4), device="cpu")
+    assert read_layer(0, changed(ODD, 0, ("mixer", "conv"), 0)["layers"][0], 3, None).mixer.conv_taps == 0
+    raw = changed(ODD, 0, ("x",), 0)["layers"][0]
+    del raw["mixer"]["conv"]  # then the tensors say
+    assert read_layer(0, raw, 3, lambda name: tuple(w[name].shape)).mixer.conv_taps == 3
     assert b.state.rows[0] == CacheRows(0, 11 + 4) and b.state.rows[1] == CacheRows(0, 90) and b.dtype == torch.bfloat16
     assert load_model(path, ExtraModelConfig(prefill_portion=4), device="cpu").max_len() == 32768  # the design sets no limit
 
